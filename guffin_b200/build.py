@@ -51,7 +51,9 @@ def build(force: bool = False, verbose: bool = False, testing: bool = False) -> 
             raise RuntimeError(f"nvcc failed on {src}")
         with open(os.path.join(out_dir, os.path.basename(src) + ".ptxas.txt"), "w") as f:
             f.write(out)
-    subprocess.run([NVCC, "-shared", "-o", lib, *objects, "-lcudart"], check=True)
+    part = f"{lib}.{os.getpid()}"
+    subprocess.run([NVCC, "-shared", "-o", part, *objects, "-lcudart"], check=True)
+    os.replace(part, lib)
     return lib
 
 

@@ -1,0 +1,401 @@
+// Products over a chunk of prompt rows and the elementwise steps between them (see dense.cuh).
+#include "dense.cuh"
+#include "tcgen05.cuh"
+
+#include <algorithm>
+#include <mutex>
+
+namespace gf {
+
+namespace {
+
+// ------------------------------------------------------------------ outputs
+
+// Column n of the result of product `index` for output row `row`.
+__device__ __forceinline__ void chunk_store(const ChunkProblem& p, uint32_t index, uint32_t row, uint32_t n, float v) {
+    if (p.output == kChunkF32) {
+        if (p.row_scale) {
+            const float s = p.row_scale[(size_t)row * p.row_scale_ld];
+            v *= p.row_scale_sigmoid ? sigmoid(s) : s;
+        }
+        p.out[(size_t)row * p.out_ld + n] = v;
+    } else if (p.output == kChunkLatentQuery) {
+        const size_t at = ((size_t)row * p.heads + index) * p.out_ld + n;
+        if (p.query_f16) reinterpret_cast<__half*>(p.out)[at] = __float2half_rn(v * p.scale);
+        else p.out[at] = v * p.scale;
+    } else {
+        const uint32_t column = (p.segment ? n / p.segment * p.segment_pad + n % p.segment : n) + index * p.column_stride;
+        store_operand(p.result, row, column, p.output == kChunkSquaredRelu ? squared_relu(v) : v);
+    }
+}
+// Column n of a paired product.
+__device__ __forceinline__ void chunk_store_gate(const ChunkProblem& p, uint32_t row, uint32_t n, float gate, float up) {
+    const float s = p.row_scale ? p.row_scale[(size_t)row * p.row_scale_ld] : 1.0f;
+    store_operand(p.result, row, n, clamped_gate(gate * s, up * s, p.limit));
+}
+
+// ------------------------------------------------------------------ bf16 products on tcgen05
+
+constexpr uint32_t kWindowMax = 256;                                   // token rows of a tile: the product's N
+constexpr uint32_t kStages = 4;
+constexpr uint32_t kStageBytes = kDenseTileBytes + kWindowMax * 128u;  // 128 weight columns, then up to 256 token rows, x 64 K
+constexpr uint32_t kEpilogueWarps = 8;
+constexpr uint32_t kChunkThreads = (kEpilogueWarps + 2u) * 32u;        // the copying and the issuing warp behind them
+constexpr uint32_t kChunkSmemBytes = kStages * kStageBytes + (2u * kStages + 1u) * 8u + 16u;
+
+// The tensor core's A operand is a tile of 128 weight columns and its B operand a window of up to 256 token rows, so
+// the product's N follows the rows there are (an expert may have few) and accumulator lanes are output columns.
+__global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const __grid_constant__ ChunkProduct p) {
+    extern __shared__ __align__(1024) uint8_t smem[];
+    __shared__ uint32_t tmem_slot, abort_flag;
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem + kStages * kStageBytes);      // [kStages] copies landed (bytes)
+    uint64_t* free_bar = full + kStages;                                             // [kStages] the stage's products have finished
+    uint64_t* done_bar = free_bar + kStages;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const volatile uint32_t* abort = &abort_flag;
+
+    uint32_t which = 0;
+    while (which + 1u < p.problems && blockIdx.x >= p.p[which + 1u].first_tile) ++which;
+    const ChunkProblem& m = p.p[which];
+    const uint32_t index = (blockIdx.x - m.first_tile) / m.tiles, tile = (blockIdx.x - m.first_tile) % m.tiles;
+    const uint32_t start = m.group_start ? m.group_start[index] : 0u, rows = m.group_rows ? m.group_rows[index] : p.rows;
+    const uint32_t first_row = blockIdx.y * p.window;
+    if (first_row >= rows) return;
+    const uint32_t live = min(p.window, rows - first_row), n_rows = (live + 15u) & ~15u, row0 = start + first_row;
+    const uint8_t* weight = m.weight + index * m.weight_stride + (size_t)tile * m.k_blocks * kDenseTileBytes;
+    const uint8_t* rows_at = static_cast<const uint8_t*>(m.a.data) + (size_t)(m.a_block0 + index * m.a_block_stride) * m.a.capacity * 128u + (size_t)row0 * 128u;
+
+    uint32_t tmem_columns = 32u;
+    while (tmem_columns < n_rows) tmem_columns *= 2u;
+    if (tid == 0) {
+        abort_flag = 0u;
+        for (uint32_t i = 0; i < kStages; ++i) { mbar_init(&full[i], 1); mbar_init(&free_bar[i], 1); }
+        mbar_init(done_bar, 1);
+        fence_barrier_init();
+    }
+    if (warp == 0) tmem_alloc(&tmem_slot, tmem_columns);
+    tc_fence_before_sync();
+    __syncthreads();
+    tc_fence_after_sync();
+    const uint32_t tmem = tmem_slot, steps = m.k_blocks;
+    bool ok = true;
+
+    if (warp == kEpilogueWarps) {
+        if (lane == 0) {
+            uint32_t requested = 0;
+            for (uint32_t step = 0; step < steps; ++step) {
+                const uint32_t stage = step % kStages, use = step / kStages;
+                if (use > 0u && !wait_or_abort(&free_bar[stage], (use - 1u) & 1u, abort)) { ok = false; break; }
+                uint8_t* at = smem + stage * kStageBytes;
+                mbar_expect_tx(&full[stage], kDenseTileBytes + n_rows * 128u);
+                bulk_load(at, weight + (size_t)step * kDenseTileBytes, kDenseTileBytes, &full[stage]);
+                bulk_load(at + kDenseTileBytes, rows_at + (size_t)step * m.a.capacity * 128u, n_rows * 128u, &full[stage]);
+                requested = step + 1u;
+            }
+            if (!ok || !wait_or_abort(done_bar, 0u, abort)) {
+                // Copies already requested get a bounded chance to land before the shared memory is released.
+                ok = false;
+                abort_flag = 1u;
+                for (uint32_t step = requested > kStages ? requested - kStages : 0u; step < requested; ++step)
+                    mbar_wait(&full[step % kStages], (step / kStages) & 1u, 1u << 16);
+            }
+        }
+    } else if (warp == kEpilogueWarps + 1u) {
+        if (lane == 0) {
+            const uint32_t instruction = mma_instruction(kDenseTile, n_rows);
+            for (uint32_t step = 0; step < steps; ++step) {
+                const uint32_t stage = step % kStages;
+                if (!wait_or_abort(&full[stage], (step / kStages) & 1u, abort)) { ok = false; break; }
+                tc_fence_after_sync();
+                const uint32_t at = smem_u32(smem + stage * kStageBytes);
+#pragma unroll
+                for (uint32_t kk = 0; kk < kDenseBlockK / 16u; ++kk)
+                    mma_bf16(tmem, operand_descriptor(at + kk * 256u), operand_descriptor(at + kDenseTileBytes + kk * 256u), instruction, (step | kk) != 0u ? 1u : 0u);
+                mma_commit(&free_bar[stage]);
+            }
+            if (ok) mma_commit(done_bar);
+            else abort_flag = 1u;
+        }
+    } else {
+        if (!wait_or_abort(done_bar, 0u, abort)) { ok = false; if (lane == 0) abort_flag = 1u; }
+    }
+    const bool failed = __syncthreads_or(ok ? 0 : 1) != 0;
+    if (!failed && warp < kEpilogueWarps) {
+        tc_fence_after_sync();
+        // Warp w reads accumulator lanes 32 (w % 4) .. + 31, i.e. output columns; a warp's accumulator columns are token rows.
+        const uint32_t quarter = warp & 3u, column = tile * kDenseTile + quarter * 32u + lane;
+        const bool paired = m.output == kChunkClampedGate;
+        const uint32_t pair_column = tile * (kDenseTile / 2u) + quarter * 16u + (lane >> 4) * 8u + (lane & 7u);
+        for (uint32_t c = (warp >> 2) * 32u; c < live; c += 64u) {
+            float v[32];
+            tmem_load_32(tmem + ((quarter * 32u) << 16) + c, v);
+#pragma unroll
+            for (uint32_t i = 0; i < 32u; ++i) {
+                const uint32_t row = row0 + c + i;
+                if (paired) {
+                    const float up = __shfl_xor_sync(0xffffffffu, v[i], 8);
+                    if (c + i < live && (lane & 8u) == 0u && pair_column < m.n / 2u) chunk_store_gate(m, row, pair_column, v[i], up);
+                } else if (c + i < live && column < m.n) {
+                    chunk_store(m, index, row, column, v[i]);
+                }
+            }
+        }
+        tc_fence_before_sync();
+    } else if (failed && tid == 0) {
+        atomicExch(p.error_flag, 1);
+    }
+    __syncthreads();
+    if (warp == 0) tmem_dealloc(tmem, tmem_columns);
+}
+
+// ------------------------------------------------------------------ f32 products
+
+// 64 rows x 64 columns per CTA, 4 x 4 per thread; a thread's columns are two (gate, up) pairs of a paired matrix.
+__global__ void __launch_bounds__(256) chunk_product_f32_kernel(const __grid_constant__ ChunkProduct p) {
+    __shared__ float a_tile[32][65], w_tile[32][65];
+    const uint32_t tid = threadIdx.x;
+    uint32_t which = 0;
+    while (which + 1u < p.problems && blockIdx.x >= p.p[which + 1u].first_tile) ++which;
+    const ChunkProblem& m = p.p[which];
+    const uint32_t index = (blockIdx.x - m.first_tile) / m.tiles, tile = (blockIdx.x - m.first_tile) % m.tiles;
+    const uint32_t start = m.group_start ? m.group_start[index] : 0u, rows = m.group_rows ? m.group_rows[index] : p.rows;
+    const uint32_t first_row = blockIdx.y * 64u;
+    if (first_row >= rows) return;
+    const uint32_t live = min(64u, rows - first_row), row0 = start + first_row;
+    const uint8_t* weight = m.weight + index * m.weight_stride;
+    const float* a = static_cast<const float*>(m.a.data) + (size_t)(m.a_block0 + index * m.a_block_stride) * kDenseBlockK;
+    const uint32_t tx = tid & 15u, ty = tid >> 4, column0 = (tx >> 3) * 16u + (tx & 7u);
+    const uint32_t columns[4] = {column0, column0 + 8u, column0 + 32u, column0 + 40u};
+    float acc[4][4] = {};
+    for (uint32_t k0 = 0; k0 < m.k; k0 += 32u) {
+        for (uint32_t i = tid; i < 64u * 32u; i += 256u) {
+            const uint32_t r = i >> 5, k = i & 31u;
+            a_tile[k][r] = r < live && k0 + k < m.k ? a[(size_t)(row0 + r) * m.a.k_pad + k0 + k] : 0.0f;
+        }
+        {
+            const uint32_t n = tid & 63u, piece = tid >> 6;            // 64 columns x four pieces of eight
+            const uint4 v = *reinterpret_cast<const uint4*>(weight + dense_offset(m.k_blocks, tile * 64u + n, k0 + piece * 8u));
+            const uint32_t words[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (uint32_t j = 0; j < 4u; ++j) {
+                w_tile[piece * 8u + 2u * j][n] = __uint_as_float(words[j] << 16);
+                w_tile[piece * 8u + 2u * j + 1u][n] = __uint_as_float(words[j] & 0xffff0000u);
+            }
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (uint32_t k = 0; k < 32u; ++k) {
+            float x[4], w[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) { x[i] = a_tile[k][ty * 4u + i]; w[i] = w_tile[k][columns[i]]; }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(x[i], w[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    for (int i = 0; i < 4; ++i) {
+        const uint32_t r = ty * 4u + i;
+        if (r >= live) continue;
+        if (m.output == kChunkClampedGate) {
+            for (int j = 0; j < 4; j += 2) {
+                const uint32_t n = tile * 32u + (columns[j] >> 4) * 8u + (columns[j] & 7u);
+                if (n < m.n / 2u) chunk_store_gate(m, row0 + r, n, acc[i][j], acc[i][j + 1]);
+            }
+        } else {
+            for (int j = 0; j < 4; ++j)
+                if (tile * 64u + columns[j] < m.n) chunk_store(m, index, row0 + r, tile * 64u + columns[j], acc[i][j]);
+        }
+    }
+}
+
+// ------------------------------------------------------------------ norms, routing, cache rows
+
+__device__ __forceinline__ float block_total(float v, float* scratch) {
+    v = warp_sum(v);
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u;
+    if (lane == 0) scratch[warp] = v;
+    __syncthreads();
+    float total = 0.0f;
+    for (uint32_t w = 0; w < blockDim.x / 32u; ++w) total += scratch[w];
+    __syncthreads();
+    return total;
+}
+
+__global__ void __launch_bounds__(256) chunk_norm_kernel(const ChunkNorm p) {
+    extern __shared__ float row_values[];
+    __shared__ float scratch[8];
+    const uint32_t row = blockIdx.x;
+    float* residual = p.residual + (size_t)row * p.width;
+    float sum = 0.0f;
+    if (p.y) {
+        for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+            float v;
+            if (p.slots) {
+                v = 0.0f;
+                for (uint32_t s = 0; s < p.slots; ++s) v += p.y[(size_t)p.slot_rows[row * p.slots + s] * p.width + i];
+                if (p.shared) v += p.shared[(size_t)row * p.width + i];
+            } else v = p.y[(size_t)row * p.width + i];
+            row_values[i] = v;
+            sum = fmaf(v, v, sum);
+        }
+        const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps);
+        sum = 0.0f;
+        for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+            const float v = residual[i] + row_values[i] * inv * p.gain0[i];
+            residual[i] = v;
+            row_values[i] = v;
+            sum = fmaf(v, v, sum);
+        }
+    } else {
+        for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+            const float v = residual[i];
+            row_values[i] = v;
+            sum = fmaf(v, v, sum);
+        }
+    }
+    if (!p.gain1) return;
+    const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps);
+    for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
+        const float v = row_values[i] * inv * p.gain1[i];
+        if (p.result.data) store_operand(p.result, row, i, v);
+        if (p.normed) p.normed[(size_t)row * p.width + i] = v;
+    }
+}
+
+// One block: every warp routes rows; counts, starts and grouped rows follow from the choices.
+__global__ void __launch_bounds__(1024) chunk_route_kernel(const ChunkRoute p) {
+    __shared__ uint32_t counts[kMaxExperts], starts[kMaxExperts];
+    extern __shared__ float scores[];                                  // [warps][experts]
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, warps = blockDim.x >> 5;
+    for (uint32_t e = threadIdx.x; e < p.experts; e += blockDim.x) counts[e] = 0;
+    __syncthreads();
+    for (uint32_t row = warp; row < p.rows; row += warps)
+        route_row(p.logits + (size_t)row * p.logits_ld, p.experts, p.top, scores + warp * p.experts, [&](uint32_t slot, uint32_t e, float score) {
+            if (lane != 0) return;
+            const uint32_t at = row * p.top + slot;
+            p.slot_experts[at] = e;
+            p.slot_scores[at] = score;
+            p.slot_rows[at] = atomicAdd(&counts[e], 1u);
+        });
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        uint32_t at = 0;
+        for (uint32_t e = 0; e < p.experts; ++e) { starts[e] = at; at += (counts[e] + 7u) & ~7u; }
+    }
+    __syncthreads();
+    for (uint32_t e = threadIdx.x; e < p.experts; e += blockDim.x) { p.group_start[e] = starts[e]; p.group_rows[e] = counts[e]; }
+    for (uint32_t at = threadIdx.x; at < p.rows * p.top; at += blockDim.x) {
+        const uint32_t grouped = starts[p.slot_experts[at]] + p.slot_rows[at];
+        p.slot_rows[at] = grouped;
+        p.row_scale[grouped] = p.slot_scores[at];
+    }
+}
+
+// Copies a token's normalised row to its grouped rows, 16 bytes at a time.
+__global__ void __launch_bounds__(256) chunk_group_kernel(const ChunkRoute p) {
+    const uint32_t at = blockIdx.x, row = at / p.top, grouped = p.slot_rows[at];
+    if (p.from.f32) {
+        const float4* src = reinterpret_cast<const float4*>(static_cast<const float*>(p.from.data) + (size_t)row * p.from.k_pad);
+        float4* dst = reinterpret_cast<float4*>(static_cast<float*>(p.to.data) + (size_t)grouped * p.to.k_pad);
+        for (uint32_t i = threadIdx.x; i < p.from.k_pad / 4u; i += blockDim.x) dst[i] = src[i];
+        return;
+    }
+    for (uint32_t i = threadIdx.x; i < p.from.k_pad / 8u; i += blockDim.x)
+        *reinterpret_cast<uint4*>(static_cast<uint8_t*>(p.to.data) + operand_offset(p.to, grouped, i * 8u)) =
+            *reinterpret_cast<const uint4*>(static_cast<const uint8_t*>(p.from.data) + operand_offset(p.from, row, i * 8u));
+}
+
+__global__ void __launch_bounds__(128) chunk_latents_kernel(const float* __restrict__ raw, uint32_t raw_ld, const float* __restrict__ gain, uint32_t rank,
+                                                            float eps, void* cache_rows, uint32_t row_elements, bool f16, uint32_t* status) {
+    __shared__ float scratch[8];
+    const uint32_t row = blockIdx.x;
+    const float* x = raw + (size_t)row * raw_ld;
+    float sum = 0.0f;
+    for (uint32_t i = threadIdx.x; i < rank; i += blockDim.x) sum = fmaf(x[i], x[i], sum);
+    const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)rank + eps);
+    for (uint32_t i = threadIdx.x; i < row_elements; i += blockDim.x) {
+        const float v = i < rank ? x[i] * inv * gain[i] : 0.0f;
+        const size_t at = (size_t)row * row_elements + i;
+        if (f16) {
+            const __half h = __float2half_rn(v);
+            if (__hisinf(h) || __hisnan(h)) atomicOr(status, kStatusKvNonFinite);
+            static_cast<__half*>(cache_rows)[at] = h;
+        } else static_cast<float*>(cache_rows)[at] = v;
+    }
+}
+
+template <typename Kernel>
+int allow_smem(Kernel kernel, std::once_flag* once, uint32_t bytes) {
+    int device = 0;
+    cudaGetDevice(&device);
+    cudaError_t error = cudaSuccess;
+    std::call_once(once[device & 63], [&] { error = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes); });
+    GF_CUDA(error);
+    return GF_OK;
+}
+
+}  // namespace
+
+int launch_chunk_product(ChunkProduct p, bool f32, cudaStream_t stream) {
+    if (p.problems == 0 || p.problems > 3 || p.rows == 0 || !p.error_flag) return fail(GF_ERR_INVALID, "chunk product: bad launch");
+    const uint32_t tile_columns = f32 ? 64u : kDenseTile;
+    uint32_t total = 0;
+    for (uint32_t i = 0; i < p.problems; ++i) {
+        ChunkProblem& m = p.p[i];
+        if (!m.weight || !m.a.data || m.n == 0 || m.k == 0 || m.count == 0 || m.a.f32 != (f32 ? 1u : 0u)) return fail(GF_ERR_INVALID, "chunk product: bad problem");
+        m.k_blocks = (m.k + kDenseBlockK - 1u) / kDenseBlockK;
+        if ((m.a_block0 + (m.count - 1u) * m.a_block_stride + m.k_blocks) * kDenseBlockK > m.a.k_pad) return fail(GF_ERR_INVALID, "chunk product: the operand is narrower than K");
+        if (!m.group_rows && p.rows > m.a.capacity) return fail(GF_ERR_INVALID, "chunk product: more rows than the operand holds");
+        m.first_tile = total;
+        m.tiles = (m.n + tile_columns - 1u) / tile_columns;
+        total += m.tiles * m.count;
+    }
+    p.total_tiles = total;
+    if (f32) {
+        p.window = 64u;
+        chunk_product_f32_kernel<<<dim3(total, (p.rows + 63u) / 64u), 256, 0, stream>>>(p);
+    } else {
+        // The widest window of rows that still gives most SMs a tile.
+        p.window = kWindowMax;
+        while (p.window > 64u && (uint64_t)total * ((p.rows + p.window - 1u) / p.window) * 5u < (uint64_t)sm_count() * 4u) p.window /= 2u;
+        static std::once_flag once[64];
+        const int status = allow_smem(chunk_product_kernel, once, kChunkSmemBytes);
+        if (status != GF_OK) return status;
+        chunk_product_kernel<<<dim3(total, (p.rows + p.window - 1u) / p.window), kChunkThreads, kChunkSmemBytes, stream>>>(p);
+    }
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+int launch_chunk_norm(const ChunkNorm& p, cudaStream_t stream) {
+    if (!p.residual || p.rows == 0 || p.width == 0 || p.width > 48u * 1024u) return fail(GF_ERR_INVALID, "chunk norm: bad arguments");
+    static std::once_flag once[64];
+    const int status = allow_smem(chunk_norm_kernel, once, 200u * 1024u);
+    if (status != GF_OK) return status;
+    chunk_norm_kernel<<<p.rows, 256, p.width * 4u, stream>>>(p);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+int launch_chunk_route(const ChunkRoute& p, cudaStream_t stream) {
+    if (p.rows == 0 || p.experts == 0 || p.experts > kMaxExperts || p.top == 0 || p.top > p.experts) return fail(GF_ERR_INVALID, "chunk route: bad arguments");
+    if (grouped_rows(p.rows, p.top, p.experts) > p.to.capacity) return fail(GF_ERR_INVALID, "chunk route: the grouped operand is too small");
+    static std::once_flag once[64];
+    const int status = allow_smem(chunk_route_kernel, once, 32u * kMaxExperts * 4u);
+    if (status != GF_OK) return status;
+    chunk_route_kernel<<<1, 1024, 32u * p.experts * 4u, stream>>>(p);
+    chunk_group_kernel<<<p.rows * p.top, 256, 0, stream>>>(p);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+int launch_chunk_latents(const float* raw, uint32_t raw_ld, const float* gain, uint32_t rank, float eps, void* cache_rows, uint32_t row_elements,
+                         bool f16, uint32_t rows, uint32_t* status, cudaStream_t stream) {
+    chunk_latents_kernel<<<rows, 128, 0, stream>>>(raw, raw_ld, gain, rank, eps, cache_rows, row_elements, f16, status);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+}  // namespace gf

@@ -154,6 +154,7 @@ int Model::bind_q8_head_from_f16(const void* f16_dev, uint64_t k, uint64_t n) {
 }
 
 int Model::set_matrix(int kind, uint32_t layer, int dtype, const void* native_host, uint64_t k, uint64_t n, bool requantize) {
+    if (layered_) return fail(GF_ERR_STATE, "gf_model_set_matrix: this plan's tensors are bound by name (gf_model_set_tensor)");
     if (finalized_) return fail(GF_ERR_STATE, "gf_model_set_matrix: the plan is already finalized");
     if (!native_host) return fail(GF_ERR_INVALID, "gf_model_set_matrix: null payload");
     const gf_model_config& c = config_;
@@ -250,6 +251,7 @@ int Model::set_matrix(int kind, uint32_t layer, int dtype, const void* native_ho
 }
 
 int Model::set_vector(int kind, uint32_t layer, const float* host, uint32_t count) {
+    if (layered_) return fail(GF_ERR_STATE, "gf_model_set_vector: this plan's tensors are bound by name (gf_model_set_tensor)");
     if (finalized_) return fail(GF_ERR_STATE, "gf_model_set_vector: the plan is already finalized");
     if (!host) return fail(GF_ERR_INVALID, "gf_model_set_vector: null payload");
     if (kind != GF_VEC_OUTPUT_NORM && layer >= config_.layers) return fail(GF_ERR_INVALID, "gf_model_set_vector: layer out of range");
@@ -277,6 +279,12 @@ int Model::finalize() {
     if (finalized_) return fail(GF_ERR_STATE, "gf_model_finalize: already finalized");
     const gf_model_config& c = config_;
     if (c.row_capacity == 0 || c.row_capacity > GF_MAX_ROWS) return fail(GF_ERR_INVALID, "row_capacity must be 1..%d", GF_MAX_ROWS);
+    if (layered_) {
+        if (c.context == 0 || c.context > 1u << 24) return fail(GF_ERR_INVALID, "bad context");
+        if (!stream_) GF_CUDA(cudaStreamCreateWithFlags(&stream_, cudaStreamNonBlocking));
+        release_stager();
+        return finalize_layered();
+    }
     if (c.head_dim != 256u) return fail(GF_ERR_INVALID, "head_dim must be 256 (the reference's kernels share this limit)");
     if (c.context == 0 || c.heads % c.kv_heads) return fail(GF_ERR_INVALID, "bad context or head geometry");
     if (!token_embd_.data || !output_norm_) return fail(GF_ERR_STATE, "token embedding or output norm missing");
@@ -375,7 +383,6 @@ int Model::finalize() {
     GF_TRY(device_alloc(allocations_, &gate_, (size_t)R * c.ffn));
     GF_TRY(device_alloc(allocations_, &up_, (size_t)R * c.ffn));
     GF_TRY(device_alloc(allocations_, &gated_, (size_t)R * c.ffn));
-    GF_TRY(device_alloc(allocations_, &logits_, (size_t)R * c.vocab));
     // Split-K workspace: the largest any launch of the schedule needs, for every row count.
     size_t ws = 256, counters = 256;
     auto grow = [&](std::initializer_list<const PackedMatrix*> set, uint32_t prologue = kProloguePlain) {
@@ -384,7 +391,7 @@ int Model::finalize() {
             launch.count = 0;
             launch.prologue = prologue;              // the merge prologue narrows the planner's choice of K chunks
             for (const PackedMatrix* m : set) {
-                launch.matrices[launch.count++] = GemvMatrixDesc{m->dtype, m->data, logits_, m->n};
+                launch.matrices[launch.count++] = GemvMatrixDesc{m->dtype, m->data, gate_, m->n};
                 launch.k = m->k;
             }
             launch.rows = rows;
@@ -401,6 +408,15 @@ int Model::finalize() {
     GF_CUDA(cudaMemsetAsync(matmul_counters_, 0, counters, stream_));   // arrival counters start (and stay) at zero
     GF_TRY(device_alloc(allocations_, &bytes, attention_workspace_bytes(R, c.heads))); attention_ws_ = bytes;
     GF_CUDA(cudaMemsetAsync(attention_counters(attention_ws_, R, c.heads), 0, (size_t)R * c.heads * sizeof(uint32_t), stream_));
+    return finalize_shared();
+}
+
+// What every plan has: logits, candidate selection, token and state words.
+int Model::finalize_shared() {
+    const gf_model_config& c = config_;
+    const uint32_t R = c.row_capacity;
+    uint8_t* bytes = nullptr;
+    GF_TRY(device_alloc(allocations_, &logits_, (size_t)R * c.vocab));
     GF_TRY(device_alloc(allocations_, &bytes, candidates_workspace_bytes(R, c.vocab))); candidates_ws_ = bytes;
     GF_TRY(device_alloc(allocations_, &bytes, (size_t)R * gf_selection_request_bytes())); requests_dev_ = bytes;
     GF_TRY(device_alloc(allocations_, &bytes, (size_t)R * gf_candidate_result_bytes())); results_dev_ = bytes;
@@ -433,7 +449,7 @@ int Model::reset() {
     GF_CUDA(cudaMemsetAsync(pass_arrived_, 0, 16, stream_));       // a pass kernel that gave up leaves its barrier count short
     pass_arrivals_ = 0;
     if (matmul_counters_bytes_) GF_CUDA(cudaMemsetAsync(matmul_counters_, 0, matmul_counters_bytes_, stream_));
-    GF_CUDA(cudaMemsetAsync(attention_counters(attention_ws_, config_.row_capacity, config_.heads), 0,
+    if (attention_ws_) GF_CUDA(cudaMemsetAsync(attention_counters(attention_ws_, config_.row_capacity, config_.heads), 0,
                             (size_t)config_.row_capacity * config_.heads * sizeof(uint32_t), stream_));
     if (head_counters_) GF_CUDA(cudaMemsetAsync(head_counters_, 0, 2u * (config_.heads + 2u * config_.kv_heads) * sizeof(uint32_t), stream_));
     position_ = 0;
@@ -472,6 +488,7 @@ int Model::reduce_partial(float* buffer, size_t count) {
 // ---- the exchange fused into the projection launches (see WeightStreamParams::Scatter / Gather)
 
 int Model::shard_prepare(uint32_t rank, uint32_t size, void* ipc_handle_out) {
+    if (layered_) return fail(GF_ERR_STATE, "tensor-parallel shards are not offered for a layered plan");
     if (size == 0 || size > (uint32_t)kGemvMaxShards || rank >= size) return fail(GF_ERR_INVALID, "shard %u of %u", rank, size);
     if (shard_.arena) return fail(GF_ERR_STATE, "this plan already has an exchange arena");
     ShardExchange& x = shard_;
@@ -705,6 +722,7 @@ int Model::run_recorded(const RecordedPass& pass, uint32_t rows) {
 //   down  <- prologue: gelu_tanh(gate) * up
 // The next layer's QKV (or the head) applies the post-FFW norm and residual of this layer.
 int Model::encode_blocks(uint32_t rows, uint32_t flags) {
+    if (layered_) return encode_layers(rows, (flags & kForwardLogits) != 0, LayeredRows{layered_->rings_dev, 1u, 0u, state_dev_, logits_});
     const gf_model_config& c = config_;
     const float embedding_scale = sqrtf((float)c.hidden);     // f32, not bf16-rounded (model.cpp:599-605)
     const bool fused_exchange = shard_.connected;
@@ -888,6 +906,10 @@ constexpr uint32_t kTensorPrefillMinRows = 64;
 int Model::prefill(const uint32_t* tokens_host, uint32_t count) {
     if (!tokens_host || count == 0) return fail(GF_ERR_INVALID, "empty prompt");
     if (!finalized_) return fail(GF_ERR_STATE, "plan is not finalized");
+    if (layered_) {
+        const uint32_t last = count - 1u;
+        return extend(tokens_host, count, &last, 1, nullptr);
+    }
     uint32_t done = 0;
     // A shard that sums through a host hook keeps to the row passes (the hook sits behind their launches).
     if (tensor_prefill_ && (!reduce_hook_ || shard_.connected) && count - 1u >= kTensorPrefillMinRows) {
@@ -1068,6 +1090,7 @@ int Model::prefill_chunk(const uint32_t* tokens_host, uint32_t rows) {
 int Model::weight_sweep(uint32_t rows, uint32_t* out_launches, uint64_t* out_bytes) {
     if (!finalized_) return fail(GF_ERR_STATE, "plan is not finalized");
     if (rows == 0 || rows > config_.row_capacity) return fail(GF_ERR_INVALID, "bad row count");
+    if (layered_) return fail(GF_ERR_STATE, "the weight sweep is not offered for a layered plan");
     if (pass_mode_ != 0 && rows <= kPassMaxRows) {
         RecordedPass& pass = sweeps_[rows];
         if (!pass.ready) GF_TRY(record_pass(rows, 0, true, pass));
@@ -1230,15 +1253,16 @@ int Model::read_logits(uint32_t row, float* host) {
 
 int Model::read_kv(uint32_t layer, uint32_t first_position, uint32_t count, float* k_host, float* v_host) {
     if (!finalized_) return fail(GF_ERR_STATE, "plan is not finalized");
-    if (layer >= config_.layers || !k_host || !v_host || count == 0) return fail(GF_ERR_INVALID, "bad K/V readback");
+    if (layer >= config_.layers || !k_host || (!v_host && !layered_) || count == 0) return fail(GF_ERR_INVALID, "bad K/V readback");
     const LayerCache& cache = caches_[layer];
     if (first_position + count > position_ || position_ - first_position > cache.ring_rows)
         return fail(GF_ERR_INVALID, "K/V rows [%u, %u) are not all committed and still inside layer %u's ring", first_position,
                     first_position + count, layer);
-    const size_t kvw = (size_t)config_.kv_heads * config_.head_dim, element = config_.kv_f16 ? 2 : 4;
+    const size_t element = config_.kv_f16 ? 2 : 4, kvw = cache_row_bytes(layer) / element;
+    const int tensors = layered_ ? 1 : 2;
     std::vector<uint8_t> raw[2];
     const void* rings[2] = {cache.ring_k, cache.ring_v};
-    for (int which = 0; which < 2; ++which) {
+    for (int which = 0; which < tensors; ++which) {
         raw[which].resize((size_t)count * kvw * element);
         uint32_t done = 0;
         while (done < count) {                       // at most two contiguous runs of ring slots
@@ -1251,6 +1275,14 @@ int Model::read_kv(uint32_t layer, uint32_t first_position, uint32_t count, floa
         }
     }
     GF_TRY(synchronize());
+    if (layered_) {          // rows are stored with their rank rounded up
+        const uint32_t rank = layered_->spec().layers[layer].mixer.rank;
+        for (uint32_t r = 0; r < count; ++r)
+            for (uint32_t i = 0; i < rank; ++i)
+                k_host[(size_t)r * rank + i] = config_.kv_f16 ? __half2float(reinterpret_cast<const __half*>(raw[0].data())[r * kvw + i])
+                                                              : reinterpret_cast<const float*>(raw[0].data())[r * kvw + i];
+        return GF_OK;
+    }
     float* outs[2] = {k_host, v_host};
     for (int which = 0; which < 2; ++which) {
         if (!config_.kv_f16) { std::memcpy(outs[which], raw[which].data(), raw[which].size()); continue; }
@@ -1283,11 +1315,10 @@ size_t Model::kv_bytes_per_pass(uint32_t rows) const {
     // once -- the rows of a pass look at the same cache (the reference counts it the same way,
     // docs/archive/DEVELOPMENT_HISTORY.md: 8 global x context + 40 local x window rows of 8 KB).
     if (rows == 0) return 0;
-    const size_t row_bytes = (size_t)config_.kv_heads * config_.head_dim * (config_.kv_f16 ? 2 : 4) * 2;
     size_t total = 0;
-    for (const LayerCache& cache : caches_) {
-        const uint32_t seen = cache.window ? std::min(position_, cache.window) : position_;
-        total += (size_t)seen * row_bytes;
+    for (uint32_t l = 0; l < config_.layers; ++l) {
+        const uint32_t window = caches_[l].window, seen = window ? std::min(position_, window) : position_;
+        total += (size_t)seen * cache_row_bytes(l) * (layered_ ? 1u : 2u);
     }
     return total;
 }
@@ -1308,6 +1339,30 @@ int gf_model_create(const gf_model_config* config, gf_model** out_model) {
     *out_model = new gf_model(*config);
     return GF_OK;
 }
+int gf_model_create_described(const char* config_json, uint32_t context, uint32_t row_capacity, int precision, gf_model** out_model) {
+    if (!config_json || !out_model) return fail(GF_ERR_INVALID, "gf_model_create_described: null argument");
+    if (precision != GF_PRECISION_SERVING && precision != GF_PRECISION_F32) return fail(GF_ERR_INVALID, "gf_model_create_described: unknown precision %d", precision);
+    ArchitectureDescription description;
+    GF_TRY(describe_architecture(config_json, std::strlen(config_json), description));
+    if (!description.layered) {
+        if (precision != GF_PRECISION_SERVING) return fail(GF_ERR_INVALID, "%s runs in its quantised form only", description.name.c_str());
+        description.config.context = context;
+        description.config.row_capacity = row_capacity;
+        return gf_model_create(&description.config, out_model);
+    }
+    int count = 0;
+    if (cudaGetDeviceCount(&count) != cudaSuccess || count == 0)
+        return fail(GF_ERR_UNAVAILABLE, "no CUDA device is available; this backend has no CPU path");
+    *out_model = new gf_model(description, context, row_capacity, precision == GF_PRECISION_F32);
+    return GF_OK;
+}
+int gf_model_set_tensor(gf_model* m, const char* name, int dtype, const void* host, const uint64_t* dims, uint32_t rank) {
+    return m ? m->impl.set_tensor(name, dtype, host, dims, rank) : fail(GF_ERR_INVALID, "null model");
+}
+int gf_model_extend(gf_model* m, const uint32_t* tokens_host, uint32_t count, const uint32_t* want, uint32_t want_count, float* logits_host) {
+    return m ? m->impl.extend(tokens_host, count, want, want_count, logits_host) : fail(GF_ERR_INVALID, "null model");
+}
+uint32_t gf_model_vocab(const gf_model* m) { return m ? m->impl.config().vocab : 0u; }
 int gf_model_destroy(gf_model* model) { delete model; return GF_OK; }
 int gf_model_set_matrix(gf_model* m, int kind, uint32_t layer, int dtype, const void* native_host, uint64_t k, uint64_t n) {
     return m ? m->impl.set_matrix(kind, layer, dtype, native_host, k, n) : fail(GF_ERR_INVALID, "null model");
@@ -1396,6 +1451,7 @@ int gf_model_use_tensor_prefill(gf_model* m, int enable) {
 uint32_t gf_model_prefill_logits_row(const gf_model* m) { return m ? m->impl.prefill_logits_row() : 0; }
 int gf_model_use_pass_kernel(gf_model* m, int mode) {
     if (!m || mode < 0 || mode > 2) return fail(GF_ERR_INVALID, "gf_model_use_pass_kernel: mode must be 0, 1 or 2");
+    if (mode != 0 && m->impl.layered()) return fail(GF_ERR_STATE, "the decode pass kernel is not offered for a layered plan");
     m->impl.set_pass_mode(mode);
     return GF_OK;
 }

@@ -1,13 +1,17 @@
 // Resident Gemma model plan: packed weights, KV rings + private rows, scratch, and the block
 // schedule.  One class serves the 12B target, the Gemma 2 target and the 270M drafter; they
-// differ only in configuration (weight types, KV precision, RoPE, softcaps, QK norm).
+// differ only in configuration (weight types, KV precision, RoPE, softcaps, QK norm).  A plan built from
+// a layered description (architecture.hpp) has the same passes, publication, streams and selection over
+// schedules of its own (layered.cu).
 #pragma once
 
 #include "common.cuh"
+#include "layered.cuh"
 #include "ops.cuh"
 #include "pass.cuh"
 #include "prefill.cuh"
 
+#include <functional>
 #include <memory>
 #include <string>
 #include <vector>
@@ -68,12 +72,14 @@ struct StreamSet {
 class Model {
 public:
     explicit Model(const gf_model_config& config);
+    Model(const ArchitectureDescription& description, uint32_t context, uint32_t row_capacity, bool f32);
     ~Model();
     Model(const Model&) = delete;
     Model& operator=(const Model&) = delete;
 
     int set_matrix(int kind, uint32_t layer, int dtype, const void* native_host, uint64_t k, uint64_t n, bool requantize = false);
     int set_vector(int kind, uint32_t layer, const float* host, uint32_t count);
+    int set_tensor(const char* name, int dtype, const void* host, const uint64_t* dims, uint32_t rank);     // layered plans
     int finalize();
 
     int reset();
@@ -86,6 +92,9 @@ public:
     int synchronize();
     int status_word(uint32_t* out);
     int prefill(const uint32_t* tokens_host, uint32_t count);
+    // Ingests a portion of a prompt at the committed position; the logits of the wanted places (rising) go to
+    // logits_host [want_count][vocab].
+    int extend(const uint32_t* tokens_host, uint32_t count, const uint32_t* want, uint32_t want_count, float* logits_host);
     int truncate(uint32_t position);
     int weight_sweep(uint32_t rows, uint32_t* out_launches, uint64_t* out_bytes);
 
@@ -115,6 +124,10 @@ public:
     // Independent streams over this plan's weights (streams.cu).
     int streams_create(uint32_t count, StreamSet** out);
     int streams_prefill(StreamSet& set, uint32_t stream, const uint32_t* tokens_host, uint32_t count);
+    int streams_extend(StreamSet& set, uint32_t stream, const uint32_t* tokens_host, uint32_t count, const uint32_t* want, uint32_t want_count,
+                       float* logits_host);
+    int streams_release(StreamSet& set, uint32_t stream);
+    int streams_ingest(StreamSet& set, uint32_t stream, uint32_t count, const std::function<int()>& ingest, bool last);
     int streams_decode(StreamSet& set, const uint32_t* tokens_host);
     int streams_set_mode(StreamSet& set, int mode);
     int streams_select(StreamSet& set, const void* requests_host);
@@ -142,6 +155,11 @@ public:
         return GF_OK;
     }
     uint32_t token_vocab() const { return token_table_vocab_ ? token_table_vocab_ : config_.vocab; }
+    bool layered() const { return layered_ != nullptr; }
+    LayeredPlan* layered_plan() { return layered_.get(); }
+    size_t cache_row_bytes(uint32_t layer) const {      // of one of the cache's tensors (K, V, or the latents)
+        return layered_ ? layered_->cache_row_bytes(layer) : (size_t)config_.kv_heads * config_.head_dim * (config_.kv_f16 ? 2u : 4u);
+    }
     bool sharded() const { return reduce_hook_ != nullptr || shard_.connected; }
     // The exchange fused into the projection launches (no host hook, no separate reduction launch): every
     // shard owns an arena its peers write into over NVLink.  shard_prepare allocates it (and exports it for
@@ -215,6 +233,12 @@ private:
     int encode_stream_group(StreamSet& set, uint32_t first, uint32_t rows);
     int encode_stream_batch(StreamSet& set);
     int encode_blocks(uint32_t rows, uint32_t flags);
+    int finalize_shared();
+    int finalize_layered();
+    int encode_layers(uint32_t rows, bool logits, const LayeredRows& where);
+    int ensure_chunk_arena();
+    int chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits);
+    std::unique_ptr<LayeredPlan> layered_;
     int run_gemv(struct GemvLaunch& launch, uint32_t rows);
     int emit_embedding(uint32_t rows, float scale);
     int emit_attention(const AttentionParams& params);
@@ -313,4 +337,5 @@ private:
 struct gf_model {
     gf::Model impl;
     explicit gf_model(const gf_model_config& c) : impl(c) {}
+    gf_model(const gf::ArchitectureDescription& d, uint32_t context, uint32_t rows, bool f32) : impl(d, context, rows, f32) {}
 };

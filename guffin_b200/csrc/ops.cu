@@ -179,7 +179,7 @@ __global__ void __launch_bounds__(128) stream_publish_kernel(const StreamPublish
     uint8_t* ring_v = static_cast<uint8_t*>(const_cast<void*>(R.ring_v));
     for (uint32_t b = threadIdx.x * 16u; b < L.row_bytes; b += blockDim.x * 16u) {
         *reinterpret_cast<uint4*>(ring_k + dst + b) = *reinterpret_cast<const uint4*>(L.private_k + src + b);
-        *reinterpret_cast<uint4*>(ring_v + dst + b) = *reinterpret_cast<const uint4*>(L.private_v + src + b);
+        if (L.private_v) *reinterpret_cast<uint4*>(ring_v + dst + b) = *reinterpret_cast<const uint4*>(L.private_v + src + b);
     }
 }
 
@@ -228,7 +228,7 @@ __global__ void __launch_bounds__(128) kv_publish_kernel(const KvPublishLayer* _
     const size_t dst = (size_t)((base + row) & L.ring_mask) * L.row_bytes, src = (size_t)row * L.row_bytes;
     for (uint32_t b = threadIdx.x * 16u; b < L.row_bytes; b += blockDim.x * 16u) {
         *reinterpret_cast<uint4*>(L.ring_k + dst + b) = *reinterpret_cast<const uint4*>(L.private_k + src + b);
-        *reinterpret_cast<uint4*>(L.ring_v + dst + b) = *reinterpret_cast<const uint4*>(L.private_v + src + b);
+        if (L.private_v) *reinterpret_cast<uint4*>(L.ring_v + dst + b) = *reinterpret_cast<const uint4*>(L.private_v + src + b);
     }
 }
 

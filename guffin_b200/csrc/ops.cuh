@@ -66,7 +66,7 @@ inline uint32_t* attention_counters(void* workspace, uint32_t rows, uint32_t hea
     return reinterpret_cast<uint32_t*>(static_cast<float*>(workspace) + (size_t)rows * heads * kMaxAttentionPartitions * (256u + 2u));
 }
 
-struct KvPublishLayer {          // one per layer, device resident
+struct KvPublishLayer {          // one per layer, device resident; a cache of one row per token has no v
     uint8_t *ring_k, *ring_v;
     const uint8_t *private_k, *private_v;
     uint32_t ring_mask, row_bytes;

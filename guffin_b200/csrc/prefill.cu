@@ -1,6 +1,7 @@
 // Prefill GEMM on tcgen05 / TMEM and the elementwise steps around it (see prefill.cuh).
 #include "prefill.cuh"
 #include "ops.cuh"
+#include "tcgen05.cuh"
 
 #include <cuda_bf16.h>
 
@@ -26,54 +27,8 @@ constexpr uint32_t kBarCount = 2u * kWeightBufs + 3u * kStages + 1u;    // weigh
 constexpr uint32_t kPrefillSmemBytes = kOffBars + kBarCount * 8u + 16u;
 static_assert(kPrefillSmemBytes <= 227u * 1024u - 1024u, "the GEMM's stages do not fit in one SM's shared memory");
 
-// ---- tcgen05 wrappers (sm_100a PTX) ----
-__device__ __forceinline__ void tmem_alloc(uint32_t* slot_smem, uint32_t columns) {
-    asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(slot_smem)), "r"(columns) : "memory");
-    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
-}
-__device__ __forceinline__ void tmem_dealloc(uint32_t address, uint32_t columns) {
-    asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(address), "r"(columns) : "memory");
-}
-__device__ __forceinline__ void tc_fence_before_sync() { asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory"); }
-__device__ __forceinline__ void tc_fence_after_sync() { asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory"); }
-// Makes this thread's shared-memory stores visible to the tensor core's (asynchronous-proxy) reads.
-__device__ __forceinline__ void fence_async_smem() { asm volatile("fence.proxy.async.shared::cta;" ::: "memory"); }
-
-// Shared-memory operand descriptor, K-major, no swizzle: start address, 128 bytes between the two
-// core matrices of a 16-element K step, 1024 bytes between groups of eight rows, descriptor version 1.
-__device__ __forceinline__ uint64_t operand_descriptor(uint32_t smem_address) {
-    return (uint64_t)((smem_address >> 4) & 0x3fffu) | ((uint64_t)(128u >> 4) << 16) | ((uint64_t)(1024u >> 4) << 32) | (1ull << 46);
-}
-// Instruction descriptor: f32 accumulator, bf16 x bf16, both operands K-major, M = 128, N = kPrefillTile.
-constexpr uint32_t kInstruction = (1u << 4) | (1u << 7) | (1u << 10) | ((kPrefillTile >> 3) << 17) | ((kPrefillHalf >> 4) << 24);
+constexpr uint32_t kInstruction = mma_instruction(kPrefillHalf, kPrefillTile);
 constexpr uint32_t kTmemColumns = 2u * kPrefillTile;                    // one accumulator of kPrefillTile columns per half of the rows
-
-__device__ __forceinline__ void mma_bf16(uint32_t tmem_d, uint64_t a_desc, uint64_t b_desc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\t"
-        "setp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-        ::"r"(tmem_d), "l"(a_desc), "l"(b_desc), "r"(kInstruction), "r"(accumulate) : "memory");
-}
-// The barrier receives one arrival once every tensor-core operation issued so far by this thread has finished.
-__device__ __forceinline__ void mma_commit(uint64_t* bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(smem_u32(bar)) : "memory");
-}
-// 32 lanes x 32 consecutive columns of 32-bit accumulators: thread l of the warp gets lane (base + l).
-__device__ __forceinline__ void tmem_load_32(uint32_t address, float (&v)[32]) {
-    uint32_t r[32];
-    asm volatile(
-        "tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-        "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-        : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]),
-          "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]),
-          "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]),
-          "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-        : "r"(address) : "memory");
-    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-#pragma unroll
-    for (int i = 0; i < 32; ++i) v[i] = __uint_as_float(r[i]);
-}
 
 __device__ __forceinline__ uint32_t bf16_pair(float lo, float hi) {
     const __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
@@ -188,14 +143,6 @@ __device__ __forceinline__ void dequant_q80(const uint8_t* row, uint32_t sub, ui
     }
 }
 
-// Bounded wait that also gives up as soon as another warp of the CTA has.
-__device__ __forceinline__ bool wait_or_abort(uint64_t* bar, uint32_t parity, const volatile uint32_t* abort) {
-    for (uint32_t spin = 0; spin < kMbarWaitLimit; ++spin) {
-        if (mbar_try_wait(bar, parity)) return true;
-        if ((spin & 63u) == 63u && *abort != 0u) return false;
-    }
-    return false;
-}
 __device__ __forceinline__ void mbar_arrive(uint64_t* bar) {
     asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(bar)) : "memory");
 }
@@ -315,7 +262,7 @@ __global__ void __launch_bounds__(kPrefillThreads, 1) prefill_gemm_kernel(const 
 #pragma unroll
                     for (uint32_t kk = 0; kk < kPrefillBlockK / 16u; ++kk)
                         mma_bf16(tmem + h * kPrefillTile, operand_descriptor(a_address + h * kAHalfBytes + kk * 256u),
-                                 operand_descriptor(b_address + kk * 256u), (step | kk) != 0u ? 1u : 0u);
+                                 operand_descriptor(b_address + kk * 256u), kInstruction, (step | kk) != 0u ? 1u : 0u);
                 mma_commit(&stage_free[stage]);
             }
             if (ok) mma_commit(done_bar);

@@ -51,23 +51,24 @@ int Model::streams_create(uint32_t count, StreamSet** out) {
     set->ring_k.assign(count, std::vector<void*>(c.layers));
     set->ring_v.assign(count, std::vector<void*>(c.layers));
     set->positions_host.assign(count, 0u);
-    const size_t element = c.kv_f16 ? 2 : 4, kvw = (size_t)c.kv_heads * c.head_dim;
     std::vector<StreamRings> rings((size_t)c.layers * count);
     std::vector<StreamPublishLayer> layers(c.layers);
     for (uint32_t l = 0; l < c.layers; ++l) {
-        const size_t bytes = (size_t)caches_[l].ring_rows * kvw * element;
+        const size_t bytes = (size_t)caches_[l].ring_rows * cache_row_bytes(l);
         for (uint32_t s = 0; s < count; ++s) {
             uint8_t *k = nullptr, *v = nullptr;
             GF_TRY(stream_alloc(*set, &k, bytes));
-            GF_TRY(stream_alloc(*set, &v, bytes));
             GF_CUDA(cudaMemsetAsync(k, 0, bytes, stream_));
-            GF_CUDA(cudaMemsetAsync(v, 0, bytes, stream_));
+            if (!layered_) {
+                GF_TRY(stream_alloc(*set, &v, bytes));
+                GF_CUDA(cudaMemsetAsync(v, 0, bytes, stream_));
+            }
             set->ring_k[s][l] = k;
             set->ring_v[s][l] = v;
             rings[(size_t)l * count + s] = StreamRings{k, v};
         }
         layers[l] = StreamPublishLayer{static_cast<const uint8_t*>(caches_[l].private_k), static_cast<const uint8_t*>(caches_[l].private_v),
-                                       caches_[l].ring_rows - 1u, (uint32_t)(kvw * element)};
+                                       caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
     }
     GF_TRY(stream_alloc(*set, &set->rings_dev, rings.size()));
     GF_TRY(stream_alloc(*set, &set->publish_layers_dev, layers.size()));
@@ -90,43 +91,74 @@ int Model::streams_create(uint32_t count, StreamSet** out) {
 // rings, and recorded graphs and pass tables have the old pointers baked in.
 int Model::bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>& ring_v, uint32_t position) {
     const gf_model_config& c = config_;
-    const size_t element = c.kv_f16 ? 2 : 4, kvw = (size_t)c.kv_heads * c.head_dim;
     std::vector<KvPublishLayer> table(c.layers), prefill_table(c.layers);
+    const bool chunks = layered_ && layered_->chunk.ready;
     for (uint32_t l = 0; l < c.layers; ++l) {
         caches_[l].ring_k = ring_k[l];
         caches_[l].ring_v = ring_v[l];
         table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), static_cast<uint8_t*>(ring_v[l]), static_cast<const uint8_t*>(caches_[l].private_k),
-                                  static_cast<const uint8_t*>(caches_[l].private_v), caches_[l].ring_rows - 1u, (uint32_t)(kvw * element)};
+                                  static_cast<const uint8_t*>(caches_[l].private_v), caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
+        if (chunks)
+            prefill_table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), nullptr, static_cast<const uint8_t*>(layered_->chunk.private_rows[l]), nullptr,
+                                              caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
         if (prefill_.ready)
             prefill_table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), static_cast<uint8_t*>(ring_v[l]), static_cast<const uint8_t*>(prefill_.private_k[l]),
-                                              static_cast<const uint8_t*>(prefill_.private_v[l]), caches_[l].ring_rows - 1u, (uint32_t)(kvw * element)};
+                                              static_cast<const uint8_t*>(prefill_.private_v[l]), caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
     }
     GF_CUDA(cudaMemcpyAsync(publish_layers_, table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice, stream_));
     if (prefill_.ready)
         GF_CUDA(cudaMemcpyAsync(prefill_.publish_layers, prefill_table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice, stream_));
+    if (chunks) GF_CUDA(cudaMemcpyAsync(layered_->chunk.publish_layers, prefill_table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice, stream_));
+    std::vector<StreamRings> rings(c.layers);
+    if (layered_) {
+        for (uint32_t l = 0; l < c.layers; ++l) rings[l] = StreamRings{ring_k[l], nullptr};
+        GF_CUDA(cudaMemcpyAsync(layered_->rings_dev, rings.data(), sizeof(StreamRings) * c.layers, cudaMemcpyHostToDevice, stream_));
+    }
     GF_CUDA(cudaMemcpyAsync(state_dev_, &position, sizeof(uint32_t), cudaMemcpyHostToDevice, stream_));
     GF_CUDA(cudaStreamSynchronize(stream_));           // the tables above are pageable
+    position_ = position;
+    if (layered_) return GF_OK;                        // its passes find the rings through the device table
     for (auto& per_rows : graphs_)
         for (cudaGraphExec_t& exec : per_rows)
             if (exec) { cudaGraphExecDestroy(exec); exec = nullptr; }
     invalidate_passes();
-    position_ = position;
     return GF_OK;
 }
 
 int Model::streams_prefill(StreamSet& set, uint32_t stream, const uint32_t* tokens_host, uint32_t count) {
+    return streams_ingest(set, stream, count, [&] { return prefill(tokens_host, count); }, true);
+}
+
+int Model::streams_extend(StreamSet& set, uint32_t stream, const uint32_t* tokens_host, uint32_t count, const uint32_t* want, uint32_t want_count,
+                          float* logits_host) {
+    return streams_ingest(set, stream, count, [&] { return extend(tokens_host, count, want, want_count, logits_host); },
+                          want_count && want && want[want_count - 1u] + 1u == count);
+}
+
+// The slot's next conversation starts at position 0; what the last one left in the rings is never visible to it.
+int Model::streams_release(StreamSet& set, uint32_t stream) {
+    if (stream >= set.count) return fail(GF_ERR_INVALID, "stream %u of %u", stream, set.count);
+    set.positions_host[stream] = 0;
+    GF_CUDA(cudaMemcpyAsync(set.positions_dev + stream, &set.positions_host[stream], sizeof(uint32_t), cudaMemcpyHostToDevice, stream_));
+    GF_CUDA(cudaStreamSynchronize(stream_));
+    return GF_OK;
+}
+
+// Runs `ingest` with the stream's rings in place of the plan's own; `last` = it leaves the last token's logits.
+int Model::streams_ingest(StreamSet& set, uint32_t stream, uint32_t count, const std::function<int()>& ingest, bool last) {
     if (stream >= set.count) return fail(GF_ERR_INVALID, "stream %u of %u", stream, set.count);
     std::vector<void*> home_k(config_.layers), home_v(config_.layers);
     for (uint32_t l = 0; l < config_.layers; ++l) { home_k[l] = caches_[l].ring_k; home_v[l] = caches_[l].ring_v; }
     const uint32_t home_position = position_;
     // The tensor-core prompt path allocates its arena on first use, before the rings are exchanged, so that
     // its publication table is rebuilt with the stream's rings like the plan's own.
-    if (tensor_prefill_ && count > 64u) GF_TRY(ensure_prefill_arena());
+    if (layered_) GF_TRY(ensure_chunk_arena());
+    else if (tensor_prefill_ && count > 64u) GF_TRY(ensure_prefill_arena());
     GF_TRY(bind_rings(set.ring_k[stream], set.ring_v[stream], set.positions_host[stream]));
-    int status = prefill(tokens_host, count);
+    int status = ingest();
     if (status == GF_OK) {
         // The last prompt token's logits become the stream's row of the batch logits.
-        status = check_cuda(cudaMemcpyAsync(set.logits + (size_t)stream * config_.vocab, logits_ + (size_t)prefill_logits_row_ * config_.vocab,
+        if (last) status = check_cuda(cudaMemcpyAsync(set.logits + (size_t)stream * config_.vocab, logits_ + (size_t)prefill_logits_row_ * config_.vocab,
                                             (size_t)config_.vocab * sizeof(float), cudaMemcpyDeviceToDevice, stream_), "logits");
         set.positions_host[stream] = position_;
         if (status == GF_OK) status = check_cuda(cudaMemcpyAsync(set.positions_dev + stream, &set.positions_host[stream], sizeof(uint32_t),
@@ -140,6 +172,12 @@ int Model::streams_prefill(StreamSet& set, uint32_t stream, const uint32_t* toke
 // One pass over `rows` <= row_capacity streams starting at `first`: their token ids are in tokens_dev_.
 int Model::encode_stream_group(StreamSet& set, uint32_t first, uint32_t rows) {
     const gf_model_config& c = config_;
+    if (layered_) {
+        GF_TRY(encode_layers(rows, true, LayeredRows{set.rings_dev + first, set.count, 1u, set.positions_dev + first, set.logits + (size_t)first * c.vocab}));
+        GF_TRY(launch_stream_publish(set.publish_layers_dev, c.layers, set.rings_dev + first, set.count, set.positions_dev + first, rows, stream_));
+        launches_ += 2;
+        return GF_OK;
+    }
     GF_TRY(emit_embedding(rows, sqrtf((float)c.hidden)));
     float* x = residual_;
     float* x2 = post_attention_;
@@ -214,6 +252,7 @@ int Model::encode_stream_group(StreamSet& set, uint32_t first, uint32_t rows) {
 int Model::streams_set_mode(StreamSet& set, int mode) {
     if (mode != 0 && mode != 1) return fail(GF_ERR_INVALID, "stream decode mode %d (0: exact row passes, 1: one tensor-core pass)", mode);
     if (mode == 1) {
+        if (layered_) return fail(GF_ERR_STATE, "a layered plan's stream steps are row passes");
         if (set.count > kPrefillRows) return fail(GF_ERR_INVALID, "a tensor-core step holds at most %u streams", kPrefillRows);
         const gf_model_config& c = config_;
         if ((has_head_ ? head_ : token_embd_).n % kPrefillTile) return fail(GF_ERR_INVALID, "the tensor-core head needs a vocabulary that is a multiple of %u", kPrefillTile);
@@ -405,12 +444,11 @@ int Model::streams_read_logits(StreamSet& set, uint32_t stream, float* host) {
 
 size_t Model::streams_kv_bytes(const StreamSet& set) const {
     // K and V bytes one decode step reads: every stream's committed rows inside every layer's window.
-    const size_t element = config_.kv_f16 ? 2 : 4, row = (size_t)config_.kv_heads * config_.head_dim * element * 2u;
     size_t total = 0;
     for (uint32_t s = 0; s < set.count; ++s)
         for (uint32_t l = 0; l < config_.layers; ++l) {
             const uint32_t window = caches_[l].window, p = set.positions_host[s];
-            total += (size_t)(window ? std::min(window, p) : p) * row;
+            total += (size_t)(window ? std::min(window, p) : p) * cache_row_bytes(l) * (layered_ ? 1u : 2u);
         }
     return total;
 }
@@ -441,6 +479,12 @@ int gf_streams_destroy(gf_streams* s) {
 }
 int gf_streams_prefill(gf_streams* s, uint32_t stream, const uint32_t* tokens_host, uint32_t count) {
     return s ? s->model->impl.streams_prefill(*s->set, stream, tokens_host, count) : fail(GF_ERR_INVALID, "null streams");
+}
+int gf_streams_extend(gf_streams* s, uint32_t stream, const uint32_t* tokens_host, uint32_t count, const uint32_t* want, uint32_t want_count, float* logits_host) {
+    return s ? s->model->impl.streams_extend(*s->set, stream, tokens_host, count, want, want_count, logits_host) : fail(GF_ERR_INVALID, "null streams");
+}
+int gf_streams_release(gf_streams* s, uint32_t stream) {
+    return s ? s->model->impl.streams_release(*s->set, stream) : fail(GF_ERR_INVALID, "null streams");
 }
 int gf_streams_decode(gf_streams* s, const uint32_t* tokens_host) {
     return s ? s->model->impl.streams_decode(*s->set, tokens_host) : fail(GF_ERR_INVALID, "null streams");

@@ -259,6 +259,40 @@ class H1:
             pass
 
 
+class Batch:
+    """Several conversations decoded together: a stream and a sampler for each (gf_streams_*, gf_sampler_*)."""
+
+    def __init__(self, model: Model, prompts, options):
+        from .model import Streams
+        self.model, self.streams = model, Streams(model, len(prompts))
+        self.options = [options] * len(prompts) if isinstance(options, SamplerOptions) else list(options)
+        self.samplers = [Sampler(o) for o in self.options]
+        for i, prompt in enumerate(prompts):
+            self.streams.prefill(i, prompt)
+            self.samplers[i].observe(prompt)
+        self.history = [[int(t) for t in prompt] for prompt in prompts]
+
+    def _next(self) -> np.ndarray:
+        from .model import selection_request
+        requests = []
+        for o, seen in zip(self.options, self.history):
+            window = list(dict.fromkeys(seen[-o.repetition_window:])) if o.repetition_penalty != 1.0 else []
+            requests.append(selection_request((1 if o.temperature == 0.0 else o.top_k) + len(window), window))
+        tokens = [sampler.sample(row.pairs()) for sampler, row in zip(self.samplers, self.streams.select(requests))]
+        for i, token in enumerate(tokens):
+            self.samplers[i].observe([token])
+            self.history[i].append(token)
+        return np.array(tokens, np.uint32)
+
+    def generate(self, max_tokens: int) -> np.ndarray:
+        """[conversations, max_tokens] tokens."""
+        out = [self._next()]
+        while len(out) < max_tokens:
+            self.streams.decode(out[-1])
+            out.append(self._next())
+        return np.stack(out, axis=1)
+
+
 def verification_schedule(horizon: int, conditional: bool) -> list:
     """(drafts, rows) of every verification pass of a cycle with `horizon` drafts."""
     drafts, rows, tiles = (u32 * 4)(), (u32 * 4)(), u32()

@@ -67,6 +67,15 @@ lib.register({
     "gf_model_shard_set_wait_limit": (i32, [vp, u32]),
     "gf_model_shard_global_selection": (i32, [vp, i32]),
     "gf_add": (i32, [vp, vp, vp, u64, vp]),
+    "gf_architectures": (C.c_char_p, []),
+    "gf_model_create_described": (i32, [C.c_char_p, u32, u32, i32, C.POINTER(vp)]),
+    "gf_model_set_tensor": (i32, [vp, C.c_char_p, i32, vp, C.POINTER(u64), u32]),
+    "gf_model_load_safetensors": (i32, [vp, C.c_char_p, C.POINTER(u32)]),
+    "gf_model_open": (i32, [C.c_char_p, u32, u32, i32, C.POINTER(vp)]),
+    "gf_model_vocab": (u32, [vp]),
+    "gf_model_extend": (i32, [vp, vp, u32, vp, u32, vp]),
+    "gf_streams_extend": (i32, [vp, u32, vp, u32, vp, u32, vp]),
+    "gf_streams_release": (i32, [vp, u32]),
     "gf_model_finalize": (i32, [vp]),
     "gf_model_reset": (i32, [vp]),
     "gf_model_position": (i32, [vp, C.POINTER(u32)]),
@@ -109,6 +118,22 @@ MATRIX_KINDS = {"token_embd": 0, "output": 1, "attn_q": 2, "attn_k": 3, "attn_v"
 VECTOR_KINDS = {"output_norm": 0, "attn_norm": 1, "post_attention_norm": 2, "ffn_norm": 3, "post_ffw_norm": 4,
                 "attn_q_norm": 5, "attn_k_norm": 6}
 FORWARD_LOGITS, FORWARD_DEVICE_TOKENS = 1, 2
+PRECISIONS = {"bfloat16": 0, "float32": 1}
+
+
+def architectures() -> list:
+    """Names config.json's "architecture" may take."""
+    return load().gf_architectures().decode().split()
+
+
+def bf16_bits(values) -> np.ndarray:
+    """f32 values rounded to bfloat16 (nearest even), as uint16 bits."""
+    bits = np.ascontiguousarray(values, np.float32).view(np.uint32)
+    return ((bits + 0x7fff + ((bits >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def bf16_values(bits) -> np.ndarray:
+    return (np.ascontiguousarray(bits, np.uint16).astype(np.uint32) << 16).view(np.float32)
 
 
 def make_config(config: dict, context: int, row_capacity: int = 2) -> ModelConfig:
@@ -168,6 +193,58 @@ class Model:
                 data = np.ascontiguousarray(value, np.float32)
                 check(self.L.gf_model_set_vector(self.handle, VECTOR_KINDS[short], layer, data.ctypes.data, data.size))
         check(self.L.gf_model_finalize(self.handle))
+
+    @classmethod
+    def _adopt(cls, handle, context: int, row_capacity: int, config: dict) -> "Model":
+        model = cls.__new__(cls)
+        model.L, model.handle, model.config = load(), handle, dict(config)
+        model.cfg = ModelConfig()
+        model.cfg.vocab, model.cfg.context, model.cfg.row_capacity = model.L.gf_model_vocab(handle), context, row_capacity
+        model.cfg.kv_heads, model.cfg.head_dim = config.get("kv_heads", 0), config.get("head_dim", 0)
+        model.cfg.layers = len(config["layers"]) if isinstance(config.get("layers"), list) else config.get("layers", 0)
+        return model
+
+    @classmethod
+    def open(cls, folder, context: int, row_capacity: int = 2, precision: str = "bfloat16") -> "Model":
+        """The model of a folder: config.json beside model.safetensors or model.gguf."""
+        import json
+        import os
+        handle = vp()
+        check(load().gf_model_open(os.fsencode(folder), context, row_capacity, PRECISIONS[precision], C.byref(handle)))
+        with open(os.path.join(folder, "config.json")) as f:
+            return cls._adopt(handle.value, context, row_capacity, json.load(f))
+
+    @classmethod
+    def described(cls, config: dict, weights, context: int, row_capacity: int = 2, precision: str = "bfloat16") -> "Model":
+        """A layered model from its configuration and (name, array) pairs: uint16 arrays are bfloat16 bits, others
+        are taken as f32 (vectors) or rounded to bfloat16 (matrices)."""
+        import json
+        L = load()
+        handle = vp()
+        check(L.gf_model_create_described(json.dumps(config).encode(), context, row_capacity, PRECISIONS[precision], C.byref(handle)))
+        model = cls._adopt(handle.value, context, row_capacity, config)
+        for name, value in (weights.items() if hasattr(weights, "items") else weights):
+            value = np.asarray(value)
+            if value.dtype != np.uint16:
+                value = bf16_bits(value) if value.ndim == 2 else np.ascontiguousarray(value, np.float32)
+            value = np.ascontiguousarray(value)
+            dims = (u64 * value.ndim)(*value.shape)
+            check(L.gf_model_set_tensor(model.handle, name.encode(), 30 if value.dtype == np.uint16 else 0, value.ctypes.data, dims, value.ndim))
+        check(L.gf_model_finalize(model.handle))
+        return model
+
+    def extend(self, tokens, want=()) -> np.ndarray:
+        """Ingests a portion; logits [len(want), vocab] of the wanted places inside it."""
+        tokens, want = np.ascontiguousarray(tokens, np.uint32), np.ascontiguousarray(np.array(want, np.uint32))
+        out = np.empty((want.size, self.cfg.vocab), np.float32)
+        check(self.L.gf_model_extend(self.handle, tokens.ctypes.data, tokens.size, want.ctypes.data, want.size, out.ctypes.data))
+        return out
+
+    def read_latents(self, layer: int, first: int, count: int) -> np.ndarray:
+        """Committed cache rows of a latent-attention layer, [count, rank]."""
+        out = np.empty((count, self.config["layers"][layer]["mixer"]["kv_rank"]), np.float32)
+        check(self.L.gf_model_read_kv(self.handle, layer, first, count, out.ctypes.data, None))
+        return out
 
     @property
     def position(self) -> int:
@@ -281,6 +358,17 @@ class Streams:
     def prefill(self, stream: int, tokens) -> None:
         tokens = np.ascontiguousarray(tokens, np.uint32)
         check(self.L.gf_streams_prefill(self.handle, stream, tokens.ctypes.data, tokens.size))
+
+    def extend(self, stream: int, tokens, want=()) -> np.ndarray:
+        """Model.extend on one stream's cache."""
+        tokens, want = np.ascontiguousarray(tokens, np.uint32), np.ascontiguousarray(np.array(want, np.uint32))
+        out = np.empty((want.size, self.model.cfg.vocab), np.float32)
+        check(self.L.gf_streams_extend(self.handle, stream, tokens.ctypes.data, tokens.size, want.ctypes.data, want.size, out.ctypes.data))
+        return out
+
+    def release(self, stream: int) -> None:
+        """Gives the stream's slot back; its next conversation starts at position 0."""
+        check(self.L.gf_streams_release(self.handle, stream))
 
     def set_mode(self, mode: int) -> None:
         """0: exact row passes in groups; 1: one tensor-core pass over all streams (bf16 operands)."""

@@ -37,7 +37,7 @@ enum {
 };
 
 /* GGUF tensor type ids (include/local_gguf_engine/tensor/dtype.hpp:9-15). */
-enum { GF_F32 = 0, GF_F16 = 1, GF_Q8_0 = 8, GF_Q4_K = 12, GF_Q6_K = 14 };
+enum { GF_F32 = 0, GF_F16 = 1, GF_Q8_0 = 8, GF_Q4_K = 12, GF_Q6_K = 14, GF_BF16 = 30 };
 
 GF_API const char* gf_last_error(void);
 GF_API const char* gf_version(void);
@@ -334,6 +334,28 @@ GF_API int gf_model_shard_global_selection(gf_model* model, int enable);
  * The geometry still comes from gf_model_config; *out_bound_tensors (optional) counts the
  * tensors taken.  Call gf_model_finalize afterwards. */
 GF_API int gf_model_load_gguf(gf_model* model, const char* path, uint32_t* out_bound_tensors);
+/* ---- models described by a configuration file.  No counterpart in the reference, which serves the Gemma families
+ * only.  `config_json` is the text of a config.json whose "architecture" names an entry of the registry
+ * (gf_architectures, one name per line): "Zasevik" (a layered decoder: every layer names its mixer and its
+ * feed-forward with their sizes and constants; bf16 tensors bound by name), or "Gemma2" / "Gemma3" (the fields of
+ * gf_model_config under their own names; tensors bound by kind).  A layered plan has the same passes, publication,
+ * streams, candidate selection and generation engine as any other plan; tensor-parallel shards, the decode pass
+ * kernel, tensor-core stream steps and the weight sweep are not offered for it.
+ * precision: GF_PRECISION_SERVING = matrix products of prompt chunks in bf16 with 32-bit accumulation and a binary16
+ * cache, everything else (norms, softmax, routing, the residual stream, row passes) in 32-bit;
+ * GF_PRECISION_F32 = everything in 32-bit (layered models only).
+ * gf_model_set_tensor binds one tensor (GF_BF16 matrices [out, in]; vectors GF_BF16 or GF_F32).
+ * gf_model_load_safetensors binds every tensor of a safetensors file.  gf_model_open does it all for a folder that
+ * holds config.json beside model.safetensors or model.gguf, and finalizes. ---- */
+enum { GF_PRECISION_SERVING = 0, GF_PRECISION_F32 = 1 };
+GF_API const char* gf_architectures(void);
+GF_API int gf_model_create_described(const char* config_json, uint32_t context, uint32_t row_capacity, int precision,
+                                     gf_model** out_model);
+GF_API int gf_model_set_tensor(gf_model* model, const char* name, int dtype, const void* host, const uint64_t* dims,
+                               uint32_t rank);
+GF_API int gf_model_load_safetensors(gf_model* model, const char* path, uint32_t* out_bound_tensors);
+GF_API int gf_model_open(const char* folder, uint32_t context, uint32_t row_capacity, int precision, gf_model** out_model);
+GF_API uint32_t gf_model_vocab(const gf_model* model);
 /* Checks every tensor is bound and allocates KV rings, private rows and scratch
  * (allocate_kv_cache, gemma2_metal_plan.cpp:514-537). */
 GF_API int gf_model_finalize(gf_model* model);
@@ -353,6 +375,12 @@ GF_API int gf_model_publish(gf_model* model, uint32_t rows);
 /* Chunked prompt ingestion through the row path (run_gemma3_resident_prefill semantics,
  * gemma_target_runtime.cpp:420); logits are produced for the last token only. */
 GF_API int gf_model_prefill(gf_model* model, const uint32_t* tokens_host, uint32_t count);
+/* One portion of a prompt at the committed position, cut wherever the caller likes: publishes `count` tokens and
+ * writes the logits of the wanted places (indices into the portion, rising) to logits_host [want_count][vocab], which
+ * may be NULL.  A layered plan takes long portions as chunks on the tensor cores and short ones as row passes; other
+ * plans as exact row passes.  Synchronises, and reports what gf_model_status would, when logits_host is given. */
+GF_API int gf_model_extend(gf_model* model, const uint32_t* tokens_host, uint32_t count, const uint32_t* want,
+                           uint32_t want_count, float* logits_host);
 GF_API int gf_model_truncate(gf_model* model, uint32_t position);
 /* gf_model_prefill ingests prompts of 65 tokens or more in chunks of up to 256 rows, every projection of
  * a chunk as one bf16 tensor-core GEMM (run_gemma3_resident_prefill's 128-row chunks,
@@ -369,6 +397,7 @@ GF_API uint32_t gf_model_prefill_logits_row(const gf_model* model);
 GF_API int gf_model_select(gf_model* model, const void* requests_host, uint32_t rows);
 GF_API int gf_model_read_candidates(gf_model* model, void* results_host, uint32_t rows);
 GF_API int gf_model_read_logits(gf_model* model, uint32_t row, float* logits_host);
+/* A layered plan's cache holds one latent per position: `count` x rank values go to k_host, v_host is not written. */
 /* Committed K and V rows of one layer, positions [first_position, first_position + count), widened
  * to f32: `count` x kv_heads*head_dim values each.  Synchronises.  The rows must still be inside
  * the layer's ring (copy_tensor_from_backend on the plan's cache buffers, backend_buffer.hpp:47-68;
@@ -423,6 +452,11 @@ GF_API int gf_streams_create(gf_model* model, uint32_t count, gf_streams** out_s
 GF_API int gf_streams_destroy(gf_streams* streams);
 GF_API uint32_t gf_streams_count(const gf_streams* streams);
 GF_API int gf_streams_prefill(gf_streams* streams, uint32_t stream, const uint32_t* tokens_host, uint32_t count);
+/* gf_model_extend on one stream's cache; gf_streams_release gives a stream's slot back: its next conversation starts
+ * at position 0. */
+GF_API int gf_streams_extend(gf_streams* streams, uint32_t stream, const uint32_t* tokens_host, uint32_t count,
+                             const uint32_t* want, uint32_t want_count, float* logits_host);
+GF_API int gf_streams_release(gf_streams* streams, uint32_t stream);
 GF_API int gf_streams_decode(gf_streams* streams, const uint32_t* tokens_host /* one id per stream */);
 /* How a step computes its projections.  0 (default): the exact row passes described above.  1: ONE pass over
  * all streams of the set (at most 256) whose projections are the prompt path's bf16 tensor-core GEMMs

@@ -5,6 +5,7 @@ weights of those geometries.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
     python bench.py --workload streams [--streams S] [--prefix P] [--steps K] [--gpus N]
+    python bench.py --workload zasevik [--sizes dense-2048,...] [--steps K]      the layered design beside the Gemma 3 plan of equal size
     torchrun ... bench.py --gpus N --workload tp [--h1] [--exchange peer|nccl]     one stream, the 12B target sharded over N GPUs
     python bench.py --horizon H [--conditional]                                   chains of H drafts per cycle
     python bench.py --case matmul <dtype 8|12|14> <K> <N> <rows> [launches]
@@ -445,6 +446,123 @@ def run_streams(args) -> dict:
                      "kernel": "one decode step: weight_stream_kernel per group of streams + stream attention over every cache",
                      "step_bytes": step_bytes, "kv_bytes": kv_bytes, "weight_passes": groups},
         "clocks": clocks.summary(),
+    }
+
+
+# Sizes of the zasevik workload (layers of a real model's widths, few of them) and the Gemma 3 geometry of equal size.
+ZASEVIK_SIZES = {
+    "dense-2048": dict(width=2048, heads=16, mlps=[("dense", 8192)], gemma=(2048, 5376, 8, 4)),
+    "experts-2048": dict(width=2048, heads=16, mlps=[("dense", 8192), ("experts", 1024, 64, 6, 2048)], gemma=(2048, 5376, 8, 4)),
+    "dense-3840": dict(width=3840, heads=32, mlps=[("dense", 15360)], gemma=(3840, 10240, 16, 8)),
+}
+ZASEVIK_LAYERS, ZASEVIK_VOCAB = 8, 32768
+
+
+def zasevik_size(name: str) -> dict:
+    from guffin_b200 import synthetic as syn
+    size = ZASEVIK_SIZES[name]
+    mlps = [syn.dense_mlp(m[1]) if m[0] == "dense" else syn.expert_mlp(m[1], m[2], m[3], 7.0, m[4], 7.0) for m in size["mlps"]]
+    return syn.zasevik_config(size["width"], ZASEVIK_LAYERS, size["heads"], 128, 128, 512, ZASEVIK_VOCAB, mlps)
+
+
+def equal_gemma(name: str) -> dict:
+    from guffin_b200 import synthetic as syn
+    hidden, ffn, heads, kv_heads = ZASEVIK_SIZES[name]["gemma"]
+    return dict(syn.model_config("gemma3-12b"), hidden=hidden, ffn=ffn, heads=heads, kv_heads=kv_heads, layers=ZASEVIK_LAYERS, vocab=ZASEVIK_VOCAB,
+                sliding_window=0, sliding_pattern=0)
+
+
+def time_plan(lib, plan, prompt, steps: int, warmup: int) -> dict:
+    """Device times of one plan: prompt ingestion (median of three after a warm-up) and one-row passes behind it."""
+    start, end = lib.Event(), lib.Event()
+
+    def timed(run):
+        plan.synchronize()
+        start.record(plan.stream)
+        run()
+        end.record(plan.stream)
+        end.synchronize()
+        return start.elapsed_ms(end)
+
+    def ingest():
+        plan.reset()
+        plan.prefill(prompt)
+    ingest()
+    ingest()
+    prefill_ms = sorted(timed(ingest) for _ in range(3))[1]
+
+    def decode(n):
+        for _ in range(n):
+            plan.forward_device_tokens(1)
+            plan.publish(1)
+    decode(warmup)
+    launches = plan.kernel_launches()
+    decode_ms = timed(lambda: decode(steps)) / steps
+    return {"prefill_ms": prefill_ms, "prefill_tok_s": len(prompt) / prefill_ms * 1e3, "decode_ms": decode_ms, "decode_tok_s": 1e3 / decode_ms,
+            "launches_per_token": (plan.kernel_launches() - launches) / steps, "kv_bytes": plan.kv_bytes_per_pass(1), "status_word": plan.status()}
+
+
+def run_zasevik(args) -> dict:
+    """Prefill and decode throughput of the layered design at a few sizes, beside the Gemma 3 plan of equal size."""
+    from guffin_b200 import engine as ge, lib, model as gm, synthetic as syn
+    L = lib.load()
+    lib.check(L.gf_set_device(0))
+    peak, peak_kind = load_peaks()
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else open(os.devnull) as f:
+        text = f.read()
+    tensor_peak = float(json.loads(text)["bf16_tflops"]) if text else 1590.0
+    prefix, steps, warmup = args.prefix if args.prefix != 8192 else 2048, args.steps, max(args.warmup, 3)
+    prompt = np.random.default_rng(SEEDS["prompt"]).integers(0, ZASEVIK_VOCAB, prefix).astype(np.uint32)
+    context = prefix + 2 * (warmup + steps) + 16
+    sizes, launches = {}, 0
+    clocks = ClockSampler(0)
+    for name in args.sizes.split(","):
+        config, gemma = zasevik_size(name), equal_gemma(name)
+        plan = gm.Model.described(config, syn.iter_zasevik_weights(config, SEEDS["target"]), context, 2)
+        with clocks:
+            ours = time_plan(lib, plan, prompt, steps, warmup)
+        launches += int(ours["launches_per_token"] * steps)
+        active = syn.zasevik_active_parameters(config)
+        ours["weight_bytes_per_token"] = 2 * active
+        ours["decode_gbs"] = (2 * active + ours["kv_bytes"]) / ours["decode_ms"] / 1e6
+        ours["decode_frac"] = ours["decode_gbs"] / peak
+        head = config["vocab"] * config["width"]
+        keys = prefix * (prefix + 1) / 2
+        attention = sum(4.0 * l["mixer"]["heads"] * l["mixer"]["kv_rank"] * keys for l in config["layers"])
+        ours["prefill_tflops"] = (2.0 * (active - head) * prefix + attention) / ours["prefill_ms"] / 1e9
+        ours["prefill_frac"] = ours["prefill_tflops"] / tensor_peak
+        # End to end through the generation engine: prompt in host memory, tokens back on the host.
+        engine = ge.H1(plan, None, ge.H1Options(ge.sampler_options(0.0), 0, 0, 0.0, 0, 0))
+        engine.prefill(prompt)
+        engine.generate(warmup)
+        t0 = time.perf_counter()
+        engine.generate(steps)
+        ours["e2e_decode_tok_s"] = steps / (time.perf_counter() - t0)
+        engine.close()
+        plan.close()
+        plan = gm.Model(gemma, syn.iter_model_weights("gemma3-like", SEEDS["target"], gemma), context, 2)
+        with clocks:
+            theirs = time_plan(lib, plan, prompt, steps, warmup)
+        theirs["weight_bytes_per_token"] = plan.weight_bytes(True)
+        theirs["decode_gbs"] = (plan.weight_bytes(True) + theirs["kv_bytes"]) / theirs["decode_ms"] / 1e6
+        theirs["decode_frac"] = theirs["decode_gbs"] / peak
+        matrices = sum(k * n for k, n in syn.matrix_shapes(gemma).values()) * ZASEVIK_LAYERS
+        theirs["prefill_tflops"] = (2.0 * matrices * prefix + 4.0 * gemma["heads"] * 256 * keys * ZASEVIK_LAYERS) / theirs["prefill_ms"] / 1e9
+        theirs["prefill_frac"] = theirs["prefill_tflops"] / tensor_peak
+        plan.close()
+        sizes[name] = {"zasevik": ours, "gemma3": theirs}
+    first = sizes[args.sizes.split(",")[0]]["zasevik"]
+    return {
+        "metric": "Zasevik decode tok/s, one stream", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
+        "ms_per_step": first["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None, "dtype": "bf16 weights, f32 activations, binary16 latents",
+        "data": "synthetic",
+        "config": {"workload": f"{ZASEVIK_LAYERS} layers of each size, {prefix}-token prompt, one-row passes behind it; beside it the Gemma 3 plan (Q4_K_M) of equal width "
+                               "and parameter count, all layers global", "sizes": list(sizes), "layers": ZASEVIK_LAYERS, "vocab": ZASEVIK_VOCAB,
+                   "l2_policy": "a pass reads its weights once; sizes whose weights exceed L2 (all of them) defeat it"},
+        "e2e": {"value": first["e2e_decode_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 + 264, "d2h_bytes_per_step": 3080},
+        "gpu_launches": launches,
+        "roofline": {"bound": "hbm", "achieved": first["decode_gbs"], "peak": peak, "unit": "GB/s", "frac": first["decode_frac"], "peak_source": f"of {peak_kind}"},
+        "sizes": sizes, "clocks": clocks.summary(),
     }
 
 
@@ -891,8 +1009,10 @@ def main():
                         help="0: one kernel per operator (CUDA graph, the default); 1: persistent decode pass kernel; "
                              "2: pass kernel with attention launched separately")
     parser.add_argument("--case", nargs="+", default=None, help="run one single-kernel case instead of the benchmark")
-    parser.add_argument("--workload", choices=("h1", "streams", "tp"), default="h1",
-                        help="h1: the headline (configs[3]); streams: configs[4]; tp: one 12B stream sharded over the GPUs")
+    parser.add_argument("--workload", choices=("h1", "streams", "tp", "zasevik"), default="h1",
+                        help="h1: the headline (configs[3]); streams: configs[4]; tp: one 12B stream sharded over the GPUs; "
+                             "zasevik: prefill and decode of the layered design beside the Gemma 3 plan of equal size")
+    parser.add_argument("--sizes", default=",".join(ZASEVIK_SIZES), help="zasevik workload: sizes to run, with commas between them")
     parser.add_argument("--horizon", type=int, default=1, help="drafts per cycle of the h1 workload (1 = the headline; 2..7 = chains)")
     parser.add_argument("--conditional", action="store_true",
                         help="h1 workload with --horizon > 2: verify the chain as a cascade of passes (the reference's conditional tiles)")
@@ -911,6 +1031,10 @@ def main():
         args.steps = 64 if args.steps is None else args.steps
         args.warmup = 3 if args.warmup is None else args.warmup
         result = run_streams(args)
+    elif args.workload == "zasevik" and args.impl == "ours":
+        args.steps = 64 if args.steps is None else args.steps
+        args.warmup = 5 if args.warmup is None else args.warmup
+        result = run_zasevik(args)
     elif args.workload == "tp" and args.impl == "ours":
         args.steps = 100 if args.steps is None else args.steps
         args.warmup = 5 if args.warmup is None else args.warmup

@@ -60,6 +60,7 @@ constexpr uint32_t kRowThreads = 256, kRowWarps = kRowThreads / 32u;
 constexpr uint32_t kRowAhead = 8;                    // 512-byte loads a warp keeps in flight
 constexpr uint32_t kRowSmemLimit = 200u * 1024u;     // activations of a launch
 constexpr uint32_t kRowMaxRows = 8;
+constexpr uint32_t kNormQuads = 4;                   // 16-byte pieces of a row a thread holds: rows of up to 4096 values
 
 __device__ __forceinline__ uint4 load_weight(const uint8_t* p) {
     uint4 v;
@@ -86,6 +87,9 @@ __device__ __forceinline__ void block_sums(float (&v)[R], float* scratch) {
     }
     __syncthreads();
 }
+
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float dot4(float4 a, float4 b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
 
 __device__ __forceinline__ float norm_factor(float sum, uint32_t width, float eps) { return 1.0f / sqrtf(sum / (float)width + eps); }
 
@@ -119,8 +123,8 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
     __shared__ float route_score;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, batch = blockIdx.y;
     if (batch >= p.batches) {                                      // the cache rows of this pass
-        pdl_launch_dependents();
         pdl_wait();
+        pdl_launch_dependents();
         if (blockIdx.x < p.rows) store_latent(p, blockIdx.x, scratch);
         return;
     }
@@ -154,8 +158,23 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
     uint32_t set = set_base + blockIdx.x;
     if (set >= set_end) return;
     if (!routed) { locate(set); prefetch(); }
-    pdl_launch_dependents();
+    const bool quads = p.vector_rows != 0u;                        // widths and strides are whole 16-byte pieces
+    // The residual rows and the gains were written at least two launches back: read ahead of the wait.
+    float4 early_residual[kNormQuads], early_gain0[kNormQuads], early_gain1[kNormQuads];
+    const bool early = R == 1 && quads && (p.input == kRowNorm || p.input == kRowAddNorm) && p.width <= kNormQuads * kRowThreads * 4u;
+    if (early)
+#pragma unroll
+        for (uint32_t j = 0; j < kNormQuads; ++j) {
+            const uint32_t i = (j * kRowThreads + tid) * 4u;
+            if (i >= p.width) continue;
+            early_gain1[j] = *reinterpret_cast<const float4*>(p.gain1 + i);
+            if (p.input == kRowAddNorm) {
+                early_residual[j] = *reinterpret_cast<const float4*>(p.residual + i);
+                early_gain0[j] = *reinterpret_cast<const float4*>(p.gain0 + i);
+            }
+        }
     pdl_wait();
+    pdl_launch_dependents();
 
     // ---- the activations
     if (routed) {
@@ -176,7 +195,51 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
         prefetch();
     }
     const uint32_t k_used = p.m[which].k, k_pad = p.k_pad;
-    if (p.input == kRowNorm || p.input == kRowAddNorm) {
+    if (early) {
+        // One row held in registers: both norms without a pass through shared memory in between.
+        const bool writer = blockIdx.x == 0 && batch == 0;
+        float4 v[kNormQuads];
+        float sum[1] = {0.0f};
+#pragma unroll
+        for (uint32_t j = 0; j < kNormQuads; ++j) {
+            const uint32_t i = (j * kRowThreads + tid) * 4u;
+            v[j] = i < p.width ? *reinterpret_cast<const float4*>(p.in + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+#pragma unroll 4
+        for (uint32_t part = 1; part < p.parts; ++part)
+#pragma unroll
+            for (uint32_t j = 0; j < kNormQuads; ++j) {
+                const uint32_t i = (j * kRowThreads + tid) * 4u;
+                if (i < p.width) v[j] = add4(v[j], *reinterpret_cast<const float4*>(p.in + part * p.part_stride + i));
+            }
+#pragma unroll
+        for (uint32_t j = 0; j < kNormQuads; ++j) sum[0] += dot4(v[j], v[j]);
+        block_sums<1>(sum, scratch);
+        float inv = norm_factor(sum[0], p.width, p.eps);
+        if (p.input == kRowAddNorm) {
+            sum[0] = 0.0f;
+#pragma unroll
+            for (uint32_t j = 0; j < kNormQuads; ++j) {
+                const uint32_t i = (j * kRowThreads + tid) * 4u;
+                if (i >= p.width) continue;
+                const float4 r = early_residual[j], g = early_gain0[j];
+                v[j] = make_float4(r.x + v[j].x * inv * g.x, r.y + v[j].y * inv * g.y, r.z + v[j].z * inv * g.z, r.w + v[j].w * inv * g.w);
+                if (writer && p.residual_out) *reinterpret_cast<float4*>(p.residual_out + i) = v[j];
+                sum[0] += dot4(v[j], v[j]);
+            }
+            block_sums<1>(sum, scratch);
+            inv = norm_factor(sum[0], p.width, p.eps);
+        }
+#pragma unroll
+        for (uint32_t j = 0; j < kNormQuads; ++j) {
+            const uint32_t i = (j * kRowThreads + tid) * 4u;
+            if (i >= p.width) continue;
+            const float4 g = early_gain1[j], n = make_float4(v[j].x * inv * g.x, v[j].y * inv * g.y, v[j].z * inv * g.z, v[j].w * inv * g.w);
+            *reinterpret_cast<float4*>(act + i) = n;
+            if (writer && p.normed_out) *reinterpret_cast<float4*>(p.normed_out + i) = n;
+        }
+        for (uint32_t i = p.width + tid; i < k_pad; i += kRowThreads) act[i] = 0.0f;
+    } else if (p.input == kRowNorm || p.input == kRowAddNorm) {
         const bool writer = blockIdx.x == 0 && batch == 0;
         float sum[R];
 #pragma unroll
@@ -225,25 +288,22 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
         }
     } else if (p.input == kRowLatent) {
         for (int r = 0; r < R; ++r) {
-            const uint32_t m = r * p.heads + batch;
-            const float* ml = p.latent_ml + (size_t)m * p.attention_parts * 2u;
-            // (maximum, sum) of every partition, and of the sink, which has no value.
-            const float sink = p.sink ? p.sink[batch] : -INFINITY;
-            float top = sink;
-            for (uint32_t part = 0; part < p.attention_parts; ++part) top = fmaxf(top, ml[part * 2u]);
-            float total = p.sink ? expf(sink - top) : 0.0f;
-            for (uint32_t part = 0; part < p.attention_parts; ++part) total += ml[part * 2u + 1u] > 0.0f ? ml[part * 2u + 1u] * expf(ml[part * 2u] - top) : 0.0f;
-            for (uint32_t part = tid; part < p.attention_parts; part += kRowThreads)
-                route_scratch[part] = ml[part * 2u + 1u] > 0.0f ? expf(ml[part * 2u] - top) / total : 0.0f;
+            const uint32_t m = r * p.heads + batch, parts = p.attention_parts;
+            if (warp == 0) merge_factors(p.latent_ml + (size_t)m * parts * 2u, parts, p.sink ? p.sink[batch] : -INFINITY, route_scratch);
             __syncthreads();
-            for (uint32_t i = tid; i < k_pad; i += kRowThreads) {
-                float v = 0.0f;
-                if (i < k_used)
-                    for (uint32_t part = 0; part < p.attention_parts; ++part) {
+            const float* rows_in = p.in + (size_t)m * parts * p.latent_ld;
+            for (uint32_t i = tid * 2u; i < k_pad; i += kRowThreads * 2u) {
+                float2 v = make_float2(0.0f, 0.0f);
+                if (i < p.latent_ld) {
+#pragma unroll 8
+                    for (uint32_t part = 0; part < parts; ++part) {
+                        const float2 o = *reinterpret_cast<const float2*>(rows_in + (size_t)part * p.latent_ld + i);
                         const float f = route_scratch[part];
-                        if (f != 0.0f) v = fmaf(p.in[((size_t)m * p.attention_parts + part) * p.latent_ld + i], f, v);
+                        v.x = fmaf(o.x, f, v.x); v.y = fmaf(o.y, f, v.y);
                     }
-                act[r * k_pad + i] = v;
+                }
+                act[r * k_pad + i] = v.x;
+                act[r * k_pad + i + 1u] = v.y;
             }
             __syncthreads();
         }
@@ -253,7 +313,13 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
             if (p.input == kRowRouted) x = p.in + (size_t)(batch / p.top) * p.in_ld;
             else if (p.input == kRowExperts) x = behind ? p.in2 + (size_t)(batch - p.rows * p.top) * p.in2_ld : p.in + (size_t)batch * p.in_ld;
             else x = p.in + (size_t)(p.in_rows ? p.in_rows[r] : (uint32_t)r) * p.in_ld + (size_t)batch * p.in_batch;
-            for (uint32_t i = tid; i < k_pad; i += kRowThreads) act[r * k_pad + i] = i < k_used ? x[i] : 0.0f;
+            if (quads) {
+#pragma unroll 4
+                for (uint32_t i = tid * 4u; i < k_pad; i += kRowThreads * 4u)
+                    *reinterpret_cast<float4*>(act + r * k_pad + i) = i < k_used ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            } else {
+                for (uint32_t i = tid; i < k_pad; i += kRowThreads) act[r * k_pad + i] = i < k_used ? x[i] : 0.0f;
+            }
         }
     }
     __syncthreads();
@@ -261,35 +327,42 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
     // ---- the products
     const float* lane_act = act + (lane >> 3) * 8u;
     for (; set < set_end; ) {
-        float acc[R];
+        float acc[R][2];
 #pragma unroll
-        for (int r = 0; r < R; ++r) acc[r] = 0.0f;
-        for (uint32_t first = unit_begin; first < unit_end; first += kRowAhead) {
+        for (int r = 0; r < R; ++r) { acc[r][0] = 0.0f; acc[r][1] = 0.0f; }
+        auto consume = [&](const uint4& v, uint32_t unit) {
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const float4 x = *reinterpret_cast<const float4*>(lane_act + r * k_pad + unit * 32u);
+                const float4 y = *reinterpret_cast<const float4*>(lane_act + r * k_pad + unit * 32u + 4u);
+                float a = acc[r][0], b = acc[r][1];
+                a = fmaf(low_half(v.x), x.x, a); b = fmaf(high_half(v.x), x.y, b);
+                a = fmaf(low_half(v.y), x.z, a); b = fmaf(high_half(v.y), x.w, b);
+                a = fmaf(low_half(v.z), y.x, a); b = fmaf(high_half(v.z), y.y, b);
+                a = fmaf(low_half(v.w), y.z, a); b = fmaf(high_half(v.w), y.w, b);
+                acc[r][0] = a; acc[r][1] = b;
+            }
+        };
+        uint32_t unit = unit_begin;
+        for (; unit + 2u * kRowAhead <= unit_end; unit += kRowAhead)      // whole rounds with a whole round behind them
 #pragma unroll
             for (uint32_t i = 0; i < kRowAhead; ++i) {
-                const uint32_t unit = first + i;
-                if (unit < unit_end) {
-                    const uint4 v = w[i];
-                    if (unit + kRowAhead < unit_end) w[i] = fetch(unit + kRowAhead);
-#pragma unroll
-                    for (int r = 0; r < R; ++r) {
-                        const float4 x = *reinterpret_cast<const float4*>(lane_act + r * k_pad + unit * 32u);
-                        const float4 y = *reinterpret_cast<const float4*>(lane_act + r * k_pad + unit * 32u + 4u);
-                        float a = acc[r];
-                        a = fmaf(low_half(v.x), x.x, a); a = fmaf(high_half(v.x), x.y, a);
-                        a = fmaf(low_half(v.y), x.z, a); a = fmaf(high_half(v.y), x.w, a);
-                        a = fmaf(low_half(v.z), y.x, a); a = fmaf(high_half(v.z), y.y, a);
-                        a = fmaf(low_half(v.w), y.z, a); a = fmaf(high_half(v.w), y.w, a);
-                        acc[r] = a;
-                    }
-                }
+                consume(w[i], unit + i);
+                w[i] = fetch(unit + kRowAhead + i);
             }
-        }
+        for (; unit < unit_end; unit += kRowAhead)
+#pragma unroll
+            for (uint32_t i = 0; i < kRowAhead; ++i)
+                if (unit + i < unit_end) {
+                    consume(w[i], unit + i);
+                    if (unit + kRowAhead + i < unit_end) w[i] = fetch(unit + kRowAhead + i);
+                }
 #pragma unroll
         for (int r = 0; r < R; ++r) {
-            acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 8);
-            acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], 16);
-            if (lane < 8u) partial[warp][r][lane] = acc[r];
+            float v = acc[r][0] + acc[r][1];
+            v += __shfl_xor_sync(0xffffffffu, v, 8);
+            v += __shfl_xor_sync(0xffffffffu, v, 16);
+            if (lane < 8u) partial[warp][r][lane] = v;
         }
         const RowMatrix& m = p.m[which];
         const uint32_t here = set, split = kRowWarps / m.groups_per_cta;
@@ -374,6 +447,8 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
         while (per < kRowWarps && (uint64_t)(groups + per - 1u) / per * batches > wanted) per *= 2u;
         // A warp's slice of K should not fall below two of its 512-byte loads.
         while (per < kRowWarps && (m.k + 31u) / 32u < 2u * (kRowWarps / per)) per *= 2u;
+        // Every CTA of a head merges all of its attention partitions: few CTAs per head.
+        if (p.input == kRowLatent) while (per < kRowWarps && (groups + per - 1u) / per > 4u) per *= 2u;
         m.groups_per_cta = per;
         m.first_set = sets;
         m.sets = (groups + per - 1u) / per;
@@ -384,6 +459,11 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
     p.sets = sets;
     p.k_pad = (k_max + 31u) / 32u * 32u;
     if ((p.input == kRowNorm || p.input == kRowAddNorm) && k_max != p.width) return fail(GF_ERR_INVALID, "row product: a normalised input has the matrices' K");
+    auto whole = [](const void* pointer) { return (reinterpret_cast<uintptr_t>(pointer) & 15u) == 0u; };
+    p.vector_rows = p.in_ld % 4u == 0u && p.in_batch % 4u == 0u && p.in2_ld % 4u == 0u && p.part_stride % 4u == 0u && whole(p.in) && whole(p.in2);
+    if (p.input == kRowNorm || p.input == kRowAddNorm)
+        p.vector_rows = p.vector_rows && p.width % 4u == 0u && whole(p.residual) && whole(p.residual_out) && whole(p.gain0) && whole(p.gain1) && whole(p.normed_out);
+    for (uint32_t i = 0; i < p.count; ++i) p.vector_rows = p.vector_rows && p.m[i].k % 4u == 0u;
     const uint32_t row_bytes = p.k_pad * 4u;
     if (row_bytes > kRowSmemLimit) return fail(GF_ERR_INVALID, "row product: K = %u is too wide", k_max);
     const uint32_t per_launch = single ? 1u : std::max(1u, std::min<uint32_t>(kRowMaxRows, kRowSmemLimit / row_bytes));

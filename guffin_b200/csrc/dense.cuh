@@ -111,7 +111,7 @@ struct RowProduct {
     uint32_t latent_row_elements = 0, latent_f16 = 0;
     uint32_t* status = nullptr;
     // filled by the launcher
-    uint32_t k_pad = 0, sets = 0;
+    uint32_t k_pad = 0, sets = 0, vector_rows = 0;
 };
 // Any number of rows; launches as many kernels as the rows need (`launches` is increased by their number).
 int launch_row_product(RowProduct product, cudaStream_t stream, bool pdl, uint32_t& launches);
@@ -161,10 +161,12 @@ struct ChunkProblem {
 struct ChunkProduct {
     ChunkProblem p[3];
     uint32_t problems = 1, rows = 0;
-    uint32_t window = 0, total_tiles = 0;          // filled by the launcher
+    uint32_t window = 0, total_tiles = 0, stage_budget = 0;      // filled by the launcher
     int* error_flag = nullptr;
 };
 int launch_chunk_product(ChunkProduct product, bool f32, cudaStream_t stream);
+// f32 rows [rows][k] into an operand.
+int launch_chunk_operand(const float* x, uint32_t rows, uint32_t k, const Operand& result, cudaStream_t stream);
 
 // Rows of a chunk between products: residual + rmsnorm(y) * gain0 -> residual (in place), rmsnorm(that) * gain1 ->
 // operand and / or f32 rows.  y null: only the second norm.  y is [row][width], or with `slots` set the sum over a
@@ -191,6 +193,7 @@ struct ChunkRoute {
     Operand from, to;                   // the normalised rows, and the grouped operand
 };
 inline uint32_t grouped_rows(uint32_t rows, uint32_t top, uint32_t experts) { return (rows * top + 8u * experts + 31u) / 16u * 16u; }
+int launch_route(const ChunkRoute& route, cudaStream_t stream);      // the choices alone
 int launch_chunk_route(const ChunkRoute& route, cudaStream_t stream);
 
 // Cache rows of a chunk: rmsnorm(raw) * gain.
@@ -215,6 +218,22 @@ __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-
 __device__ __forceinline__ float clamped_gate(float gate, float up, float limit) {
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return g * sigmoid(1.702f * g) * (u + 1.0f);
+}
+// One warp turns the (maximum, sum) pairs of a query's key partitions, and its sink, into the factors of the merge.
+__device__ __forceinline__ void merge_factors(const float* ml, uint32_t parts, float sink, float* factors) {
+    const uint32_t lane = threadIdx.x & 31u;
+    float top = sink;
+    for (uint32_t part = lane; part < parts; part += 32u) top = fmaxf(top, ml[part * 2u]);
+#pragma unroll
+    for (int offset = 16; offset > 0; offset >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, offset));
+    float total = 0.0f;
+    for (uint32_t part = lane; part < parts; part += 32u) {
+        const float f = ml[part * 2u + 1u] > 0.0f ? expf(ml[part * 2u] - top) : 0.0f;      // an empty partition has no maximum
+        factors[part] = f;
+        total += f * ml[part * 2u + 1u];
+    }
+    total = warp_sum(total) + (sink == -INFINITY ? 0.0f : expf(sink - top));
+    for (uint32_t part = lane; part < parts; part += 32u) factors[part] /= total;
 }
 // One warp picks the `slots` best experts of a row of router logits in order; `scores` is a warp's scratch of
 // `experts` floats in shared memory.  pick(slot, expert, score) is called on every lane.

@@ -37,20 +37,19 @@ __device__ __forceinline__ void chunk_store_gate(const ChunkProblem& p, uint32_t
 // ------------------------------------------------------------------ bf16 products on tcgen05
 
 constexpr uint32_t kWindowMax = 256;                                   // token rows of a tile: the product's N
-constexpr uint32_t kStages = 4;
-constexpr uint32_t kStageBytes = kDenseTileBytes + kWindowMax * 128u;  // 128 weight columns, then up to 256 token rows, x 64 K
+constexpr uint32_t kMaxStages = 8;                                     // a stage: 128 weight columns, then the window's token rows, x 64 K
 constexpr uint32_t kEpilogueWarps = 8;
 constexpr uint32_t kChunkThreads = (kEpilogueWarps + 2u) * 32u;        // the copying and the issuing warp behind them
-constexpr uint32_t kChunkSmemBytes = kStages * kStageBytes + (2u * kStages + 1u) * 8u + 16u;
+constexpr uint32_t kSmemAlone = 208u * 1024u, kSmemPaired = 104u * 1024u;      // stages of a CTA that has its SM alone, or shares it with another
 
 // The tensor core's A operand is a tile of 128 weight columns and its B operand a window of up to 256 token rows, so
 // the product's N follows the rows there are (an expert may have few) and accumulator lanes are output columns.
 __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const __grid_constant__ ChunkProduct p) {
     extern __shared__ __align__(1024) uint8_t smem[];
     __shared__ uint32_t tmem_slot, abort_flag;
-    uint64_t* full = reinterpret_cast<uint64_t*>(smem + kStages * kStageBytes);      // [kStages] copies landed (bytes)
-    uint64_t* free_bar = full + kStages;                                             // [kStages] the stage's products have finished
-    uint64_t* done_bar = free_bar + kStages;
+    __shared__ __align__(8) uint64_t full[kMaxStages];                  // copies landed (bytes)
+    __shared__ __align__(8) uint64_t free_bar[kMaxStages];              // the stage's products have finished
+    __shared__ __align__(8) uint64_t done_bar[1];
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
     const volatile uint32_t* abort = &abort_flag;
 
@@ -65,11 +64,12 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
     const uint8_t* weight = m.weight + index * m.weight_stride + (size_t)tile * m.k_blocks * kDenseTileBytes;
     const uint8_t* rows_at = static_cast<const uint8_t*>(m.a.data) + (size_t)(m.a_block0 + index * m.a_block_stride) * m.a.capacity * 128u + (size_t)row0 * 128u;
 
+    const uint32_t stage_bytes = kDenseTileBytes + n_rows * 128u, stages = min(kMaxStages, p.stage_budget / stage_bytes);
     uint32_t tmem_columns = 32u;
     while (tmem_columns < n_rows) tmem_columns *= 2u;
     if (tid == 0) {
         abort_flag = 0u;
-        for (uint32_t i = 0; i < kStages; ++i) { mbar_init(&full[i], 1); mbar_init(&free_bar[i], 1); }
+        for (uint32_t i = 0; i < kMaxStages; ++i) { mbar_init(&full[i], 1); mbar_init(&free_bar[i], 1); }
         mbar_init(done_bar, 1);
         fence_barrier_init();
     }
@@ -84,9 +84,9 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
         if (lane == 0) {
             uint32_t requested = 0;
             for (uint32_t step = 0; step < steps; ++step) {
-                const uint32_t stage = step % kStages, use = step / kStages;
+                const uint32_t stage = step % stages, use = step / stages;
                 if (use > 0u && !wait_or_abort(&free_bar[stage], (use - 1u) & 1u, abort)) { ok = false; break; }
-                uint8_t* at = smem + stage * kStageBytes;
+                uint8_t* at = smem + stage * stage_bytes;
                 mbar_expect_tx(&full[stage], kDenseTileBytes + n_rows * 128u);
                 bulk_load(at, weight + (size_t)step * kDenseTileBytes, kDenseTileBytes, &full[stage]);
                 bulk_load(at + kDenseTileBytes, rows_at + (size_t)step * m.a.capacity * 128u, n_rows * 128u, &full[stage]);
@@ -96,18 +96,18 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
                 // Copies already requested get a bounded chance to land before the shared memory is released.
                 ok = false;
                 abort_flag = 1u;
-                for (uint32_t step = requested > kStages ? requested - kStages : 0u; step < requested; ++step)
-                    mbar_wait(&full[step % kStages], (step / kStages) & 1u, 1u << 16);
+                for (uint32_t step = requested > stages ? requested - stages : 0u; step < requested; ++step)
+                    mbar_wait(&full[step % stages], (step / stages) & 1u, 1u << 16);
             }
         }
     } else if (warp == kEpilogueWarps + 1u) {
         if (lane == 0) {
             const uint32_t instruction = mma_instruction(kDenseTile, n_rows);
             for (uint32_t step = 0; step < steps; ++step) {
-                const uint32_t stage = step % kStages;
-                if (!wait_or_abort(&full[stage], (step / kStages) & 1u, abort)) { ok = false; break; }
+                const uint32_t stage = step % stages;
+                if (!wait_or_abort(&full[stage], (step / stages) & 1u, abort)) { ok = false; break; }
                 tc_fence_after_sync();
-                const uint32_t at = smem_u32(smem + stage * kStageBytes);
+                const uint32_t at = smem_u32(smem + stage * stage_bytes);
 #pragma unroll
                 for (uint32_t kk = 0; kk < kDenseBlockK / 16u; ++kk)
                     mma_bf16(tmem, operand_descriptor(at + kk * 256u), operand_descriptor(at + kDenseTileBytes + kk * 256u), instruction, (step | kk) != 0u ? 1u : 0u);
@@ -264,25 +264,38 @@ __global__ void __launch_bounds__(256) chunk_norm_kernel(const ChunkNorm p) {
     }
 }
 
-// One block: every warp routes rows; counts, starts and grouped rows follow from the choices.
-__global__ void __launch_bounds__(1024) chunk_route_kernel(const ChunkRoute p) {
-    __shared__ uint32_t counts[kMaxExperts], starts[kMaxExperts];
+// A warp per row chooses its experts.
+__global__ void __launch_bounds__(128) chunk_route_kernel(const ChunkRoute p) {
     extern __shared__ float scores[];                                  // [warps][experts]
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, warps = blockDim.x >> 5;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, row = blockIdx.x * 4u + warp;
+    if (row >= p.rows) return;
+    route_row(p.logits + (size_t)row * p.logits_ld, p.experts, p.top, scores + warp * p.experts, [&](uint32_t slot, uint32_t e, float score) {
+        if (lane != 0) return;
+        p.slot_experts[row * p.top + slot] = e;
+        p.slot_scores[row * p.top + slot] = score;
+    });
+}
+
+// One block: the experts' counts, their starts, and every choice's grouped row.
+__global__ void __launch_bounds__(1024) chunk_starts_kernel(const ChunkRoute p) {
+    __shared__ uint32_t counts[kMaxExperts], starts[kMaxExperts];
     for (uint32_t e = threadIdx.x; e < p.experts; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    for (uint32_t row = warp; row < p.rows; row += warps)
-        route_row(p.logits + (size_t)row * p.logits_ld, p.experts, p.top, scores + warp * p.experts, [&](uint32_t slot, uint32_t e, float score) {
-            if (lane != 0) return;
-            const uint32_t at = row * p.top + slot;
-            p.slot_experts[at] = e;
-            p.slot_scores[at] = score;
-            p.slot_rows[at] = atomicAdd(&counts[e], 1u);
-        });
+    for (uint32_t at = threadIdx.x; at < p.rows * p.top; at += blockDim.x) p.slot_rows[at] = atomicAdd(&counts[p.slot_experts[at]], 1u);
     __syncthreads();
-    if (threadIdx.x == 0) {
-        uint32_t at = 0;
-        for (uint32_t e = 0; e < p.experts; ++e) { starts[e] = at; at += (counts[e] + 7u) & ~7u; }
+    if (threadIdx.x < 32u) {                                           // prefix sums of the counts, rounded up to eight
+        uint32_t before = 0;
+        for (uint32_t first = 0; first < p.experts; first += 32u) {
+            const uint32_t e = first + threadIdx.x, padded = e < p.experts ? (counts[e] + 7u) & ~7u : 0u;
+            uint32_t sum = padded;
+#pragma unroll
+            for (int offset = 1; offset < 32; offset <<= 1) {
+                const uint32_t other = __shfl_up_sync(0xffffffffu, sum, offset);
+                if (threadIdx.x >= (uint32_t)offset) sum += other;
+            }
+            if (e < p.experts) starts[e] = before + sum - padded;
+            before += __shfl_sync(0xffffffffu, sum, 31);
+        }
     }
     __syncthreads();
     for (uint32_t e = threadIdx.x; e < p.experts; e += blockDim.x) { p.group_start[e] = starts[e]; p.group_rows[e] = counts[e]; }
@@ -305,6 +318,10 @@ __global__ void __launch_bounds__(256) chunk_group_kernel(const ChunkRoute p) {
     for (uint32_t i = threadIdx.x; i < p.from.k_pad / 8u; i += blockDim.x)
         *reinterpret_cast<uint4*>(static_cast<uint8_t*>(p.to.data) + operand_offset(p.to, grouped, i * 8u)) =
             *reinterpret_cast<const uint4*>(static_cast<const uint8_t*>(p.from.data) + operand_offset(p.from, row, i * 8u));
+}
+
+__global__ void __launch_bounds__(256) chunk_operand_kernel(const float* __restrict__ x, uint32_t k, const Operand result) {
+    for (uint32_t i = threadIdx.x; i < result.k_pad; i += blockDim.x) store_operand(result, blockIdx.x, i, i < k ? x[(size_t)blockIdx.x * k + i] : 0.0f);
 }
 
 __global__ void __launch_bounds__(128) chunk_latents_kernel(const float* __restrict__ raw, uint32_t raw_ld, const float* __restrict__ gain, uint32_t rank,
@@ -361,9 +378,11 @@ int launch_chunk_product(ChunkProduct p, bool f32, cudaStream_t stream) {
         p.window = kWindowMax;
         while (p.window > 64u && (uint64_t)total * ((p.rows + p.window - 1u) / p.window) * 5u < (uint64_t)sm_count() * 4u) p.window /= 2u;
         static std::once_flag once[64];
-        const int status = allow_smem(chunk_product_kernel, once, kChunkSmemBytes);
+        const int status = allow_smem(chunk_product_kernel, once, kSmemAlone);
         if (status != GF_OK) return status;
-        chunk_product_kernel<<<dim3(total, (p.rows + p.window - 1u) / p.window), kChunkThreads, kChunkSmemBytes, stream>>>(p);
+        // Many tiles: two CTAs share an SM, so that one's start and output overlap the other's products.
+        p.stage_budget = (uint64_t)total * ((p.rows + p.window - 1u) / p.window) > 3u * (uint64_t)sm_count() ? kSmemPaired : kSmemAlone;
+        chunk_product_kernel<<<dim3(total, (p.rows + p.window - 1u) / p.window), kChunkThreads, p.stage_budget, stream>>>(p);
     }
     GF_CUDA(cudaGetLastError());
     return GF_OK;
@@ -379,14 +398,26 @@ int launch_chunk_norm(const ChunkNorm& p, cudaStream_t stream) {
     return GF_OK;
 }
 
+int launch_route(const ChunkRoute& p, cudaStream_t stream) {
+    if (p.rows == 0 || p.experts == 0 || p.experts > kMaxExperts || p.top == 0 || p.top > p.experts) return fail(GF_ERR_INVALID, "route: bad arguments");
+    chunk_route_kernel<<<(p.rows + 3u) / 4u, 128, 4u * p.experts * 4u, stream>>>(p);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
 int launch_chunk_route(const ChunkRoute& p, cudaStream_t stream) {
-    if (p.rows == 0 || p.experts == 0 || p.experts > kMaxExperts || p.top == 0 || p.top > p.experts) return fail(GF_ERR_INVALID, "chunk route: bad arguments");
     if (grouped_rows(p.rows, p.top, p.experts) > p.to.capacity) return fail(GF_ERR_INVALID, "chunk route: the grouped operand is too small");
-    static std::once_flag once[64];
-    const int status = allow_smem(chunk_route_kernel, once, 32u * kMaxExperts * 4u);
+    const int status = launch_route(p, stream);
     if (status != GF_OK) return status;
-    chunk_route_kernel<<<1, 1024, 32u * p.experts * 4u, stream>>>(p);
+    chunk_starts_kernel<<<1, 1024, 0, stream>>>(p);
     chunk_group_kernel<<<p.rows * p.top, 256, 0, stream>>>(p);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+int launch_chunk_operand(const float* x, uint32_t rows, uint32_t k, const Operand& result, cudaStream_t stream) {
+    if (!x || !result.data || rows == 0 || rows > result.capacity || k > result.k_pad) return fail(GF_ERR_INVALID, "chunk operand: bad arguments");
+    chunk_operand_kernel<<<rows, 256, 0, stream>>>(x, k, result);
     GF_CUDA(cudaGetLastError());
     return GF_OK;
 }

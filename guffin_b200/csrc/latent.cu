@@ -61,8 +61,8 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
     float* correction = run_sum + kQueries;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, g = lane >> 2, t = lane & 3u;
 
-    pdl_launch_dependents();
     pdl_wait();
+    pdl_launch_dependents();
     const bool chain = p.ring_stride == 0u;
     const uint32_t z = blockIdx.z, queries = chain ? p.rows * p.heads : p.heads;      // this sequence's queries
     const uint32_t first_query = blockIdx.x * kQueries, part = blockIdx.y;
@@ -275,8 +275,8 @@ __global__ void __launch_bounds__(kThreads) latent_attention_plain_kernel(const 
     float* query = plain;
     float* out = plain + p.row_elements;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    pdl_launch_dependents();
     pdl_wait();
+    pdl_launch_dependents();
     const bool chain = p.ring_stride == 0u;
     const uint32_t m = blockIdx.x, row = m / p.heads, head = m % p.heads, part = blockIdx.y;
     const uint32_t base = p.positions[chain ? 0u : row], end = chain ? base + row + 1u : base + 1u;
@@ -330,17 +330,12 @@ __global__ void __launch_bounds__(kThreads) latent_attention_plain_kernel(const 
 __global__ void __launch_bounds__(128) latent_merge_kernel(const LatentAttention p) {
     __shared__ float factors[kLatentMaxParts];
     const uint32_t m = blockIdx.x, row = m / p.heads, head = m % p.heads;
-    const float* ml = p.partial_ml + (size_t)m * p.parts * 2u;
-    float top = p.sink ? p.sink[head] : -INFINITY;
-    for (uint32_t part = 0; part < p.parts; ++part) top = fmaxf(top, ml[part * 2u]);
-    float total = p.sink ? expf(p.sink[head] - top) : 0.0f;
-    for (uint32_t part = 0; part < p.parts; ++part) total += ml[part * 2u + 1u] > 0.0f ? ml[part * 2u + 1u] * expf(ml[part * 2u] - top) : 0.0f;
-    for (uint32_t part = threadIdx.x; part < p.parts; part += blockDim.x) factors[part] = ml[part * 2u + 1u] > 0.0f ? expf(ml[part * 2u] - top) / total : 0.0f;
+    if (threadIdx.x < 32u) merge_factors(p.partial_ml + (size_t)m * p.parts * 2u, p.parts, p.sink ? p.sink[head] : -INFINITY, factors);
     __syncthreads();
     for (uint32_t i = threadIdx.x; i < p.row_elements; i += blockDim.x) {
         float v = 0.0f;
-        for (uint32_t part = 0; part < p.parts; ++part)
-            if (factors[part] != 0.0f) v = fmaf(p.partial_out[((size_t)m * p.parts + part) * p.row_elements + i], factors[part], v);
+#pragma unroll 8
+        for (uint32_t part = 0; part < p.parts; ++part) v = fmaf(p.partial_out[((size_t)m * p.parts + part) * p.row_elements + i], factors[part], v);
         store_operand(p.result, row, head * p.result_stride + i, v);
     }
 }

@@ -538,7 +538,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         groups.logits = a.router_logits; groups.logits_ld = f.experts; groups.rows = rows; groups.experts = f.experts; groups.top = f.top;
         groups.group_start = a.group_start; groups.group_rows = a.group_rows; groups.slot_rows = a.slot_rows; groups.slot_experts = a.slot_experts;
         groups.slot_scores = a.slot_scores; groups.row_scale = a.row_scale; groups.from = normed; groups.to = group;
-        launches_ += 2;
+        launches_ += 3;
         GF_TRY(launch_chunk_route(groups, stream_));
         ChunkProduct up;
         up.p[0] = chunk_problem(w.expert_up, group);

@@ -67,6 +67,14 @@ lib.register({
     "gf_model_shard_set_wait_limit": (i32, [vp, u32]),
     "gf_model_shard_global_selection": (i32, [vp, i32]),
     "gf_add": (i32, [vp, vp, vp, u64, vp]),
+    "gf_dense_packed_bytes": (sz, [u32, u32]),
+    "gf_dense_pack": (i32, [vp, u32, u32, vp, vp]),
+    "gf_dense_matmul": (i32, [vp, vp, vp, u32, u32, u32, vp]),
+    "gf_dense_chunk_workspace_bytes": (sz, [u32, u32, i32]),
+    "gf_dense_chunk_matmul": (i32, [vp, vp, vp, u32, u32, u32, i32, vp, vp]),
+    "gf_latent_attention_workspace_bytes": (sz, [u32, u32, u32, u32]),
+    "gf_latent_attention": (i32, [vp, vp, vp, vp, vp, vp, u32, u32, u32, u32, u32, i32, vp, vp]),
+    "gf_route": (i32, [vp, u32, u32, u32, vp, vp, vp]),
     "gf_architectures": (C.c_char_p, []),
     "gf_model_create_described": (i32, [C.c_char_p, u32, u32, i32, C.POINTER(vp)]),
     "gf_model_set_tensor": (i32, [vp, C.c_char_p, i32, vp, C.POINTER(u64), u32]),

@@ -175,6 +175,80 @@ def make_model_weights(name: str, seed: int, config: dict | None = None) -> dict
     return dict(iter_model_weights(name, seed, config))
 
 
+# ---------------------------------------------------------------------------- layered models
+
+def zasevik_config(width, layers, heads, dim, vdim, rank, vocab, mlps, eps=1e-6) -> dict:
+    """A Zasevik configuration with one attention geometry; layer i takes mlps[i % len(mlps)] (dense_mlp / expert_mlp / None)."""
+    mixer = dict(heads=heads, dim=dim, vdim=vdim, kv_rank=rank, scale=1.0 / math.sqrt(dim))
+    return dict(architecture="Zasevik", embedding=dict(scale=math.sqrt(width)), norm=dict(eps=eps), vocab=vocab, width=width,
+                layers=[dict(type="latent_attention", mixer=dict(mixer), mlp=mlps[i % len(mlps)]) for i in range(layers)])
+
+
+def dense_mlp(ff) -> dict:
+    return dict(kind="dense", ff=ff)
+
+
+def expert_mlp(ff, experts, top, limit, shared_ff=0, shared_limit=0.0) -> dict:
+    mlp = dict(kind="moe", expert=dict(ff=ff, limit=limit), router=dict(experts=experts, top=top))
+    if shared_ff:
+        mlp["shared"] = dict(ff=shared_ff, limit=shared_limit)
+    return mlp
+
+
+def zasevik_shapes(config: dict) -> dict:
+    """Tensor name -> shape of every tensor of a Zasevik configuration."""
+    W, shapes = config["width"], {"embed": (config["vocab"], config["width"]), "final.norm": (config["width"],)}
+    for i, layer in enumerate(config["layers"]):
+        p, m, f = f"l{i}", layer["mixer"], layer.get("mlp")
+        H, R = m["heads"], m["kv_rank"]
+        shapes.update({f"{p}.norm1": (W,), f"{p}.norm1b": (W,), f"{p}.ls1": (W,), f"{p}.mix.q": (H * m["dim"], W), f"{p}.mix.dkv": (R, W),
+                       f"{p}.mix.dkv.norm": (R,), f"{p}.mix.uk": (H * m["dim"], R), f"{p}.mix.uv": (H * m["vdim"], R), f"{p}.mix.sink": (H,),
+                       f"{p}.mix.o": (W, H * m["vdim"])})
+        if not f:
+            continue
+        shapes.update({f"{p}.norm2": (W,), f"{p}.norm2b": (W,), f"{p}.ls2": (W,)})
+        if f["kind"] == "dense":
+            shapes.update({f"{p}.mlp.up": (f["ff"], W), f"{p}.mlp.down": (W, f["ff"])})
+            continue
+        for e in range(f["router"]["experts"]):
+            shapes.update({f"{p}.mlp.e{e}.gate": (f["expert"]["ff"], W), f"{p}.mlp.e{e}.up": (f["expert"]["ff"], W), f"{p}.mlp.e{e}.down": (W, f["expert"]["ff"])})
+        shapes[f"{p}.mlp.router"] = (f["router"]["experts"], W)
+        if f.get("shared"):
+            ff = f["shared"]["ff"]
+            shapes.update({f"{p}.mlp.shared.gate": (ff, W), f"{p}.mlp.shared.up": (ff, W), f"{p}.mlp.shared.down": (W, ff), f"{p}.mlp.shared.sg": (1, W)})
+    return shapes
+
+
+def iter_zasevik_weights(config: dict, seed: int):
+    """Yields (name, array): matrices as bfloat16 bits with entries of variance 1 / inputs, vectors as f32."""
+    rng = np.random.default_rng(seed)
+    for name, shape in zasevik_shapes(config).items():
+        if len(shape) == 2:
+            values = rng.standard_normal(shape, dtype=np.float32) * np.float32(1.0 / math.sqrt(shape[1]))
+            bits = values.view(np.uint32)
+            yield name, ((bits + 0x7fff + ((bits >> 16) & 1)) >> 16).astype(np.uint16)
+        elif name.endswith(".sink"):
+            yield name, rng.normal(1.0, 1.0, shape).astype(np.float32)
+        elif ".ls" in name or name.endswith("dkv.norm"):
+            yield name, rng.uniform(0.5, 1.5, shape).astype(np.float32)
+        else:
+            yield name, rng.normal(0.0, 0.2, shape).astype(np.float32)
+
+
+def zasevik_active_parameters(config: dict) -> int:
+    """Matrix elements one token's pass multiplies with (chosen experts only; the head included)."""
+    total = 0
+    for name, shape in zasevik_shapes(config).items():
+        if len(shape) != 2:
+            continue
+        parts, share = name.split("."), 1.0
+        if len(parts) > 2 and parts[1] == "mlp" and parts[2][0] == "e" and parts[2][1:].isdigit():
+            router = config["layers"][int(parts[0][1:])]["mlp"]["router"]
+            share = router["top"] / router["experts"]
+        total += share * shape[0] * shape[1]
+    return int(round(total))
+
+
 def model_weight_bytes(name: str, config: dict | None = None) -> int:
     """Native GGUF bytes one decode pass streams: every matrix once, the tied head included."""
     config = config or model_config(name)

@@ -334,6 +334,29 @@ GF_API int gf_model_shard_global_selection(gf_model* model, int enable);
  * The geometry still comes from gf_model_config; *out_bound_tensors (optional) counts the
  * tensors taken.  Call gf_model_finalize afterwards. */
 GF_API int gf_model_load_gguf(gf_model* model, const char* path, uint32_t* out_bound_tensors);
+/* ---- operators of layered models.  No counterpart in the reference.  A bf16 matrix [n][k] (out x in) is packed once
+ * (gf_dense_pack) into the order the tensor core reads; gf_dense_matmul multiplies any number of f32 rows with it in
+ * 32-bit (the product of row passes, tuned for up to GF_MAX_ROWS); gf_dense_chunk_matmul is the product of prompt
+ * chunks: bf16 operands on tcgen05 with f32 accumulation, or with precision GF_PRECISION_F32 everything in 32-bit.
+ * It synchronises the stream and reports GF_ERR_TIMEOUT.
+ * gf_latent_attention: causal attention of `rows` tokens x `heads` over cached latents of `rank` values, which serve
+ * as keys and values.  q_dev holds the scaled queries already in latent space, [rows * heads][rank rounded up to 16];
+ * ring_dev [ring_rows][..] the committed rows, private_dev [rows][..] the pass's own; binary16, or f32 with precision
+ * GF_PRECISION_F32.  The rows follow position *position_dev as a chain.  sink_dev (may be NULL): a logit per head in the
+ * denominator.  out_dev f32 [rows * heads][rank rounded up to 16].  parts = partitions of the keys, 1..64.
+ * gf_route: the `top` largest sigmoid scores of every row, lower index first among equals. ---- */
+GF_API size_t gf_dense_packed_bytes(uint32_t k, uint32_t n);
+GF_API int gf_dense_pack(const uint16_t* bf16_dev, uint32_t k, uint32_t n, void* packed_dev, void* stream);
+GF_API int gf_dense_matmul(const void* packed_dev, const float* x_dev, float* y_dev, uint32_t rows, uint32_t k, uint32_t n, void* stream);
+GF_API size_t gf_dense_chunk_workspace_bytes(uint32_t rows, uint32_t k, int precision);
+GF_API int gf_dense_chunk_matmul(const void* packed_dev, const float* x_dev, float* y_dev, uint32_t rows, uint32_t k, uint32_t n, int precision,
+                                 void* workspace_dev, void* stream);
+GF_API size_t gf_latent_attention_workspace_bytes(uint32_t rows, uint32_t heads, uint32_t rank, uint32_t parts);
+GF_API int gf_latent_attention(const void* q_dev, const void* ring_dev, const void* private_dev, const uint32_t* position_dev, const float* sink_dev,
+                               float* out_dev, uint32_t rows, uint32_t heads, uint32_t rank, uint32_t ring_rows, uint32_t parts, int precision,
+                               void* workspace_dev, void* stream);
+GF_API int gf_route(const float* logits_dev, uint32_t rows, uint32_t experts, uint32_t top, uint32_t* ids_dev, float* scores_dev, void* stream);
+
 /* ---- models described by a configuration file.  No counterpart in the reference, which serves the Gemma families
  * only.  `config_json` is the text of a config.json whose "architecture" names an entry of the registry
  * (gf_architectures, one name per line): "Zasevik" (a layered decoder: every layer names its mixer and its

@@ -528,7 +528,7 @@ def run_zasevik(args) -> dict:
         ours["decode_frac"] = ours["decode_gbs"] / peak
         head = config["vocab"] * config["width"]
         keys = prefix * (prefix + 1) / 2
-        attention = sum(4.0 * l["mixer"]["heads"] * l["mixer"]["kv_rank"] * keys for l in config["layers"])
+        attention = sum(2.0 * l["mixer"]["heads"] * (l["mixer"]["dim"] + l["mixer"]["vdim"]) * keys for l in config["layers"])
         ours["prefill_tflops"] = (2.0 * (active - head) * prefix + attention) / ours["prefill_ms"] / 1e9
         ours["prefill_frac"] = ours["prefill_tflops"] / tensor_peak
         # End to end through the generation engine: prompt in host memory, tokens back on the host.

@@ -134,6 +134,7 @@ enum ChunkOutput : uint32_t {
     kChunkSquaredRelu = 2,    // operand(row, n) = max(product, 0)^2
     kChunkClampedGate = 3,    // paired matrix: operand(row, n) = clamped gate of (gate, up) * row scale
     kChunkLatentQuery = 4,    // out[(row * heads + index) * out_ld + n] = product * scale, f16 or f32
+    kChunkHalfRows = 5,       // f16 out[row * out_ld + column(n)] = product * scale
 };
 
 // `count` products of the same shape: heads of one matrix, or experts.

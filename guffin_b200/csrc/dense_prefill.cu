@@ -23,6 +23,12 @@ __device__ __forceinline__ void chunk_store(const ChunkProblem& p, uint32_t inde
         const size_t at = ((size_t)row * p.heads + index) * p.out_ld + n;
         if (p.query_f16) reinterpret_cast<__half*>(p.out)[at] = __float2half_rn(v * p.scale);
         else p.out[at] = v * p.scale;
+    } else if (p.output == kChunkHalfRows) {
+        const uint32_t column = (p.segment ? n / p.segment * p.segment_pad + n % p.segment : n) + index * p.column_stride;
+        __half* out = reinterpret_cast<__half*>(p.out) + (size_t)row * p.out_ld + column;
+        *out = __float2half_rn(v * p.scale);
+        if (p.segment && n % p.segment + 1u == p.segment)               // the padding takes part in scores
+            for (uint32_t i = 1; i <= p.segment_pad - p.segment; ++i) out[i] = __float2half_rn(0.0f);
     } else {
         const uint32_t column = (p.segment ? n / p.segment * p.segment_pad + n % p.segment : n) + index * p.column_stride;
         store_operand(p.result, row, column, p.output == kChunkSquaredRelu ? squared_relu(v) : v);
@@ -34,11 +40,66 @@ __device__ __forceinline__ void chunk_store_gate(const ChunkProblem& p, uint32_t
     store_operand(p.result, row, n, clamped_gate(gate * s, up * s, p.limit));
 }
 
+__device__ __forceinline__ uint4 bf16_octet(const float (&v)[8]) {
+    uint4 r;
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r.x) : "f"(v[1]), "f"(v[0]));
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r.y) : "f"(v[3]), "f"(v[2]));
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r.z) : "f"(v[5]), "f"(v[4]));
+    asm("cvt.rn.bf16x2.f32 %0, %1, %2;" : "=r"(r.w) : "f"(v[7]), "f"(v[6]));
+    return r;
+}
+__device__ __forceinline__ uint4 half_octet(const float (&v)[8], float scale) {
+    uint4 r;
+    uint32_t* w = &r.x;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const __half2 h = __floats2half2_rn(v[2 * i] * scale, v[2 * i + 1] * scale);
+        w[i] = *reinterpret_cast<const uint32_t*>(&h);
+    }
+    return r;
+}
+
+// Columns n .. n + 7 (n a multiple of eight) of an output row at once where they stay together in the result and start
+// on a 16-byte boundary; one by one otherwise.
+__device__ __forceinline__ void chunk_store8(const ChunkProblem& p, uint32_t index, uint32_t row, uint32_t n, float (&v)[8]) {
+    const bool whole = n + 8u <= p.n && p.segment % 8u == 0u;
+    const uint32_t column = (p.segment ? n / p.segment * p.segment_pad + n % p.segment : n) + index * p.column_stride;
+    if (whole && p.output == kChunkF32 && p.out_ld % 4u == 0u) {
+        float s = 1.0f;
+        if (p.row_scale) {
+            s = p.row_scale[(size_t)row * p.row_scale_ld];
+            if (p.row_scale_sigmoid) s = sigmoid(s);
+        }
+        float* out = p.out + (size_t)row * p.out_ld + n;
+        *reinterpret_cast<float4*>(out) = make_float4(v[0] * s, v[1] * s, v[2] * s, v[3] * s);
+        *reinterpret_cast<float4*>(out + 4) = make_float4(v[4] * s, v[5] * s, v[6] * s, v[7] * s);
+        return;
+    }
+    if (whole && column % 8u == 0u && (p.output == kChunkOperand || p.output == kChunkSquaredRelu)) {
+        if (p.output == kChunkSquaredRelu)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) v[i] = squared_relu(v[i]);
+        *reinterpret_cast<uint4*>(static_cast<uint8_t*>(p.result.data) + operand_offset(p.result, row, column)) = bf16_octet(v);
+        return;
+    }
+    if (whole && p.out_ld % 8u == 0u && p.output == kChunkLatentQuery && p.query_f16) {
+        *reinterpret_cast<uint4*>(reinterpret_cast<__half*>(p.out) + ((size_t)row * p.heads + index) * p.out_ld + n) = half_octet(v, p.scale);
+        return;
+    }
+    if (whole && p.out_ld % 8u == 0u && column % 8u == 0u && p.output == kChunkHalfRows && p.segment == p.segment_pad) {
+        *reinterpret_cast<uint4*>(reinterpret_cast<__half*>(p.out) + (size_t)row * p.out_ld + column) = half_octet(v, p.scale);
+        return;
+    }
+#pragma unroll 1
+    for (uint32_t i = 0; i < 8u && n + i < p.n; ++i) chunk_store(p, index, row, n + i, v[i]);
+}
+
 // ------------------------------------------------------------------ bf16 products on tcgen05
 
 constexpr uint32_t kWindowMax = 256;                                   // token rows of a tile: the product's N
 constexpr uint32_t kMaxStages = 8;                                     // a stage: 128 weight columns, then the window's token rows, x 64 K
 constexpr uint32_t kEpilogueWarps = 8;
+constexpr uint32_t kStagedLd = kDenseTile + 4u;                        // floats between staged output rows
 constexpr uint32_t kChunkThreads = (kEpilogueWarps + 2u) * 32u;        // the copying and the issuing warp behind them
 constexpr uint32_t kSmemAlone = 208u * 1024u, kSmemPaired = 104u * 1024u;      // stages of a CTA that has its SM alone, or shares it with another
 
@@ -120,30 +181,47 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
         if (!wait_or_abort(done_bar, 0u, abort)) { ok = false; if (lane == 0) abort_flag = 1u; }
     }
     const bool failed = __syncthreads_or(ok ? 0 : 1) != 0;
-    if (!failed && warp < kEpilogueWarps) {
-        tc_fence_after_sync();
-        // Warp w reads accumulator lanes 32 (w % 4) .. + 31, i.e. output columns; a warp's accumulator columns are token rows.
-        const uint32_t quarter = warp & 3u, column = tile * kDenseTile + quarter * 32u + lane;
-        const bool paired = m.output == kChunkClampedGate;
-        const uint32_t pair_column = tile * (kDenseTile / 2u) + quarter * 16u + (lane >> 4) * 8u + (lane & 7u);
-        for (uint32_t c = (warp >> 2) * 32u; c < live; c += 64u) {
-            float v[32];
-            tmem_load_32(tmem + ((quarter * 32u) << 16) + c, v);
+    // Output, 64 token rows at a time: the accumulators go through shared memory (the stages are free again), so that a
+    // thread holds eight neighbouring columns of a row.
+    float* staged = reinterpret_cast<float*>(smem);                     // [64][kStagedLd]
+    for (uint32_t c0 = 0; c0 < live && !failed; c0 += 64u) {
+        if (warp < kEpilogueWarps) {
+            // Warp w reads accumulator lanes 32 (w % 4) .. + 31, i.e. output columns; a warp's accumulator columns are token rows.
+            tc_fence_after_sync();
+            const uint32_t quarter = warp & 3u, c = c0 + (warp >> 2) * 32u;
+            if (c < live) {
+                float v[32];
+                tmem_load_32(tmem + ((quarter * 32u) << 16) + c, v);
 #pragma unroll
-            for (uint32_t i = 0; i < 32u; ++i) {
-                const uint32_t row = row0 + c + i;
-                if (paired) {
-                    const float up = __shfl_xor_sync(0xffffffffu, v[i], 8);
-                    if (c + i < live && (lane & 8u) == 0u && pair_column < m.n / 2u) chunk_store_gate(m, row, pair_column, v[i], up);
-                } else if (c + i < live && column < m.n) {
-                    chunk_store(m, index, row, column, v[i]);
-                }
+                for (uint32_t i = 0; i < 32u; ++i) staged[((warp >> 2) * 32u + i) * kStagedLd + quarter * 32u + lane] = v[i];
             }
+            tc_fence_before_sync();
         }
-        tc_fence_before_sync();
-    } else if (failed && tid == 0) {
-        atomicExch(p.error_flag, 1);
+        __syncthreads();
+        const bool paired = m.output == kChunkClampedGate;
+        const uint32_t octets = paired ? 8u : 16u, count = min(64u, live - c0) * octets;
+#pragma unroll 1
+        for (uint32_t i = tid; i < count; i += kChunkThreads) {
+            const uint32_t r = i / octets, octet = i % octets, row = row0 + c0 + r;
+            const float* src = staged + r * kStagedLd + octet * (paired ? 16u : 8u);
+            float v[8];
+#pragma unroll
+            for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4*>(v + j) = *reinterpret_cast<const float4*>(src + j);
+            if (!paired) {
+                const uint32_t n = tile * kDenseTile + octet * 8u;
+                if (n < m.n) chunk_store8(m, index, row, n, v);
+                continue;
+            }
+            const uint32_t n = tile * (kDenseTile / 2u) + octet * 8u;
+            if (n >= m.n / 2u) continue;
+            const float s = m.row_scale ? m.row_scale[(size_t)row * m.row_scale_ld] : 1.0f;
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = clamped_gate(v[j] * s, src[8 + j] * s, m.limit);
+            *reinterpret_cast<uint4*>(static_cast<uint8_t*>(m.result.data) + operand_offset(m.result, row, n)) = bf16_octet(v);
+        }
+        __syncthreads();
     }
+    if (failed && tid == 0) atomicExch(p.error_flag, 1);
     __syncthreads();
     if (warp == 0) tmem_dealloc(tmem, tmem_columns);
 }

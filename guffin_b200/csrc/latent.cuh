@@ -37,4 +37,26 @@ int launch_latent_attention(LatentAttention p, cudaStream_t stream, bool pdl);
 // Merges partial results (and the sink) into the operand `result`.
 int launch_latent_merge(const LatentAttention& p, cudaStream_t stream);
 
+// ---- the same attention with the latents expanded into keys and values per head: fewer operations once a chunk has
+// many rows for the keys it sees, since a score then costs a head's `dim` instead of the latent's rank.
+constexpr uint32_t kHeadAttentionMaxDim = 256;
+struct HeadAttention {
+    const __half* q = nullptr;           // [rows][heads][dim_pad], scaled
+    const __half* k = nullptr;           // [positions][heads][dim_pad], positions from 0
+    const __half* v = nullptr;           // [positions][heads][vdim_pad]
+    const uint32_t* position = nullptr;  // of row 0
+    const float* sink = nullptr;
+    uint32_t rows = 0, heads = 0, dim_pad = 0, vdim = 0, vdim_pad = 0;      // pads: multiples of 16
+    Operand result;                      // (row, head * vdim + d), bf16 or f32
+};
+int launch_head_attention(const HeadAttention& p, cudaStream_t stream);
+// The first `positions` cache rows of a sequence as a bf16 operand.
+int launch_latent_operand(const StreamRings* rings, const void* own, const uint32_t* position, uint32_t positions, uint32_t row_elements, uint32_t ring_mask,
+                          const Operand& result, cudaStream_t stream);
+// Rows of a chunk from which expanding pays: expansion costs every key rank x (dim + vdim) per head, and saves every
+// (row, key) pair 2 x rank - (dim + vdim).
+inline bool latent_expansion_pays(uint32_t rows, uint32_t rank, uint32_t dim, uint32_t vdim) {
+    return 2u * rank > dim + vdim && (uint64_t)rows * (2u * rank - dim - vdim) > (uint64_t)rank * (dim + vdim);
+}
+
 }  // namespace gf

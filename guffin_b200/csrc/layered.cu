@@ -144,6 +144,13 @@ int Model::set_tensor(const char* name, int dtype, const void* host, const uint6
     pack.dst_stride = dst->bytes();
     pack.k_blocks = dst->k_blocks();
     GF_TRY(launch_dense_pack(pack, stream_));
+    if (slot.role == TensorRole::kLatentUpKey && !p.f32) {
+        GF_TRY(ensure_matrix(allocations_, l.expand_key, m.rank, m.heads * m.dim, 1, weight_bytes_));
+        DensePack plain = pack;
+        plain.dst = l.expand_key.data; plain.count = 1; plain.count_stride = 0; plain.n = m.heads * m.dim; plain.k = m.rank;
+        plain.n_stride = m.rank; plain.k_stride = 1; plain.k_blocks = l.expand_key.k_blocks();
+        GF_TRY(launch_dense_pack(plain, stream_));
+    }
     GF_CUDA(cudaEventRecord(stager_.packed[staging], stream_));
     native_weight_bytes_ += bytes;
     p.bound[name] = true;
@@ -400,6 +407,20 @@ int Model::ensure_chunk_arena() {
     GF_TRY(plan_alloc(allocations_, &a.final_rows, (size_t)rows * s.width));
     GF_TRY(plan_alloc(allocations_, &a.raw_latent, (size_t)rows * latent));
     GF_TRY(bytes_alloc(allocations_, &a.latent_q, (size_t)rows * query_elements * (p.f32 ? 4u : 2u)));
+    if (!p.f32) {
+        size_t per_key = 0, q_elements = 0;
+        for (const LayerSpec& l : s.layers) {
+            const size_t dims = round_up(l.mixer.dim, 16u), vdims = round_up(l.mixer.vdim, 16u);
+            per_key = std::max(per_key, l.mixer.heads * std::max(dims, vdims));
+            q_elements = std::max(q_elements, l.mixer.heads * dims);
+        }
+        // At most 1 GiB for either; chunks that see more positions than fit attend the latents themselves.
+        a.expand_keys = (uint32_t)std::min<size_t>(round_up(c.context, 16u), ((size_t)1 << 30) / (per_key * 2u) / 16u * 16u);
+        GF_TRY(bytes_alloc(allocations_, &a.latent_rows, (size_t)a.expand_keys * round_up(latent, kDenseBlockK) * 2u));
+        GF_TRY(plan_alloc(allocations_, &a.keys, a.expand_keys * per_key));
+        GF_TRY(plan_alloc(allocations_, &a.values, a.expand_keys * per_key));
+        GF_TRY(plan_alloc(allocations_, &a.head_q, rows * q_elements));
+    }
     a.partial_rows = std::max((uint32_t)sm_count() * 64u, heads * 16u);
     GF_TRY(plan_alloc(allocations_, &a.partial_out, (size_t)a.partial_rows * row_elements));
     GF_TRY(plan_alloc(allocations_, &a.partial_ml, (size_t)a.partial_rows * 2u));
@@ -450,7 +471,8 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         return launch_chunk_norm(n, stream_);
     };
     auto run = [&](ChunkProduct& product) -> int {
-        product.rows = rows; product.error_flag = error_flag_;
+        if (product.rows == 0) product.rows = rows;
+        product.error_flag = error_flag_;
         ++launches_;
         return launch_chunk_product(product, f32, stream_);
     };
@@ -465,8 +487,16 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         ChunkProduct down;
         down.p[0] = chunk_problem(w.latent_down, normed);
         down.p[0].out = a.raw_latent; down.p[0].out_ld = m.rank;
-        const Operand query = operand_view(a.query, m.heads * dim_pad);
-        if (!last) {
+        const Operand query = operand_view(a.query, m.heads * dim_pad), heads_out = operand_view(a.heads_out, m.heads * m.vdim);
+        const uint32_t positions = position_ + rows, head_pad = round_up(m.dim, 16u), value_pad = round_up(m.vdim, 16u);
+        const bool expand = !f32 && positions <= a.expand_keys && head_pad <= kHeadAttentionMaxDim && value_pad <= kHeadAttentionMaxDim
+                            && latent_expansion_pays(rows, m.rank, m.dim, m.vdim);
+        if (!last && expand) {
+            down.problems = 2;
+            down.p[1] = chunk_problem(w.q, normed);
+            down.p[1].output = kChunkHalfRows; down.p[1].out = reinterpret_cast<float*>(a.head_q); down.p[1].out_ld = m.heads * head_pad;
+            down.p[1].segment = m.dim; down.p[1].segment_pad = head_pad; down.p[1].scale = m.scale;
+        } else if (!last) {
             down.problems = 2;
             down.p[1] = chunk_problem(w.q, normed);
             down.p[1].output = kChunkOperand; down.p[1].result = query; down.p[1].segment = m.dim; down.p[1].segment_pad = dim_pad;
@@ -475,32 +505,54 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         ++launches_;
         GF_TRY(launch_chunk_latents(a.raw_latent, m.rank, w.latent_gain, m.rank, s.eps, a.private_rows[l], row_elements, !f32, rows, status_dev_, stream_));
         if (last) break;
-        ChunkProduct absorb;
-        absorb.p[0] = chunk_problem(w.up_key, query);
-        absorb.p[0].count = m.heads; absorb.p[0].a_block_stride = dim_pad / kDenseBlockK;
-        absorb.p[0].output = kChunkLatentQuery; absorb.p[0].out = static_cast<float*>(a.latent_q); absorb.p[0].out_ld = row_elements;
-        absorb.p[0].heads = m.heads; absorb.p[0].scale = m.scale; absorb.p[0].query_f16 = f32 ? 0u : 1u;
-        GF_TRY(run(absorb));
-        LatentAttention attention;
-        attention.q = a.latent_q; attention.rings = p.rings_dev + l; attention.ring_stride = 0;
-        attention.private_rows = a.private_rows[l]; attention.positions = state_dev_;
-        attention.rows = rows; attention.heads = m.heads; attention.row_elements = row_elements; attention.ring_mask = caches_[l].ring_rows - 1u;
-        attention.cache_f32 = f32 ? 1u : 0u; attention.sink = w.sink;
-        attention.partial_out = a.partial_out; attention.partial_ml = a.partial_ml;
-        attention.parts = std::max(1u, std::min(latent_attention_parts(rows, m.heads, position_ + rows, true), a.partial_rows / (rows * m.heads)));
-        const Operand latent_out = operand_view(a.latent_out, m.heads * rank_pad);
-        const bool merge = attention.parts > 1u;
-        LatentAttention merged = attention;
-        merged.result = latent_out; merged.result_stride = rank_pad;
-        ++launches_;
-        GF_TRY(launch_latent_attention(merge ? attention : merged, stream_, false));
-        if (merge) { ++launches_; GF_TRY(launch_latent_merge(merged, stream_)); }
-        const Operand heads_out = operand_view(a.heads_out, m.heads * m.vdim);
-        ChunkProduct value;
-        value.p[0] = chunk_problem(w.up_value, latent_out);
-        value.p[0].count = m.heads; value.p[0].a_block_stride = rank_pad / kDenseBlockK;
-        value.p[0].output = kChunkOperand; value.p[0].result = heads_out; value.p[0].column_stride = m.vdim;
-        GF_TRY(run(value));
+        if (expand) {
+            Operand latents;
+            latents.data = a.latent_rows; latents.capacity = round_up(positions, 16u); latents.k_pad = rank_pad;
+            ++launches_;
+            GF_TRY(launch_latent_operand(p.rings_dev + l, a.private_rows[l], state_dev_, positions, row_elements, caches_[l].ring_rows - 1u, latents, stream_));
+            ChunkProduct expansion;
+            expansion.problems = 2;
+            expansion.p[0] = chunk_problem(w.expand_key, latents);
+            expansion.p[0].output = kChunkHalfRows; expansion.p[0].out = reinterpret_cast<float*>(a.keys); expansion.p[0].out_ld = m.heads * head_pad;
+            expansion.p[0].segment = m.dim; expansion.p[0].segment_pad = head_pad;
+            expansion.p[1] = chunk_problem(w.up_value, latents);
+            expansion.p[1].count = m.heads; expansion.p[1].output = kChunkHalfRows; expansion.p[1].out = reinterpret_cast<float*>(a.values);
+            expansion.p[1].out_ld = m.heads * value_pad; expansion.p[1].column_stride = value_pad;
+            expansion.rows = positions;
+            GF_TRY(run(expansion));
+            HeadAttention attention;
+            attention.q = a.head_q; attention.k = a.keys; attention.v = a.values; attention.position = state_dev_; attention.sink = w.sink;
+            attention.rows = rows; attention.heads = m.heads; attention.dim_pad = head_pad; attention.vdim = m.vdim; attention.vdim_pad = value_pad;
+            attention.result = heads_out;
+            ++launches_;
+            GF_TRY(launch_head_attention(attention, stream_));
+        } else {
+            ChunkProduct absorb;
+            absorb.p[0] = chunk_problem(w.up_key, query);
+            absorb.p[0].count = m.heads; absorb.p[0].a_block_stride = dim_pad / kDenseBlockK;
+            absorb.p[0].output = kChunkLatentQuery; absorb.p[0].out = static_cast<float*>(a.latent_q); absorb.p[0].out_ld = row_elements;
+            absorb.p[0].heads = m.heads; absorb.p[0].scale = m.scale; absorb.p[0].query_f16 = f32 ? 0u : 1u;
+            GF_TRY(run(absorb));
+            LatentAttention attention;
+            attention.q = a.latent_q; attention.rings = p.rings_dev + l; attention.ring_stride = 0;
+            attention.private_rows = a.private_rows[l]; attention.positions = state_dev_;
+            attention.rows = rows; attention.heads = m.heads; attention.row_elements = row_elements; attention.ring_mask = caches_[l].ring_rows - 1u;
+            attention.cache_f32 = f32 ? 1u : 0u; attention.sink = w.sink;
+            attention.partial_out = a.partial_out; attention.partial_ml = a.partial_ml;
+            attention.parts = std::max(1u, std::min(latent_attention_parts(rows, m.heads, position_ + rows, true), a.partial_rows / (rows * m.heads)));
+            const Operand latent_out = operand_view(a.latent_out, m.heads * rank_pad);
+            const bool merge = attention.parts > 1u;
+            LatentAttention merged = attention;
+            merged.result = latent_out; merged.result_stride = rank_pad;
+            ++launches_;
+            GF_TRY(launch_latent_attention(merge ? attention : merged, stream_, false));
+            if (merge) { ++launches_; GF_TRY(launch_latent_merge(merged, stream_)); }
+            ChunkProduct value;
+            value.p[0] = chunk_problem(w.up_value, latent_out);
+            value.p[0].count = m.heads; value.p[0].a_block_stride = rank_pad / kDenseBlockK;
+            value.p[0].output = kChunkOperand; value.p[0].result = heads_out; value.p[0].column_stride = m.vdim;
+            GF_TRY(run(value));
+        }
         ChunkProduct out;
         out.p[0] = chunk_problem(w.o, heads_out);
         out.p[0].out = a.y; out.p[0].out_ld = s.width;

@@ -18,6 +18,7 @@ struct LayeredLayer {
     float *latent_gain = nullptr, *sink = nullptr;
     DenseMatrix q, latent_down, o;
     DenseMatrix up_key, up_value;             // per head: [rank x dim] and [vdim x rank]
+    DenseMatrix expand_key;                   // [heads * dim x rank]: the same weights as up_key for chunks that expand their keys
     DenseMatrix up, down;                     // dense feed-forward
     DenseMatrix expert_up, expert_down;       // per expert, gate and up paired
     DenseMatrix router, shared_up, shared_down, shared_weight;
@@ -60,6 +61,10 @@ struct LayeredPlan {
         float *residual = nullptr, *raw_latent = nullptr, *y = nullptr, *shared_y = nullptr, *group_y = nullptr, *router_logits = nullptr, *shared_logit = nullptr;
         float *final_rows = nullptr, *partial_out = nullptr, *partial_ml = nullptr, *slot_scores = nullptr, *row_scale = nullptr;
         void* latent_q = nullptr;
+        // Keys and values of a chunk that expands its latents (16-bit plans): up to expand_keys positions.
+        uint32_t expand_keys = 0;
+        void *latent_rows = nullptr;          // a bf16 operand of that many rows
+        __half *keys = nullptr, *values = nullptr, *head_q = nullptr;
         uint32_t *group_start = nullptr, *group_rows = nullptr, *slot_rows = nullptr, *slot_experts = nullptr, *tokens = nullptr, *wanted = nullptr;
         std::vector<void*> private_rows;
         KvPublishLayer* publish_layers = nullptr;

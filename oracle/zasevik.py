@@ -72,6 +72,12 @@ def route(h, router, top):
     return chosen, np.take_along_axis(scores, chosen, axis=-1)
 
 
+def routing_margin(h, router, top):
+    """How far the router's logits are from choosing other experts, per token."""
+    z = -np.sort(-(h @ router.T), axis=-1)
+    return z[:, top - 1] - z[:, top] if top < z.shape[1] else np.full(z.shape[0], np.inf)
+
+
 def mixture(h, weights, prefix, spec):
     chosen, scores = route(h, weights[prefix + ".router"], spec["router"]["top"])
     limit = spec["expert"]["limit"]
@@ -99,12 +105,13 @@ class Reference:
         self.latents = [None] * len(self.config["layers"])
         self.position = 0
         self.residuals = []
+        self.margins = np.zeros(0)             # per token seen: the closest routing decision of any layer
 
     def extend(self, tokens):
         """Logits of every token of the portion; self.residuals holds the stream behind each layer."""
         c, w, eps = self.config, self.w, self.config["norm"]["eps"]
         x = w["embed"][np.asarray(tokens)] * c["embedding"]["scale"]
-        self.residuals = []
+        self.residuals, margins = [], np.full(len(tokens), np.inf)
         for i, layer in enumerate(c["layers"]):
             p, m = f"l{i}", layer["mixer"]
             h = centred_rms_norm(x, w[p + ".norm1"], eps)
@@ -118,8 +125,10 @@ class Reference:
                 if layer["mlp"]["kind"] == "dense":
                     y = dense_feed_forward(h, w[p + ".mlp.up"], w[p + ".mlp.down"])
                 else:
+                    margins = np.minimum(margins, routing_margin(h, w[p + ".mlp.router"], layer["mlp"]["router"]["top"]))
                     y = mixture(h, w, p + ".mlp", layer["mlp"])
                 x = x + centred_rms_norm(y, w[p + ".norm2b"], eps) * w[p + ".ls2"]
             self.residuals.append(x)
         self.position += len(tokens)
+        self.margins = np.concatenate([self.margins, margins])
         return centred_rms_norm(x, w["final.norm"], eps) @ w["embed"].T

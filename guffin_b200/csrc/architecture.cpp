@@ -35,8 +35,8 @@ struct ConfigReader {
     }
 };
 
-// ---- Zasevik: latent attention without positions in every layer, dense or routed feed-forward layers, norms
-// before and after each sublayer with layer scales, tied embedding.
+// ---- Zasevik: every layer attends cached latents (no rotation), its feed-forward is dense, routed or absent; each
+// sublayer has a pre-norm, a post-norm and a per-channel scale; the token table is also the output head.
 
 bool read_mixer(ConfigReader& r, const Json* layer, const std::string& path, MixerSpec& out) {
     const Json* type = r.member(layer, path, "type", Json::kString);

@@ -370,7 +370,9 @@ uint32_t latent_attention_parts(uint32_t rows, uint32_t heads, uint32_t position
     const uint32_t queries = chain ? rows * heads : heads, wide = queries > 16u ? 64u : 16u;
     const uint32_t blocks = (queries + wide - 1u) / wide * (chain ? 1u : rows);
     const uint32_t tiles = (positions + kKeys - 1u) / kKeys;
-    return std::max(1u, std::min(std::min(tiles, kLatentMaxParts), (uint32_t)sm_count() / std::max(1u, blocks)));
+    // Every partition is read again by the merge: more than 64 only where each has many tiles.
+    const uint32_t most = std::min(kLatentMaxParts, std::max(64u, tiles / 8u));
+    return std::max(1u, std::min(std::min(tiles, most), (uint32_t)sm_count() / std::max(1u, blocks)));
 }
 
 int launch_latent_attention(LatentAttention p, cudaStream_t stream, bool pdl) {

@@ -6,7 +6,7 @@
 
 namespace gf {
 
-constexpr uint32_t kLatentMaxParts = 64;
+constexpr uint32_t kLatentMaxParts = 128;
 
 // Elements of a cache row: the rank rounded up so that a row is whole 32-byte pieces.
 __host__ __device__ inline uint32_t latent_row_elements(uint32_t rank) { return (rank + 15u) / 16u * 16u; }

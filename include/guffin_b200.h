@@ -343,7 +343,7 @@ GF_API int gf_model_load_gguf(gf_model* model, const char* path, uint32_t* out_b
  * as keys and values.  q_dev holds the scaled queries already in latent space, [rows * heads][rank rounded up to 16];
  * ring_dev [ring_rows][..] the committed rows, private_dev [rows][..] the pass's own; binary16, or f32 with precision
  * GF_PRECISION_F32.  The rows follow position *position_dev as a chain.  sink_dev (may be NULL): a logit per head in the
- * denominator.  out_dev f32 [rows * heads][rank rounded up to 16].  parts = partitions of the keys, 1..64.
+ * denominator.  out_dev f32 [rows * heads][rank rounded up to 16].  parts = partitions of the keys, 1..128.
  * gf_route: the `top` largest sigmoid scores of every row, lower index first among equals. ---- */
 GF_API size_t gf_dense_packed_bytes(uint32_t k, uint32_t n);
 GF_API int gf_dense_pack(const uint16_t* bf16_dev, uint32_t k, uint32_t n, void* packed_dev, void* stream);

@@ -8,12 +8,22 @@ from __future__ import annotations
 import numpy as np
 
 
+def exact(x):
+    return x
+
+
+def bf16(x):
+    """Rounded to bfloat16 (nearest even), in the precision it came in."""
+    bits = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    return ((bits + 0x7fff + ((bits >> 16) & 1)) & np.uint32(0xffff0000)).view(np.float32).astype(np.asarray(x).dtype)
+
+
 def rms_norm(x, gain, eps):
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * gain
 
 
 def centred_rms_norm(x, weight, eps):
-    """The weight is stored around zero."""
+    """The gain is one plus the stored weight."""
     return rms_norm(x, 1.0 + weight, eps)
 
 
@@ -42,27 +52,27 @@ def latent(h, down, gain, eps):
     return rms_norm(h @ down.T, gain, eps)
 
 
-def latent_attention(q, c, first, heads, up_k, up_v, sink, scale):
+def latent_attention(q, c, first, heads, up_k, up_v, sink, scale, cast=exact):
     """q [T, heads * dim] at positions first.., c [S, rank] every latent from position 0 on; returns [T, heads * vdim]."""
     T, S = q.shape[0], c.shape[0]
     dim, vdim = q.shape[1] // heads, up_v.shape[0] // heads
-    k = (c @ up_k.T).reshape(S, heads, dim)
-    v = (c @ up_v.T).reshape(S, heads, vdim)
-    q = q.reshape(T, heads, dim)
+    k = cast(c @ up_k.T).reshape(S, heads, dim)
+    v = cast(c @ up_v.T).reshape(S, heads, vdim)
+    q = cast(q).reshape(T, heads, dim)
     seen = np.arange(S)[None, :] <= first + np.arange(T)[:, None]
     out = np.empty((T, heads, vdim), q.dtype)
     for n in range(heads):
         scores = np.where(seen, (q[:, n] @ k[:, n].T) * scale, -np.inf)
-        out[:, n] = softmax_with_sink(scores, sink[n]) @ v[:, n]
+        out[:, n] = cast(softmax_with_sink(scores, sink[n])) @ v[:, n]
     return out.reshape(T, heads * vdim)
 
 
-def dense_feed_forward(h, up, down):
-    return squared_relu(h @ up.T) @ down.T
+def dense_feed_forward(h, up, down, cast=exact):
+    return cast(squared_relu(h @ up.T)) @ down.T
 
 
-def expert(h, gate, up, down, limit):
-    return clamped_gate(h @ gate.T, h @ up.T, limit) @ down.T
+def expert(h, gate, up, down, limit, cast=exact):
+    return cast(clamped_gate(h @ gate.T, h @ up.T, limit)) @ down.T
 
 
 def route(h, router, top):
@@ -72,32 +82,27 @@ def route(h, router, top):
     return chosen, np.take_along_axis(scores, chosen, axis=-1)
 
 
-def routing_margin(h, router, top):
-    """How far the router's logits are from choosing other experts, per token."""
-    z = -np.sort(-(h @ router.T), axis=-1)
-    return z[:, top - 1] - z[:, top] if top < z.shape[1] else np.full(z.shape[0], np.inf)
-
-
-def mixture(h, weights, prefix, spec):
+def mixture(h, weights, prefix, spec, cast=exact):
     chosen, scores = route(h, weights[prefix + ".router"], spec["router"]["top"])
     limit = spec["expert"]["limit"]
     out = np.zeros((h.shape[0], h.shape[1]), h.dtype)
     for t in range(h.shape[0]):
         for e, s in zip(chosen[t], scores[t]):
             p = f"{prefix}.e{e}"
-            out[t] += expert(s * h[t:t + 1], weights[p + ".gate"], weights[p + ".up"], weights[p + ".down"], limit)[0]
+            out[t] += expert(s * h[t:t + 1], weights[p + ".gate"], weights[p + ".up"], weights[p + ".down"], limit, cast)[0]
     if spec.get("shared"):
         p = prefix + ".shared"
-        y = expert(h, weights[p + ".gate"], weights[p + ".up"], weights[p + ".down"], spec["shared"]["limit"])
+        y = expert(h, weights[p + ".gate"], weights[p + ".up"], weights[p + ".down"], spec["shared"]["limit"], cast)
         out += sigmoid(h @ weights[p + ".sg"].T) * y
     return out
 
 
 class Reference:
-    """A whole model fed in portions; keeps every latent it has seen."""
+    """A whole model fed in portions; keeps every latent it has seen.  `cast` is applied to what enters a matrix product
+    or the cache: with bf16 it shows what rounding alone does."""
 
-    def __init__(self, config, weights, dtype=np.float64):
-        self.config = config
+    def __init__(self, config, weights, dtype=np.float64, cast=exact):
+        self.config, self.cast = config, cast
         self.w = {k: np.asarray(v, dtype) for k, v in weights.items()}
         self.reset()
 
@@ -105,30 +110,27 @@ class Reference:
         self.latents = [None] * len(self.config["layers"])
         self.position = 0
         self.residuals = []
-        self.margins = np.zeros(0)             # per token seen: the closest routing decision of any layer
 
     def extend(self, tokens):
         """Logits of every token of the portion; self.residuals holds the stream behind each layer."""
-        c, w, eps = self.config, self.w, self.config["norm"]["eps"]
+        c, w, eps, cast = self.config, self.w, self.config["norm"]["eps"], self.cast
         x = w["embed"][np.asarray(tokens)] * c["embedding"]["scale"]
-        self.residuals, margins = [], np.full(len(tokens), np.inf)
+        self.residuals = []
         for i, layer in enumerate(c["layers"]):
             p, m = f"l{i}", layer["mixer"]
-            h = centred_rms_norm(x, w[p + ".norm1"], eps)
-            new = latent(h, w[p + ".mix.dkv"], w[p + ".mix.dkv.norm"], eps)
+            h = cast(centred_rms_norm(x, w[p + ".norm1"], eps))
+            new = cast(latent(h, w[p + ".mix.dkv"], w[p + ".mix.dkv.norm"], eps))
             self.latents[i] = new if self.latents[i] is None else np.concatenate([self.latents[i], new])
-            y = latent_attention(h @ w[p + ".mix.q"].T, self.latents[i], self.position, m["heads"], w[p + ".mix.uk"],
-                                 w[p + ".mix.uv"], w[p + ".mix.sink"], m["scale"]) @ w[p + ".mix.o"].T
+            y = cast(latent_attention(h @ w[p + ".mix.q"].T, self.latents[i], self.position, m["heads"], w[p + ".mix.uk"],
+                                      w[p + ".mix.uv"], w[p + ".mix.sink"], m["scale"], cast)) @ w[p + ".mix.o"].T
             x = x + centred_rms_norm(y, w[p + ".norm1b"], eps) * w[p + ".ls1"]
             if layer.get("mlp"):
-                h = centred_rms_norm(x, w[p + ".norm2"], eps)
+                h = cast(centred_rms_norm(x, w[p + ".norm2"], eps))
                 if layer["mlp"]["kind"] == "dense":
-                    y = dense_feed_forward(h, w[p + ".mlp.up"], w[p + ".mlp.down"])
+                    y = dense_feed_forward(h, w[p + ".mlp.up"], w[p + ".mlp.down"], cast)
                 else:
-                    margins = np.minimum(margins, routing_margin(h, w[p + ".mlp.router"], layer["mlp"]["router"]["top"]))
-                    y = mixture(h, w, p + ".mlp", layer["mlp"])
+                    y = mixture(h, w, p + ".mlp", layer["mlp"], cast)
                 x = x + centred_rms_norm(y, w[p + ".norm2b"], eps) * w[p + ".ls2"]
             self.residuals.append(x)
         self.position += len(tokens)
-        self.margins = np.concatenate([self.margins, margins])
-        return centred_rms_norm(x, w["final.norm"], eps) @ w["embed"].T
+        return cast(centred_rms_norm(x, w["final.norm"], eps)) @ w["embed"].T

@@ -291,19 +291,24 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
             const uint32_t m = r * p.heads + batch, parts = p.attention_parts;
             if (warp == 0) merge_factors(p.latent_ml + (size_t)m * parts * 2u, parts, p.sink ? p.sink[batch] : -INFINITY, route_scratch);
             __syncthreads();
+            // Two halves of the block take the even and the odd partitions, a thread four dimensions at a time.
             const float* rows_in = p.in + (size_t)m * parts * p.latent_ld;
-            for (uint32_t i = tid * 2u; i < k_pad; i += kRowThreads * 2u) {
-                float2 v = make_float2(0.0f, 0.0f);
+            const uint32_t odd = tid / (kRowThreads / 2u), first = (tid % (kRowThreads / 2u)) * 4u;
+            for (uint32_t i0 = 0; i0 < k_pad; i0 += kRowThreads * 2u) {
+                const uint32_t i = i0 + first;
+                float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
                 if (i < p.latent_ld) {
 #pragma unroll 8
-                    for (uint32_t part = 0; part < parts; ++part) {
-                        const float2 o = *reinterpret_cast<const float2*>(rows_in + (size_t)part * p.latent_ld + i);
+                    for (uint32_t part = odd; part < parts; part += 2u) {
+                        const float4 o = *reinterpret_cast<const float4*>(rows_in + (size_t)part * p.latent_ld + i);
                         const float f = route_scratch[part];
-                        v.x = fmaf(o.x, f, v.x); v.y = fmaf(o.y, f, v.y);
+                        v.x = fmaf(o.x, f, v.x); v.y = fmaf(o.y, f, v.y); v.z = fmaf(o.z, f, v.z); v.w = fmaf(o.w, f, v.w);
                     }
                 }
-                act[r * k_pad + i] = v.x;
-                act[r * k_pad + i + 1u] = v.y;
+                float4* dst = reinterpret_cast<float4*>(act + r * k_pad + i);
+                if (odd && i < k_pad) *dst = v;
+                __syncthreads();
+                if (!odd && i < k_pad) *dst = add4(*dst, v);
             }
             __syncthreads();
         }
@@ -456,7 +461,6 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
         widest = std::max(widest, m.sets);
         k_max = std::max(k_max, m.k);
     }
-    p.sets = sets;
     p.k_pad = (k_max + 31u) / 32u * 32u;
     if ((p.input == kRowNorm || p.input == kRowAddNorm) && k_max != p.width) return fail(GF_ERR_INVALID, "row product: a normalised input has the matrices' K");
     auto whole = [](const void* pointer) { return (reinterpret_cast<uintptr_t>(pointer) & 15u) == 0u; };

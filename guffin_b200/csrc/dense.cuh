@@ -111,7 +111,7 @@ struct RowProduct {
     uint32_t latent_row_elements = 0, latent_f16 = 0;
     uint32_t* status = nullptr;
     // filled by the launcher
-    uint32_t k_pad = 0, sets = 0, vector_rows = 0;
+    uint32_t k_pad = 0, vector_rows = 0;
 };
 // Any number of rows; launches as many kernels as the rows need (`launches` is increased by their number).
 int launch_row_product(RowProduct product, cudaStream_t stream, bool pdl, uint32_t& launches);
@@ -162,7 +162,7 @@ struct ChunkProblem {
 struct ChunkProduct {
     ChunkProblem p[3];
     uint32_t problems = 1, rows = 0;
-    uint32_t window = 0, total_tiles = 0, stage_budget = 0;      // filled by the launcher
+    uint32_t window = 0, stage_budget = 0;      // filled by the launcher
     int* error_flag = nullptr;
 };
 int launch_chunk_product(ChunkProduct product, bool f32, cudaStream_t stream);

@@ -447,7 +447,6 @@ int launch_chunk_product(ChunkProduct p, bool f32, cudaStream_t stream) {
         m.tiles = (m.n + tile_columns - 1u) / tile_columns;
         total += m.tiles * m.count;
     }
-    p.total_tiles = total;
     if (f32) {
         p.window = 64u;
         chunk_product_f32_kernel<<<dim3(total, (p.rows + 63u) / 64u), 256, 0, stream>>>(p);

@@ -9,7 +9,9 @@ namespace gf {
 namespace {
 
 constexpr uint32_t kKeys = 64;                       // cache rows per tile
+constexpr uint32_t kNarrowKeys = 32;                 // of the kernel for up to sixteen queries
 constexpr uint32_t kThreads = 256;
+constexpr uint32_t kSmemLimit = 226u * 1024u;
 
 __device__ __forceinline__ void copy16(void* dst_smem, const void* src, bool valid) {      // zero-fills when not valid
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst_smem)), "l"(src), "r"(valid ? 16u : 0u) : "memory");
@@ -30,32 +32,35 @@ __device__ __forceinline__ void mma_f16(float (&d)[4], const uint32_t (&a)[4], u
 }
 
 struct LatentSmem { uint32_t q, cache, scores, weights, stats, bytes; };
-__host__ __device__ inline LatentSmem latent_smem(uint32_t queries, uint32_t row_elements) {
+template <int MT>
+__host__ __device__ inline LatentSmem latent_smem(uint32_t row_elements) {
+    constexpr uint32_t queries = 16u * MT, keys = MT == 1 ? kNarrowKeys : kKeys, slots = MT == 1 ? 4u : 2u, planes = MT == 1 ? 2u : 1u;
     const uint32_t stride = (row_elements + 8u) * 2u;
     LatentSmem s;
     s.q = 0;
     s.cache = queries * stride;
-    s.scores = s.cache + 2u * kKeys * stride;
-    s.weights = s.scores + queries * (kKeys + 4u) * 4u;
-    s.stats = s.weights + queries * (kKeys + 8u) * 2u;
+    s.scores = s.cache + slots * keys * stride;
+    s.weights = s.scores + planes * queries * (keys + 4u) * 4u;
+    s.stats = s.weights + queries * (keys + 8u) * 2u;
     s.bytes = s.stats + queries * 3u * 4u;
     return s;
 }
 
 // A block serves 16 * MT queries -- (row, head) pairs in order, heads fastest -- against one partition of the cache
-// rows they see.  Per tile of 64 rows: scores on the tensor cores (the eight warps split the tile's keys and, for
-// MT = 4, the queries), an online softmax over shared-memory scores, then the outputs, warp w accumulating the
-// dimension groups w, w + 8, .. of sixteen.  The next tile's rows are copied meanwhile.
+// rows they see.  Per tile of cache rows: scores on the tensor cores, an online softmax over shared-memory scores, then
+// the outputs, warp w accumulating the dimension groups w, w + 8, .. of sixteen; later tiles' rows are copied meanwhile.
+// MT = 4 (prompts): tiles of 64 rows, the eight warps split the queries and the tile's rows.  MT = 1 (decoding, bound
+// by the cache): tiles of 32 rows, three of them in flight, the warps split the rows and the dimensions of a score.
 template <int MT, int NP>
 __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __grid_constant__ LatentAttention p) {
     extern __shared__ __align__(16) uint8_t smem[];
-    constexpr uint32_t kQueries = 16u * MT;
-    const LatentSmem at = latent_smem(kQueries, p.row_elements);
+    constexpr uint32_t kQueries = 16u * MT, kTile = MT == 1 ? kNarrowKeys : kKeys, kSlots = MT == 1 ? 4u : 2u;
+    const LatentSmem at = latent_smem<MT>(p.row_elements);
     const uint32_t stride = p.row_elements + 8u;                     // halves; rows land in different banks
     __half* q_tile = reinterpret_cast<__half*>(smem + at.q);
     __half* cache_tiles = reinterpret_cast<__half*>(smem + at.cache);
-    float* scores = reinterpret_cast<float*>(smem + at.scores);      // [queries][kKeys + 4]
-    __half* weights = reinterpret_cast<__half*>(smem + at.weights);  // [queries][kKeys + 8]
+    float* scores = reinterpret_cast<float*>(smem + at.scores);      // [queries][kTile + 4], two of them for MT = 1
+    __half* weights = reinterpret_cast<__half*>(smem + at.weights);  // [queries][kTile + 8]
     float* run_max = reinterpret_cast<float*>(smem + at.stats);
     float* run_sum = run_max + kQueries;
     float* correction = run_sum + kQueries;
@@ -73,27 +78,30 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
     const uint32_t out_query = chain ? 0u : z * p.heads;
     const uint32_t last_query = min(first_query + kQueries, queries) - 1u;
     const uint32_t end = base + last_query / p.heads + 1u;           // cache rows the block's last query sees
-    const uint32_t tiles = (end + kKeys - 1u) / kKeys;
+    const uint32_t tiles = (end + kTile - 1u) / kTile;
     const uint32_t tile_begin = (uint32_t)((uint64_t)tiles * part / p.parts), tile_end = (uint32_t)((uint64_t)tiles * (part + 1u) / p.parts);
 
     const uint32_t pieces = p.row_elements / 8u;
     auto load_tile = [&](uint32_t tile, uint32_t slot) {
-        __half* dst = cache_tiles + (size_t)slot * kKeys * stride;
-        for (uint32_t i = tid; i < kKeys * pieces; i += kThreads) {
-            const uint32_t r = i / pieces, piece = i % pieces, position = tile * kKeys + r;
-            const bool valid = position < end;
-            const __half* src = !valid ? own : position < base ? ring + (size_t)(position & p.ring_mask) * p.row_elements
-                                                              : own + (size_t)(position - base) * p.row_elements;
-            copy16(dst + r * stride + piece * 8u, src + piece * 8u, valid);
-        }
+        constexpr uint32_t kPerRow = kThreads / kTile;                // threads that share a row, alternating pieces
+        const uint32_t r = tid / kPerRow, position = tile * kTile + r;
+        const bool valid = position < end;
+        const __half* src = !valid ? own : position < base ? ring + (size_t)(position & p.ring_mask) * p.row_elements
+                                                          : own + (size_t)(position - base) * p.row_elements;
+        __half* dst = cache_tiles + (size_t)slot * kTile * stride + r * stride;
+#pragma unroll 4
+        for (uint32_t piece = tid % kPerRow; piece < pieces; piece += kPerRow) copy16(dst + piece * 8u, src + piece * 8u, valid);
     };
     for (uint32_t i = tid; i < kQueries * pieces; i += kThreads) {
         const uint32_t m = i / pieces, piece = i % pieces;
         const bool valid = first_query + m < queries;
         copy16(q_tile + m * stride + piece * 8u, q + (size_t)(valid ? first_query + m : 0u) * p.row_elements + piece * 8u, valid);
     }
-    if (tile_begin < tile_end) load_tile(tile_begin, 0u);
-    copies_commit();
+#pragma unroll
+    for (uint32_t i = 0; i + 1u < kSlots; ++i) {                      // one copy group per tile, the queries with the first
+        if (tile_begin + i < tile_end) load_tile(tile_begin + i, i);
+        copies_commit();
+    }
     for (uint32_t m = tid; m < kQueries; m += kThreads) { run_max[m] = -INFINITY; run_sum[m] = 0.0f; correction[m] = 1.0f; }
 
     float acc[MT][NP][2][4];
@@ -108,18 +116,20 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
 
     const uint32_t steps = p.row_elements / 16u;
     for (uint32_t tile = tile_begin; tile < tile_end; ++tile) {
-        const uint32_t slot = (tile - tile_begin) & 1u;
-        if (tile + 1u < tile_end) load_tile(tile + 1u, slot ^ 1u);
+        const uint32_t slot = (tile - tile_begin) % kSlots;
+        if (tile + kSlots - 1u < tile_end) load_tile(tile + kSlots - 1u, (slot + kSlots - 1u) % kSlots);
         copies_commit();
-        copies_wait<1>();
+        copies_wait<(int)kSlots - 1>();
         __syncthreads();
-        const __half* cache = cache_tiles + (size_t)slot * kKeys * stride;
-        // ---- scores: MT = 4: two query tiles x sixteen keys per warp; MT = 1: one query tile x eight keys.
+        const __half* cache = cache_tiles + (size_t)slot * kTile * stride;
+        // ---- scores: MT = 4: two query tiles x sixteen keys per warp; MT = 1: sixteen queries x eight keys x half of the
+        // dimensions.
         if (MT == 4) {
             const uint32_t m0 = (warp & 1u) * 32u, n0 = (warp >> 1) * 16u;
             float s[2][2][4] = {};
             const __half* a_row = q_tile + (m0 + (lane & 15u)) * stride + (lane >> 4) * 8u;
             const __half* b_row = cache + (n0 + (lane & 7u) + (lane >> 4) * 8u) * stride + ((lane >> 3) & 1u) * 8u;
+#pragma unroll 4
             for (uint32_t k = 0; k < steps; ++k) {
                 uint32_t a0[4], a1[4], b[4];
                 ldmatrix4(a0, a_row + k * 16u);
@@ -134,17 +144,18 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
             for (int a = 0; a < 2; ++a)
 #pragma unroll
                 for (int b = 0; b < 2; ++b) {
-                    float* out = scores + (m0 + 16u * a + g) * (kKeys + 4u) + n0 + 8u * b + 2u * t;
+                    float* out = scores + (m0 + 16u * a + g) * (kTile + 4u) + n0 + 8u * b + 2u * t;
                     *reinterpret_cast<float2*>(out) = make_float2(s[a][b][0], s[a][b][1]);
-                    *reinterpret_cast<float2*>(out + 8u * (kKeys + 4u)) = make_float2(s[a][b][2], s[a][b][3]);
+                    *reinterpret_cast<float2*>(out + 8u * (kTile + 4u)) = make_float2(s[a][b][2], s[a][b][3]);
                 }
         } else {
-            const uint32_t n0 = warp * 8u;
+            const uint32_t n0 = (warp & 3u) * 8u, half = warp >> 2, k_end = steps * (half + 1u) / 2u;
             float s[2][4] = {};
             const __half* a_row = q_tile + (lane & 15u) * stride + (lane >> 4) * 8u;
             const __half* b_row = cache + (n0 + (lane & 7u)) * stride + (lane >> 3) * 8u;      // 32 dimensions of eight keys
-            uint32_t k = 0;
-            for (; k + 2u <= steps; k += 2u) {
+            uint32_t k = steps * half / 2u;
+#pragma unroll 4
+            for (; k + 2u <= k_end; k += 2u) {
                 uint32_t a0[4], a1[4], b[4];
                 ldmatrix4(a0, a_row + k * 16u);
                 ldmatrix4(a1, a_row + k * 16u + 16u);
@@ -152,28 +163,29 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
                 mma_f16(s[0], a0, b[0], b[1]);
                 mma_f16(s[1], a1, b[2], b[3]);
             }
-            if (k < steps) {
+            if (k < k_end) {
                 uint32_t a0[4], b[4];
                 ldmatrix4(a0, a_row + k * 16u);
                 ldmatrix4(b, cache + (n0 + (lane & 7u)) * stride + ((lane >> 3) & 1u) * 8u + k * 16u);
                 mma_f16(s[0], a0, b[0], b[1]);
             }
-            float* out = scores + g * (kKeys + 4u) + n0 + 2u * t;
+            float* out = scores + (half * kQueries + g) * (kTile + 4u) + n0 + 2u * t;
             *reinterpret_cast<float2*>(out) = make_float2(s[0][0] + s[1][0], s[0][1] + s[1][1]);
-            *reinterpret_cast<float2*>(out + 8u * (kKeys + 4u)) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
+            *reinterpret_cast<float2*>(out + 8u * (kTile + 4u)) = make_float2(s[0][2] + s[1][2], s[0][3] + s[1][3]);
         }
         __syncthreads();
         // ---- softmax: 16 / MT threads per query.
         {
-            constexpr uint32_t kPer = kThreads / kQueries, kEach = kKeys / kPer;
+            constexpr uint32_t kPer = kThreads / kQueries, kEach = kTile / kPer;
             const uint32_t m = tid / kPer, sub = tid % kPer;
             const uint32_t sees = base + min(first_query + m, queries - 1u) / p.heads;      // last visible position
-            const float* row = scores + m * (kKeys + 4u);
+            const float* row = scores + m * (kTile + 4u);
             float v[kEach], top = -INFINITY;
 #pragma unroll
             for (uint32_t j = 0; j < kEach; ++j) {
                 const uint32_t key = j * kPer + sub;
-                v[j] = tile * kKeys + key <= sees ? row[key] : -INFINITY;
+                const float score = MT == 1 ? row[key] + row[kQueries * (kTile + 4u) + key] : row[key];
+                v[j] = tile * kTile + key <= sees ? score : -INFINITY;
                 top = fmaxf(top, v[j]);
             }
 #pragma unroll
@@ -184,7 +196,7 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
             for (uint32_t j = 0; j < kEach; ++j) {
                 const float w = v[j] == -INFINITY ? 0.0f : expf(v[j] - now);
                 sum += w;
-                weights[m * (kKeys + 8u) + j * kPer + sub] = __float2half_rn(w);
+                weights[m * (kTile + 8u) + j * kPer + sub] = __float2half_rn(w);
             }
 #pragma unroll
             for (uint32_t o = kPer / 2u; o > 0u; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
@@ -207,10 +219,10 @@ __global__ void __launch_bounds__(kThreads, 1) latent_attention_kernel(const __g
                 for (int c = 0; c < 2; ++c) { acc[a][b][c][0] *= c0; acc[a][b][c][1] *= c0; acc[a][b][c][2] *= c1; acc[a][b][c][3] *= c1; }
         }
 #pragma unroll
-        for (uint32_t k = 0; k < kKeys / 16u; ++k) {
+        for (uint32_t k = 0; k < kTile / 16u; ++k) {
             uint32_t w[MT][4];
 #pragma unroll
-            for (int a = 0; a < MT; ++a) ldmatrix4(w[a], weights + (16u * a + (lane & 15u)) * (kKeys + 8u) + k * 16u + (lane >> 4) * 8u);
+            for (int a = 0; a < MT; ++a) ldmatrix4(w[a], weights + (16u * a + (lane & 15u)) * (kTile + 8u) + k * 16u + (lane >> 4) * 8u);
 #pragma unroll
             for (int b = 0; b < NP; ++b) {
                 const uint32_t d0 = (b * 8u + warp) * 16u;
@@ -354,12 +366,12 @@ template <int MT, int NP>
 int launch_tensor(const LatentAttention& p, cudaStream_t stream, bool pdl) {
     constexpr uint32_t kQueries = 16u * MT;
     static std::once_flag once[64];
-    const int status = allow_smem(latent_attention_kernel<MT, NP>, once, 226u * 1024u);
+    const int status = allow_smem(latent_attention_kernel<MT, NP>, once, kSmemLimit);
     if (status != GF_OK) return status;
     const bool chain = p.ring_stride == 0u;
     const uint32_t queries = chain ? p.rows * p.heads : p.heads;
     return launch_kernel(latent_attention_kernel<MT, NP>, dim3((queries + kQueries - 1u) / kQueries, p.parts, chain ? 1u : p.rows), dim3(kThreads),
-                         latent_smem(kQueries, p.row_elements).bytes, stream, pdl, p);
+                         latent_smem<MT>(p.row_elements).bytes, stream, pdl, p);
 }
 
 }  // namespace
@@ -369,9 +381,9 @@ bool latent_attention_on_tensor_cores(const LatentAttention& p) { return !p.cach
 uint32_t latent_attention_parts(uint32_t rows, uint32_t heads, uint32_t positions, bool chain) {
     const uint32_t queries = chain ? rows * heads : heads, wide = queries > 16u ? 64u : 16u;
     const uint32_t blocks = (queries + wide - 1u) / wide * (chain ? 1u : rows);
-    const uint32_t tiles = (positions + kKeys - 1u) / kKeys;
-    // Every partition is read again by the merge: more than 64 only where each has many tiles.
-    const uint32_t most = std::min(kLatentMaxParts, std::max(64u, tiles / 8u));
+    const uint32_t keys = wide > 16u ? kKeys : kNarrowKeys, tiles = (positions + keys - 1u) / keys;
+    // Every partition is read again by the merge: more than 64 only where each has several tiles.
+    const uint32_t most = std::min(kLatentMaxParts, std::max(64u, tiles / 4u));
     return std::max(1u, std::min(std::min(tiles, most), (uint32_t)sm_count() / std::max(1u, blocks)));
 }
 

@@ -248,6 +248,21 @@ def test_portions_of_every_size(gm, name, precision):
         assert at == 200 and within(np.concatenate(rows), want, limits), cuts
 
 
+@pytest.mark.parametrize("name", ["sharp attention", "experts"])
+@pytest.mark.parametrize("precision", PRECISIONS)
+def test_prompts_longer_than_a_chunk(gm, name, precision):
+    """The second chunk of a long prompt sees the first one's cache rows; only some logits are wanted."""
+    config, bits, weights = make(gm, name)
+    tokens = tokens_for(config, 1100, 5)
+    want, limits = plain(config, weights, tokens, precision)
+    places = [0, 1, 511, 1022, 1023, 1024, 1025, 1060, 1099]
+    plan = gm.Model.described(config, bits, 1100, 8, precision)
+    assert within(plan.extend(tokens, places), want[places], limits[places])
+    plan.reset()
+    plan.extend(tokens[:1090])
+    assert within(plan.extend(tokens[1090:], [0, 9]), want[[1090, 1099]], limits[[1090, 1099]])
+
+
 @pytest.mark.parametrize("precision", PRECISIONS)
 def test_decoding_behind_a_prompt(gm, precision):
     """Token by token for longer than the prompt, through the captured passes, up to the last position of the context."""

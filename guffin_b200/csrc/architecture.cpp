@@ -29,10 +29,11 @@ struct ConfigReader {
         }
         return (uint32_t)v->number;
     }
-    float real(const Json* from, const std::string& path, const char* key) {
+    double number(const Json* from, const std::string& path, const char* key) {
         const Json* v = member(from, path, key, Json::kNumber);
-        return v ? (float)v->number : 0.0f;
+        return v ? v->number : 0.0;
     }
+    float real(const Json* from, const std::string& path, const char* key) { return (float)number(from, path, key); }
 };
 
 // ---- Zasevik: every layer attends cached latents (no rotation), its feed-forward is dense, routed or absent; each
@@ -86,7 +87,7 @@ bool read_feed_forward(ConfigReader& r, const Json* layer, const std::string& pa
 
 void list_tensors(const LayeredSpec& s, std::vector<TensorSlot>& out) {
     auto add = [&](const std::string& name, TensorRole role, uint32_t layer, uint32_t index, uint32_t rows, uint32_t columns) {
-        out.push_back(TensorSlot{name, role, layer, index, rows, columns});
+        out.push_back(TensorSlot{name, role, layer, index, rows, columns, false});
     };
     add("embed", TensorRole::kEmbedding, 0, 0, s.vocab, s.width);
     add("final.norm", TensorRole::kFinalNorm, 0, 0, 0, s.width);
@@ -129,6 +130,24 @@ void list_tensors(const LayeredSpec& s, std::vector<TensorSlot>& out) {
     }
 }
 
+// Follows every layer's source to the layer that has the tensors, which must be a layer of the same shape.
+void resolve_sources(ConfigReader& r, LayeredSpec& s) {
+    for (uint32_t l = 0; l < s.layers.size(); ++l) {
+        uint32_t at = s.layers[l].source;
+        for (size_t steps = 0; s.layers[at].source != at; at = s.layers[at].source)
+            if (++steps > s.layers.size()) { r.complain("layers[" + std::to_string(l) + "].weights_of", "leads round in a circle"); return; }
+        const MixerSpec &a = s.layers[l].mixer, &b = s.layers[at].mixer;
+        const FeedForwardSpec &f = s.layers[l].mlp, &g = s.layers[at].mlp;
+        if (a.kind != b.kind || a.heads != b.heads || a.dim != b.dim || a.vdim != b.vdim || a.kv_heads != b.kv_heads || a.rank != b.rank || a.state != b.state
+            || a.groups != b.groups || a.taps != b.taps || a.norm_parts != b.norm_parts || f.kind != g.kind || f.ff != g.ff)
+            r.complain("layers[" + std::to_string(l) + "].weights_of", "names a layer of another shape");
+    }
+    std::vector<uint32_t> owners(s.layers.size());
+    for (uint32_t l = 0; l < s.layers.size(); ++l)
+        for (owners[l] = l; s.layers[owners[l]].source != owners[l];) owners[l] = s.layers[owners[l]].source;
+    for (uint32_t l = 0; l < s.layers.size(); ++l) s.layers[l].source = owners[l];
+}
+
 void describe_zasevik(ConfigReader& r, const Json& config, ArchitectureDescription& out) {
     LayeredSpec& s = out.spec;
     out.layered = true;
@@ -143,10 +162,122 @@ void describe_zasevik(ConfigReader& r, const Json& config, ArchitectureDescripti
     for (size_t i = 0; i < layers->items.size(); ++i) {
         LayerSpec layer;
         const std::string path = "layers[" + std::to_string(i) + "].";
+        layer.source = (uint32_t)i;
         if (!read_mixer(r, &layers->items[i], path, layer.mixer) || !read_feed_forward(r, &layers->items[i], path, layer.mlp)) return;
         s.layers.push_back(layer);
     }
     list_tensors(s, out.tensors);
+}
+
+// ---- Tufirax: layers of grouped-query attention (rotated, capped scores, sinks, a gate per head, values that are the
+// projected keys) and of state-space mixers, dense gated feed-forward layers or none; sublayers read the residual stream
+// itself and are normalised behind; layers may use another layer's tensors; the output head is a matrix of its own.
+
+void read_grouped_attention(ConfigReader& r, const Json* m, const std::string& at, MixerSpec& out) {
+    out.kind = MixerKind::kGroupedAttention;
+    out.heads = r.count(m, at, "heads", 1, 4096);
+    out.kv_heads = r.count(m, at, "kv_heads", 1, 4096);
+    out.dim = r.count(m, at, "dim", 1, 4096);
+    out.vdim = r.count(m, at, "vdim", 1, 4096);
+    out.scale = r.real(m, at, "scale");
+    out.softcap = r.real(m, at, "softcap");
+    out.sink = out.head_gate = true;
+    const Json* rotation = r.member(m, at, "rot", Json::kObject);
+    out.rotated = r.count(rotation, at + "rot.", "dims", 0, 4096);
+    out.rotation_base = r.number(rotation, at + "rot.", "base");
+    if (!r.ok()) return;
+    if (out.heads % out.kv_heads) r.complain(at + "kv_heads", "does not divide heads");
+    if (out.vdim != out.dim) r.complain(at + "vdim", "differs from dim, but the values are the keys");
+    if (out.rotated % 2u || out.rotated > out.dim) r.complain(at + "rot.dims", "must be even and at most dim");
+    if (out.rotated && !(out.rotation_base > 0.0)) r.complain(at + "rot.base", "must be positive");
+    if (!(out.softcap > 0.0f)) r.complain(at + "softcap", "must be positive");
+}
+
+void read_state_space(ConfigReader& r, const Json* m, const std::string& at, MixerSpec& out) {
+    out.kind = MixerKind::kStateSpace;
+    out.heads = r.count(m, at, "heads", 1, 4096);
+    out.vdim = r.count(m, at, "vdim", 1, 4096);
+    out.state = r.count(m, at, "state", 1, 1024);
+    out.groups = r.count(m, at, "groups", 1, 4096);
+    out.taps = r.count(m, at, "conv", 1, 256);
+    out.norm_parts = r.count(m, at, "norm_groups", 1, 1024);
+    if (!r.ok()) return;
+    if (out.heads % out.groups) r.complain(at + "groups", "does not divide heads");
+    if (out.inner() % out.norm_parts) r.complain(at + "norm_groups", "does not divide heads * vdim");
+}
+
+void list_tufirax_tensors(const LayeredSpec& s, std::vector<TensorSlot>& out) {
+    auto add = [&](const std::string& name, TensorRole role, uint32_t layer, uint32_t rows, uint32_t columns, bool table = false) {
+        out.push_back(TensorSlot{name, role, layer, 0, rows, columns, table});
+    };
+    add("embed", TensorRole::kEmbedding, 0, s.vocab, s.width);
+    add("head", TensorRole::kHead, 0, s.vocab, s.width);
+    add("final.norm", TensorRole::kFinalNorm, 0, 0, s.width);
+    for (uint32_t l = 0; l < s.layers.size(); ++l) {
+        if (s.layers[l].source != l) continue;
+        const MixerSpec& m = s.layers[l].mixer;
+        const FeedForwardSpec& f = s.layers[l].mlp;
+        const std::string p = "l" + std::to_string(l) + ".";
+        add(p + "norm1", TensorRole::kNorm1b, l, 0, s.width);
+        if (m.kind == MixerKind::kGroupedAttention) {
+            add(p + "mix.q", TensorRole::kQuery, l, m.heads * m.dim, s.width);
+            add(p + "mix.k", TensorRole::kKey, l, m.kv_heads * m.dim, s.width);
+            add(p + "mix.q.norm", TensorRole::kQueryNorm, l, 0, m.heads * m.dim);
+            add(p + "mix.k.norm", TensorRole::kKeyNorm, l, 0, m.kv_heads * m.dim);
+            add(p + "mix.sink", TensorRole::kSink, l, 0, m.heads);
+            add(p + "mix.g", TensorRole::kHeadGate, l, m.heads, s.width);
+        } else {
+            add(p + "mix.in", TensorRole::kStateIn, l, m.state_inputs(), s.width);
+            add(p + "mix.conv", TensorRole::kTaps, l, m.channels(), m.taps, true);
+            add(p + "mix.conv.b", TensorRole::kTapBias, l, 0, m.channels());
+            add(p + "mix.dt_bias", TensorRole::kStepBias, l, 0, m.heads);
+            add(p + "mix.A_log", TensorRole::kDecayLog, l, 0, m.heads);
+            add(p + "mix.D", TensorRole::kSkip, l, 0, m.heads);
+            add(p + "mix.norm", TensorRole::kMixerNorm, l, 0, m.inner());
+        }
+        add(p + "mix.o", TensorRole::kMixerOut, l, s.width, m.inner());
+        if (f.kind == FeedForwardSpec::kNone) continue;
+        add(p + "norm2", TensorRole::kNorm2b, l, 0, s.width);
+        add(p + "mlp.gate", TensorRole::kGate, l, f.ff, s.width);
+        add(p + "mlp.up", TensorRole::kUp, l, f.ff, s.width);
+        add(p + "mlp.down", TensorRole::kDown, l, s.width, f.ff);
+    }
+}
+
+void describe_tufirax(ConfigReader& r, const Json& config, ArchitectureDescription& out) {
+    LayeredSpec& s = out.spec;
+    out.layered = true;
+    s.width = r.count(&config, "", "width", 1, 1u << 20);
+    s.vocab = r.count(&config, "", "vocab");
+    s.eps = r.real(r.member(&config, "", "norm", Json::kObject), "norm.", "eps");
+    s.pre_norm = s.tied_head = false;
+    const Json* layers = r.member(&config, "", "layers", Json::kArray);
+    if (!layers) return;
+    if (layers->items.empty()) { r.complain("layers", "is empty"); return; }
+    for (size_t i = 0; i < layers->items.size(); ++i) {
+        const Json* entry = &layers->items[i];
+        const std::string path = "layers[" + std::to_string(i) + "].";
+        LayerSpec layer;
+        layer.source = (uint32_t)i;
+        if (entry->find("weights_of") && !entry->find("weights_of")->is_null()) layer.source = r.count(entry, path, "weights_of", 0, (uint32_t)layers->items.size() - 1u);
+        const Json* type = r.member(entry, path, "type", Json::kString);
+        const Json* m = r.member(entry, path, "mixer", Json::kObject);
+        if (!r.ok()) return;
+        if (type->text == "attention") read_grouped_attention(r, m, path + "mixer.", layer.mixer);
+        else if (type->text == "mamba2") read_state_space(r, m, path + "mixer.", layer.mixer);
+        else r.complain(path + "type", ("names the unknown mixer '" + type->text + "'").c_str());
+        if (const Json* f = r.member(entry, path, "mlp", Json::kObject, false)) {
+            const Json* kind = r.member(f, path + "mlp.", "kind", Json::kString);
+            if (kind && kind->text != "dense") r.complain(path + "mlp.kind", ("names the unknown feed-forward '" + kind->text + "'").c_str());
+            layer.mlp.kind = FeedForwardSpec::kDense;
+            layer.mlp.activation = Activation::kGeluGate;
+            layer.mlp.ff = r.count(f, path + "mlp.", "ff");
+        }
+        if (!r.ok()) return;
+        s.layers.push_back(layer);
+    }
+    resolve_sources(r, s);
+    if (r.ok()) list_tufirax_tensors(s, out.tensors);
 }
 
 // ---- the quantised Gemma families: the fields of gf_model_config under their own names (weights in model.gguf).
@@ -168,6 +299,7 @@ struct Architecture { const char* name; void (*describe)(ConfigReader&, const Js
 const Architecture kArchitectures[] = {
     {"Gemma2", describe_gemma},
     {"Gemma3", describe_gemma},
+    {"Tufirax", describe_tufirax},
     {"Zasevik", describe_zasevik},
 };
 

@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
         for (uint32_t j = 0; j < kNormQuads; ++j) {
             const uint32_t i = (j * kRowThreads + tid) * 4u;
             if (i >= p.width) continue;
-            early_gain1[j] = *reinterpret_cast<const float4*>(p.gain1 + i);
+            if (p.gain1) early_gain1[j] = *reinterpret_cast<const float4*>(p.gain1 + i);
             if (p.input == kRowAddNorm) {
                 early_residual[j] = *reinterpret_cast<const float4*>(p.residual + i);
                 early_gain0[j] = *reinterpret_cast<const float4*>(p.gain0 + i);
@@ -227,14 +227,20 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
                 if (writer && p.residual_out) *reinterpret_cast<float4*>(p.residual_out + i) = v[j];
                 sum[0] += dot4(v[j], v[j]);
             }
-            block_sums<1>(sum, scratch);
-            inv = norm_factor(sum[0], p.width, p.eps);
+            if (p.gain1) {
+                block_sums<1>(sum, scratch);
+                inv = norm_factor(sum[0], p.width, p.eps);
+            }
         }
 #pragma unroll
         for (uint32_t j = 0; j < kNormQuads; ++j) {
             const uint32_t i = (j * kRowThreads + tid) * 4u;
             if (i >= p.width) continue;
-            const float4 g = early_gain1[j], n = make_float4(v[j].x * inv * g.x, v[j].y * inv * g.y, v[j].z * inv * g.z, v[j].w * inv * g.w);
+            float4 n = v[j];
+            if (p.gain1) {
+                const float4 g = early_gain1[j];
+                n = make_float4(n.x * inv * g.x, n.y * inv * g.y, n.z * inv * g.z, n.w * inv * g.w);
+            }
             *reinterpret_cast<float4*>(act + i) = n;
             if (writer && p.normed_out) *reinterpret_cast<float4*>(p.normed_out + i) = n;
         }
@@ -271,20 +277,50 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
                     next[r] = fmaf(v, v, next[r]);
                 }
             }
-            block_sums<R>(next, scratch);
+            if (p.gain1) block_sums<R>(next, scratch);
 #pragma unroll
             for (int r = 0; r < R; ++r) sum[r] = next[r];
         }
 #pragma unroll
-        for (int r = 0; r < R; ++r) sum[r] = norm_factor(sum[r], p.width, p.eps);
+        for (int r = 0; r < R; ++r) sum[r] = p.gain1 ? norm_factor(sum[r], p.width, p.eps) : 1.0f;
         for (uint32_t i = tid; i < k_pad; i += kRowThreads) {
-            const float gain = i < p.width ? p.gain1[i] : 0.0f;
+            const float gain = i >= p.width ? 0.0f : p.gain1 ? p.gain1[i] : 1.0f;
 #pragma unroll
             for (int r = 0; r < R; ++r) {
                 const float v = i < p.width ? act[r * k_pad + i] * sum[r] * gain : 0.0f;
                 act[r * k_pad + i] = v;
                 if (writer && p.normed_out && i < p.width) p.normed_out[(size_t)r * p.width + i] = v;
             }
+        }
+    } else if (p.input == kRowPartNorm) {
+        // Warps share the parts: several to a part where there are fewer parts than warps.
+        const uint32_t part = p.width / p.norm_parts;
+        uint32_t per = kRowWarps;
+        while (per > 1u && per * p.norm_parts > kRowWarps) per /= 2u;
+        for (int r = 0; r < R; ++r) {
+            const float* x = p.in + (size_t)r * p.in_ld;
+            for (uint32_t unit = warp; unit < per * p.norm_parts; unit += kRowWarps) {
+                const uint32_t first = unit / per * part;
+                float sum = 0.0f;
+                for (uint32_t i = (unit % per) * 32u + lane; i < part; i += per * 32u) {
+                    const float v = x[first + i];
+                    act[r * k_pad + first + i] = v;
+                    sum = fmaf(v, v, sum);
+                }
+                sum = warp_sum(sum);
+                if (lane == 0) route_scratch[unit] = sum;
+            }
+            __syncthreads();
+            for (uint32_t i = tid; i < k_pad; i += kRowThreads) {
+                float v = 0.0f;
+                if (i < p.width) {
+                    float sum = 0.0f;
+                    for (uint32_t s = 0; s < per; ++s) sum += route_scratch[i / part * per + s];
+                    v = act[r * k_pad + i] * norm_factor(sum, part, p.eps) * p.gain1[i];
+                }
+                act[r * k_pad + i] = v;
+            }
+            __syncthreads();
         }
     } else if (p.input == kRowLatent) {
         for (int r = 0; r < R; ++r) {
@@ -375,7 +411,7 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
         if (set < set_end) { locate(set); prefetch(); }            // the next set's loads overlap the hand-over
         __syncthreads();
         // ---- K slices summed in order, then the output
-        const bool paired = m.output == kOutClampedGate;
+        const bool paired = paired_output(m.output);
         const uint32_t outputs = m.groups_per_cta * 8u / (paired ? 2u : 1u);
         for (uint32_t i = tid; i < outputs * R; i += kRowThreads) {
             const uint32_t column = i % outputs, r = i / outputs;
@@ -390,7 +426,8 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
                 if (n >= m.n / 2u) continue;
                 const float score = p.input == kRowRouted ? route_score : 1.0f;
                 const uint32_t pair = column >> 3;
-                const float v = clamped_gate(sum_group(2u * pair) * score, sum_group(2u * pair + 1u) * score, m.limit);
+                const float gate = sum_group(2u * pair) * score, up = sum_group(2u * pair + 1u) * score;
+                const float v = m.output == kOutGeluGate ? gelu_tanh(gate) * up : clamped_gate(gate, up, m.limit);
                 static_cast<float*>(m.out)[(size_t)r * m.out_ld + (size_t)batch * m.out_batch + n] = v;
                 continue;
             }
@@ -448,7 +485,7 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
         if (!m.weight || !m.out || m.k == 0 || m.n == 0) return fail(GF_ERR_INVALID, "row product: bad matrix");
         m.k_blocks = (m.k + kDenseBlockK - 1u) / kDenseBlockK;
         const uint32_t groups = (m.n + 7u) / 8u, batches = single ? 4u : p.batches;
-        uint32_t per = m.output == kOutClampedGate ? 2u : 1u;
+        uint32_t per = paired_output(m.output) ? 2u : 1u;
         while (per < kRowWarps && (uint64_t)(groups + per - 1u) / per * batches > wanted) per *= 2u;
         // A warp's slice of K should not fall below two of its 512-byte loads.
         while (per < kRowWarps && (m.k + 31u) / 32u < 2u * (kRowWarps / per)) per *= 2u;
@@ -462,7 +499,8 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
         k_max = std::max(k_max, m.k);
     }
     p.k_pad = (k_max + 31u) / 32u * 32u;
-    if ((p.input == kRowNorm || p.input == kRowAddNorm) && k_max != p.width) return fail(GF_ERR_INVALID, "row product: a normalised input has the matrices' K");
+    if ((p.input == kRowNorm || p.input == kRowAddNorm || p.input == kRowPartNorm) && k_max != p.width) return fail(GF_ERR_INVALID, "row product: a normalised input has the matrices' K");
+    if (p.input == kRowPartNorm && (p.norm_parts == 0 || p.norm_parts > kMaxNormParts || p.width % p.norm_parts)) return fail(GF_ERR_INVALID, "row product: %u norm parts of %u", p.norm_parts, p.width);
     auto whole = [](const void* pointer) { return (reinterpret_cast<uintptr_t>(pointer) & 15u) == 0u; };
     p.vector_rows = p.in_ld % 4u == 0u && p.in_batch % 4u == 0u && p.in2_ld % 4u == 0u && p.part_stride % 4u == 0u && whole(p.in) && whole(p.in2);
     if (p.input == kRowNorm || p.input == kRowAddNorm)

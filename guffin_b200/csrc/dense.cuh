@@ -55,17 +55,20 @@ constexpr uint32_t kMaxExperts = 1024;
 enum RowInput : uint32_t {
     kRowPlain = 0,        // in[row * in_ld + batch * in_batch + k]
     kRowNorm = 1,         // rmsnorm(in) * gain1
-    kRowAddNorm = 2,      // residual + rmsnorm(sum of the parts of in) * gain0 -> residual_out; rmsnorm(that) * gain1
+    kRowAddNorm = 2,      // residual + rmsnorm(sum of the parts of in) * gain0 -> residual_out; rmsnorm(that) * gain1 (that alone without gain1)
     kRowLatent = 3,       // batch = head: merge of the attention partitions of (row, head)
     kRowRouted = 4,       // batch = row * top + slot: row `batch / top` of in, plain; the product is multiplied by the slot's score
     kRowExperts = 5,      // batch < rows * top: in[batch * in_ld + k]; the batches behind them: row `batch - rows * top` of in2
+    kRowPartNorm = 6,     // rmsnorm(in) * gain1, every one of norm_parts equal parts of the row by its own root mean square
 };
 enum RowOutput : uint32_t {
     kOutF32 = 0,          // out[row * ld + batch * out_batch + n]
     kOutSquaredRelu = 1,
     kOutClampedGate = 2,  // paired matrix: n halves
     kOutLatentQuery = 3,  // out[(row * heads + batch) * ld + n] = product * scale, f16 or f32
+    kOutGeluGate = 4,     // paired matrix: gelu(gate) * up
 };
+__host__ __device__ inline bool paired_output(uint32_t output) { return output == kOutClampedGate || output == kOutGeluGate; }
 
 struct RowMatrix {
     const uint8_t* weight = nullptr;
@@ -86,7 +89,7 @@ struct RowProduct {
     uint32_t in_ld = 0, in_batch = 0;
     const uint32_t* in_rows = nullptr;  // kRowPlain: optional row indices
     // norms
-    uint32_t width = 0, parts = 1;
+    uint32_t width = 0, parts = 1, norm_parts = 1;
     size_t part_stride = 0;             // floats between parts
     const float *residual = nullptr, *gain0 = nullptr, *gain1 = nullptr;
     float *residual_out = nullptr, *normed_out = nullptr;
@@ -135,7 +138,10 @@ enum ChunkOutput : uint32_t {
     kChunkClampedGate = 3,    // paired matrix: operand(row, n) = clamped gate of (gate, up) * row scale
     kChunkLatentQuery = 4,    // out[(row * heads + index) * out_ld + n] = product * scale, f16 or f32
     kChunkHalfRows = 5,       // f16 out[row * out_ld + column(n)] = product * scale
+    kChunkGeluGate = 6,       // paired matrix: operand(row, n) = gelu(gate) * up
 };
+__host__ __device__ inline bool paired_chunk(uint32_t output) { return output == kChunkClampedGate || output == kChunkGeluGate; }
+constexpr uint32_t kMaxNormParts = 1024;           // of kRowPartNorm and launch_chunk_part_norm
 
 // `count` products of the same shape: heads of one matrix, or experts.
 struct ChunkProblem {
@@ -170,8 +176,8 @@ int launch_chunk_product(ChunkProduct product, bool f32, cudaStream_t stream);
 int launch_chunk_operand(const float* x, uint32_t rows, uint32_t k, const Operand& result, cudaStream_t stream);
 
 // Rows of a chunk between products: residual + rmsnorm(y) * gain0 -> residual (in place), rmsnorm(that) * gain1 ->
-// operand and / or f32 rows.  y null: only the second norm.  y is [row][width], or with `slots` set the sum over a
-// token's slots of y[slot_rows[row * slots + slot]] and of shared[row].
+// operand and / or f32 rows.  y null: only the second norm.  gain1 null: the residual itself instead of its norm.  y is
+// [row][width], or with `slots` set the sum over a token's slots of y[slot_rows[row * slots + slot]] and of shared[row].
 struct ChunkNorm {
     float* residual = nullptr;
     const float *y = nullptr, *shared = nullptr, *gain0 = nullptr, *gain1 = nullptr;
@@ -182,6 +188,9 @@ struct ChunkNorm {
     float* normed = nullptr;
 };
 int launch_chunk_norm(const ChunkNorm& norm, cudaStream_t stream);
+// rmsnorm(x * silu(gate)) * gain into an operand, every one of `parts` equal parts of a row by its own root mean square.
+int launch_chunk_part_norm(const float* x, uint32_t x_ld, const float* gate, uint32_t gate_ld, uint32_t width, uint32_t parts, const float* gain, float eps, const Operand& result, uint32_t rows,
+                           cudaStream_t stream);
 
 // Routing of a chunk: rows grouped by expert.  Expert e's rows are [start[e], start[e] + count[e]) of the grouped
 // operand, every start a multiple of eight; slot_rows maps (token, slot) to its grouped row.
@@ -220,6 +229,8 @@ __device__ __forceinline__ float clamped_gate(float gate, float up, float limit)
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return g * sigmoid(1.702f * g) * (u + 1.0f);
 }
+__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
 // One warp turns the (maximum, sum) pairs of a query's key partitions, and its sink, into the factors of the merge.
 __device__ __forceinline__ void merge_factors(const float* ml, uint32_t parts, float sink, float* factors) {
     const uint32_t lane = threadIdx.x & 31u;

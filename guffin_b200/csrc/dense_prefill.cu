@@ -35,9 +35,12 @@ __device__ __forceinline__ void chunk_store(const ChunkProblem& p, uint32_t inde
     }
 }
 // Column n of a paired product.
+__device__ __forceinline__ float chunk_gate(const ChunkProblem& p, float gate, float up) {
+    return p.output == kChunkGeluGate ? gelu_tanh(gate) * up : clamped_gate(gate, up, p.limit);
+}
 __device__ __forceinline__ void chunk_store_gate(const ChunkProblem& p, uint32_t row, uint32_t n, float gate, float up) {
     const float s = p.row_scale ? p.row_scale[(size_t)row * p.row_scale_ld] : 1.0f;
-    store_operand(p.result, row, n, clamped_gate(gate * s, up * s, p.limit));
+    store_operand(p.result, row, n, chunk_gate(p, gate * s, up * s));
 }
 
 __device__ __forceinline__ uint4 bf16_octet(const float (&v)[8]) {
@@ -198,7 +201,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
             tc_fence_before_sync();
         }
         __syncthreads();
-        const bool paired = m.output == kChunkClampedGate;
+        const bool paired = paired_chunk(m.output);
         const uint32_t octets = paired ? 8u : 16u, count = min(64u, live - c0) * octets;
 #pragma unroll 1
         for (uint32_t i = tid; i < count; i += kChunkThreads) {
@@ -216,7 +219,7 @@ __global__ void __launch_bounds__(kChunkThreads, 1) chunk_product_kernel(const _
             if (n >= m.n / 2u) continue;
             const float s = m.row_scale ? m.row_scale[(size_t)row * m.row_scale_ld] : 1.0f;
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = clamped_gate(v[j] * s, src[8 + j] * s, m.limit);
+            for (int j = 0; j < 8; ++j) v[j] = chunk_gate(m, v[j] * s, src[8 + j] * s);
             *reinterpret_cast<uint4*>(static_cast<uint8_t*>(m.result.data) + operand_offset(m.result, row, n)) = bf16_octet(v);
         }
         __syncthreads();
@@ -276,7 +279,7 @@ __global__ void __launch_bounds__(256) chunk_product_f32_kernel(const __grid_con
     for (int i = 0; i < 4; ++i) {
         const uint32_t r = ty * 4u + i;
         if (r >= live) continue;
-        if (m.output == kChunkClampedGate) {
+        if (paired_chunk(m.output)) {
             for (int j = 0; j < 4; j += 2) {
                 const uint32_t n = tile * 32u + (columns[j] >> 4) * 8u + (columns[j] & 7u);
                 if (n < m.n / 2u) chunk_store_gate(m, row0 + r, n, acc[i][j], acc[i][j + 1]);
@@ -333,13 +336,29 @@ __global__ void __launch_bounds__(256) chunk_norm_kernel(const ChunkNorm p) {
             sum = fmaf(v, v, sum);
         }
     }
-    if (!p.gain1) return;
-    const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps);
+    const float inv = p.gain1 ? 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps) : 1.0f;
     for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
-        const float v = row_values[i] * inv * p.gain1[i];
+        const float v = p.gain1 ? row_values[i] * inv * p.gain1[i] : row_values[i];
         if (p.result.data) store_operand(p.result, row, i, v);
         if (p.normed) p.normed[(size_t)row * p.width + i] = v;
     }
+}
+
+// Block = (row, part): the part by its own root mean square.
+__global__ void __launch_bounds__(256) chunk_part_norm_kernel(const float* __restrict__ x, uint32_t x_ld, const float* __restrict__ gate, uint32_t gate_ld, uint32_t part, const float* __restrict__ gain, float eps,
+                                                              const Operand result) {
+    extern __shared__ float row_values[];
+    __shared__ float scratch[8];
+    const uint32_t row = blockIdx.x, first = blockIdx.y * part;
+    const float *in = x + (size_t)row * x_ld + first, *z = gate + (size_t)row * gate_ld + first;
+    float sum = 0.0f;
+    for (uint32_t i = threadIdx.x; i < part; i += blockDim.x) {
+        const float v = in[i] * silu(z[i]);
+        row_values[i] = v;
+        sum = fmaf(v, v, sum);
+    }
+    const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)part + eps);
+    for (uint32_t i = threadIdx.x; i < part; i += blockDim.x) store_operand(result, row, first + i, row_values[i] * inv * gain[first + i]);
 }
 
 // A warp per row chooses its experts.
@@ -471,6 +490,20 @@ int launch_chunk_norm(const ChunkNorm& p, cudaStream_t stream) {
     const int status = allow_smem(chunk_norm_kernel, once, 200u * 1024u);
     if (status != GF_OK) return status;
     chunk_norm_kernel<<<p.rows, 256, p.width * 4u, stream>>>(p);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+int launch_chunk_part_norm(const float* x, uint32_t x_ld, const float* gate, uint32_t gate_ld, uint32_t width, uint32_t parts, const float* gain, float eps, const Operand& result, uint32_t rows,
+                           cudaStream_t stream) {
+    if (!x || !gate || !gain || !result.data || rows == 0 || rows > result.capacity || parts == 0 || parts > kMaxNormParts || width % parts || width > result.k_pad
+        || width / parts > 48u * 1024u)
+        return fail(GF_ERR_INVALID, "chunk part norm: bad arguments");
+    const uint32_t part = width / parts;
+    static std::once_flag once[64];
+    const int status = allow_smem(chunk_part_norm_kernel, once, 200u * 1024u);
+    if (status != GF_OK) return status;
+    chunk_part_norm_kernel<<<dim3(rows, parts), part >= 256u ? 256u : (part + 31u) / 32u * 32u, part * 4u, stream>>>(x, x_ld, gate, gate_ld, part, gain, eps, result);
     GF_CUDA(cudaGetLastError());
     return GF_OK;
 }

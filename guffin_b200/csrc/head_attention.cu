@@ -1,5 +1,5 @@
-// Causal attention of a prompt chunk over expanded keys and values (see latent.cuh): every head has keys and values
-// of its own, one row per position from 0 on, binary16.
+// Causal attention of a prompt chunk over keys and values per head or per group of heads, binary16 (see latent.cuh).
+#include "grouped.cuh"
 #include "latent.cuh"
 
 #include <mutex>
@@ -33,7 +33,8 @@ __device__ __forceinline__ uint32_t half_pair(float lo, float hi) {
 
 // Block = (64 chunk rows, head).  Tiles of 64 keys and values, the next one copied while this one is used; a warp's
 // scores, weights and outputs stay in its registers.  G = groups of sixteen dimensions a head has at most.
-template <int G>
+// kCap: capped scores.
+template <int G, bool kCap>
 __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_constant__ HeadAttention p) {
     extern __shared__ __align__(16) uint8_t smem[];
     const uint32_t q_stride = p.dim_pad + 8u, v_stride = p.vdim_pad + 8u;
@@ -44,9 +45,17 @@ __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_c
     const uint32_t head = blockIdx.y, first_row = (gridDim.x - 1u - blockIdx.x) * kRows;      // the longest blocks first
     const uint32_t base = *p.position, end = base + min(first_row + kRows, p.rows), tiles = (end + kKeys - 1u) / kKeys;
     const __half* q = p.q + (size_t)head * p.dim_pad;
-    const __half* keys = p.k + (size_t)head * p.dim_pad;
-    const __half* values = p.v + (size_t)head * p.vdim_pad;
-    const size_t k_ld = (size_t)p.heads * p.dim_pad, v_ld = (size_t)p.heads * p.vdim_pad;
+    const uint32_t kv = head / (p.heads / p.kv_heads);
+    const __half* keys = p.k + (size_t)kv * p.dim_pad;
+    const __half* values = p.v + (size_t)kv * p.vdim_pad;
+    const size_t q_ld = (size_t)p.heads * p.dim_pad, k_ld = (size_t)p.kv_heads * p.dim_pad, v_ld = (size_t)p.kv_heads * p.vdim_pad;
+    // Keys before the chunk lie in the rings, or ahead of the chunk's own where there are none.
+    const uint32_t own_from = p.rings ? base : 0u;
+    const __half *ring_k = nullptr, *ring_v = nullptr;
+    if (p.rings) {
+        ring_k = static_cast<const __half*>(p.rings->ring_k) + (size_t)kv * p.dim_pad;
+        ring_v = static_cast<const __half*>(p.rings->ring_v) + (size_t)kv * p.vdim_pad;
+    }
     const uint32_t k_pieces = p.dim_pad / 8u, v_pieces = p.vdim_pad / 8u;
 
     auto load_tile = [&](uint32_t tile, uint32_t slot) {
@@ -54,16 +63,17 @@ __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_c
         __half* vd = v_tiles + slot * kKeys * v_stride;
         // Two threads per key, alternating pieces.
         const uint32_t r = tid >> 1, position = tile * kKeys + r;
-        const bool valid = position < end;
-        const __half* ks = keys + (valid ? position : 0u) * k_ld;
-        const __half* vs = values + (valid ? position : 0u) * v_ld;
+        const bool valid = position < end, cached = position < own_from;
+        const size_t at = !valid ? 0u : cached ? position & p.ring_mask : position - own_from;
+        const __half* ks = (cached ? ring_k : keys) + at * k_ld;
+        const __half* vs = (cached ? ring_v : values) + at * v_ld;
         for (uint32_t piece = tid & 1u; piece < k_pieces; piece += 2u) copy16(kd + r * q_stride + piece * 8u, ks + piece * 8u, valid);
         for (uint32_t piece = tid & 1u; piece < v_pieces; piece += 2u) copy16(vd + r * v_stride + piece * 8u, vs + piece * 8u, valid);
     };
     {
         const uint32_t r = tid >> 1, row = first_row + r;
         const bool valid = row < p.rows;
-        const __half* src = q + (valid ? row : 0u) * k_ld;
+        const __half* src = q + (valid ? row : 0u) * q_ld;
         for (uint32_t piece = tid & 1u; piece < k_pieces; piece += 2u) copy16(q_tile + r * q_stride + piece * 8u, src + piece * 8u, valid);
     }
     load_tile(0u, 0u);
@@ -78,6 +88,7 @@ __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_c
     const uint32_t sees[2] = {base + first_row + warp * 16u + g, base + first_row + warp * 16u + g + 8u};      // last visible position
     const __half* a_row = q_tile + (warp * 16u + (lane & 15u)) * q_stride + (lane >> 4) * 8u;
     constexpr float kLog2e = 1.4426950408889634f;
+    const float inverse_cap = kCap ? 1.0f / p.softcap : 0.0f;
 
     for (uint32_t tile = 0; tile < tiles; ++tile) {
         if (tile + 1u < tiles) load_tile(tile + 1u, (tile + 1u) & 1u);
@@ -111,6 +122,11 @@ __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_c
                 mma_f16(s[2 * n + 1], a, b[2], b[3]);
             }
         }
+        if (kCap)
+#pragma unroll
+            for (int n = 0; n < 8; ++n)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[n][e] = soft_cap(s[n][e], p.softcap, inverse_cap);
         if (tile * kKeys + kKeys > base + first_row + warp * 16u + 1u)      // some key of the tile lies behind some row
 #pragma unroll
             for (int n = 0; n < 8; ++n)
@@ -166,6 +182,7 @@ __global__ void __launch_bounds__(kThreads) head_attention_kernel(const __grid_c
             const float sink = p.sink[head], most = fmaxf(top[i], sink);
             factor = expf(top[i] - most) / (sum[i] * expf(top[i] - most) + expf(sink - most));
         }
+        if (p.gate) factor *= sigmoid(p.gate[(size_t)row * p.heads + head]);
 #pragma unroll
         for (int o = 0; o < 2 * G; ++o) {
             const uint32_t d = o * 8u + 2u * t;
@@ -197,31 +214,36 @@ __global__ void __launch_bounds__(64) latent_operand_kernel(const StreamRings* r
     }
 }
 
-template <int G>
+template <int G, bool kCap>
 int launch_groups(const HeadAttention& p, cudaStream_t stream) {
     const uint32_t smem = (kRows + 2u * kKeys) * (p.dim_pad + 8u) * 2u + 2u * kKeys * (p.vdim_pad + 8u) * 2u;
     static std::once_flag once[64];
     int device = 0;
     cudaGetDevice(&device);
     cudaError_t error = cudaSuccess;
-    std::call_once(once[device & 63], [&] { error = cudaFuncSetAttribute(head_attention_kernel<G>, cudaFuncAttributeMaxDynamicSharedMemorySize, 180 * 1024); });
+    std::call_once(once[device & 63], [&] { error = cudaFuncSetAttribute(head_attention_kernel<G, kCap>, cudaFuncAttributeMaxDynamicSharedMemorySize, 180 * 1024); });
     GF_CUDA(error);
-    head_attention_kernel<G><<<dim3((p.rows + kRows - 1u) / kRows, p.heads), kThreads, smem, stream>>>(p);
+    head_attention_kernel<G, kCap><<<dim3((p.rows + kRows - 1u) / kRows, p.heads), kThreads, smem, stream>>>(p);
     GF_CUDA(cudaGetLastError());
     return GF_OK;
+}
+
+template <bool kCap>
+int launch_by_dim(const HeadAttention& p, cudaStream_t stream) {
+    const uint32_t groups = (p.dim_pad > p.vdim_pad ? p.dim_pad : p.vdim_pad) / 16u;
+    if (groups <= 2u) return launch_groups<2, kCap>(p, stream);
+    if (groups <= 4u) return launch_groups<4, kCap>(p, stream);
+    if (groups <= 8u) return launch_groups<8, kCap>(p, stream);
+    return launch_groups<16, kCap>(p, stream);
 }
 
 }  // namespace
 
 int launch_head_attention(const HeadAttention& p, cudaStream_t stream) {
-    if (!p.q || !p.k || !p.v || !p.position || !p.result.data || p.rows == 0 || p.heads == 0 || p.dim_pad % 16u || p.vdim_pad % 16u || p.dim_pad == 0
+    if (!p.q || !p.k || !p.v || !p.position || !p.result.data || p.rows == 0 || p.heads == 0 || p.kv_heads == 0 || p.heads % p.kv_heads || p.dim_pad % 16u || p.vdim_pad % 16u || p.dim_pad == 0
         || p.vdim_pad == 0 || p.dim_pad > kHeadAttentionMaxDim || p.vdim_pad > kHeadAttentionMaxDim || p.vdim > p.vdim_pad)
         return fail(GF_ERR_INVALID, "head attention: bad arguments");
-    const uint32_t groups = (p.dim_pad > p.vdim_pad ? p.dim_pad : p.vdim_pad) / 16u;
-    if (groups <= 2u) return launch_groups<2>(p, stream);
-    if (groups <= 4u) return launch_groups<4>(p, stream);
-    if (groups <= 8u) return launch_groups<8>(p, stream);
-    return launch_groups<16>(p, stream);
+    return p.softcap > 0.0f ? launch_by_dim<true>(p, stream) : launch_by_dim<false>(p, stream);
 }
 
 int launch_latent_operand(const StreamRings* rings, const void* own, const uint32_t* position, uint32_t positions, uint32_t row_elements, uint32_t ring_mask,

@@ -37,16 +37,21 @@ int launch_latent_attention(LatentAttention p, cudaStream_t stream, bool pdl);
 // Merges partial results (and the sink) into the operand `result`.
 int launch_latent_merge(const LatentAttention& p, cudaStream_t stream);
 
-// ---- the same attention with the latents expanded into keys and values per head: fewer operations once a chunk has
-// many rows for the keys it sees, since a score then costs a head's `dim` instead of the latent's rank.
+// ---- attention of a chunk over keys and values per head.  For latents: the same attention with the latents expanded,
+// fewer operations once a chunk has many rows for the keys it sees, since a score then costs a head's `dim` instead of
+// the latent's rank.  For grouped-query attention: over the cache rows themselves.
 constexpr uint32_t kHeadAttentionMaxDim = 256;
 struct HeadAttention {
     const __half* q = nullptr;           // [rows][heads][dim_pad], scaled
-    const __half* k = nullptr;           // [positions][heads][dim_pad], positions from 0
-    const __half* v = nullptr;           // [positions][heads][vdim_pad]
+    const __half* k = nullptr;           // [positions][kv_heads][dim_pad], positions from 0; with rings: the chunk's own rows
+    const __half* v = nullptr;           // [positions][kv_heads][vdim_pad]
+    const StreamRings* rings = nullptr;  // the rows before the chunk, or null
+    uint32_t ring_mask = 0;
     const uint32_t* position = nullptr;  // of row 0
-    const float* sink = nullptr;
-    uint32_t rows = 0, heads = 0, dim_pad = 0, vdim = 0, vdim_pad = 0;      // pads: multiples of 16
+    const float* sink = nullptr;         // per head, or null
+    const float* gate = nullptr;         // [rows][heads], ahead of the sigmoid, or null
+    float softcap = 0.0f;                // of the scores; 0: none
+    uint32_t rows = 0, heads = 0, kv_heads = 0, dim_pad = 0, vdim = 0, vdim_pad = 0;      // pads: multiples of 16
     Operand result;                      // (row, head * vdim + d), bf16 or f32
 };
 int launch_head_attention(const HeadAttention& p, cudaStream_t stream);

@@ -1,18 +1,29 @@
 // Layered models: weight binding and the schedules of a pass and of a prompt chunk (see layered.cuh).
 //
-// A pass of up to GF_MAX_ROWS rows, per layer (row_product launches unless said otherwise):
+// A pass of up to GF_MAX_ROWS rows, per layer (row_product launches unless said otherwise).  Latent attention:
 //   q, latent     <- prologue: [residual + norm(previous sublayer)]; norm
 //   latent query  <- per head, with the new cache rows stored beside it
 //   attention over the cached latents (split over the keys)
 //   values        <- per head; prologue: merge of the attention partitions and the sink
 //   mixer output
-//   dense:   up (squared relu) <- prologue: residual + norm(mixer); norm          down
+// Grouped-query attention:
+//   q, k, gates of the heads <- the same prologue
+//   norm, rotation and the new cache rows
+//   attention over the cached keys and values (split over the keys; the last block merges, with sink and gate)
+//   mixer output
+// State space:
+//   input projection <- the same prologue
+//   convolution, recurrence, gate
+//   mixer output  <- prologue: norm in parts
+// Feed-forward:
+//   dense:   up (squared relu, or gate and up) <- prologue: residual + norm(mixer); norm          down
 //   mixture: router, shared gate / up <- the same prologue     routed gate / up     routed and shared down
 // A chunk of prompt rows runs the same steps as products over all its rows with small kernels between them.
 #include "layered.cuh"
 #include "model.cuh"
 
 #include <algorithm>
+#include <cmath>
 #include <cstring>
 
 #define GF_TRY(expr) do { const int gf_s_ = (expr); if (gf_s_ != GF_OK) return gf_s_; } while (0)
@@ -55,6 +66,7 @@ Model::Model(const ArchitectureDescription& description, uint32_t context, uint3
     for (const TensorSlot& slot : p.description.tensors) p.slots[slot.name] = &slot;
     config_.hidden = s.width; config_.vocab = s.vocab; config_.layers = (uint32_t)s.layers.size();
     config_.heads = s.layers[0].mixer.heads; config_.kv_heads = 1;
+    p.own_slots = row_capacity + 1u;
     config_.rms_eps = s.eps; config_.kv_f16 = f32 ? 0 : 1; config_.attention_scale = s.layers[0].mixer.scale;
     config_.context = context; config_.row_capacity = row_capacity;
     layers_.resize(config_.layers);
@@ -79,21 +91,21 @@ int Model::set_tensor(const char* name, int dtype, const void* host, const uint6
     if (found == p.slots.end()) return fail(GF_ERR_INVALID, "gf_model_set_tensor: this model has no tensor '%s'", name);
     const TensorSlot& slot = *found->second;
     if (p.bound[name]) return fail(GF_ERR_STATE, "gf_model_set_tensor: tensor '%s' bound twice", name);
-    const bool vector = slot.rows == 0;
+    const bool vector = slot.rows == 0, constants = vector || slot.table;
     if (rank != (vector ? 1u : 2u) || dims[rank - 1u] != slot.columns || (!vector && dims[0] != slot.rows))
         return fail(GF_ERR_INVALID, "gf_model_set_tensor: tensor '%s' should have shape [%s%u]", name,
                     vector ? "" : (std::to_string(slot.rows) + ", ").c_str(), slot.columns);
-    if (vector) {
+    if (constants) {
         if (dtype != GF_BF16 && dtype != GF_F32) return fail(GF_ERR_INVALID, "gf_model_set_tensor: vector '%s' must be bf16 or f32", name);
-        std::vector<float> values(slot.columns);
+        std::vector<float> values(slot.values());
         if (dtype == GF_F32) std::memcpy(values.data(), host, values.size() * 4u);
         else
-            for (uint32_t i = 0; i < slot.columns; ++i) {
+            for (size_t i = 0; i < values.size(); ++i) {
                 const uint32_t bits = (uint32_t)static_cast<const uint16_t*>(host)[i] << 16;
                 std::memcpy(&values[i], &bits, 4u);
             }
         native_weight_bytes_ += values.size() * 4u;
-        p.vectors[name] = std::move(values);
+        p.vectors[{slot.role, slot.layer}] = std::move(values);
         p.bound[name] = true;
         return GF_OK;
     }
@@ -111,7 +123,11 @@ int Model::set_tensor(const char* name, int dtype, const void* host, const uint6
     auto half = [&](uint32_t stored, uint32_t first) { columns = stored; pack.group_step = 2; pack.group_first = first; };
     switch (slot.role) {
         case TensorRole::kEmbedding: dst = &p.table; break;
+        case TensorRole::kHead: dst = &p.output_head; break;
         case TensorRole::kQuery: dst = &l.q; break;
+        case TensorRole::kKey: dst = &l.k; break;
+        case TensorRole::kHeadGate: dst = &l.head_gate; break;
+        case TensorRole::kStateIn: dst = &l.state_in; break;
         case TensorRole::kLatentDown: dst = &l.latent_down; break;
         case TensorRole::kLatentUpKey:        // per head the transposed matrix: latent from query
             dst = &l.up_key; count = m.heads; k = m.dim; columns = m.rank;
@@ -122,7 +138,8 @@ int Model::set_tensor(const char* name, int dtype, const void* host, const uint6
             pack.count = m.heads; pack.n = m.vdim; pack.count_stride = (size_t)m.vdim * m.rank;
             break;
         case TensorRole::kMixerOut: dst = &l.o; break;
-        case TensorRole::kUp: dst = &l.up; break;
+        case TensorRole::kGate: dst = &l.up; half(paired, 0); break;
+        case TensorRole::kUp: dst = &l.up; if (f.activation == Activation::kGeluGate) half(paired, 1); break;
         case TensorRole::kDown: dst = &l.down; break;
         case TensorRole::kExpertGate: dst = &l.expert_up; index = slot.index; count = f.experts; half(paired, 0); break;
         case TensorRole::kExpertUp: dst = &l.expert_up; index = slot.index; count = f.experts; half(paired, 1); break;
@@ -168,32 +185,70 @@ int Model::finalize_layered() {
         GF_CUDA(cudaMemcpy(*out, v.data(), v.size() * 4u, cudaMemcpyHostToDevice));
         return GF_OK;
     };
-    auto gain = [&](const std::string& norm, const std::string& scale, float offset, float** out) -> int {
-        std::vector<float> v = p.vectors[norm];
+    // offset + stored weight, times the layer scale where there is one; tensors the design does not have stay null.
+    auto gain = [&](TensorRole norm, uint32_t l, float offset, float** out, TensorRole scale = TensorRole::kFinalNorm) -> int {
+        const auto found = p.vectors.find({norm, l});
+        if (found == p.vectors.end()) return GF_OK;
+        std::vector<float> v = found->second;
+        const auto scales = p.vectors.find({scale, l});
         for (size_t i = 0; i < v.size(); ++i) {
             v[i] = offset + v[i];
-            if (!scale.empty()) v[i] *= p.vectors[scale][i];
+            if (scale != TensorRole::kFinalNorm && scales != p.vectors.end()) v[i] *= scales->second[i];
         }
         return upload(v, out);
     };
-    GF_TRY(gain("final.norm", "", s.norm_offset, &p.final_gain));
-    uint32_t q_width = 0, latent = 0, row_elements = 0, heads = 0, values = 0, ff = 0, top = 0, experts = 0, expert_ff = 0, shared_ff = 0, query_elements = 0;
+    auto plain = [&](TensorRole role, uint32_t l, float** out) { return gain(role, l, 0.0f, out); };
+    GF_TRY(gain(TensorRole::kFinalNorm, 0, s.norm_offset, &p.final_gain));
+    uint32_t q_width = 0, latent = 0, heads = 0, values = 0, ff = 0, top = 0, experts = 0, expert_ff = 0, shared_ff = 0, query_elements = 0;
+    uint32_t k_width = 0, prepared = 0;
+    size_t partial = 0, partial_pairs = 0;             // elements per row
+    p.frequencies.assign(s.layers.size(), nullptr);
     for (uint32_t l = 0; l < s.layers.size(); ++l) {
         LayeredLayer& w = p.layers[l];
         const MixerSpec& m = s.layers[l].mixer;
         const FeedForwardSpec& f = s.layers[l].mlp;
-        const std::string t = "l" + std::to_string(l) + ".";
-        GF_TRY(gain(t + "norm1", "", s.norm_offset, &w.gain1));
-        GF_TRY(gain(t + "norm1b", t + "ls1", s.norm_offset, &w.gain1b));
-        GF_TRY(gain(t + "mix.dkv.norm", "", 0.0f, &w.latent_gain));
-        if (m.sink) GF_TRY(upload(p.vectors[t + "mix.sink"], &w.sink));
-        q_width = std::max(q_width, m.heads * m.dim); latent = std::max(latent, m.rank); heads = std::max(heads, m.heads);
-        row_elements = std::max(row_elements, latent_row_elements(m.rank)); values = std::max(values, m.heads * m.vdim);
-        query_elements = std::max(query_elements, m.heads * latent_row_elements(m.rank));
+        if (s.layers[l].source == l) {
+            GF_TRY(gain(TensorRole::kNorm1, l, s.norm_offset, &w.gain1));
+            GF_TRY(gain(TensorRole::kNorm1b, l, s.norm_offset, &w.gain1b, TensorRole::kScale1));
+            GF_TRY(gain(TensorRole::kNorm2, l, s.norm_offset, &w.gain2));
+            GF_TRY(gain(TensorRole::kNorm2b, l, s.norm_offset, &w.gain2b, TensorRole::kScale2));
+            GF_TRY(plain(TensorRole::kLatentNorm, l, &w.latent_gain));
+            GF_TRY(plain(TensorRole::kSink, l, &w.sink));
+            GF_TRY(plain(TensorRole::kQueryNorm, l, &w.q_gain));
+            GF_TRY(plain(TensorRole::kKeyNorm, l, &w.k_gain));
+            GF_TRY(plain(TensorRole::kTaps, l, &w.taps));
+            GF_TRY(plain(TensorRole::kTapBias, l, &w.tap_bias));
+            GF_TRY(plain(TensorRole::kStepBias, l, &w.step_bias));
+            GF_TRY(plain(TensorRole::kSkip, l, &w.skip));
+            GF_TRY(plain(TensorRole::kMixerNorm, l, &w.mixer_gain));
+            const auto logs = p.vectors.find({TensorRole::kDecayLog, l});
+            if (logs != p.vectors.end()) {
+                for (float& v : logs->second) v = -std::exp(v);
+                GF_TRY(plain(TensorRole::kDecayLog, l, &w.decay));
+            }
+        }
+        values = std::max(values, m.inner());
+        if (m.kind == MixerKind::kLatentAttention) {
+            const size_t row_elements = latent_row_elements(m.rank);
+            q_width = std::max(q_width, m.heads * m.dim); latent = std::max(latent, m.rank);
+            query_elements = std::max(query_elements, m.heads * latent_row_elements(m.rank));
+            partial = std::max(partial, m.heads * kLatentMaxParts * row_elements);
+            partial_pairs = std::max<size_t>(partial_pairs, m.heads * kLatentMaxParts * 2u);
+        } else if (m.kind == MixerKind::kGroupedAttention) {
+            const uint32_t row_head = grouped_row_head(m.dim, m.vdim);
+            q_width = std::max(q_width, m.heads * m.dim); k_width = std::max(k_width, m.kv_heads * m.dim); heads = std::max(heads, m.heads);
+            prepared = std::max(prepared, m.heads * row_head);
+            partial = std::max(partial, (size_t)m.heads * kGroupedMaxParts * row_head);
+            partial_pairs = std::max<size_t>(partial_pairs, m.heads * kGroupedMaxParts * 2u);
+            std::vector<double> frequencies(std::max(1u, m.rotated / 2u), 0.0);
+            for (uint32_t i = 0; i < m.rotated / 2u; ++i) frequencies[i] = std::pow(m.rotation_base, -2.0 * (double)i / (double)m.rotated);
+            GF_TRY(plan_alloc(allocations_, &p.frequencies[l], frequencies.size()));
+            GF_CUDA(cudaMemcpy(p.frequencies[l], frequencies.data(), frequencies.size() * sizeof(double), cudaMemcpyHostToDevice));
+        } else {
+            q_width = std::max(q_width, state_inputs_ld(m));
+        }
         if (f.kind == FeedForwardSpec::kNone) continue;
-        GF_TRY(gain(t + "norm2", "", s.norm_offset, &w.gain2));
-        GF_TRY(gain(t + "norm2b", t + "ls2", s.norm_offset, &w.gain2b));
-        if (f.kind == FeedForwardSpec::kDense) ff = std::max(ff, f.ff);
+        if (f.kind == FeedForwardSpec::kDense) ff = std::max(ff, round_up(f.ff, 8u));
         else {
             top = std::max(top, f.top); experts = std::max(experts, f.experts);
             expert_ff = std::max(expert_ff, f.top * round_up(f.ff, 8u)); shared_ff = std::max(shared_ff, round_up(f.shared_ff, 8u));
@@ -207,11 +262,18 @@ int Model::finalize_layered() {
         LayerCache& cache = caches_[l];
         const size_t row = p.cache_row_bytes(l);
         cache.window = 0;
-        cache.ring_rows = ring_rows;
-        GF_TRY(bytes_alloc(allocations_, &cache.ring_k, row * ring_rows));
-        GF_TRY(bytes_alloc(allocations_, &cache.private_k, row * R));
-        table[l] = KvPublishLayer{static_cast<uint8_t*>(cache.ring_k), nullptr, static_cast<const uint8_t*>(cache.private_k), nullptr, ring_rows - 1u, (uint32_t)row};
-        rings[l] = StreamRings{cache.ring_k, nullptr};
+        // A recurrent layer's ring holds the rows a convolution looks back at, those of a pass, and as many again to go
+        // back to.
+        cache.ring_rows = p.recurrent(l) ? next_pow2(s.layers[l].mixer.taps - 1u + 2u * R) : ring_rows;
+        void** ring[2] = {&cache.ring_k, &cache.ring_v};
+        void** own[2] = {&cache.private_k, &cache.private_v};
+        for (uint32_t which = 0; which < 2u; ++which) {
+            const size_t bytes = p.ring_bytes(l, which, cache.ring_rows, p.own_slots);
+            if (bytes) GF_TRY(bytes_alloc(allocations_, ring[which], bytes));
+            if (which < p.cache_tensors(l)) GF_TRY(bytes_alloc(allocations_, own[which], row * R));
+        }
+        table[l] = publish_layer(l, cache.ring_k, cache.ring_v, cache.private_k, cache.private_v);
+        rings[l] = StreamRings{cache.ring_k, cache.ring_v};
     }
     GF_TRY(plan_alloc(allocations_, &publish_layers_, c.layers));
     GF_CUDA(cudaMemcpy(publish_layers_, table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice));
@@ -224,8 +286,17 @@ int Model::finalize_layered() {
     GF_TRY(plan_alloc(allocations_, &p.heads_out, (size_t)R * values));
     GF_TRY(plan_alloc(allocations_, &p.projected, (size_t)R * s.width));
     GF_TRY(bytes_alloc(allocations_, &p.latent_q, (size_t)R * query_elements * 4u));
-    GF_TRY(plan_alloc(allocations_, &p.partial_out, (size_t)R * heads * kLatentMaxParts * row_elements));
-    GF_TRY(plan_alloc(allocations_, &p.partial_ml, (size_t)R * heads * kLatentMaxParts * 2u));
+    GF_TRY(plan_alloc(allocations_, &p.partial_out, R * partial));
+    GF_TRY(plan_alloc(allocations_, &p.partial_ml, R * partial_pairs));
+    if (heads) {
+        GF_TRY(plan_alloc(allocations_, &p.raw_k, (size_t)R * k_width));
+        GF_TRY(plan_alloc(allocations_, &p.raw_gate, (size_t)R * heads));
+        GF_TRY(bytes_alloc(allocations_, &p.query, (size_t)R * prepared * 4u));
+        GF_TRY(plan_alloc(allocations_, &p.counters, (size_t)R * heads));
+    }
+    GF_TRY(plan_alloc(allocations_, &p.slots_dev, 2u));
+    const uint32_t slots[2] = {p.own_slots, LayeredPlan::kStreamSlots};
+    GF_CUDA(cudaMemcpy(p.slots_dev, slots, sizeof slots, cudaMemcpyHostToDevice));
     if (ff) GF_TRY(plan_alloc(allocations_, &p.hidden, (size_t)R * ff));
     if (top) {
         GF_TRY(plan_alloc(allocations_, &p.expert_hidden, (size_t)R * expert_ff));
@@ -237,6 +308,17 @@ int Model::finalize_layered() {
         GF_TRY(plan_alloc(allocations_, &p.route_scores, (size_t)R * top));
     }
     return finalize_shared();
+}
+
+// A layer's entry of a publication table: its cache rows, or nothing to publish (recurrent layers).
+KvPublishLayer Model::publish_layer(uint32_t l, void* ring_k, void* ring_v, const void* own_k, const void* own_v) const {
+    const uint32_t tensors = layered_->cache_tensors(l);
+    KvPublishLayer entry {};
+    entry.ring_mask = caches_[l].ring_rows - 1u;
+    entry.row_bytes = (uint32_t)layered_->cache_row_bytes(l);
+    if (tensors > 0u) { entry.ring_k = static_cast<uint8_t*>(ring_k); entry.private_k = static_cast<const uint8_t*>(own_k); }
+    if (tensors > 1u) { entry.ring_v = static_cast<uint8_t*>(ring_v); entry.private_v = static_cast<const uint8_t*>(own_v); }
+    return entry;
 }
 
 // ------------------------------------------------------------------ a pass of a few rows
@@ -257,17 +339,14 @@ int Model::encode_layers(uint32_t rows, bool logits, const LayeredRows& where) {
     struct { const float *y = nullptr, *gain = nullptr; uint32_t parts = 1; size_t stride = 0; } pending;      // a sublayer's output not yet in the residual
     auto run = [&](RowProduct& r) { r.rows = rows; r.eps = s.eps; r.status = status_dev_; return launch_row_product(r, stream_, true, launches_); };
     auto normalised = [&](RowProduct& r, const float* gain) {
-        r.width = s.width; r.in_ld = s.width; r.gain1 = gain;
-        if (!pending.y) { r.input = kRowNorm; r.in = x; return; }
+        r.width = s.width; r.in_ld = s.width; r.gain1 = gain;      // without a gain the residual itself
+        if (!pending.y) { r.input = gain ? kRowNorm : kRowPlain; r.in = x; return; }
         r.input = kRowAddNorm; r.in = pending.y; r.parts = pending.parts; r.part_stride = pending.stride; r.gain0 = pending.gain;
         r.residual = x; r.residual_out = other;
         std::swap(x, other);
         pending = {};
     };
-    for (uint32_t l = 0; l < s.layers.size(); ++l) {
-        const LayeredLayer& w = p.layers[l];
-        const MixerSpec& m = s.layers[l].mixer;
-        const FeedForwardSpec& f = s.layers[l].mlp;
+    auto latent_attention = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m) -> int {
         const uint32_t row_elements = latent_row_elements(m.rank);
         RowProduct down;
         down.count = 2;
@@ -300,19 +379,77 @@ int Model::encode_layers(uint32_t rows, bool logits, const LayeredRows& where) {
         value.m[0] = row_matrix(w.up_value, p.heads_out, m.heads * m.vdim);
         value.m[0].weight_batch = w.up_value.bytes(); value.m[0].out_batch = m.vdim;
         GF_TRY(run(value));
+        return GF_OK;
+    };
+    auto grouped_attention = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m) -> int {
+        const uint32_t row_head = grouped_row_head(m.dim, m.vdim);
+        RowProduct in;
+        in.count = 3;
+        in.m[0] = row_matrix(w.q, p.raw_q, m.heads * m.dim);
+        in.m[1] = row_matrix(w.k, p.raw_k, m.kv_heads * m.dim);
+        in.m[2] = row_matrix(w.head_gate, p.raw_gate, m.heads);
+        normalised(in, w.gain1);
+        GF_TRY(run(in));
+        QueryKey prepare;
+        prepare.raw_q = p.raw_q; prepare.raw_k = prepare.raw_v = p.raw_k;
+        prepare.q_ld = m.heads * m.dim; prepare.k_ld = prepare.v_ld = m.kv_heads * m.dim;
+        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.frequencies = p.frequencies[l];
+        prepare.positions = where.positions; prepare.chain = where.ring_stride == 0u;
+        prepare.q = p.query; prepare.keys = caches_[l].private_k; prepare.values = caches_[l].private_v;
+        prepare.rows = rows; prepare.heads = m.heads; prepare.kv_heads = m.kv_heads; prepare.dim = m.dim; prepare.vdim = m.vdim;
+        prepare.row_head = row_head; prepare.rotated = m.rotated; prepare.f32 = p.f32 ? 1u : 0u;
+        prepare.eps = s.eps; prepare.scale = m.scale; prepare.status = status_dev_;
+        ++launches_;
+        GF_TRY(launch_query_key(prepare, stream_, true));
+        GroupedAttention attention;
+        attention.q = p.query;
+        attention.rings = where.rings + (size_t)l * where.layer_stride; attention.ring_stride = where.ring_stride;
+        attention.own_k = caches_[l].private_k; attention.own_v = caches_[l].private_v; attention.positions = where.positions;
+        attention.rows = rows; attention.heads = m.heads; attention.kv_heads = m.kv_heads; attention.row_head = row_head; attention.vdim = m.vdim;
+        attention.ring_mask = caches_[l].ring_rows - 1u; attention.f32 = p.f32 ? 1u : 0u;
+        attention.softcap = m.softcap; attention.sink = w.sink; attention.gate = p.raw_gate;
+        attention.partial_out = p.partial_out; attention.partial_ml = p.partial_ml; attention.counters = p.counters;
+        attention.parts = grouped_attention_parts(rows, m.heads, m.kv_heads, config_.context, where.ring_stride == 0u);
+        attention.result.data = p.heads_out; attention.result.capacity = R; attention.result.k_pad = m.inner(); attention.result.f32 = 1u;
+        ++launches_;
+        return launch_grouped_attention(attention, stream_, true);
+    };
+    auto state_space = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m) -> int {
+        RowProduct in;
+        in.m[0] = row_matrix(w.state_in, p.raw_q, state_inputs_ld(m));
+        normalised(in, w.gain1);
+        GF_TRY(run(in));
+        StateSpace step = p.state_space(l);
+        step.raw = p.raw_q; step.raw_ld = state_inputs_ld(m);
+        step.taps = w.taps; step.tap_bias = w.tap_bias; step.step_bias = w.step_bias; step.decay = w.decay; step.skip = w.skip;
+        step.rings = where.rings + (size_t)l * where.layer_stride; step.ring_stride = where.ring_stride;
+        step.positions = where.positions; step.slots = where.slots; step.rows = rows; step.input_mask = caches_[l].ring_rows - 1u;
+        step.out = p.heads_out;
+        ++launches_;
+        return launch_state_space_rows(step, stream_, true);
+    };
+    for (uint32_t l = 0; l < s.layers.size(); ++l) {
+        const LayeredLayer& w = p.weights(l);
+        const MixerSpec& m = s.layers[l].mixer;
+        const FeedForwardSpec& f = s.layers[l].mlp;
+        if (m.kind == MixerKind::kLatentAttention) GF_TRY(latent_attention(l, w, m));
+        else if (m.kind == MixerKind::kGroupedAttention) GF_TRY(grouped_attention(l, w, m));
+        else GF_TRY(state_space(l, w, m));
         RowProduct out;
-        out.in = p.heads_out; out.in_ld = m.heads * m.vdim;
+        out.in = p.heads_out; out.in_ld = m.inner();
+        if (m.kind == MixerKind::kStateSpace) { out.input = kRowPartNorm; out.width = m.inner(); out.norm_parts = m.norm_parts; out.gain1 = w.mixer_gain; }
         out.m[0] = row_matrix(w.o, p.projected, s.width);
         GF_TRY(run(out));
         pending.y = p.projected; pending.gain = w.gain1b;
         if (f.kind == FeedForwardSpec::kNone) continue;
         if (f.kind == FeedForwardSpec::kDense) {
             RowProduct up;
-            up.m[0] = row_matrix(w.up, p.hidden, f.ff, kOutSquaredRelu);
+            const uint32_t ff = round_up(f.ff, 8u);
+            up.m[0] = row_matrix(w.up, p.hidden, ff, f.activation == Activation::kGeluGate ? kOutGeluGate : kOutSquaredRelu);
             normalised(up, w.gain2);
             GF_TRY(run(up));
             RowProduct d;
-            d.in = p.hidden; d.in_ld = f.ff;
+            d.in = p.hidden; d.in_ld = ff;
             d.m[0] = row_matrix(w.down, p.projected, s.width);
             GF_TRY(run(d));
             pending.y = p.projected; pending.gain = w.gain2b;
@@ -348,7 +485,7 @@ int Model::encode_layers(uint32_t rows, bool logits, const LayeredRows& where) {
     }
     if (logits) {
         RowProduct head;
-        head.m[0] = row_matrix(p.table, where.logits, s.vocab);
+        head.m[0] = row_matrix(p.head(), where.logits, s.vocab);
         normalised(head, p.final_gain);
         GF_TRY(run(head));
     }
@@ -370,11 +507,23 @@ int Model::ensure_chunk_arena() {
         return bytes_alloc(allocations_, &o.data, o.bytes());
     };
     uint32_t query = 0, latent_out = 0, values = 0, latent = 0, query_elements = 0, row_elements = 0, ff = 0, shared_ff = 0, expert_ff = 0, experts = 0, top = 0, heads = 0;
+    size_t raw_q = 0, raw_k = 0, gates = 0, prepared = 0, x_elements = 0, bc_elements = 0, step_elements = 0, y_elements = 0;      // per row
     for (const LayerSpec& l : s.layers) {
         const MixerSpec& m = l.mixer;
-        query = std::max(query, m.heads * round_up(m.dim, kDenseBlockK)); latent_out = std::max(latent_out, m.heads * round_up(m.rank, kDenseBlockK));
-        values = std::max(values, m.heads * m.vdim); latent = std::max(latent, m.rank); heads = std::max(heads, m.heads);
-        query_elements = std::max(query_elements, m.heads * latent_row_elements(m.rank)); row_elements = std::max(row_elements, latent_row_elements(m.rank));
+        values = std::max(values, m.inner());
+        if (m.kind == MixerKind::kLatentAttention) {
+            query = std::max(query, m.heads * round_up(m.dim, kDenseBlockK)); latent_out = std::max(latent_out, m.heads * round_up(m.rank, kDenseBlockK));
+            latent = std::max(latent, m.rank); heads = std::max(heads, m.heads);
+            query_elements = std::max(query_elements, m.heads * latent_row_elements(m.rank)); row_elements = std::max(row_elements, latent_row_elements(m.rank));
+        } else if (m.kind == MixerKind::kGroupedAttention) {
+            raw_q = std::max<size_t>(raw_q, m.heads * m.dim); raw_k = std::max<size_t>(raw_k, m.kv_heads * m.dim); gates = std::max<size_t>(gates, m.heads);
+            prepared = std::max<size_t>(prepared, m.heads * grouped_row_head(m.dim, m.vdim));
+        } else {
+            const StateSpace shape = p.state_space((uint32_t)(&l - s.layers.data()));
+            raw_q = std::max<size_t>(raw_q, state_inputs_ld(m)); y_elements = std::max<size_t>(y_elements, m.inner());
+            x_elements = std::max<size_t>(x_elements, m.heads * shape.x_row()); bc_elements = std::max<size_t>(bc_elements, m.groups * shape.state_row());
+            step_elements = std::max<size_t>(step_elements, m.heads);
+        }
         const FeedForwardSpec& f = l.mlp;
         if (f.kind == FeedForwardSpec::kDense) ff = std::max(ff, f.ff);
         if (f.kind == FeedForwardSpec::kExperts) {
@@ -383,9 +532,20 @@ int Model::ensure_chunk_arena() {
         }
     }
     GF_TRY(operand(a.normed, s.width, rows));
-    GF_TRY(operand(a.query, query, rows));
-    GF_TRY(operand(a.latent_out, latent_out, rows));
     GF_TRY(operand(a.heads_out, values, rows));
+    if (raw_q) GF_TRY(plan_alloc(allocations_, &a.raw_q, rows * raw_q));
+    if (raw_k) {
+        GF_TRY(plan_alloc(allocations_, &a.raw_k, rows * raw_k));
+        GF_TRY(plan_alloc(allocations_, &a.raw_gate, rows * gates));
+        GF_TRY(bytes_alloc(allocations_, &a.prepared_q, rows * prepared * (p.f32 ? 4u : 2u)));
+    }
+    if (y_elements) {
+        GF_TRY(plan_alloc(allocations_, &a.state_x, rows * x_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_b, rows * bc_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_c, rows * bc_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_steps, rows * step_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_y, rows * y_elements));
+    }
     if (ff) GF_TRY(operand(a.hidden, ff, rows));
     if (experts) {
         if (shared_ff) GF_TRY(operand(a.shared_hidden, shared_ff, rows));
@@ -405,11 +565,19 @@ int Model::ensure_chunk_arena() {
     GF_TRY(plan_alloc(allocations_, &a.residual, (size_t)rows * s.width));
     GF_TRY(plan_alloc(allocations_, &a.y, (size_t)rows * s.width));
     GF_TRY(plan_alloc(allocations_, &a.final_rows, (size_t)rows * s.width));
-    GF_TRY(plan_alloc(allocations_, &a.raw_latent, (size_t)rows * latent));
-    GF_TRY(bytes_alloc(allocations_, &a.latent_q, (size_t)rows * query_elements * (p.f32 ? 4u : 2u)));
-    if (!p.f32) {
+    if (latent) {
+        GF_TRY(operand(a.query, query, rows));
+        GF_TRY(operand(a.latent_out, latent_out, rows));
+        GF_TRY(plan_alloc(allocations_, &a.raw_latent, (size_t)rows * latent));
+        GF_TRY(bytes_alloc(allocations_, &a.latent_q, (size_t)rows * query_elements * (p.f32 ? 4u : 2u)));
+        a.partial_rows = std::max((uint32_t)sm_count() * 64u, heads * 16u);
+        GF_TRY(plan_alloc(allocations_, &a.partial_out, (size_t)a.partial_rows * row_elements));
+        GF_TRY(plan_alloc(allocations_, &a.partial_ml, (size_t)a.partial_rows * 2u));
+    }
+    if (latent && !p.f32) {
         size_t per_key = 0, q_elements = 0;
         for (const LayerSpec& l : s.layers) {
+            if (l.mixer.kind != MixerKind::kLatentAttention) continue;
             const size_t dims = round_up(l.mixer.dim, 16u), vdims = round_up(l.mixer.vdim, 16u);
             per_key = std::max(per_key, l.mixer.heads * std::max(dims, vdims));
             q_elements = std::max(q_elements, l.mixer.heads * dims);
@@ -421,17 +589,15 @@ int Model::ensure_chunk_arena() {
         GF_TRY(plan_alloc(allocations_, &a.values, a.expand_keys * per_key));
         GF_TRY(plan_alloc(allocations_, &a.head_q, rows * q_elements));
     }
-    a.partial_rows = std::max((uint32_t)sm_count() * 64u, heads * 16u);
-    GF_TRY(plan_alloc(allocations_, &a.partial_out, (size_t)a.partial_rows * row_elements));
-    GF_TRY(plan_alloc(allocations_, &a.partial_ml, (size_t)a.partial_rows * 2u));
     GF_TRY(plan_alloc(allocations_, &a.tokens, rows));
     GF_TRY(plan_alloc(allocations_, &a.wanted, rows));
     std::vector<KvPublishLayer> table(c.layers);
-    a.private_rows.resize(c.layers);
+    a.private_rows.assign(c.layers, nullptr);
+    a.private_values.assign(c.layers, nullptr);
     for (uint32_t l = 0; l < c.layers; ++l) {
-        GF_TRY(bytes_alloc(allocations_, &a.private_rows[l], p.cache_row_bytes(l) * rows));
-        table[l] = KvPublishLayer{static_cast<uint8_t*>(caches_[l].ring_k), nullptr, static_cast<const uint8_t*>(a.private_rows[l]), nullptr,
-                                  caches_[l].ring_rows - 1u, (uint32_t)p.cache_row_bytes(l)};
+        if (p.cache_tensors(l) > 0u) GF_TRY(bytes_alloc(allocations_, &a.private_rows[l], p.cache_row_bytes(l) * rows));
+        if (p.cache_tensors(l) > 1u) GF_TRY(bytes_alloc(allocations_, &a.private_values[l], p.cache_row_bytes(l) * rows));
+        table[l] = publish_layer(l, caches_[l].ring_k, caches_[l].ring_v, a.private_rows[l], a.private_values[l]);
     }
     GF_TRY(plan_alloc(allocations_, &a.publish_layers, c.layers));
     GF_CUDA(cudaMemcpy(a.publish_layers, table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice));
@@ -476,18 +642,13 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         ++launches_;
         return launch_chunk_product(product, f32, stream_);
     };
-    for (uint32_t l = 0; l < s.layers.size(); ++l) {
-        const LayeredLayer& w = p.layers[l];
-        const MixerSpec& m = s.layers[l].mixer;
-        const FeedForwardSpec& f = s.layers[l].mlp;
-        const bool last = l + 1u == s.layers.size() && !logits;      // nothing downstream of the last layer's cache rows is needed
+    const Operand normed = operand_view(a.normed, s.width);
+    auto latent_attention = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m, const Operand& heads_out, bool last) -> int {
         const uint32_t row_elements = latent_row_elements(m.rank), dim_pad = round_up(m.dim, kDenseBlockK), rank_pad = round_up(m.rank, kDenseBlockK);
-        GF_TRY(normalise(w.gain1, false));
-        const Operand normed = operand_view(a.normed, s.width);
         ChunkProduct down;
         down.p[0] = chunk_problem(w.latent_down, normed);
         down.p[0].out = a.raw_latent; down.p[0].out_ld = m.rank;
-        const Operand query = operand_view(a.query, m.heads * dim_pad), heads_out = operand_view(a.heads_out, m.heads * m.vdim);
+        const Operand query = operand_view(a.query, m.heads * dim_pad);
         const uint32_t positions = position_ + rows, head_pad = round_up(m.dim, 16u), value_pad = round_up(m.vdim, 16u);
         const bool expand = !f32 && positions <= a.expand_keys && head_pad <= kHeadAttentionMaxDim && value_pad <= kHeadAttentionMaxDim
                             && latent_expansion_pays(rows, m.rank, m.dim, m.vdim);
@@ -504,7 +665,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         GF_TRY(run(down));
         ++launches_;
         GF_TRY(launch_chunk_latents(a.raw_latent, m.rank, w.latent_gain, m.rank, s.eps, a.private_rows[l], row_elements, !f32, rows, status_dev_, stream_));
-        if (last) break;
+        if (last) return GF_OK;
         if (expand) {
             Operand latents;
             latents.data = a.latent_rows; latents.capacity = round_up(positions, 16u); latents.k_pad = rank_pad;
@@ -522,7 +683,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
             GF_TRY(run(expansion));
             HeadAttention attention;
             attention.q = a.head_q; attention.k = a.keys; attention.v = a.values; attention.position = state_dev_; attention.sink = w.sink;
-            attention.rows = rows; attention.heads = m.heads; attention.dim_pad = head_pad; attention.vdim = m.vdim; attention.vdim_pad = value_pad;
+            attention.rows = rows; attention.heads = attention.kv_heads = m.heads; attention.dim_pad = head_pad; attention.vdim = m.vdim; attention.vdim_pad = value_pad;
             attention.result = heads_out;
             ++launches_;
             GF_TRY(launch_head_attention(attention, stream_));
@@ -553,6 +714,78 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
             value.p[0].output = kChunkOperand; value.p[0].result = heads_out; value.p[0].column_stride = m.vdim;
             GF_TRY(run(value));
         }
+        return GF_OK;
+    };
+    auto grouped_attention = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m, const Operand& heads_out, bool last) -> int {
+        const uint32_t row_head = grouped_row_head(m.dim, m.vdim);
+        ChunkProduct in;
+        in.p[0] = chunk_problem(w.k, normed);
+        in.p[0].out = a.raw_k; in.p[0].out_ld = m.kv_heads * m.dim;
+        if (!last) {
+            in.problems = 3;
+            in.p[1] = chunk_problem(w.q, normed);
+            in.p[1].out = a.raw_q; in.p[1].out_ld = m.heads * m.dim;
+            in.p[2] = chunk_problem(w.head_gate, normed);
+            in.p[2].out = a.raw_gate; in.p[2].out_ld = m.heads;
+        }
+        GF_TRY(run(in));
+        QueryKey prepare;
+        prepare.raw_q = last ? nullptr : a.raw_q; prepare.raw_k = prepare.raw_v = a.raw_k;
+        prepare.q_ld = m.heads * m.dim; prepare.k_ld = prepare.v_ld = m.kv_heads * m.dim;
+        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.frequencies = p.frequencies[l]; prepare.positions = state_dev_;
+        prepare.q = a.prepared_q; prepare.keys = a.private_rows[l]; prepare.values = a.private_values[l];
+        prepare.rows = rows; prepare.heads = m.heads; prepare.kv_heads = m.kv_heads; prepare.dim = m.dim; prepare.vdim = m.vdim;
+        prepare.row_head = row_head; prepare.rotated = m.rotated; prepare.f32 = f32 ? 1u : 0u;
+        prepare.eps = s.eps; prepare.scale = m.scale; prepare.status = status_dev_;
+        ++launches_;
+        GF_TRY(launch_query_key(prepare, stream_, false));
+        if (last) return GF_OK;
+        ++launches_;
+        if (!f32 && row_head <= kHeadAttentionMaxDim) {
+            HeadAttention attention;
+            attention.q = static_cast<const __half*>(a.prepared_q);
+            attention.k = static_cast<const __half*>(a.private_rows[l]); attention.v = static_cast<const __half*>(a.private_values[l]);
+            attention.rings = p.rings_dev + l; attention.ring_mask = caches_[l].ring_rows - 1u; attention.position = state_dev_;
+            attention.sink = w.sink; attention.gate = a.raw_gate; attention.softcap = m.softcap;
+            attention.rows = rows; attention.heads = m.heads; attention.kv_heads = m.kv_heads;
+            attention.dim_pad = attention.vdim_pad = row_head; attention.vdim = m.vdim; attention.result = heads_out;
+            return launch_head_attention(attention, stream_);
+        }
+        GroupedAttention attention;
+        attention.q = a.prepared_q; attention.rings = p.rings_dev + l;
+        attention.own_k = a.private_rows[l]; attention.own_v = a.private_values[l]; attention.positions = state_dev_;
+        attention.rows = rows; attention.heads = m.heads; attention.kv_heads = m.kv_heads; attention.row_head = row_head; attention.vdim = m.vdim;
+        attention.ring_mask = caches_[l].ring_rows - 1u; attention.f32 = f32 ? 1u : 0u;
+        attention.softcap = m.softcap; attention.sink = w.sink; attention.gate = a.raw_gate; attention.result = heads_out;
+        return launch_grouped_attention(attention, stream_, false);
+    };
+    auto state_space = [&](uint32_t l, const LayeredLayer& w, const MixerSpec& m, const Operand& heads_out, bool last) -> int {
+        ChunkProduct in;
+        in.p[0] = chunk_problem(w.state_in, normed);
+        in.p[0].out = a.raw_q; in.p[0].out_ld = state_inputs_ld(m);
+        GF_TRY(run(in));
+        StateSpace step = p.state_space(l);
+        step.raw = a.raw_q; step.raw_ld = state_inputs_ld(m);
+        step.taps = w.taps; step.tap_bias = w.tap_bias; step.step_bias = w.step_bias; step.decay = w.decay; step.skip = w.skip;
+        step.rings = p.rings_dev + l; step.positions = state_dev_; step.slots = p.slots_dev; step.rows = rows; step.input_mask = caches_[l].ring_rows - 1u;
+        step.out = a.state_y; step.x = a.state_x; step.b = a.state_b; step.c = a.state_c; step.steps = a.state_steps;
+        launches_ += 2;
+        GF_TRY(launch_state_space_chunk(step, stream_));
+        if (last) return GF_OK;
+        ++launches_;
+        return launch_chunk_part_norm(a.state_y, m.inner(), a.raw_q, state_inputs_ld(m), m.inner(), m.norm_parts, w.mixer_gain, s.eps, heads_out, rows, stream_);
+    };
+    for (uint32_t l = 0; l < s.layers.size(); ++l) {
+        const LayeredLayer& w = p.weights(l);
+        const MixerSpec& m = s.layers[l].mixer;
+        const FeedForwardSpec& f = s.layers[l].mlp;
+        const bool last = l + 1u == s.layers.size() && !logits;      // nothing downstream of the last layer's cache rows and state is needed
+        const Operand heads_out = operand_view(a.heads_out, m.inner());
+        GF_TRY(normalise(w.gain1, false));
+        if (m.kind == MixerKind::kLatentAttention) GF_TRY(latent_attention(l, w, m, heads_out, last));
+        else if (m.kind == MixerKind::kGroupedAttention) GF_TRY(grouped_attention(l, w, m, heads_out, last));
+        else GF_TRY(state_space(l, w, m, heads_out, last));
+        if (last) break;
         ChunkProduct out;
         out.p[0] = chunk_problem(w.o, heads_out);
         out.p[0].out = a.y; out.p[0].out_ld = s.width;
@@ -564,7 +797,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
             const Operand hidden = operand_view(a.hidden, f.ff);
             ChunkProduct up;
             up.p[0] = chunk_problem(w.up, normed);
-            up.p[0].output = kChunkSquaredRelu; up.p[0].result = hidden;
+            up.p[0].output = f.activation == Activation::kGeluGate ? kChunkGeluGate : kChunkSquaredRelu; up.p[0].result = hidden;
             GF_TRY(run(up));
             ChunkProduct d;
             d.p[0] = chunk_problem(w.down, hidden);
@@ -614,6 +847,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
     GF_TRY(launch_kv_publish(a.publish_layers, config_.layers, state_dev_, rows, stream_));
     launches_ += 2;
     position_ += rows;
+    state_floor_ = state_frontier_ = position_;          // a chunk leaves its last state alone
     return GF_OK;
 }
 
@@ -653,7 +887,7 @@ int Model::extend(const uint32_t* tokens_host, uint32_t count, const uint32_t* w
                     RowProduct head;
                     head.rows = std::min(config_.row_capacity, (uint32_t)places.size() - i);
                     head.in = p.chunk.final_rows; head.in_ld = config_.hidden; head.in_rows = p.chunk.wanted + i;
-                    head.m[0] = row_matrix(p.table, logits_, config_.vocab);
+                    head.m[0] = row_matrix(p.head(), logits_, config_.vocab);
                     GF_TRY(launch_row_product(head, stream_, false, launches_));
                     for (uint32_t r = 0; r < head.rows; ++r) GF_TRY(keep(r));
                 }

@@ -452,7 +452,13 @@ int Model::reset() {
     if (attention_ws_) GF_CUDA(cudaMemsetAsync(attention_counters(attention_ws_, config_.row_capacity, config_.heads), 0,
                             (size_t)config_.row_capacity * config_.heads * sizeof(uint32_t), stream_));
     if (head_counters_) GF_CUDA(cudaMemsetAsync(head_counters_, 0, 2u * (config_.heads + 2u * config_.kv_heads) * sizeof(uint32_t), stream_));
+    if (layered_ && layered_->counters) {
+        uint32_t heads = 0;
+        for (const LayerSpec& l : layered_->spec().layers) heads = std::max(heads, l.mixer.kind == MixerKind::kGroupedAttention ? l.mixer.heads : 0u);
+        GF_CUDA(cudaMemsetAsync(layered_->counters, 0, (size_t)config_.row_capacity * heads * sizeof(uint32_t), stream_));
+    }
     position_ = 0;
+    state_floor_ = state_frontier_ = 0;
     poisoned_ = false;
     return GF_OK;
 }
@@ -722,7 +728,7 @@ int Model::run_recorded(const RecordedPass& pass, uint32_t rows) {
 //   down  <- prologue: gelu_tanh(gate) * up
 // The next layer's QKV (or the head) applies the post-FFW norm and residual of this layer.
 int Model::encode_blocks(uint32_t rows, uint32_t flags) {
-    if (layered_) return encode_layers(rows, (flags & kForwardLogits) != 0, LayeredRows{layered_->rings_dev, 1u, 0u, state_dev_, logits_});
+    if (layered_) return encode_layers(rows, (flags & kForwardLogits) != 0, LayeredRows{layered_->rings_dev, 1u, 0u, state_dev_, logits_, layered_->slots_dev});
     const gf_model_config& c = config_;
     const float embedding_scale = sqrtf((float)c.hidden);     // f32, not bf16-rounded (model.cpp:599-605)
     const bool fused_exchange = shard_.connected;
@@ -874,6 +880,7 @@ int Model::forward(const uint32_t* tokens_host, uint32_t rows, uint32_t flags) {
         GF_CUDA(cudaMemcpyAsync(tokens_dev_, tokens_pinned_, rows * sizeof(uint32_t), cudaMemcpyHostToDevice, stream_));
         GF_CUDA(cudaEventRecord(tokens_copied_, stream_));
     }
+    state_frontier_ = std::max(state_frontier_, position_ + rows);
     return run_graph_or_encode(rows, flags);
 }
 
@@ -892,6 +899,9 @@ int Model::truncate(uint32_t position) {
     if (position > position_) return fail(GF_ERR_INVALID, "cannot truncate forward");
     if (position_ - position > config_.row_capacity)
         return fail(GF_ERR_INVALID, "published sliding-window rows older than one pass cannot be restored");
+    if (layered_ && layered_->any_recurrent() && position != position_ && position != 0u
+        && (position < state_floor_ || state_frontier_ - position >= layered_->own_slots))
+        return fail(GF_ERR_INVALID, "the recurrent state after %u tokens is no longer held", position);
     if (position != position_) {
         GF_CUDA(cudaMemcpyAsync(state_dev_, &position, sizeof(uint32_t), cudaMemcpyHostToDevice, stream_));
         GF_CUDA(cudaStreamSynchronize(stream_));
@@ -1253,13 +1263,15 @@ int Model::read_logits(uint32_t row, float* host) {
 
 int Model::read_kv(uint32_t layer, uint32_t first_position, uint32_t count, float* k_host, float* v_host) {
     if (!finalized_) return fail(GF_ERR_STATE, "plan is not finalized");
-    if (layer >= config_.layers || !k_host || (!v_host && !layered_) || count == 0) return fail(GF_ERR_INVALID, "bad K/V readback");
+    if (layer >= config_.layers || !k_host || count == 0) return fail(GF_ERR_INVALID, "bad K/V readback");
+    const int tensors = layered_ ? (int)layered_->cache_tensors(layer) : 2;
+    if (tensors == 0) return fail(GF_ERR_INVALID, "layer %u is recurrent: it has a state (gf_model_read_state) and no rows", layer);
+    if (!v_host && tensors > 1) return fail(GF_ERR_INVALID, "bad K/V readback");
     const LayerCache& cache = caches_[layer];
     if (first_position + count > position_ || position_ - first_position > cache.ring_rows)
         return fail(GF_ERR_INVALID, "K/V rows [%u, %u) are not all committed and still inside layer %u's ring", first_position,
                     first_position + count, layer);
     const size_t element = config_.kv_f16 ? 2 : 4, kvw = cache_row_bytes(layer) / element;
-    const int tensors = layered_ ? 1 : 2;
     std::vector<uint8_t> raw[2];
     const void* rings[2] = {cache.ring_k, cache.ring_v};
     for (int which = 0; which < tensors; ++which) {
@@ -1275,20 +1287,39 @@ int Model::read_kv(uint32_t layer, uint32_t first_position, uint32_t count, floa
         }
     }
     GF_TRY(synchronize());
-    if (layered_) {          // rows are stored with their rank rounded up
-        const uint32_t rank = layered_->spec().layers[layer].mixer.rank;
-        for (uint32_t r = 0; r < count; ++r)
-            for (uint32_t i = 0; i < rank; ++i)
-                k_host[(size_t)r * rank + i] = config_.kv_f16 ? __half2float(reinterpret_cast<const __half*>(raw[0].data())[r * kvw + i])
-                                                              : reinterpret_cast<const float*>(raw[0].data())[r * kvw + i];
+    float* outs[2] = {k_host, v_host};
+    if (layered_) {          // rows are stored with a head's size, or the latent's, rounded up
+        const MixerSpec& m = layered_->spec().layers[layer].mixer;
+        const bool grouped = m.kind == MixerKind::kGroupedAttention;
+        const uint32_t groups = grouped ? m.kv_heads : 1u, wide = (uint32_t)(kvw / groups);
+        for (int which = 0; which < tensors; ++which) {
+            const uint32_t used = !grouped ? m.rank : which ? m.vdim : m.dim;
+            for (size_t i = 0; i < (size_t)count * groups; ++i)
+                for (uint32_t d = 0; d < used; ++d)
+                    outs[which][i * used + d] = config_.kv_f16 ? __half2float(reinterpret_cast<const __half*>(raw[which].data())[i * wide + d])
+                                                               : reinterpret_cast<const float*>(raw[which].data())[i * wide + d];
+        }
         return GF_OK;
     }
-    float* outs[2] = {k_host, v_host};
     for (int which = 0; which < 2; ++which) {
         if (!config_.kv_f16) { std::memcpy(outs[which], raw[which].data(), raw[which].size()); continue; }
         const __half* src = reinterpret_cast<const __half*>(raw[which].data());
         for (size_t i = 0; i < (size_t)count * kvw; ++i) outs[which][i] = __half2float(src[i]);
     }
+    return GF_OK;
+}
+
+int Model::read_state(uint32_t layer, float* state_host) {
+    if (!finalized_) return fail(GF_ERR_STATE, "plan is not finalized");
+    if (!state_host || !layered_ || layer >= config_.layers || !layered_->recurrent(layer)) return fail(GF_ERR_INVALID, "state readback: not a recurrent layer");
+    const StateSpace shape = layered_->state_space(layer);
+    const uint32_t wide = shape.state_row();
+    std::vector<float> raw(shape.slot_elements(), 0.0f);
+    if (position_)
+        GF_CUDA(cudaMemcpyAsync(raw.data(), static_cast<const float*>(caches_[layer].ring_k) + (position_ % layered_->own_slots) * shape.slot_elements(),
+                                raw.size() * sizeof(float), cudaMemcpyDeviceToHost, stream_));
+    GF_TRY(synchronize());
+    for (size_t i = 0; i < raw.size() / wide; ++i) std::memcpy(state_host + i * shape.state, raw.data() + i * wide, shape.state * sizeof(float));
     return GF_OK;
 }
 
@@ -1318,7 +1349,8 @@ size_t Model::kv_bytes_per_pass(uint32_t rows) const {
     size_t total = 0;
     for (uint32_t l = 0; l < config_.layers; ++l) {
         const uint32_t window = caches_[l].window, seen = window ? std::min(position_, window) : position_;
-        total += (size_t)seen * cache_row_bytes(l) * (layered_ ? 1u : 2u);
+        total += (size_t)seen * cache_row_bytes(l) * (layered_ ? layered_->cache_tensors(l) : 2u);
+        if (layered_) total += 2u * layered_->state_bytes(l);          // read and written
     }
     return total;
 }
@@ -1424,6 +1456,9 @@ int gf_model_read_logits(gf_model* m, uint32_t row, float* logits_host) {
 }
 int gf_model_read_kv(gf_model* m, uint32_t layer, uint32_t first_position, uint32_t count, float* k_host, float* v_host) {
     return m ? m->impl.read_kv(layer, first_position, count, k_host, v_host) : fail(GF_ERR_INVALID, "null model");
+}
+int gf_model_read_state(gf_model* m, uint32_t layer, float* state_host) {
+    return m ? m->impl.read_state(layer, state_host) : fail(GF_ERR_INVALID, "null model");
 }
 int gf_model_synchronize(gf_model* m) { return m ? m->impl.synchronize() : fail(GF_ERR_INVALID, "null model"); }
 int gf_model_status(gf_model* m, uint32_t* out_status) { return m ? m->impl.status_word(out_status) : fail(GF_ERR_INVALID, "null model"); }

@@ -89,6 +89,7 @@ public:
     int read_candidates(void* results_host, uint32_t rows);
     int read_logits(uint32_t row, float* host);
     int read_kv(uint32_t layer, uint32_t first_position, uint32_t count, float* k_host, float* v_host);
+    int read_state(uint32_t layer, float* state_host);     // recurrent layers: [heads][vdim][N] after the committed tokens
     int synchronize();
     int status_word(uint32_t* out);
     int prefill(const uint32_t* tokens_host, uint32_t count);
@@ -229,16 +230,20 @@ private:
     gf_reduce_fn reduce_hook_ = nullptr;
     void* reduce_user_ = nullptr;
     int bind_q8_head_from_f16(const void* f16_dev, uint64_t k, uint64_t n);
-    int bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>& ring_v, uint32_t position);
+    int bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>& ring_v, uint32_t position, uint32_t slots);
     int encode_stream_group(StreamSet& set, uint32_t first, uint32_t rows);
     int encode_stream_batch(StreamSet& set);
     int encode_blocks(uint32_t rows, uint32_t flags);
     int finalize_shared();
     int finalize_layered();
+    KvPublishLayer publish_layer(uint32_t layer, void* ring_k, void* ring_v, const void* own_k, const void* own_v) const;
     int encode_layers(uint32_t rows, bool logits, const LayeredRows& where);
     int ensure_chunk_arena();
     int chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits);
     std::unique_ptr<LayeredPlan> layered_;
+    // Recurrent layers hold the states after the last few positions only: those above state_frontier_ (the furthest a pass
+    // has gone) less the slots, and none below state_floor_ (the end of the last chunk).
+    uint32_t state_floor_ = 0, state_frontier_ = 0;
     int run_gemv(struct GemvLaunch& launch, uint32_t rows);
     int emit_embedding(uint32_t rows, float scale);
     int emit_attention(const AttentionParams& params);

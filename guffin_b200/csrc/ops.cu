@@ -173,6 +173,7 @@ __global__ void __launch_bounds__(128) stream_publish_kernel(const StreamPublish
                                                              uint32_t stride, const uint32_t* __restrict__ positions) {
     const uint32_t row = blockIdx.x, layer = blockIdx.y;
     const StreamPublishLayer L = layers[layer];
+    if (!L.private_k) return;                                          // a layer without cache rows
     const StreamRings R = rings[(size_t)layer * stride + row];
     const size_t dst = (size_t)(positions[row] & L.ring_mask) * L.row_bytes, src = (size_t)row * L.row_bytes;
     uint8_t* ring_k = static_cast<uint8_t*>(const_cast<void*>(R.ring_k));
@@ -224,6 +225,7 @@ __global__ void __launch_bounds__(128) kv_publish_kernel(const KvPublishLayer* _
     pdl_wait();
     const uint32_t row = blockIdx.x, layer = blockIdx.y;
     const KvPublishLayer L = layers[layer];
+    if (!L.private_k) return;                                          // a layer without cache rows
     const uint32_t base = *base_position;
     const size_t dst = (size_t)((base + row) & L.ring_mask) * L.row_bytes, src = (size_t)row * L.row_bytes;
     for (uint32_t b = threadIdx.x * 16u; b < L.row_bytes; b += blockDim.x * 16u) {

@@ -54,18 +54,18 @@ int Model::streams_create(uint32_t count, StreamSet** out) {
     std::vector<StreamRings> rings((size_t)c.layers * count);
     std::vector<StreamPublishLayer> layers(c.layers);
     for (uint32_t l = 0; l < c.layers; ++l) {
-        const size_t bytes = (size_t)caches_[l].ring_rows * cache_row_bytes(l);
         for (uint32_t s = 0; s < count; ++s) {
-            uint8_t *k = nullptr, *v = nullptr;
-            GF_TRY(stream_alloc(*set, &k, bytes));
-            GF_CUDA(cudaMemsetAsync(k, 0, bytes, stream_));
-            if (!layered_) {
-                GF_TRY(stream_alloc(*set, &v, bytes));
-                GF_CUDA(cudaMemsetAsync(v, 0, bytes, stream_));
+            uint8_t* tensors[2] = {nullptr, nullptr};
+            for (uint32_t which = 0; which < 2u; ++which) {
+                const size_t bytes = layered_ ? layered_->ring_bytes(l, which, caches_[l].ring_rows, LayeredPlan::kStreamSlots)
+                                              : (size_t)caches_[l].ring_rows * cache_row_bytes(l);
+                if (bytes == 0u) continue;
+                GF_TRY(stream_alloc(*set, &tensors[which], bytes));
+                GF_CUDA(cudaMemsetAsync(tensors[which], 0, bytes, stream_));
             }
-            set->ring_k[s][l] = k;
-            set->ring_v[s][l] = v;
-            rings[(size_t)l * count + s] = StreamRings{k, v};
+            set->ring_k[s][l] = tensors[0];
+            set->ring_v[s][l] = tensors[1];
+            rings[(size_t)l * count + s] = StreamRings{tensors[0], tensors[1]};
         }
         layers[l] = StreamPublishLayer{static_cast<const uint8_t*>(caches_[l].private_k), static_cast<const uint8_t*>(caches_[l].private_v),
                                        caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
@@ -89,18 +89,17 @@ int Model::streams_create(uint32_t count, StreamSet** out) {
 
 // Points the plan's cache at other rings (a stream's, or its own again): the publication tables name the
 // rings, and recorded graphs and pass tables have the old pointers baked in.
-int Model::bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>& ring_v, uint32_t position) {
+int Model::bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>& ring_v, uint32_t position, uint32_t slots) {
     const gf_model_config& c = config_;
     std::vector<KvPublishLayer> table(c.layers), prefill_table(c.layers);
     const bool chunks = layered_ && layered_->chunk.ready;
     for (uint32_t l = 0; l < c.layers; ++l) {
         caches_[l].ring_k = ring_k[l];
         caches_[l].ring_v = ring_v[l];
-        table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), static_cast<uint8_t*>(ring_v[l]), static_cast<const uint8_t*>(caches_[l].private_k),
-                                  static_cast<const uint8_t*>(caches_[l].private_v), caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
-        if (chunks)
-            prefill_table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), nullptr, static_cast<const uint8_t*>(layered_->chunk.private_rows[l]), nullptr,
-                                              caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
+        table[l] = layered_ ? publish_layer(l, ring_k[l], ring_v[l], caches_[l].private_k, caches_[l].private_v)
+                            : KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), static_cast<uint8_t*>(ring_v[l]), static_cast<const uint8_t*>(caches_[l].private_k),
+                                             static_cast<const uint8_t*>(caches_[l].private_v), caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
+        if (chunks) prefill_table[l] = publish_layer(l, ring_k[l], ring_v[l], layered_->chunk.private_rows[l], layered_->chunk.private_values[l]);
         if (prefill_.ready)
             prefill_table[l] = KvPublishLayer{static_cast<uint8_t*>(ring_k[l]), static_cast<uint8_t*>(ring_v[l]), static_cast<const uint8_t*>(prefill_.private_k[l]),
                                               static_cast<const uint8_t*>(prefill_.private_v[l]), caches_[l].ring_rows - 1u, (uint32_t)cache_row_bytes(l)};
@@ -111,8 +110,9 @@ int Model::bind_rings(const std::vector<void*>& ring_k, const std::vector<void*>
     if (chunks) GF_CUDA(cudaMemcpyAsync(layered_->chunk.publish_layers, prefill_table.data(), sizeof(KvPublishLayer) * c.layers, cudaMemcpyHostToDevice, stream_));
     std::vector<StreamRings> rings(c.layers);
     if (layered_) {
-        for (uint32_t l = 0; l < c.layers; ++l) rings[l] = StreamRings{ring_k[l], nullptr};
+        for (uint32_t l = 0; l < c.layers; ++l) rings[l] = StreamRings{ring_k[l], ring_v[l]};
         GF_CUDA(cudaMemcpyAsync(layered_->rings_dev, rings.data(), sizeof(StreamRings) * c.layers, cudaMemcpyHostToDevice, stream_));
+        GF_CUDA(cudaMemcpyAsync(layered_->slots_dev, &slots, sizeof slots, cudaMemcpyHostToDevice, stream_));
     }
     GF_CUDA(cudaMemcpyAsync(state_dev_, &position, sizeof(uint32_t), cudaMemcpyHostToDevice, stream_));
     GF_CUDA(cudaStreamSynchronize(stream_));           // the tables above are pageable
@@ -149,12 +149,12 @@ int Model::streams_ingest(StreamSet& set, uint32_t stream, uint32_t count, const
     if (stream >= set.count) return fail(GF_ERR_INVALID, "stream %u of %u", stream, set.count);
     std::vector<void*> home_k(config_.layers), home_v(config_.layers);
     for (uint32_t l = 0; l < config_.layers; ++l) { home_k[l] = caches_[l].ring_k; home_v[l] = caches_[l].ring_v; }
-    const uint32_t home_position = position_;
+    const uint32_t home_position = position_, home_floor = state_floor_, home_frontier = state_frontier_;
     // The tensor-core prompt path allocates its arena on first use, before the rings are exchanged, so that
     // its publication table is rebuilt with the stream's rings like the plan's own.
     if (layered_) GF_TRY(ensure_chunk_arena());
     else if (tensor_prefill_ && count > 64u) GF_TRY(ensure_prefill_arena());
-    GF_TRY(bind_rings(set.ring_k[stream], set.ring_v[stream], set.positions_host[stream]));
+    GF_TRY(bind_rings(set.ring_k[stream], set.ring_v[stream], set.positions_host[stream], LayeredPlan::kStreamSlots));
     int status = ingest();
     if (status == GF_OK) {
         // The last prompt token's logits become the stream's row of the batch logits.
@@ -165,7 +165,9 @@ int Model::streams_ingest(StreamSet& set, uint32_t stream, uint32_t count, const
                                                                  cudaMemcpyHostToDevice, stream_), "position");
         if (status == GF_OK) status = check_cuda(cudaStreamSynchronize(stream_), "prefill");
     }
-    const int restored = bind_rings(home_k, home_v, home_position);
+    const int restored = bind_rings(home_k, home_v, home_position, layered_ ? layered_->own_slots : 0u);
+    state_floor_ = home_floor;
+    state_frontier_ = home_frontier;
     return status != GF_OK ? status : restored;
 }
 
@@ -173,7 +175,8 @@ int Model::streams_ingest(StreamSet& set, uint32_t stream, uint32_t count, const
 int Model::encode_stream_group(StreamSet& set, uint32_t first, uint32_t rows) {
     const gf_model_config& c = config_;
     if (layered_) {
-        GF_TRY(encode_layers(rows, true, LayeredRows{set.rings_dev + first, set.count, 1u, set.positions_dev + first, set.logits + (size_t)first * c.vocab}));
+        GF_TRY(encode_layers(rows, true, LayeredRows{set.rings_dev + first, set.count, 1u, set.positions_dev + first, set.logits + (size_t)first * c.vocab,
+                                                     layered_->slots_dev + 1}));
         GF_TRY(launch_stream_publish(set.publish_layers_dev, c.layers, set.rings_dev + first, set.count, set.positions_dev + first, rows, stream_));
         launches_ += 2;
         return GF_OK;
@@ -448,7 +451,8 @@ size_t Model::streams_kv_bytes(const StreamSet& set) const {
     for (uint32_t s = 0; s < set.count; ++s)
         for (uint32_t l = 0; l < config_.layers; ++l) {
             const uint32_t window = caches_[l].window, p = set.positions_host[s];
-            total += (size_t)(window ? std::min(window, p) : p) * cache_row_bytes(l) * (layered_ ? 1u : 2u);
+            total += (size_t)(window ? std::min(window, p) : p) * cache_row_bytes(l) * (layered_ ? layered_->cache_tensors(l) : 2u);
+            if (layered_) total += 2u * layered_->state_bytes(l);
         }
     return total;
 }

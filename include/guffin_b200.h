@@ -420,7 +420,10 @@ GF_API uint32_t gf_model_prefill_logits_row(const gf_model* model);
 GF_API int gf_model_select(gf_model* model, const void* requests_host, uint32_t rows);
 GF_API int gf_model_read_candidates(gf_model* model, void* results_host, uint32_t rows);
 GF_API int gf_model_read_logits(gf_model* model, uint32_t row, float* logits_host);
-/* A layered plan's cache holds one latent per position: `count` x rank values go to k_host, v_host is not written. */
+/* A layered plan's cache: a layer of latent attention holds one latent per position (`count` x rank values go to k_host,
+ * v_host is not written), one of grouped-query attention keys and values (`count` x kv_heads * dim and * vdim), a
+ * recurrent one a state instead: gf_model_read_state, [heads][vdim][N] f32 after the committed tokens. */
+GF_API int gf_model_read_state(gf_model* model, uint32_t layer, float* state_host);
 /* Committed K and V rows of one layer, positions [first_position, first_position + count), widened
  * to f32: `count` x kv_heads*head_dim values each.  Synchronises.  The rows must still be inside
  * the layer's ring (copy_tensor_from_backend on the plan's cache buffers, backend_buffer.hpp:47-68;

@@ -5,7 +5,8 @@ weights of those geometries.
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--impl ours|reference]
     python bench.py --workload streams [--streams S] [--prefix P] [--steps K] [--gpus N]
-    python bench.py --workload zasevik [--sizes dense-2048,...] [--steps K]      the layered design beside the Gemma 3 plan of equal size
+    python bench.py --workload zasevik [--sizes dense-2048,...] [--steps K]      a layered design beside the Gemma 3 plan of equal size
+    python bench.py --workload tufirax [--sizes hybrid-2048,...] [--steps K]     another one beside the Zasevik plan of equal size
     torchrun ... bench.py --gpus N --workload tp [--h1] [--exchange peer|nccl]     one stream, the 12B target sharded over N GPUs
     python bench.py --horizon H [--conditional]                                   chains of H drafts per cycle
     python bench.py --case matmul <dtype 8|12|14> <K> <N> <rows> [launches]
@@ -566,6 +567,105 @@ def run_zasevik(args) -> dict:
     }
 
 
+# Sizes of the tufirax workload: attention layers with a feed-forward, state-space layers, or the two in turn.
+TUFIRAX_SIZES = {
+    "hybrid-2048": dict(width=2048, kinds="as", heads=16, kv_heads=4, ff=8192, state_heads=64),
+    "attention-2048": dict(width=2048, kinds="a", heads=16, kv_heads=4, ff=8192, state_heads=64),
+    "state-2048": dict(width=2048, kinds="s", heads=16, kv_heads=4, ff=8192, state_heads=64),
+    "hybrid-4096": dict(width=4096, kinds="as", heads=32, kv_heads=8, ff=14336, state_heads=128),
+}
+
+
+def tufirax_size(name: str) -> dict:
+    from guffin_b200 import synthetic as syn
+    size = TUFIRAX_SIZES[name]
+    layers = {"a": syn.tufirax_attention(size["heads"], size["kv_heads"], 128, ff=size["ff"]),
+              "s": syn.tufirax_state_space(size["state_heads"], 64, 128, groups=8, norm_groups=8)}
+    return syn.tufirax_config(size["width"], ZASEVIK_VOCAB, [layers[size["kinds"][i % len(size["kinds"])]] for i in range(ZASEVIK_LAYERS)])
+
+
+def equal_zasevik(config: dict) -> dict:
+    """The Zasevik configuration of equal width whose layers have as many matrix elements."""
+    from guffin_b200 import synthetic as syn
+    width, heads = config["width"], config["width"] // 128
+    per_layer = (syn.tufirax_active_parameters(config) - config["vocab"] * width) / ZASEVIK_LAYERS
+    attention = 2 * heads * 128 * width + 512 * width + 2 * heads * 128 * 512
+    ff = max(64, int(round((per_layer - attention) / (2 * width) / 64)) * 64)
+    return syn.zasevik_config(width, ZASEVIK_LAYERS, heads, 128, 128, 512, ZASEVIK_VOCAB, [syn.dense_mlp(ff)])
+
+
+def tufirax_prefill_flops(config: dict, prefix: int) -> float:
+    """Products of every token, scores and outputs of attention, and six operations per element of a state."""
+    from guffin_b200 import synthetic as syn
+    total = 2.0 * (syn.tufirax_active_parameters(config) - config["vocab"] * config["width"]) * prefix
+    for layer in config["layers"]:
+        m = layer["mixer"]
+        if layer["type"] == "attention":
+            total += 4.0 * m["heads"] * m["dim"] * prefix * (prefix + 1) / 2
+        else:
+            total += 6.0 * m["heads"] * m["vdim"] * m["state"] * prefix
+    return total
+
+
+def run_tufirax(args) -> dict:
+    """Prefill and decode throughput at a few sizes, beside the Zasevik plan of equal width and parameter count."""
+    from guffin_b200 import engine as ge, lib, model as gm, synthetic as syn
+    L = lib.load()
+    lib.check(L.gf_set_device(0))
+    peak, peak_kind = load_peaks()
+    with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")) else open(os.devnull) as f:
+        text = f.read()
+    tensor_peak = float(json.loads(text)["bf16_tflops"]) if text else 1590.0
+    prefix, steps, warmup = args.prefix if args.prefix != 8192 else 2048, args.steps, max(args.warmup, 3)
+    names = (args.sizes or ",".join(TUFIRAX_SIZES)).split(",")
+    prompt = np.random.default_rng(SEEDS["prompt"]).integers(0, ZASEVIK_VOCAB, prefix).astype(np.uint32)
+    context = prefix + 2 * (warmup + steps) + 16
+    sizes, launches = {}, 0
+    clocks = ClockSampler(0)
+    for name in names:
+        config = tufirax_size(name)
+        other = equal_zasevik(config)
+        keys = prefix * (prefix + 1) / 2
+        flops = {"tufirax": tufirax_prefill_flops(config, prefix),
+                 "zasevik": 2.0 * (syn.zasevik_active_parameters(other) - other["vocab"] * other["width"]) * prefix
+                 + sum(2.0 * l["mixer"]["heads"] * (l["mixer"]["dim"] + l["mixer"]["vdim"]) * keys for l in other["layers"])}
+        active = {"tufirax": syn.tufirax_active_parameters(config), "zasevik": syn.zasevik_active_parameters(other)}
+        sizes[name] = {}
+        for kind, described, weights in (("tufirax", config, syn.iter_tufirax_weights), ("zasevik", other, syn.iter_zasevik_weights)):
+            plan = gm.Model.described(described, weights(described, SEEDS["target"]), context, 2)
+            with clocks:
+                row = time_plan(lib, plan, prompt, steps, warmup)
+            row["weight_bytes_per_token"] = 2 * active[kind]
+            row["decode_gbs"] = (2 * active[kind] + row["kv_bytes"]) / row["decode_ms"] / 1e6
+            row["decode_frac"] = row["decode_gbs"] / peak
+            row["prefill_tflops"] = flops[kind] / row["prefill_ms"] / 1e9
+            row["prefill_frac"] = row["prefill_tflops"] / tensor_peak
+            if kind == "tufirax":
+                launches += int(row["launches_per_token"] * steps)
+                engine = ge.H1(plan, None, ge.H1Options(ge.sampler_options(0.0), 0, 0, 0.0, 0, 0))
+                engine.prefill(prompt)
+                engine.generate(warmup)
+                t0 = time.perf_counter()
+                engine.generate(steps)
+                row["e2e_decode_tok_s"] = steps / (time.perf_counter() - t0)
+                engine.close()
+            plan.close()
+            sizes[name][kind] = row
+    first = sizes[names[0]]["tufirax"]
+    return {
+        "metric": "Tufirax decode tok/s, one stream", "value": first["decode_tok_s"], "unit": "tok/s", "n_gpus": 1, "steps": steps, "warmup": warmup,
+        "ms_per_step": first["decode_ms"], "higher_is_better": True, "scaling": "weak", "vs_baseline": None,
+        "dtype": "bf16 weights, f32 activations and states, binary16 keys and values", "data": "synthetic",
+        "config": {"workload": f"{ZASEVIK_LAYERS} layers of each size, {prefix}-token prompt, one-row passes behind it; beside it the Zasevik plan of equal width and "
+                               "parameter count", "sizes": names, "layers": ZASEVIK_LAYERS, "vocab": ZASEVIK_VOCAB,
+                   "l2_policy": "a pass reads its weights once; sizes whose weights exceed L2 (all of them) defeat it"},
+        "e2e": {"value": first["e2e_decode_tok_s"], "unit": "tok/s", "h2d_bytes_per_step": 4 + 264, "d2h_bytes_per_step": 3080},
+        "gpu_launches": launches,
+        "roofline": {"bound": "hbm", "achieved": first["decode_gbs"], "peak": peak, "unit": "GB/s", "frac": first["decode_frac"], "peak_source": f"of {peak_kind}"},
+        "sizes": sizes, "clocks": clocks.summary(),
+    }
+
+
 def run_tensor_parallel_h1(args, plan, shard, dist, world, rank, local, context, prompt, load_s, prefill_s) -> dict:
     """The headline's H1 cycle with the target sharded over the ranks: every rank runs its own engine on its shard
     and its own replica of the drafter, with the same seeds; the shards' merged candidate rows are identical, so
@@ -1009,10 +1109,10 @@ def main():
                         help="0: one kernel per operator (CUDA graph, the default); 1: persistent decode pass kernel; "
                              "2: pass kernel with attention launched separately")
     parser.add_argument("--case", nargs="+", default=None, help="run one single-kernel case instead of the benchmark")
-    parser.add_argument("--workload", choices=("h1", "streams", "tp", "zasevik"), default="h1",
+    parser.add_argument("--workload", choices=("h1", "streams", "tp", "zasevik", "tufirax"), default="h1",
                         help="h1: the headline (configs[3]); streams: configs[4]; tp: one 12B stream sharded over the GPUs; "
-                             "zasevik: prefill and decode of the layered design beside the Gemma 3 plan of equal size")
-    parser.add_argument("--sizes", default=",".join(ZASEVIK_SIZES), help="zasevik workload: sizes to run, with commas between them")
+                             "zasevik, tufirax: prefill and decode of a layered design beside another plan of equal size")
+    parser.add_argument("--sizes", default=None, help="zasevik and tufirax workloads: sizes to run, with commas between them (default: all)")
     parser.add_argument("--horizon", type=int, default=1, help="drafts per cycle of the h1 workload (1 = the headline; 2..7 = chains)")
     parser.add_argument("--conditional", action="store_true",
                         help="h1 workload with --horizon > 2: verify the chain as a cascade of passes (the reference's conditional tiles)")
@@ -1034,7 +1134,12 @@ def main():
     elif args.workload == "zasevik" and args.impl == "ours":
         args.steps = 64 if args.steps is None else args.steps
         args.warmup = 5 if args.warmup is None else args.warmup
+        args.sizes = args.sizes or ",".join(ZASEVIK_SIZES)
         result = run_zasevik(args)
+    elif args.workload == "tufirax" and args.impl == "ours":
+        args.steps = 64 if args.steps is None else args.steps
+        args.warmup = 5 if args.warmup is None else args.warmup
+        result = run_tufirax(args)
     elif args.workload == "tp" and args.impl == "ours":
         args.steps = 100 if args.steps is None else args.steps
         args.warmup = 5 if args.warmup is None else args.warmup

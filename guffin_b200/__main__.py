@@ -47,7 +47,8 @@ def info(args) -> None:
         print(f"width {config['width']}, {len(layers)} layers")
         for i, layer in enumerate(layers):
             mlp = layer.get("mlp") or {"kind": "none"}
-            print(f"  {i}: {layer['type']} {json.dumps(layer['mixer'])}  {mlp['kind']} {json.dumps({k: v for k, v in mlp.items() if k != 'kind'})}")
+            shared = f"  tensors of layer {layer['weights_of']}" if "weights_of" in layer else ""
+            print(f"  {i}: {layer['type']} {json.dumps(layer['mixer'])}  {mlp['kind']} {json.dumps({k: v for k, v in mlp.items() if k != 'kind'})}{shared}")
     else:
         print(json.dumps({k: v for k, v in config.items() if k not in ("architecture", "vocab")}))
 

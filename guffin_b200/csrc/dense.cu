@@ -293,8 +293,39 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
             }
         }
     } else if (p.input == kRowPartNorm) {
-        // Warps share the parts: several to a part where there are fewer parts than warps.
         const uint32_t part = p.width / p.norm_parts;
+        if (quads && part % 128u == 0u && p.norm_parts <= kRowThreads && p.width <= kMaxExperts * 128u) {
+            // Sums of 128 values at a time, a warp's 16-byte pieces.
+            for (int r = 0; r < R; ++r) {
+                const float* x = p.in + (size_t)r * p.in_ld;
+#pragma unroll 8
+                for (uint32_t i = tid * 4u; i < p.width; i += kRowThreads * 4u) {
+                    const float4 v = *reinterpret_cast<const float4*>(x + i);
+                    *reinterpret_cast<float4*>(act + r * k_pad + i) = v;
+                    const float sum = warp_sum(dot4(v, v));
+                    if (lane == 0) route_scratch[i / 128u] = sum;
+                }
+                __syncthreads();
+                float inv = 0.0f;
+                if (tid < p.norm_parts) {
+                    for (uint32_t s = 0; s < part / 128u; ++s) inv += route_scratch[tid * (part / 128u) + s];
+                    inv = norm_factor(inv, part, p.eps);
+                }
+                __syncthreads();
+                if (tid < p.norm_parts) route_scratch[tid] = inv;
+                __syncthreads();
+#pragma unroll 4
+                for (uint32_t i = tid * 4u; i < p.width; i += kRowThreads * 4u) {
+                    const float4 g = *reinterpret_cast<const float4*>(p.gain1 + i);
+                    float4* at = reinterpret_cast<float4*>(act + r * k_pad + i);
+                    const float f = route_scratch[i / part];
+                    *at = make_float4(at->x * f * g.x, at->y * f * g.y, at->z * f * g.z, at->w * f * g.w);
+                }
+                for (uint32_t i = p.width + tid; i < k_pad; i += kRowThreads) act[r * k_pad + i] = 0.0f;
+                __syncthreads();
+            }
+        } else {
+        // Warps share the parts: several to a part where there are fewer parts than warps.
         uint32_t per = kRowWarps;
         while (per > 1u && per * p.norm_parts > kRowWarps) per /= 2u;
         for (int r = 0; r < R; ++r) {
@@ -321,6 +352,7 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
                 act[r * k_pad + i] = v;
             }
             __syncthreads();
+        }
         }
     } else if (p.input == kRowLatent) {
         for (int r = 0; r < R; ++r) {
@@ -503,7 +535,7 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
     if (p.input == kRowPartNorm && (p.norm_parts == 0 || p.norm_parts > kMaxNormParts || p.width % p.norm_parts)) return fail(GF_ERR_INVALID, "row product: %u norm parts of %u", p.norm_parts, p.width);
     auto whole = [](const void* pointer) { return (reinterpret_cast<uintptr_t>(pointer) & 15u) == 0u; };
     p.vector_rows = p.in_ld % 4u == 0u && p.in_batch % 4u == 0u && p.in2_ld % 4u == 0u && p.part_stride % 4u == 0u && whole(p.in) && whole(p.in2);
-    if (p.input == kRowNorm || p.input == kRowAddNorm)
+    if (p.input == kRowNorm || p.input == kRowAddNorm || p.input == kRowPartNorm)
         p.vector_rows = p.vector_rows && p.width % 4u == 0u && whole(p.residual) && whole(p.residual_out) && whole(p.gain0) && whole(p.gain1) && whole(p.normed_out);
     for (uint32_t i = 0; i < p.count; ++i) p.vector_rows = p.vector_rows && p.m[i].k % 4u == 0u;
     const uint32_t row_bytes = p.k_pad * 4u;

@@ -305,11 +305,57 @@ __device__ __forceinline__ float block_total(float v, float* scratch) {
 }
 
 __global__ void __launch_bounds__(256) chunk_norm_kernel(const ChunkNorm p) {
-    extern __shared__ float row_values[];
+    extern __shared__ __align__(16) float row_values[];
     __shared__ float scratch[8];
     const uint32_t row = blockIdx.x;
     float* residual = p.residual + (size_t)row * p.width;
     float sum = 0.0f;
+    if (p.width % 8u == 0u && !p.slots && !p.result.f32) {             // whole 16-byte pieces
+        auto octet = [](float* to, const float* from) {
+#pragma unroll
+            for (int j = 0; j < 8; j += 4) *reinterpret_cast<float4*>(to + j) = *reinterpret_cast<const float4*>(from + j);
+        };
+        float v[8], g[8];
+        if (p.y) {
+            for (uint32_t i = threadIdx.x * 8u; i < p.width; i += blockDim.x * 8u) {
+                octet(v, p.y + (size_t)row * p.width + i);
+                octet(row_values + i, v);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) sum = fmaf(v[j], v[j], sum);
+            }
+            const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps);
+            sum = 0.0f;
+            for (uint32_t i = threadIdx.x * 8u; i < p.width; i += blockDim.x * 8u) {
+                float x[8];
+                octet(v, residual + i);
+                octet(x, row_values + i);
+                octet(g, p.gain0 + i);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) { v[j] += x[j] * inv * g[j]; sum = fmaf(v[j], v[j], sum); }
+                octet(residual + i, v);
+                octet(row_values + i, v);
+            }
+        } else {
+            for (uint32_t i = threadIdx.x * 8u; i < p.width; i += blockDim.x * 8u) {
+                octet(v, residual + i);
+                octet(row_values + i, v);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) sum = fmaf(v[j], v[j], sum);
+            }
+        }
+        const float inv = p.gain1 ? 1.0f / sqrtf(block_total(sum, scratch) / (float)p.width + p.eps) : 1.0f;
+        for (uint32_t i = threadIdx.x * 8u; i < p.width; i += blockDim.x * 8u) {
+            octet(v, row_values + i);
+            if (p.gain1) {
+                octet(g, p.gain1 + i);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = v[j] * inv * g[j];
+            }
+            if (p.result.data) *reinterpret_cast<uint4*>(static_cast<uint8_t*>(p.result.data) + operand_offset(p.result, row, i)) = bf16_octet(v);
+            if (p.normed) octet(p.normed + (size_t)row * p.width + i, v);
+        }
+        return;
+    }
     if (p.y) {
         for (uint32_t i = threadIdx.x; i < p.width; i += blockDim.x) {
             float v;
@@ -347,7 +393,7 @@ __global__ void __launch_bounds__(256) chunk_norm_kernel(const ChunkNorm p) {
 // Block = (row, part): the part by its own root mean square.
 __global__ void __launch_bounds__(256) chunk_part_norm_kernel(const float* __restrict__ x, uint32_t x_ld, const float* __restrict__ gate, uint32_t gate_ld, uint32_t part, const float* __restrict__ gain, float eps,
                                                               const Operand result) {
-    extern __shared__ float row_values[];
+    extern __shared__ __align__(16) float row_values[];
     __shared__ float scratch[8];
     const uint32_t row = blockIdx.x, first = blockIdx.y * part;
     const float *in = x + (size_t)row * x_ld + first, *z = gate + (size_t)row * gate_ld + first;
@@ -359,6 +405,36 @@ __global__ void __launch_bounds__(256) chunk_part_norm_kernel(const float* __res
     }
     const float inv = 1.0f / sqrtf(block_total(sum, scratch) / (float)part + eps);
     for (uint32_t i = threadIdx.x; i < part; i += blockDim.x) store_operand(result, row, first + i, row_values[i] * inv * gain[first + i]);
+}
+
+// The same for parts of whole 256 values, bf16: block = row, a thread takes eight values at a time.
+__global__ void __launch_bounds__(256) chunk_part_norm_octets_kernel(const float* __restrict__ x, uint32_t x_ld, const float* __restrict__ gate, uint32_t gate_ld,
+                                                                     uint32_t width, uint32_t part, const float* __restrict__ gain, float eps, const Operand result) {
+    extern __shared__ __align__(16) float row_values[];                // [width], then a sum per 256 values
+    float* sums = row_values + width;
+    const uint32_t row = blockIdx.x;
+    for (uint32_t i = threadIdx.x * 8u; i < width; i += blockDim.x * 8u) {
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = 0; j < 8; j += 4) {
+            const float4 v = *reinterpret_cast<const float4*>(x + (size_t)row * x_ld + i + j), z = *reinterpret_cast<const float4*>(gate + (size_t)row * gate_ld + i + j);
+            const float4 y = make_float4(v.x * silu(z.x), v.y * silu(z.y), v.z * silu(z.z), v.w * silu(z.w));
+            *reinterpret_cast<float4*>(row_values + i + j) = y;
+            sum = fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, fmaf(y.w, y.w, sum))));
+        }
+        sum = warp_sum(sum);
+        if ((threadIdx.x & 31u) == 0u) sums[i / 256u] = sum;
+    }
+    __syncthreads();
+    for (uint32_t i = threadIdx.x * 8u; i < width; i += blockDim.x * 8u) {
+        const uint32_t first = i / part * (part / 256u);
+        float sum = 0.0f, v[8];
+        for (uint32_t s = 0; s < part / 256u; ++s) sum += sums[first + s];
+        const float inv = 1.0f / sqrtf(sum / (float)part + eps);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = row_values[i + j] * inv * gain[i + j];
+        *reinterpret_cast<uint4*>(static_cast<uint8_t*>(result.data) + operand_offset(result, row, i)) = bf16_octet(v);
+    }
 }
 
 // A warp per row chooses its experts.
@@ -500,9 +576,15 @@ int launch_chunk_part_norm(const float* x, uint32_t x_ld, const float* gate, uin
         || width / parts > 48u * 1024u)
         return fail(GF_ERR_INVALID, "chunk part norm: bad arguments");
     const uint32_t part = width / parts;
-    static std::once_flag once[64];
-    const int status = allow_smem(chunk_part_norm_kernel, once, 200u * 1024u);
+    static std::once_flag once[2][64];
+    int status = allow_smem(chunk_part_norm_kernel, once[0], 200u * 1024u);
+    if (status == GF_OK) status = allow_smem(chunk_part_norm_octets_kernel, once[1], 200u * 1024u);
     if (status != GF_OK) return status;
+    if (part % 256u == 0u && x_ld % 4u == 0u && gate_ld % 4u == 0u && width <= 40u * 1024u && !result.f32) {
+        chunk_part_norm_octets_kernel<<<rows, 256, (width + width / 256u) * 4u, stream>>>(x, x_ld, gate, gate_ld, width, part, gain, eps, result);
+        GF_CUDA(cudaGetLastError());
+        return GF_OK;
+    }
     chunk_part_norm_kernel<<<dim3(rows, parts), part >= 256u ? 256u : (part + 31u) / 32u * 32u, part * 4u, stream>>>(x, x_ld, gate, gate_ld, part, gain, eps, result);
     GF_CUDA(cudaGetLastError());
     return GF_OK;

@@ -33,12 +33,30 @@ __device__ __forceinline__ uint32_t half_pair(float lo, float hi) {
 
 constexpr uint32_t kPrepareThreads = 256;
 
-// Cosine and sine of position * frequency: the angle in double, its remainder of a turn in f32.
+// Cosine and sine of position * frequency: the turns in double, their remainder in f32.
 __device__ __forceinline__ float2 rotation(uint32_t position, double frequency) {
-    const double angle = (double)position * frequency, turns = rint(angle * 0.15915494309189535);
+    const double turns = (double)position * frequency * 0.15915494309189535;      // 1 / (2 pi)
     float s, c;
-    sincosf((float)fma(turns, -6.283185307179586, angle), &s, &c);
+    sincospif((float)(2.0 * (turns - rint(turns))), &s, &c);
     return make_float2(c, s);
+}
+
+// Dimension d of a head that starts at `first` of a projected row: normalised, turned.
+__device__ __forceinline__ float turned(const QueryKey& p, const float* x, const float* gain, float inv, const float2* turn, uint32_t first, uint32_t d) {
+    const float here = x[first + d] * inv * gain[first + d];
+    if (d >= p.rotated) return here;
+    const uint32_t half = p.rotated / 2u, i = d < half ? d : d - half, other = first + (d < half ? d + half : i);
+    const float there = x[other] * inv * gain[other];
+    return d < half ? here * turn[i].x - there * turn[i].y : here * turn[i].x + there * turn[i].y;
+}
+__device__ __forceinline__ __half cache_half(const QueryKey& p, float value) {
+    const __half h = __float2half_rn(value);
+    if (__hisinf(h) || __hisnan(h)) atomicOr(p.status, kStatusKvNonFinite);
+    return h;
+}
+__device__ __forceinline__ void store_cache(const QueryKey& p, void* to, size_t at, float value) {
+    if (p.f32) static_cast<float*>(to)[at] = value;
+    else static_cast<__half*>(to)[at] = cache_half(p, value);
 }
 
 __global__ void __launch_bounds__(kPrepareThreads) query_key_kernel(const __grid_constant__ QueryKey p) {
@@ -64,30 +82,49 @@ __global__ void __launch_bounds__(kPrepareThreads) query_key_kernel(const __grid
     q_sum = k_sum = 0.0f;
     for (uint32_t w = 0; w < kPrepareThreads / 32u; ++w) { q_sum += sums[w][0]; k_sum += sums[w][1]; }
     const float q_inv = 1.0f / sqrtf(q_sum / (float)q_width + p.eps), k_inv = 1.0f / sqrtf(k_sum / (float)k_width + p.eps);
-    auto turned = [&](const float* x, const float* gain, float inv, uint32_t first, uint32_t d) {
-        const float here = x[first + d] * inv * gain[first + d];
+    // Dimensions d and d + 1 of a head that starts at `first`.
+    auto turned2 = [&](const float* x, const float* gain, float inv, uint32_t first, uint32_t d) {
+        const float2 v = *reinterpret_cast<const float2*>(x + first + d), w = *reinterpret_cast<const float2*>(gain + first + d);
+        const float2 here = make_float2(v.x * inv * w.x, v.y * inv * w.y);
         if (d >= p.rotated) return here;
-        const uint32_t i = d < half ? d : d - half, other = first + (d < half ? d + half : i);
-        const float there = x[other] * inv * gain[other];
-        return d < half ? here * turn[i].x - there * turn[i].y : here * turn[i].x + there * turn[i].y;
+        const bool lower = d < half;
+        const uint32_t i = lower ? d : d - half, other = first + (lower ? d + half : i);
+        const float2 ov = *reinterpret_cast<const float2*>(x + other), ow = *reinterpret_cast<const float2*>(gain + other);
+        const float2 there = make_float2(ov.x * inv * ow.x, ov.y * inv * ow.y), a = turn[i], c = turn[i + 1u];
+        return lower ? make_float2(here.x * a.x - there.x * a.y, here.y * c.x - there.y * c.y) : make_float2(here.x * a.x + there.x * a.y, here.y * c.x + there.y * c.y);
     };
-    auto store = [&](void* to, size_t at, float value) {
-        if (p.f32) { static_cast<float*>(to)[at] = value; return; }
-        const __half h = __float2half_rn(value);
-        if (__hisinf(h) || __hisnan(h)) atomicOr(p.status, kStatusKvNonFinite);
-        static_cast<__half*>(to)[at] = h;
-    };
-    if (q)
+    if (!p.f32 && p.pairs) {
+        auto store2 = [&](void* to, size_t at, float2 v) {
+            const __half2 h = __floats2half2_rn(v.x, v.y);
+            if (__hisinf(h.x) || __hisnan(h.x) || __hisinf(h.y) || __hisnan(h.y)) atomicOr(p.status, kStatusKvNonFinite);
+            *reinterpret_cast<__half2*>(static_cast<__half*>(to) + at) = h;
+        };
+        const float2 zero = make_float2(0.0f, 0.0f);
+        if (q)
 #pragma unroll 4
+            for (uint32_t i = tid * 2u; i < p.heads * p.row_head; i += kPrepareThreads * 2u) {
+                const uint32_t head = i / p.row_head, d = i % p.row_head;
+                float2 v = d < p.dim ? turned2(q, p.q_gain, q_inv, head * p.dim, d) : zero;
+                store2(p.q, (size_t)row * p.heads * p.row_head + i, make_float2(v.x * p.scale, v.y * p.scale));
+            }
+        for (uint32_t i = tid * 2u; i < p.kv_heads * p.row_head; i += kPrepareThreads * 2u) {
+            const uint32_t head = i / p.row_head, d = i % p.row_head;
+            const size_t at = (size_t)row * p.kv_heads * p.row_head + i;
+            store2(p.keys, at, d < p.dim ? turned2(k, p.k_gain, k_inv, head * p.dim, d) : zero);
+            store2(p.values, at, d < p.vdim ? *reinterpret_cast<const float2*>(v + head * p.vdim + d) : zero);
+        }
+        return;
+    }
+    if (q)
         for (uint32_t i = tid; i < p.heads * p.row_head; i += kPrepareThreads) {
             const uint32_t head = i / p.row_head, d = i % p.row_head;
-            store(p.q, (size_t)row * p.heads * p.row_head + i, d < p.dim ? turned(q, p.q_gain, q_inv, head * p.dim, d) * p.scale : 0.0f);
+            store_cache(p, p.q, (size_t)row * p.heads * p.row_head + i, d < p.dim ? turned(p, q, p.q_gain, q_inv, turn, head * p.dim, d) * p.scale : 0.0f);
         }
     for (uint32_t i = tid; i < p.kv_heads * p.row_head; i += kPrepareThreads) {
         const uint32_t head = i / p.row_head, d = i % p.row_head;
         const size_t at = (size_t)row * p.kv_heads * p.row_head + i;
-        store(p.keys, at, d < p.dim ? turned(k, p.k_gain, k_inv, head * p.dim, d) : 0.0f);
-        store(p.values, at, d < p.vdim ? v[head * p.vdim + d] : 0.0f);
+        store_cache(p, p.keys, at, d < p.dim ? turned(p, k, p.k_gain, k_inv, turn, head * p.dim, d) : 0.0f);
+        store_cache(p, p.values, at, d < p.vdim ? v[head * p.vdim + d] : 0.0f);
     }
 }
 
@@ -122,13 +159,76 @@ __device__ __forceinline__ void merge_query(const GroupedAttention& p, uint32_t 
     merge_factors(pairs, p.parts, p.sink ? p.sink[head] : -INFINITY, factors);
     __syncwarp();
     const float gate = head_gate(p, row, head);
-    for (uint32_t d = lane; d < p.vdim; d += 32u) {
-        float v = 0.0f;
-#pragma unroll 8
-        for (uint32_t part = 0; part < p.parts; ++part) v = fmaf(__ldcg(p.partial_out + (query * p.parts + part) * p.row_head + d), factors[part], v);
-        store_operand(p.result, row, head * p.vdim + d, v * gate);
+    for (uint32_t d = lane * 4u; d < p.vdim; d += 128u) {              // a row's head is whole 16-byte pieces
+        const float4* from = reinterpret_cast<const float4*>(p.partial_out + query * p.parts * p.row_head + d);
+        float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 16
+        for (uint32_t part = 0; part < p.parts; ++part) {
+            const float4 x = __ldcg(from + part * (p.row_head / 4u));
+            const float f = factors[part];
+            v = make_float4(fmaf(x.x, f, v.x), fmaf(x.y, f, v.y), fmaf(x.z, f, v.z), fmaf(x.w, f, v.w));
+        }
+        const float four[4] = {v.x * gate, v.y * gate, v.z * gate, v.w * gate};
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j)
+            if (d + j < p.vdim) store_operand(p.result, row, head * p.vdim + d + j, four[j]);
     }
     __syncwarp();
+}
+
+// The prologue of a fused pass: the block's queries (zeros behind them) and the pass's own keys and values of key/value
+// head `kv`, prepared from the projections.  Rows [first_row, first_row + query_rows) have queries here; with `own` all
+// of `rows` leave their cache rows in own_k and own_v, and with `publish` in the private rows too.
+struct FusedRows { uint32_t first_row, query_rows, rows, row0; bool own, publish; };
+template <int kThreads>
+__device__ __forceinline__ void prepare_fused(const GroupedAttention& p, const FusedRows& f, const float2* turns, uint32_t kv, uint32_t first_query, uint32_t queries,
+                                              __half* q_tile, __half* own_k, __half* own_v, uint32_t stride) {
+    constexpr uint32_t kWarps = kThreads / 32u, kItems = 16u + kGroupedFusedRows;
+    __shared__ float sums[kItems][kWarps];
+    const QueryKey& in = p.prepare;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, group = p.heads / p.kv_heads, half = in.rotated / 2u;
+    const uint32_t q_width = in.heads * in.dim, k_width = in.kv_heads * in.dim, items = f.query_rows + (f.own ? f.rows : 0u);
+    for (uint32_t item = 0; item < items; ++item) {
+        const bool query = item < f.query_rows;
+        const uint32_t row = f.row0 + (query ? f.first_row + item : item - f.query_rows), width = query ? q_width : k_width;
+        const float* x = query ? in.raw_q + (size_t)row * in.q_ld : in.raw_k + (size_t)row * in.k_ld;
+        float sum = 0.0f;
+#pragma unroll 8
+        for (uint32_t i = threadIdx.x; i < width; i += kThreads) sum = fmaf(x[i], x[i], sum);
+        sum = warp_sum(sum);
+        if (lane == 0) sums[item][warp] = sum;
+    }
+    __syncthreads();
+    auto inverse = [&](uint32_t item, uint32_t width) {
+        float sum = 0.0f;
+#pragma unroll
+        for (uint32_t w = 0; w < kWarps; ++w) sum += sums[item][w];
+        return 1.0f / sqrtf(sum / (float)width + in.eps);
+    };
+    for (uint32_t m = warp; m < 16u; m += kWarps) {
+        const uint32_t query = first_query + m;
+        const bool valid = query < queries;
+        const uint32_t r = valid ? query / group : 0u, first = (kv * group + query % group) * in.dim;
+        const float inv = valid ? inverse(r - f.first_row, q_width) : 0.0f;
+        const float* x = in.raw_q + (size_t)(f.row0 + r) * in.q_ld;
+#pragma unroll 4
+        for (uint32_t d = lane; d < p.row_head; d += 32u)
+            q_tile[m * stride + d] = valid && d < in.dim ? cache_half(in, turned(in, x, in.q_gain, inv, turns + r * half, first, d) * in.scale) : __float2half_rn(0.0f);
+    }
+    if (!f.own) return;
+    for (uint32_t r = warp; r < f.rows; r += kWarps) {
+        const float inv = inverse(f.query_rows + r, k_width);
+        const float *x = in.raw_k + (size_t)(f.row0 + r) * in.k_ld, *v = in.raw_v + (size_t)(f.row0 + r) * in.v_ld + kv * in.vdim;
+        const size_t to = ((size_t)(f.row0 + r) * p.kv_heads + kv) * p.row_head;
+#pragma unroll 4
+        for (uint32_t d = lane; d < p.row_head; d += 32u) {
+            const __half key = d < in.dim ? cache_half(in, turned(in, x, in.k_gain, inv, turns + r * half, kv * in.dim, d)) : __float2half_rn(0.0f);
+            const __half value = d < in.vdim ? cache_half(in, v[d]) : __float2half_rn(0.0f);
+            own_k[r * stride + d] = key;
+            own_v[r * stride + d] = value;
+            if (f.publish) { static_cast<__half*>(in.keys)[to + d] = key; static_cast<__half*>(in.values)[to + d] = value; }
+        }
+    }
 }
 
 constexpr uint32_t kRowsWarps = 4;
@@ -146,25 +246,27 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
     __half* q_tile = reinterpret_cast<__half*>(smem);
     __half* tiles = q_tile + 16u * stride;                             // [warps][2][keys, values][kTile][stride]
     __half* mine = tiles + (size_t)warp * 4u * kTile * stride;
+    __half* own_rows = tiles + (size_t)kRowsWarps * 4u * kTile * stride;           // fused: [keys, values][rows][stride], then the turns
     const bool chain = p.ring_stride == 0u;
     const uint32_t kv = blockIdx.z % p.kv_heads, z = blockIdx.z / p.kv_heads, part = blockIdx.y;
     const uint32_t group = p.heads / p.kv_heads, queries = (chain ? p.rows : 1u) * group, first_query = blockIdx.x * 16u;
     const uint32_t base = p.positions[z], cache_row = p.kv_heads * p.row_head;
     const StreamRings rings = p.rings[(size_t)z * p.ring_stride];
     const uint32_t end = base + min(first_query + 15u, queries - 1u) / group + 1u;      // keys the block's last query sees
-    const uint32_t all = (end + kTile - 1u) / kTile, step = kRowsWarps;
+    const uint32_t all = (end + kTile - 1u) / kTile;
+    constexpr uint32_t step = kRowsWarps;
     const uint32_t tile_begin = (uint32_t)((uint64_t)all * part / p.parts), tile_end = (uint32_t)((uint64_t)all * (part + 1u) / p.parts);
     const __half *ring_k = static_cast<const __half*>(rings.ring_k) + kv * p.row_head, *ring_v = static_cast<const __half*>(rings.ring_v) + kv * p.row_head;
     const size_t own_at = (size_t)(chain ? 0u : z) * cache_row + kv * p.row_head;
     const __half *own_k = static_cast<const __half*>(p.own_k) + own_at, *own_v = static_cast<const __half*>(p.own_v) + own_at;
 
+    const uint32_t copied = p.fused ? base : end;                      // a fused pass has its own rows in shared memory
     auto load_tile = [&](uint32_t tile, uint32_t slot) {
         __half *kd = mine + slot * 2u * kTile * stride, *vd = kd + kTile * stride;
 #pragma unroll
         for (uint32_t r0 = 0; r0 < kTile; r0 += 4u) {                  // four rows at a time, eight lanes each
             const uint32_t r = r0 + (lane >> 3), position = tile * kTile + r;
-            const bool valid = position < end;
-            const bool cached = position < base;
+            const bool valid = position < copied, cached = position < base;
             const size_t at = valid ? (size_t)(cached ? position & p.ring_mask : position - base) * cache_row : 0u;
             const __half *ks = (cached ? ring_k : own_k) + at, *vs = (cached ? ring_v : own_v) + at;
             for (uint32_t piece = lane & 7u; piece < pieces; piece += 8u) {
@@ -173,11 +275,28 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
             }
         }
     };
-    pdl_wait();
-    pdl_launch_dependents();
-    if (tile_begin + warp < tile_end) load_tile(tile_begin + warp, 0u);
-    copies_commit();
-    {
+    const uint32_t rows = chain ? p.rows : 1u;
+    __half *my_k = own_rows, *my_v = own_rows + rows * stride;
+    if (p.fused) {
+        // Cached rows and positions were written at least two launches back: read ahead of the wait.
+        if (tile_begin + warp < tile_end) load_tile(tile_begin + warp, 0u);
+        copies_commit();
+        float2* turns = reinterpret_cast<float2*>(own_rows + 2u * rows * stride);
+        const uint32_t half = p.prepare.rotated / 2u;
+        for (uint32_t i = tid; i < rows * half; i += kRowsWarps * 32u) turns[i] = rotation(base + i / half, p.prepare.frequencies[i % half]);
+        const uint32_t last_query = min(first_query + 15u, queries - 1u);
+        FusedRows f;
+        f.first_row = first_query / group; f.query_rows = last_query / group - f.first_row + 1u; f.rows = rows; f.row0 = chain ? 0u : z;
+        f.publish = part + 1u == p.parts && blockIdx.x + 1u == gridDim.x;
+        f.own = tile_end * kTile > base;
+        pdl_wait();
+        pdl_launch_dependents();
+        prepare_fused<kRowsWarps * 32>(p, f, turns, kv, first_query, queries, q_tile, my_k, my_v, stride);
+    } else {
+        pdl_wait();
+        pdl_launch_dependents();
+        if (tile_begin + warp < tile_end) load_tile(tile_begin + warp, 0u);
+        copies_commit();
         const __half* q = static_cast<const __half*>(p.q);
         for (uint32_t m = tid >> 3; m < 16u; m += kRowsWarps * 4u) {
             const uint32_t query = first_query + m;
@@ -205,7 +324,15 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         copies_commit();
         copies_wait<1>();
         __syncwarp();
-        const __half *k_tile = mine + slot * 2u * kTile * stride, *v_tile = k_tile + kTile * stride;
+        __half *k_tile = mine + slot * 2u * kTile * stride, *v_tile = k_tile + kTile * stride;
+        if (p.fused && (tile + 1u) * kTile > base) {
+            for (uint32_t r = max(base, tile * kTile); r < min(end, (tile + 1u) * kTile); ++r)
+                for (uint32_t piece = lane; piece < pieces; piece += 32u) {
+                    *reinterpret_cast<uint4*>(k_tile + (r - tile * kTile) * stride + piece * 8u) = *reinterpret_cast<const uint4*>(my_k + (r - base) * stride + piece * 8u);
+                    *reinterpret_cast<uint4*>(v_tile + (r - tile * kTile) * stride + piece * 8u) = *reinterpret_cast<const uint4*>(my_v + (r - base) * stride + piece * 8u);
+                }
+            __syncwarp();
+        }
         float s[kTile / 8u][4];
 #pragma unroll
         for (uint32_t n = 0; n < kTile / 8u; ++n) { s[n][0] = 0.0f; s[n][1] = 0.0f; s[n][2] = 0.0f; s[n][3] = 0.0f; }
@@ -399,19 +526,21 @@ template <int G>
 int launch_rows(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
     constexpr uint32_t kTile = G <= 8 ? 32u : 16u;
     static std::once_flag once[64];
-    const int status = allow_smem(grouped_attention_kernel<G>, once, 180u * 1024u);
+    const int status = allow_smem(grouped_attention_kernel<G>, once, 200u * 1024u);
     if (status != GF_OK) return status;
     const bool chain = p.ring_stride == 0u;
-    const uint32_t queries = (chain ? p.rows : 1u) * (p.heads / p.kv_heads), smem = (16u + kRowsWarps * 4u * kTile) * (p.row_head + 8u) * 2u;
+    const uint32_t rows = chain ? p.rows : 1u, queries = rows * (p.heads / p.kv_heads);
+    const uint32_t smem = (16u + kRowsWarps * 4u * kTile + (p.fused ? 2u * rows : 0u)) * (p.row_head + 8u) * 2u + (p.fused ? rows * p.prepare.rotated * 4u : 0u);
     return launch_kernel(grouped_attention_kernel<G>, dim3((queries + 15u) / 16u, p.parts, p.kv_heads * (chain ? 1u : p.rows)), dim3(kRowsWarps * 32u), smem, stream, pdl, p);
 }
 
 }  // namespace
 
-int launch_query_key(const QueryKey& p, cudaStream_t stream, bool pdl) {
+int launch_query_key(QueryKey p, cudaStream_t stream, bool pdl) {
     if (!p.raw_k || !p.raw_v || (p.raw_q && (!p.q_gain || !p.q)) || !p.k_gain || !p.positions || !p.keys || !p.values || p.rows == 0 || p.heads == 0 || p.kv_heads == 0
         || p.dim == 0 || p.vdim == 0 || p.row_head < p.dim || p.row_head < p.vdim || p.rotated > p.dim || p.rotated % 2u || (p.rotated && !p.frequencies))
         return fail(GF_ERR_INVALID, "query and key preparation: bad arguments");
+    p.pairs = p.dim % 2u == 0u && p.vdim % 2u == 0u && p.rotated % 4u == 0u && p.q_ld % 2u == 0u && p.k_ld % 2u == 0u && p.v_ld % 2u == 0u ? 1u : 0u;
     return launch_kernel(query_key_kernel, dim3(p.rows), dim3(kPrepareThreads), p.rotated / 2u * sizeof(float2), stream, pdl, p);
 }
 
@@ -423,11 +552,15 @@ uint32_t grouped_attention_parts(uint32_t rows, uint32_t heads, uint32_t kv_head
 }
 
 int launch_grouped_attention(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
-    if (!p.q || !p.rings || !p.own_k || !p.own_v || !p.positions || !p.result.data || p.rows == 0 || p.heads == 0 || p.kv_heads == 0 || p.heads % p.kv_heads
+    if (p.fused ? (!grouped_attention_on_tensor_cores(p.row_head, p.f32 != 0u) || p.rows > kGroupedFusedRows || !p.prepare.raw_q || !p.prepare.raw_k || !p.prepare.raw_v
+                   || !p.prepare.keys || !p.prepare.values || p.prepare.row_head != p.row_head || p.prepare.vdim != p.vdim || (p.prepare.rotated && !p.prepare.frequencies))
+                : !p.q)
+        return fail(GF_ERR_INVALID, "grouped attention: bad arguments");
+    if (!p.rings || !p.own_k || !p.own_v || !p.positions || !p.result.data || p.rows == 0 || p.heads == 0 || p.kv_heads == 0 || p.heads % p.kv_heads
         || p.row_head == 0 || p.row_head % 16u || p.vdim > p.row_head || p.parts == 0 || p.parts > kGroupedMaxParts
         || (p.parts > 1u && (!p.partial_out || !p.partial_ml || !p.counters)))
         return fail(GF_ERR_INVALID, "grouped attention: bad arguments");
-    if (!p.f32 && p.row_head <= 256u) {
+    if (grouped_attention_on_tensor_cores(p.row_head, p.f32 != 0u)) {
         const uint32_t groups = p.row_head / 16u;
         if (groups <= 2u) return launch_rows<2>(p, stream, pdl);
         if (groups <= 4u) return launch_rows<4>(p, stream, pdl);

@@ -25,8 +25,9 @@ struct QueryKey {
     uint32_t rows = 0, heads = 0, kv_heads = 0, dim = 0, vdim = 0, row_head = 0, rotated = 0, f32 = 0;
     float eps = 0.0f, scale = 1.0f;
     uint32_t* status = nullptr;
+    uint32_t pairs = 0;                            // filled by the launcher: every row and head starts on an even value
 };
-int launch_query_key(const QueryKey& p, cudaStream_t stream, bool pdl);
+int launch_query_key(QueryKey p, cudaStream_t stream, bool pdl);
 
 constexpr uint32_t kGroupedMaxParts = 64;
 struct GroupedAttention {
@@ -45,7 +46,14 @@ struct GroupedAttention {
     uint32_t* counters = nullptr;
     uint32_t parts = 1;
     Operand result;                      // (row, head * vdim + d)
+    // With `fused` the blocks prepare their queries and the pass's own cache rows from the projections themselves (q is
+    // not read; own_k and own_v are written): passes of the tensor-core kernel alone.
+    uint32_t fused = 0;
+    QueryKey prepare;
 };
+// Whether the tensor-core kernel takes this shape (binary16, heads of up to 256); else a plain f32 kernel runs.
+inline bool grouped_attention_on_tensor_cores(uint32_t row_head, bool f32) { return !f32 && row_head <= 256u; }
+constexpr uint32_t kGroupedFusedRows = GF_MAX_ROWS;
 // Partitions of the keys worth launching for a pass of `rows` rows over up to `positions` cached rows.
 uint32_t grouped_attention_parts(uint32_t rows, uint32_t heads, uint32_t kv_heads, uint32_t positions, bool chain);
 int launch_grouped_attention(const GroupedAttention& p, cudaStream_t stream, bool pdl);

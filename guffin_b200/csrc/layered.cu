@@ -8,8 +8,8 @@
 //   mixer output
 // Grouped-query attention:
 //   q, k, gates of the heads <- the same prologue
-//   norm, rotation and the new cache rows
-//   attention over the cached keys and values (split over the keys; the last block merges, with sink and gate)
+//   norm, rotation and the new cache rows; attention over the cached keys and values (split over the keys; the last block
+//   merges, with sink and gate) -- one launch, two in 32-bit plans
 //   mixer output
 // State space:
 //   input projection <- the same prologue
@@ -399,10 +399,10 @@ int Model::encode_layers(uint32_t rows, bool logits, const LayeredRows& where) {
         prepare.rows = rows; prepare.heads = m.heads; prepare.kv_heads = m.kv_heads; prepare.dim = m.dim; prepare.vdim = m.vdim;
         prepare.row_head = row_head; prepare.rotated = m.rotated; prepare.f32 = p.f32 ? 1u : 0u;
         prepare.eps = s.eps; prepare.scale = m.scale; prepare.status = status_dev_;
-        ++launches_;
-        GF_TRY(launch_query_key(prepare, stream_, true));
         GroupedAttention attention;
-        attention.q = p.query;
+        attention.q = p.query; attention.prepare = prepare;
+        attention.fused = grouped_attention_on_tensor_cores(row_head, p.f32) ? 1u : 0u;
+        if (!attention.fused) { ++launches_; GF_TRY(launch_query_key(prepare, stream_, true)); }
         attention.rings = where.rings + (size_t)l * where.layer_stride; attention.ring_stride = where.ring_stride;
         attention.own_k = caches_[l].private_k; attention.own_v = caches_[l].private_v; attention.positions = where.positions;
         attention.rows = rows; attention.heads = m.heads; attention.kv_heads = m.kv_heads; attention.row_head = row_head; attention.vdim = m.vdim;
@@ -507,7 +507,7 @@ int Model::ensure_chunk_arena() {
         return bytes_alloc(allocations_, &o.data, o.bytes());
     };
     uint32_t query = 0, latent_out = 0, values = 0, latent = 0, query_elements = 0, row_elements = 0, ff = 0, shared_ff = 0, expert_ff = 0, experts = 0, top = 0, heads = 0;
-    size_t raw_q = 0, raw_k = 0, gates = 0, prepared = 0, x_elements = 0, bc_elements = 0, step_elements = 0, y_elements = 0;      // per row
+    size_t raw_q = 0, raw_k = 0, gates = 0, prepared = 0, x_elements = 0, bc_elements = 0, cb_elements = 0, step_elements = 0, y_elements = 0;      // per row
     for (const LayerSpec& l : s.layers) {
         const MixerSpec& m = l.mixer;
         values = std::max(values, m.inner());
@@ -522,7 +522,7 @@ int Model::ensure_chunk_arena() {
             const StateSpace shape = p.state_space((uint32_t)(&l - s.layers.data()));
             raw_q = std::max<size_t>(raw_q, state_inputs_ld(m)); y_elements = std::max<size_t>(y_elements, m.inner());
             x_elements = std::max<size_t>(x_elements, m.heads * shape.x_row()); bc_elements = std::max<size_t>(bc_elements, m.groups * shape.state_row());
-            step_elements = std::max<size_t>(step_elements, m.heads);
+            step_elements = std::max<size_t>(step_elements, m.heads); cb_elements = std::max<size_t>(cb_elements, m.groups * 4u);
         }
         const FeedForwardSpec& f = l.mlp;
         if (f.kind == FeedForwardSpec::kDense) ff = std::max(ff, f.ff);
@@ -543,6 +543,7 @@ int Model::ensure_chunk_arena() {
         GF_TRY(plan_alloc(allocations_, &a.state_x, rows * x_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_b, rows * bc_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_c, rows * bc_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_cb, rows * cb_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_steps, rows * step_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_y, rows * y_elements));
     }
@@ -768,7 +769,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         step.raw = a.raw_q; step.raw_ld = state_inputs_ld(m);
         step.taps = w.taps; step.tap_bias = w.tap_bias; step.step_bias = w.step_bias; step.decay = w.decay; step.skip = w.skip;
         step.rings = p.rings_dev + l; step.positions = state_dev_; step.slots = p.slots_dev; step.rows = rows; step.input_mask = caches_[l].ring_rows - 1u;
-        step.out = a.state_y; step.x = a.state_x; step.b = a.state_b; step.c = a.state_c; step.steps = a.state_steps;
+        step.out = a.state_y; step.x = a.state_x; step.b = a.state_b; step.c = a.state_c; step.cb = a.state_cb; step.steps = a.state_steps;
         launches_ += 2;
         GF_TRY(launch_state_space_chunk(step, stream_));
         if (last) return GF_OK;

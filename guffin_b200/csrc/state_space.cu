@@ -46,274 +46,498 @@ __device__ __forceinline__ Pair pair_mul(Pair a, Pair b) {
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.0f) + log1pf(expf(-fabsf(z))); }
 
 // The convolution of one channel at row r of a portion that starts at `base`: rows of the portion come from `raw`,
-// earlier ones from the ring.
+// earlier ones from the ring.  kFew: up to four taps, whose reads are issued together.
+template <bool kFew>
 __device__ __forceinline__ float convolve(const StateSpace& p, const float* raw, const float* ring, uint32_t base, uint32_t r, uint32_t channel) {
     const float* taps = p.taps + (size_t)channel * p.tap_count;
     const uint32_t inner = p.inner(), row = p.input_row();
+    auto value = [&](uint32_t back) {                                  // `back` rows behind row r
+        if (base + r < back) return 0.0f;
+        return back <= r ? raw[(size_t)(r - back) * p.raw_ld + inner + channel] : ring[(size_t)((base + r - back) & p.input_mask) * row + channel];
+    };
     float sum = 0.0f;
-    for (uint32_t j = 0; j < p.tap_count; ++j) {
-        const uint32_t back = p.tap_count - 1u - j;                    // rows behind row r
-        if (base + r < back) continue;
-        const float v = back <= r ? raw[(size_t)(r - back) * p.raw_ld + inner + channel] : ring[(size_t)((base + r - back) & p.input_mask) * row + channel];
-        sum = fmaf(taps[j], v, sum);
+    if (kFew) {
+        float v[4], w[4];
+#pragma unroll
+        for (uint32_t j = 0; j < 4u; ++j) {                            // j taps before the last one
+            v[j] = j < p.tap_count ? value(j) : 0.0f;
+            w[j] = j < p.tap_count ? taps[p.tap_count - 1u - j] : 0.0f;
+        }
+        const float bias = p.tap_bias[channel];
+#pragma unroll
+        for (int j = 3; j >= 0; --j) sum = fmaf(w[j], v[j], sum);
+        return silu(sum + bias);
     }
+    for (uint32_t j = 0; j < p.tap_count; ++j) sum = fmaf(taps[j], value(p.tap_count - 1u - j), sum);
     return silu(sum + p.tap_bias[channel]);
 }
+// dt and the logarithm of the decay.
 __device__ __forceinline__ float2 step_of(const StateSpace& p, const float* raw, uint32_t r, uint32_t head) {
     const float dt = softplus(raw[(size_t)r * p.raw_ld + p.inner() + p.channels() + head] + p.step_bias[head]);
-    return make_float2(dt, expf(p.decay[head] * dt));
+    return make_float2(dt, p.decay[head] * dt);
 }
 
-struct TileLayout { uint32_t b, c, x, steps, stage, doubled, gate, bytes; };
-// Offsets in bytes: `stages` stages of B, C, x and steps for `tile` tokens, then (x * dt) twice and the gates.
-__host__ __device__ inline TileLayout tile_layout(uint32_t tile, uint32_t wide, uint32_t columns, uint32_t stages) {
-    TileLayout t;
-    t.b = 0;
-    t.c = t.b + tile * wide * 4u;
-    t.x = t.c + tile * wide * 4u;
-    t.steps = t.x + tile * columns * 4u;
-    t.stage = (t.steps + tile * 8u + 15u) & ~15u;
-    t.doubled = stages * t.stage;
-    t.gate = t.doubled + tile * columns * 8u;
-    t.bytes = t.gate + (stages == 1u ? tile * columns * 4u : 0u);
-    return t;
+// Sums part[0 .. 4 V) over the L lanes that share a column: every round halves the values a lane is left with.  Returns
+// how many it has, from `index` on.
+template <int L, int V>
+__device__ __forceinline__ uint32_t lane_sums(float (&part)[4 * V], uint32_t lane, uint32_t& index) {
+    uint32_t count = 4u * V;
+    index = 0u;
+#pragma unroll
+    for (uint32_t o = L / 2u; o > 0u; o >>= 1) {
+        const bool upper = (lane & o) != 0u;
+        if (count > 1u) {
+            count /= 2u;
+            if (upper) index += count;
+#pragma unroll
+            for (uint32_t i = 0; i < 2u * V; ++i) {
+                if (i >= count) break;
+                const float keep = upper ? part[i + count] : part[i], send = upper ? part[i] : part[i + count];
+                part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
+            }
+        } else part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
+    }
+    return count;
 }
-template <int NL> constexpr uint32_t tile_tokens() { return NL <= 256 ? 16u : NL <= 512 ? 8u : 4u; }
+// Whether a lane writes what lane_sums leaves it with (of lanes left with the same value, the first).
+template <int L, int V>
+__device__ __forceinline__ bool sums_writer(uint32_t ln) {
+    constexpr uint32_t kSame = L > 4 * V ? L / (4 * V) : 1;
+    return ln % kSame == 0u;
+}
 
 // A block holds some columns (of vdim) of one head's state in registers while it walks the tokens: L lanes share a
-// column's N values, four apart in turn, NQ fours each; a lane holds V columns.  kPass: the convolution is computed here and the gate
-// applied (rows of a pass); else the inputs come convolved.
-template <int L, int NQ, int V, bool kPass>
-__global__ void __launch_bounds__(kMaxWarps * 32) state_space_kernel(const __grid_constant__ StateSpace p) {
-    extern __shared__ __align__(16) uint8_t smem[];
-    constexpr uint32_t kWide = L * NQ * 4, kTile = tile_tokens<(int)kWide>(), kStages = kPass ? 1u : 2u, kThreadsPer = 32u / L;
-    const uint32_t tid = threadIdx.x, threads = blockDim.x, warp = tid >> 5, lane = tid & 31u, ln = lane % L;
-    const uint32_t columns = threads / L * V, c0 = blockIdx.y * columns, local = (warp * kThreadsPer + lane / L) * V, column = c0 + local;
-    const TileLayout at = tile_layout(kTile, kWide, columns, kStages);
-    const bool chain = p.ring_stride == 0u;
-    const uint32_t head = blockIdx.x, z = blockIdx.z, rows = chain ? p.rows : 1u, row0 = chain ? 0u : z;
-    const uint32_t group = head / (p.heads / p.groups), np = p.state_row(), inner = p.inner(), input_row = p.input_row();
-    // The state, the position and the ring were written at least two launches back: read ahead of the wait.
-    const uint32_t base = p.positions[chain ? 0u : z], slots = *p.slots;
-    const StreamRings rings = p.rings[(size_t)z * p.ring_stride];
-    float* states = static_cast<float*>(const_cast<void*>(rings.ring_k)) + (size_t)head * p.vdim * np;
-    float* ring = static_cast<float*>(const_cast<void*>(rings.ring_v));
-    const size_t slot_elements = p.slot_elements();
-    Pair s[V][2 * NQ];
-    {
-        const float* from = states + (base % slots) * slot_elements;
+// column's N values, four apart in turn, NQ fours each; a lane holds V columns.
+template <int L, int NQ, int V>
+struct Columns {
+    static constexpr uint32_t kWide = L * NQ * 4;                      // N with its padding
+    uint32_t count, first, local, ln, np, vdim;                        // count columns from `first` on; this lane's from first + local on
+    __device__ Columns(const StateSpace& p) {
+        const uint32_t lane = threadIdx.x & 31u;
+        count = blockDim.x / L * V; first = blockIdx.y * count;
+        ln = lane % L; local = ((threadIdx.x >> 5) * (32u / L) + lane / L) * V;
+        np = p.state_row(); vdim = p.vdim;
+    }
+    __device__ uint32_t column(int v) const { return first + local + v; }
+    __device__ uint32_t n(int j) const { return (j * L + ln) * 4u; }
+    __device__ void load(Pair (&s)[V][2 * NQ], const float* head_state, bool any) const {
 #pragma unroll
         for (int v = 0; v < V; ++v)
 #pragma unroll
             for (int j = 0; j < NQ; ++j) {
-                const uint32_t n = (j * L + ln) * 4u;
                 float4 q = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-                if (base > 0u && column + v < p.vdim && n < np) q = *reinterpret_cast<const float4*>(from + (size_t)(column + v) * np + n);
+                if (any && column(v) < vdim && n(j) < np) q = *reinterpret_cast<const float4*>(head_state + (size_t)column(v) * np + n(j));
                 s[v][2 * j] = pair_of(q.x, q.y);
                 s[v][2 * j + 1] = pair_of(q.z, q.w);
             }
     }
-    if (kPass) {
-        pdl_wait();
-        pdl_launch_dependents();
+    __device__ void store(const Pair (&s)[V][2 * NQ], float* head_state) const {
+#pragma unroll
+        for (int v = 0; v < V; ++v)
+#pragma unroll
+            for (int j = 0; j < NQ; ++j)
+                if (column(v) < vdim && n(j) < np) *reinterpret_cast<ulonglong2*>(head_state + (size_t)column(v) * np + n(j)) = make_ulonglong2(s[v][2 * j], s[v][2 * j + 1]);
     }
-    const float* raw = p.raw + (size_t)row0 * p.raw_ld;
-    const float skip = p.skip[head];
+};
 
-    auto fill = [&](uint32_t tile, uint32_t stage) {
-        uint8_t* to = smem + stage * at.stage;
-        float *b = reinterpret_cast<float*>(to + at.b), *c = reinterpret_cast<float*>(to + at.c), *x = reinterpret_cast<float*>(to + at.x);
-        float2* steps = reinterpret_cast<float2*>(to + at.steps);
-        const uint32_t first = tile * kTile;
-        if (kPass) {
-            float* gate = reinterpret_cast<float*>(smem + at.gate);
-            const uint32_t live = min(kTile, rows - first);
-            for (uint32_t i = tid; i < live * kWide; i += threads) {
-                const uint32_t t = i / kWide, n = i % kWide;
-                const uint32_t channel = inner + group * p.state + n;
-                b[i] = n < p.state ? convolve(p, raw, ring, base, first + t, channel) : 0.0f;
-                c[i] = n < p.state ? convolve(p, raw, ring, base, first + t, channel + p.groups * p.state) : 0.0f;
-            }
-            for (uint32_t t = 0; t < live; ++t)
-                for (uint32_t i = tid; i < columns; i += threads) {
-                    const bool valid = c0 + i < p.vdim;
-                    x[t * columns + i] = valid ? convolve(p, raw, ring, base, first + t, head * p.vdim + c0 + i) : 0.0f;
-                    gate[t * columns + i] = valid ? raw[(size_t)(first + t) * p.raw_ld + head * p.vdim + c0 + i] : 0.0f;
-                }
-            if (tid < live) steps[tid] = step_of(p, raw, first + tid, head);
-            return;
-        }
-        const uint32_t x_row = p.x_row();
-        for (uint32_t i = tid; i < kTile * (kWide / 4u); i += threads) {
-            const uint32_t t = i / (kWide / 4u), n = i % (kWide / 4u) * 4u, row = first + t;
-            const bool valid = row < rows && n < np;
-            const size_t from = valid ? ((size_t)row * p.groups + group) * np + n : 0u;
-            copy16(b + t * kWide + n, p.b + from, valid);
-            copy16(c + t * kWide + n, p.c + from, valid);
-        }
-        for (uint32_t i = tid; i < kTile * (columns / 4u); i += threads) {
-            const uint32_t t = i / (columns / 4u), k = i % (columns / 4u) * 4u, row = first + t;
-            const bool valid = row < rows && c0 + k < x_row;
-            copy16(x + t * columns + k, p.x + (valid ? ((size_t)row * p.heads + head) * x_row + c0 + k : 0u), valid);
-        }
-        if (tid < kTile) copy8(steps + tid, p.steps + (first + tid < rows ? (size_t)(first + tid) * p.heads + head : 0u), first + tid < rows);
-    };
-
-    const uint32_t tiles = (rows + kTile - 1u) / kTile;
-    // States kept: all of them where the slots hold them besides the one that was read, else the last.
-    const uint32_t kept = kPass ? rows - min(rows, slots - 1u) : rows - 1u;
-    if (!kPass) { fill(0u, 0u); copies_commit(); }
-    for (uint32_t tile = 0; tile < tiles; ++tile) {
-        const uint32_t stage = kPass ? 0u : tile & 1u, first = tile * kTile;
-        if (kPass) fill(tile, 0u);
-        else {
-            if (tile + 1u < tiles) fill(tile + 1u, stage ^ 1u);
-            copies_commit();
-            copies_wait<1>();
-        }
-        __syncthreads();
-        const uint8_t* from = smem + stage * at.stage;
-        const float *b = reinterpret_cast<const float*>(from + at.b), *c = reinterpret_cast<const float*>(from + at.c), *x = reinterpret_cast<const float*>(from + at.x);
-        const float2* steps = reinterpret_cast<const float2*>(from + at.steps);
-        Pair* doubled = reinterpret_cast<Pair*>(smem + at.doubled);
-        for (uint32_t i = tid; i < kTile * columns; i += threads) {
-            const float v = x[i] * steps[i / columns].x;
-            doubled[i] = pair_of(v, v);
-        }
-        __syncthreads();
-#pragma unroll 1
-        for (uint32_t t4 = 0; t4 < kTile && first + t4 < rows; t4 += 4u) {
-            float part[4 * V];
-#pragma unroll
-            for (int q = 0; q < 4; ++q) {
-                const uint32_t t = t4 + q;
-                const float decay = steps[t].y;
-                const Pair a = pair_of(decay, decay);
-                Pair xd[V], sum[V];
-#pragma unroll
-                for (int v = 0; v < V; v += 2) {
-                    const ulonglong2 two = *reinterpret_cast<const ulonglong2*>(doubled + t * columns + local + v);
-                    xd[v] = two.x;
-                    xd[v + 1] = two.y;
-                }
-#pragma unroll
-                for (int j = 0; j < NQ; ++j) {
-                    const ulonglong2 bq = *reinterpret_cast<const ulonglong2*>(b + t * kWide + (j * L + ln) * 4u);
-                    const ulonglong2 cq = *reinterpret_cast<const ulonglong2*>(c + t * kWide + (j * L + ln) * 4u);
-#pragma unroll
-                    for (int v = 0; v < V; ++v) {
-                        s[v][2 * j] = pair_fma(bq.x, xd[v], pair_mul(s[v][2 * j], a));
-                        s[v][2 * j + 1] = pair_fma(bq.y, xd[v], pair_mul(s[v][2 * j + 1], a));
-                        sum[v] = j == 0 ? pair_mul(s[v][0], cq.x) : pair_fma(s[v][2 * j], cq.x, sum[v]);
-                        sum[v] = pair_fma(s[v][2 * j + 1], cq.y, sum[v]);
-                    }
-                }
-#pragma unroll
-                for (int v = 0; v < V; ++v) part[q * V + v] = pair_sum(sum[v]);
-                const uint32_t row = first + t;
-                if (row >= kept && row < rows) {
-                    float* to = states + ((base + row + 1u) % slots) * slot_elements;
-#pragma unroll
-                    for (int v = 0; v < V; ++v)
-#pragma unroll
-                        for (int j = 0; j < NQ; ++j) {
-                            const uint32_t n = (j * L + ln) * 4u;
-                            if (column + v < p.vdim && n < np) *reinterpret_cast<ulonglong2*>(to + (size_t)(column + v) * np + n) = make_ulonglong2(s[v][2 * j], s[v][2 * j + 1]);
-                        }
-                }
-            }
-            // Sums over the L lanes: every round halves the values a lane is left with.
-            uint32_t count = 4u * V, index = 0;
-#pragma unroll
-            for (uint32_t o = L / 2u; o > 0u; o >>= 1) {
-                const bool upper = (lane & o) != 0u;
-                if (count > 1u) {
-                    count /= 2u;
-                    if (upper) index += count;
-#pragma unroll
-                    for (uint32_t i = 0; i < 2u * V; ++i) {
-                        if (i >= count) break;
-                        const float keep = upper ? part[i + count] : part[i], send = upper ? part[i] : part[i + count];
-                        part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
-                    }
-                } else part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
-            }
-            const bool writer = (uint32_t)L <= 4u * V || ln % (L / (4u * V) > 0u ? L / (4u * V) : 1u) == 0u;
-#pragma unroll
-            for (uint32_t i = 0; i < 4u * V; ++i) {
-                if (i >= count) break;
-                const uint32_t t = t4 + (index + i) / V, k = local + (index + i) % V, row = first + t;
-                if (!writer || row >= rows || c0 + k >= p.vdim) continue;
-                float y = fmaf(skip, x[t * columns + k], part[i]);
-                if (kPass) y *= silu(reinterpret_cast<const float*>(smem + at.gate)[t * columns + k]);
-                p.out[(size_t)(row0 + row) * inner + head * p.vdim + c0 + k] = y;
-            }
-        }
-        __syncthreads();                                               // the tile's buffers are free again
-    }
-    // The convolution's inputs of the rows that later tokens look back at: every block its own columns, the first one
-    // of a group the shared channels.
-    const uint32_t first_kept = kPass ? 0u : rows - min(rows, p.tap_count - 1u);
-    const bool shared = head % (p.heads / p.groups) == 0u && blockIdx.y == 0u;
-    for (uint32_t r = first_kept; r < rows; ++r) {
+// The convolution's inputs of the rows from `first` on, which later tokens look back at: every block its own columns,
+// the first one of a group the shared channels.
+__device__ __forceinline__ void keep_inputs(const StateSpace& p, const float* raw, float* ring, uint32_t base, uint32_t first, uint32_t rows, uint32_t head,
+                                            uint32_t first_column, uint32_t columns) {
+    const uint32_t per_group = p.heads / p.groups, inner = p.inner();
+    const bool shared = head % per_group == 0u && blockIdx.y == 0u;
+    for (uint32_t r = first; r < rows; ++r) {
         const float* from = raw + (size_t)r * p.raw_ld + inner;
-        float* to = ring + (size_t)((base + r) & p.input_mask) * input_row;
-        for (uint32_t i = tid; i < columns; i += threads)
-            if (c0 + i < p.vdim) to[head * p.vdim + c0 + i] = from[head * p.vdim + c0 + i];
+        float* to = ring + (size_t)((base + r) & p.input_mask) * p.input_row();
+        for (uint32_t i = threadIdx.x; i < columns; i += blockDim.x)
+            if (first_column + i < p.vdim) to[head * p.vdim + first_column + i] = from[head * p.vdim + first_column + i];
         if (shared)
-            for (uint32_t i = tid; i < p.state; i += threads) {
-                const uint32_t channel = inner + group * p.state + i;
+            for (uint32_t i = threadIdx.x; i < p.state; i += blockDim.x) {
+                const uint32_t channel = inner + head / per_group * p.state + i;
                 to[channel] = from[channel];
                 to[channel + p.groups * p.state] = from[channel + p.groups * p.state];
             }
     }
 }
 
-// The convolved inputs of a chunk, padding included.
-constexpr uint32_t kConvolveRows = 8;
-__global__ void __launch_bounds__(128) convolve_chunk_kernel(const __grid_constant__ StateSpace p) {
-    const uint32_t np = p.state_row(), x_row = p.x_row(), all_x = p.heads * x_row, all_n = p.groups * np;
-    const uint32_t base = p.positions[0], end = min(p.rows, (blockIdx.y + 1u) * kConvolveRows);
-    const float* ring = static_cast<const float*>(p.rings->ring_v);
-    uint32_t i = blockIdx.x * blockDim.x + threadIdx.x;
-    float* out = nullptr;
-    uint32_t ld = 0, channel = 0;
-    bool valid = false;
-    if (i < all_x) {
-        const uint32_t k = i % x_row;
-        out = p.x + i; ld = all_x; channel = i / x_row * p.vdim + k; valid = k < p.vdim;
-    } else if (i - all_x < 2u * all_n) {
-        i -= all_x;
-        const uint32_t which = i / all_n, j = i % all_n, n = j % np;
-        out = (which ? p.c : p.b) + j; ld = all_n; channel = p.inner() + (which * p.groups + j / np) * p.state + n; valid = n < p.state;
-    } else if (i - all_x - 2u * all_n < p.heads) {
-        const uint32_t head = i - all_x - 2u * all_n;
-        for (uint32_t r = blockIdx.y * kConvolveRows; r < end; ++r) p.steps[(size_t)r * p.heads + head] = step_of(p, p.raw, r, head);
+// ------------------------------------------------------------------ rows of a pass
+
+constexpr uint32_t kPassTile = 4;
+__host__ __device__ inline uint32_t pass_smem(uint32_t wide, uint32_t columns) { return kPassTile * (2u * wide + 4u * columns) * 4u + kPassTile * 8u; }
+
+// Token by token, the convolution computed here and the gate applied.
+template <int L, int NQ, int V>
+__global__ void __launch_bounds__(kMaxWarps * 32, 3) state_space_rows_kernel(const __grid_constant__ StateSpace p) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    const Columns<L, NQ, V> mine(p);
+    constexpr uint32_t kWide = Columns<L, NQ, V>::kWide;
+    const uint32_t tid = threadIdx.x, threads = blockDim.x, lane = tid & 31u, columns = mine.count, c0 = mine.first;
+    Pair* doubled = reinterpret_cast<Pair*>(smem);                     // [tile][columns]: x * dt, twice
+    float* b = reinterpret_cast<float*>(doubled + kPassTile * columns);            // [tile][kWide]
+    float *c = b + kPassTile * kWide, *x = c + kPassTile * kWide, *gate = x + kPassTile * columns;
+    float2* steps = reinterpret_cast<float2*>(gate + kPassTile * columns);         // dt, decay
+    const bool chain = p.ring_stride == 0u;
+    const uint32_t head = blockIdx.x, z = blockIdx.z, rows = chain ? p.rows : 1u, row0 = chain ? 0u : z, inner = p.inner(), group = head / (p.heads / p.groups);
+    // The state, the position and the ring were written at least two launches back: read ahead of the wait.
+    const uint32_t base = p.positions[chain ? 0u : z], slots = *p.slots;
+    const StreamRings rings = p.rings[(size_t)z * p.ring_stride];
+    const size_t slot_elements = p.slot_elements();
+    float* states = static_cast<float*>(const_cast<void*>(rings.ring_k)) + (size_t)head * p.vdim * mine.np;
+    float* ring = static_cast<float*>(const_cast<void*>(rings.ring_v));
+    Pair s[V][2 * NQ];
+    mine.load(s, states + (base % slots) * slot_elements, base > 0u);
+    pdl_wait();
+    pdl_launch_dependents();
+    const float* raw = p.raw + (size_t)row0 * p.raw_ld;
+    const float skip = p.skip[head];
+
+    auto fill = [&](uint32_t first, uint32_t live, auto convolved) {
+        for (uint32_t t = 0; t < live; ++t) {
+            const uint32_t r = first + t, all = 2u * kWide + columns;
+#pragma unroll 3
+            for (uint32_t i = tid; i < all; i += threads) {
+                const uint32_t n = i % kWide, k = i - 2u * kWide;
+                const bool vectors = i < 2u * kWide, valid = vectors ? n < p.state : c0 + k < p.vdim;
+                const uint32_t channel = vectors ? inner + (i < kWide ? 0u : p.groups * p.state) + group * p.state + n : head * p.vdim + c0 + k;
+                const float v = valid ? convolved(r, channel) : 0.0f;
+                if (vectors) (i < kWide ? b : c)[t * kWide + n] = v;
+                else x[t * columns + k] = v;
+            }
+            for (uint32_t i = tid; i < columns; i += threads) gate[t * columns + i] = c0 + i < p.vdim ? raw[(size_t)r * p.raw_ld + head * p.vdim + c0 + i] : 0.0f;
+        }
+        if (tid < live) {
+            const float2 step = step_of(p, raw, first + tid, head);
+            steps[tid] = make_float2(step.x, expf(step.y));
+        }
+    };
+    // States kept: all of them where the slots hold them besides the one that was read, else the last.
+    const uint32_t kept = rows - min(rows, slots - 1u);
+    for (uint32_t first = 0; first < rows; first += kPassTile) {
+        const uint32_t live = min(kPassTile, rows - first);
+        if (p.tap_count <= 4u) fill(first, live, [&](uint32_t r, uint32_t channel) { return convolve<true>(p, raw, ring, base, r, channel); });
+        else fill(first, live, [&](uint32_t r, uint32_t channel) { return convolve<false>(p, raw, ring, base, r, channel); });
+        __syncthreads();
+        for (uint32_t i = tid; i < live * columns; i += threads) {
+            const float v = x[i] * steps[i / columns].x;
+            doubled[i] = pair_of(v, v);
+        }
+        __syncthreads();
+        float part[4 * V];
+#pragma unroll
+        for (int i = 0; i < 4 * V; ++i) part[i] = 0.0f;
+#pragma unroll
+        for (int t = 0; t < 4; ++t) {
+            if ((uint32_t)t >= live) break;
+            const float decay = steps[t].y;
+            const Pair a = pair_of(decay, decay);
+            Pair sum[V];
+#pragma unroll
+            for (int j = 0; j < NQ; ++j) {
+                const ulonglong2 bq = *reinterpret_cast<const ulonglong2*>(b + t * kWide + mine.n(j)), cq = *reinterpret_cast<const ulonglong2*>(c + t * kWide + mine.n(j));
+#pragma unroll
+                for (int v = 0; v < V; ++v) {
+                    const Pair xd = doubled[t * columns + mine.local + v];
+                    s[v][2 * j] = pair_fma(bq.x, xd, pair_mul(s[v][2 * j], a));
+                    s[v][2 * j + 1] = pair_fma(bq.y, xd, pair_mul(s[v][2 * j + 1], a));
+                    sum[v] = j == 0 ? pair_mul(s[v][0], cq.x) : pair_fma(s[v][2 * j], cq.x, sum[v]);
+                    sum[v] = pair_fma(s[v][2 * j + 1], cq.y, sum[v]);
+                }
+            }
+#pragma unroll
+            for (int v = 0; v < V; ++v) part[t * V + v] = pair_sum(sum[v]);
+            const uint32_t row = first + t;
+            if (row >= kept) mine.store(s, states + ((base + row + 1u) % slots) * slot_elements);
+        }
+        uint32_t index;
+        const uint32_t count = lane_sums<L, V>(part, lane, index);
+#pragma unroll
+        for (uint32_t i = 0; i < 4u * V; ++i) {
+            if (i >= count) break;
+            const uint32_t t = (index + i) / V, k = mine.local + (index + i) % V;
+            if (!sums_writer<L, V>(mine.ln) || t >= live || c0 + k >= p.vdim) continue;
+            p.out[(size_t)(row0 + first + t) * inner + head * p.vdim + c0 + k] = fmaf(skip, x[t * columns + k], part[i]) * silu(gate[t * columns + k]);
+        }
+        __syncthreads();                                               // the tile's buffers are free again
+    }
+    keep_inputs(p, raw, ring, base, 0u, rows, head, c0, columns);
+}
+
+// ------------------------------------------------------------------ chunks
+
+// Four tokens at a time.  With a_t the logarithm of token t's decay and A_t their sums within the four,
+//   y_t = exp(A_t) C_t . S + sum over s <= t of exp(A_t - A_s) dt_s (C_t . B_s) x_s + skip x_t
+//   S  <- exp(A_3) S + sum over s of exp(A_3 - A_s) dt_s B_s x_s^T
+// so that a state's element costs nine multiply-adds per four tokens; the products C_t . B_s come with the inputs.
+template <int NL> constexpr uint32_t chunk_tile() { return NL <= 128 ? 32u : NL <= 256 ? 16u : NL <= 512 ? 8u : 4u; }
+struct ChunkLayout { uint32_t c, x, steps, cb, stage, doubled, m, u, w, whole, bytes; };
+__host__ __device__ inline ChunkLayout chunk_layout(uint32_t tile, uint32_t wide, uint32_t columns) {      // bytes; two stages, then one of each
+    ChunkLayout t;
+    t.c = tile * wide * 4u;
+    t.x = 2u * t.c;
+    t.cb = t.x + tile * columns * 4u;
+    t.steps = t.cb + tile * 16u;
+    t.stage = t.steps + tile * 8u;
+    t.doubled = 2u * t.stage;
+    t.m = t.doubled + tile * columns * 8u;
+    t.u = t.m + tile * 16u;
+    t.w = t.u + tile * 4u;
+    t.whole = t.w + tile * 4u;
+    t.bytes = t.whole + tile * 4u;
+    return t;
+}
+
+template <int L, int NQ, int V>
+__global__ void __launch_bounds__(kMaxWarps * 32) state_space_chunk_kernel(const __grid_constant__ StateSpace p) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    const Columns<L, NQ, V> mine(p);
+    constexpr uint32_t kWide = Columns<L, NQ, V>::kWide, kTile = chunk_tile<(int)kWide>();
+    const uint32_t tid = threadIdx.x, threads = blockDim.x, lane = tid & 31u, columns = mine.count, c0 = mine.first, rows = p.rows;
+    const ChunkLayout at = chunk_layout(kTile, kWide, columns);
+    const uint32_t head = blockIdx.x, group = head / (p.heads / p.groups), np = mine.np, inner = p.inner(), x_row = p.x_row();
+    const uint32_t base = *p.positions, slots = *p.slots;
+    const size_t slot_elements = p.slot_elements();
+    float* states = static_cast<float*>(const_cast<void*>(p.rings->ring_k)) + (size_t)head * p.vdim * np;
+    Pair s[V][2 * NQ];
+    mine.load(s, states + (base % slots) * slot_elements, base > 0u);
+    const float skip = p.skip[head];
+
+    auto fill = [&](uint32_t tile, uint32_t stage) {                   // zeros behind the chunk's rows
+        uint8_t* to = smem + stage * at.stage;
+        const uint32_t first = tile * kTile;
+        for (uint32_t i = tid; i < kTile * (kWide / 4u); i += threads) {
+            const uint32_t t = i / (kWide / 4u), n = i % (kWide / 4u) * 4u, row = first + t;
+            const bool valid = row < rows && n < np;
+            const size_t from = valid ? ((size_t)row * p.groups + group) * np + n : 0u;
+            copy16(to + (t * kWide + n) * 4u, p.b + from, valid);
+            copy16(to + at.c + (t * kWide + n) * 4u, p.c + from, valid);
+        }
+        for (uint32_t i = tid; i < kTile * (columns / 4u); i += threads) {
+            const uint32_t t = i / (columns / 4u), k = i % (columns / 4u) * 4u, row = first + t;
+            const bool valid = row < rows && c0 + k < x_row;
+            copy16(to + at.x + (t * columns + k) * 4u, p.x + (valid ? ((size_t)row * p.heads + head) * x_row + c0 + k : 0u), valid);
+        }
+        if (tid < kTile) {
+            const bool valid = first + tid < rows;
+            const size_t row = valid ? first + tid : 0u;
+            copy16(to + at.cb + tid * 16u, p.cb + (row * p.groups + group) * 4u, valid);
+            copy8(to + at.steps + tid * 8u, p.steps + row * p.heads + head, valid);
+        }
+        copies_commit();
+    };
+    const uint32_t tiles = (rows + kTile - 1u) / kTile;
+    fill(0u, 0u);
+    for (uint32_t tile = 0; tile < tiles; ++tile) {
+        const uint32_t first = tile * kTile;
+        if (tile + 1u < tiles) fill(tile + 1u, (tile + 1u) & 1u);
+        else copies_commit();
+        copies_wait<1>();
+        __syncthreads();
+        const uint8_t* from = smem + (tile & 1u) * at.stage;
+        const float *b = reinterpret_cast<const float*>(from), *c = reinterpret_cast<const float*>(from + at.c), *x = reinterpret_cast<const float*>(from + at.x);
+        float4* m = reinterpret_cast<float4*>(smem + at.m);            // of x_0 .. x_3 of the four tokens, in y_t
+        float *u = reinterpret_cast<float*>(smem + at.u), *w = reinterpret_cast<float*>(smem + at.w), *whole = reinterpret_cast<float*>(smem + at.whole);
+        Pair* doubled = reinterpret_cast<Pair*>(smem + at.doubled);    // w_t x_t, twice
+        if (tid < kTile) {
+            const float2* steps = reinterpret_cast<const float2*>(from + at.steps) + (tid & ~3u);
+            const float* cb = reinterpret_cast<const float*>(from + at.cb) + tid * 4u;
+            const uint32_t q = tid & 3u;
+            float factors[4], behind = 0.0f, rest = 0.0f;              // sums of logarithms: (s, q], and (q, 3]
+#pragma unroll
+            for (int i = 3; i >= 0; --i) {
+                factors[i] = 0.0f;
+                if ((uint32_t)i > q) { rest += steps[i].y; continue; }
+                factors[i] = cb[i] * expf(behind) * steps[i].x;
+                if ((uint32_t)i == q) factors[i] += skip;
+                behind += steps[i].y;
+            }
+            m[tid] = make_float4(factors[0], factors[1], factors[2], factors[3]);
+            u[tid] = expf(behind);
+            w[tid] = expf(rest) * steps[q].x;
+            whole[tid] = expf(behind + rest);
+        }
+        __syncthreads();
+        for (uint32_t i = tid; i < kTile * columns; i += threads) {
+            const float v = x[i] * w[i / columns];
+            doubled[i] = pair_of(v, v);
+        }
+        __syncthreads();
+#pragma unroll 1
+        for (uint32_t t4 = 0; t4 < kTile && first + t4 < rows; t4 += 4u) {
+            Pair xw[4][V], sum[4][V];
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+#pragma unroll
+                for (int v = 0; v < V; v += 2) {
+                    const ulonglong2 two = *reinterpret_cast<const ulonglong2*>(doubled + (t4 + q) * columns + mine.local + v);
+                    xw[q][v] = two.x;
+                    xw[q][v + 1] = two.y;
+                }
+            const float decay = whole[t4 + 3u];
+            const Pair a = pair_of(decay, decay);
+#pragma unroll
+            for (int j = 0; j < NQ; ++j) {
+                ulonglong2 bq[4], cq[4];
+#pragma unroll
+                for (int q = 0; q < 4; ++q) {
+                    cq[q] = *reinterpret_cast<const ulonglong2*>(c + (t4 + q) * kWide + mine.n(j));
+                    bq[q] = *reinterpret_cast<const ulonglong2*>(b + (t4 + q) * kWide + mine.n(j));
+                }
+#pragma unroll
+                for (int v = 0; v < V; ++v) {
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        sum[q][v] = j == 0 ? pair_mul(s[v][0], cq[q].x) : pair_fma(s[v][2 * j], cq[q].x, sum[q][v]);
+                        sum[q][v] = pair_fma(s[v][2 * j + 1], cq[q].y, sum[q][v]);
+                    }
+                    s[v][2 * j] = pair_mul(s[v][2 * j], a);
+                    s[v][2 * j + 1] = pair_mul(s[v][2 * j + 1], a);
+#pragma unroll
+                    for (int q = 0; q < 4; ++q) {
+                        s[v][2 * j] = pair_fma(bq[q].x, xw[q][v], s[v][2 * j]);
+                        s[v][2 * j + 1] = pair_fma(bq[q].y, xw[q][v], s[v][2 * j + 1]);
+                    }
+                }
+            }
+            float part[4 * V];
+#pragma unroll
+            for (int i = 0; i < 4 * V; ++i) part[i] = pair_sum(sum[i / V][i % V]);
+            uint32_t index;
+            const uint32_t count = lane_sums<L, V>(part, lane, index);
+#pragma unroll
+            for (uint32_t i = 0; i < 4u * V; ++i) {
+                if (i >= count) break;
+                const uint32_t t = t4 + (index + i) / V, k = mine.local + (index + i) % V, row = first + t;
+                if (!sums_writer<L, V>(mine.ln) || row >= rows || c0 + k >= p.vdim) continue;
+                const float4 f = m[t];
+                const float* x4 = x + t4 * columns + k;
+                float y = u[t] * part[i];
+                y = fmaf(f.x, x4[0], y);
+                y = fmaf(f.y, x4[columns], y);
+                y = fmaf(f.z, x4[2u * columns], y);
+                p.out[(size_t)row * inner + head * p.vdim + c0 + k] = fmaf(f.w, x4[3u * columns], y);
+            }
+        }
+        __syncthreads();                                               // the tile's buffers are free again
+    }
+    mine.store(s, states + ((base + rows) % slots) * slot_elements);
+    keep_inputs(p, p.raw, static_cast<float*>(const_cast<void*>(p.rings->ring_v)), base, rows - min(rows, p.tap_count - 1u), rows, head, c0, columns);
+}
+
+// The convolved inputs of eight rows, padding included: the first blocks take a group's B and C, its heads' steps, and
+// the products C_t . B_s within every four tokens; the others columns of x.
+constexpr uint32_t kConvolveRows = 8, kConvolveThreads = 256;
+
+// Eight rows of one channel: emit(row, value).  T: taps at most (0: any number).
+template <int T, typename Emit>
+__device__ __forceinline__ void convolve_rows(const StateSpace& p, const float* ring, uint32_t base, uint32_t row, uint32_t live, uint32_t channel, Emit emit) {
+    if (T == 0) {
+        for (uint32_t r = 0; r < live; ++r) emit(r, convolve<false>(p, p.raw, ring, base, row + r, channel));
         return;
-    } else return;
-    for (uint32_t r = blockIdx.y * kConvolveRows; r < end; ++r) out[(size_t)r * ld] = valid ? convolve(p, p.raw, ring, base, r, channel) : 0.0f;
+    }
+    constexpr int kBack = T > 0 ? T - 1 : 0;
+    float v[kBack + (int)kConvolveRows], w[T > 0 ? T : 1];
+    const float* raw = p.raw + p.inner() + channel;
+#pragma unroll
+    for (int i = 0; i < kBack + (int)kConvolveRows; ++i) {
+        const int r = (int)row + i - kBack;                            // a row of the chunk, or behind it
+        v[i] = 0.0f;
+        if (i < kBack && (uint32_t)(kBack - i) >= p.tap_count) continue;
+        if (r >= 0) { if ((uint32_t)r < row + live) v[i] = raw[(size_t)r * p.raw_ld]; }
+        else if (base >= (uint32_t)-r) v[i] = ring[(size_t)((base + (uint32_t)r) & p.input_mask) * p.input_row() + channel];
+    }
+#pragma unroll
+    for (int j = 0; j < T; ++j) w[j] = (uint32_t)j < p.tap_count ? p.taps[(size_t)channel * p.tap_count + p.tap_count - 1u - j] : 0.0f;
+    const float bias = p.tap_bias[channel];
+#pragma unroll
+    for (int r = 0; r < (int)kConvolveRows; ++r) {
+        if ((uint32_t)r >= live) break;
+        float sum = 0.0f;
+#pragma unroll
+        for (int j = T - 1; j >= 0; --j) sum = fmaf(w[j], v[kBack + r - j], sum);
+        emit((uint32_t)r, silu(sum + bias));
+    }
+}
+
+template <int T>
+__global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const __grid_constant__ StateSpace p) {
+    extern __shared__ float vectors[];                                 // [2][8][np]: B, C
+    const uint32_t np = p.state_row(), x_row = p.x_row(), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const uint32_t base = p.positions[0], row = blockIdx.y * kConvolveRows, live = min(kConvolveRows, p.rows - row);
+    const float* ring = static_cast<const float*>(p.rings->ring_v);
+    if (blockIdx.x >= p.groups) {
+        const uint32_t i = (blockIdx.x - p.groups) * kConvolveThreads + tid, all = p.heads * x_row, k = i % x_row;
+        if (i >= all) return;
+        float* out = p.x + (size_t)row * all + i;
+        if (k >= p.vdim) {
+            for (uint32_t r = 0; r < live; ++r) out[(size_t)r * all] = 0.0f;
+            return;
+        }
+        convolve_rows<T>(p, ring, base, row, live, i / x_row * p.vdim + k, [&](uint32_t r, float v) { out[(size_t)r * all] = v; });
+        return;
+    }
+    const uint32_t group = blockIdx.x, per_group = p.heads / p.groups;
+    for (uint32_t i = tid; i < 2u * np; i += kConvolveThreads) {
+        const uint32_t which = i / np, n = i % np;
+        float *out = (which ? p.c : p.b) + ((size_t)row * p.groups + group) * np + n, *here = vectors + which * kConvolveRows * np + n;
+        if (n >= p.state) {
+            for (uint32_t r = 0; r < kConvolveRows; ++r) { here[r * np] = 0.0f; if (r < live) out[(size_t)r * p.groups * np] = 0.0f; }
+            continue;
+        }
+        for (uint32_t r = live; r < kConvolveRows; ++r) here[r * np] = 0.0f;
+        convolve_rows<T>(p, ring, base, row, live, p.inner() + (which * p.groups + group) * p.state + n, [&](uint32_t r, float v) {
+            here[r * np] = v;
+            out[(size_t)r * p.groups * np] = v;
+        });
+    }
+    for (uint32_t i = tid; i < live * per_group; i += kConvolveThreads) {
+        const uint32_t r = row + i / per_group, head = group * per_group + i % per_group;
+        p.steps[(size_t)r * p.heads + head] = step_of(p, p.raw, r, head);
+    }
+    __syncthreads();
+    for (uint32_t i = warp; i < kConvolveRows * 4u; i += kConvolveThreads / 32u) {
+        const uint32_t t = i / 4u, s = i % 4u;
+        if (t >= live) break;
+        const float *b = vectors + ((t & ~3u) + s) * np, *c = vectors + (kConvolveRows + t) * np;
+        float sum = 0.0f;
+        if (s <= (t & 3u))
+            for (uint32_t n = lane; n < np; n += 32u) sum = fmaf(c[n], b[n], sum);
+        sum = warp_sum(sum);
+        if (lane == 0) p.cb[((size_t)(row + t) * p.groups + group) * 4u + s] = sum;
+    }
+}
+
+// ------------------------------------------------------------------ launches
+
+template <typename Kernel>
+int allow_smem(Kernel kernel, std::once_flag* once, uint32_t bytes) {
+    int device = 0;
+    cudaGetDevice(&device);
+    cudaError_t error = cudaSuccess;
+    std::call_once(once[device & 63], [&] { error = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes); });
+    GF_CUDA(error);
+    return GF_OK;
 }
 
 template <int L, int NQ, int V, bool kPass>
 int launch_recurrence(const StateSpace& p, cudaStream_t stream, bool pdl) {
     constexpr uint32_t kWide = L * NQ * 4, per_warp = 32u / L * V;
     static std::once_flag once[64];
-    int device = 0;
-    cudaGetDevice(&device);
-    cudaError_t error = cudaSuccess;
-    std::call_once(once[device & 63], [&] {
-        error = cudaFuncSetAttribute(state_space_kernel<L, NQ, V, kPass>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemLimit);
-    });
-    GF_CUDA(error);
-    // As many warps per block as still give every SM a block; the block's columns are whole 16-byte pieces.
+    int status = GF_OK;
+    if constexpr (kPass) status = allow_smem(state_space_rows_kernel<L, NQ, V>, once, kSmemLimit);
+    else status = allow_smem(state_space_chunk_kernel<L, NQ, V>, once, kSmemLimit);
+    if (status != GF_OK) return status;
+    // As many warps per block as still give most SMs a block; the block's columns are whole 16-byte pieces.
     const uint32_t sequences = p.ring_stride ? p.rows : 1u;
     uint32_t warps = kMaxWarps;
     while (warps > 1u && (warps / 2u) * per_warp % 4u == 0u
-           && ((uint64_t)p.heads * sequences * ((p.vdim + warps * per_warp - 1u) / (warps * per_warp)) < (uint64_t)sm_count() || (warps / 2u) * per_warp >= p.vdim))
+           && ((uint64_t)p.heads * sequences * ((p.vdim + warps * per_warp - 1u) / (warps * per_warp)) * 5u < (uint64_t)sm_count() * 4u
+               || (warps / 2u) * per_warp >= p.vdim))
         warps /= 2u;
+    while (!kPass && warps > 1u && chunk_layout(chunk_tile<(int)kWide>(), kWide, warps * per_warp).bytes > kSmemLimit) warps /= 2u;
     const uint32_t columns = warps * per_warp;
-    const TileLayout layout = tile_layout(tile_tokens<(int)kWide>(), kWide, columns, kPass ? 1u : 2u);
-    return launch_kernel(state_space_kernel<L, NQ, V, kPass>, dim3(p.heads, (p.vdim + columns - 1u) / columns, sequences), dim3(warps * 32u), layout.bytes, stream, pdl, p);
+    const dim3 grid(p.heads, (p.vdim + columns - 1u) / columns, sequences);
+    if constexpr (kPass) return launch_kernel(state_space_rows_kernel<L, NQ, V>, grid, dim3(warps * 32u), pass_smem(kWide, columns), stream, pdl, p);
+    else return launch_kernel(state_space_chunk_kernel<L, NQ, V>, grid, dim3(warps * 32u), chunk_layout(chunk_tile<(int)kWide>(), kWide, columns).bytes, stream, pdl, p);
 }
 
 template <bool kPass>
@@ -345,9 +569,17 @@ int launch_state_space_rows(const StateSpace& p, cudaStream_t stream, bool pdl) 
 }
 
 int launch_state_space_chunk(const StateSpace& p, cudaStream_t stream) {
-    if (!usable(p) || p.ring_stride || !p.x || !p.b || !p.c || !p.steps || p.input_mask + 1u < p.tap_count - 1u) return fail(GF_ERR_INVALID, "state space: bad arguments");
-    const uint32_t items = p.heads * p.x_row() + 2u * p.groups * p.state_row() + p.heads;
-    convolve_chunk_kernel<<<dim3((items + 127u) / 128u, (p.rows + kConvolveRows - 1u) / kConvolveRows), 128, 0, stream>>>(p);
+    if (!usable(p) || p.ring_stride || !p.x || !p.b || !p.c || !p.steps || !p.cb || p.input_mask + 1u < p.tap_count - 1u) return fail(GF_ERR_INVALID, "state space: bad arguments");
+    const dim3 grid(p.groups + (p.heads * p.x_row() + kConvolveThreads - 1u) / kConvolveThreads, (p.rows + kConvolveRows - 1u) / kConvolveRows);
+    const uint32_t smem = 2u * kConvolveRows * p.state_row() * 4u;
+    static std::once_flag once[3][64];
+    int status = allow_smem(convolve_chunk_kernel<4>, once[0], 2u * kConvolveRows * kMaxStateSize * 4u);
+    if (status == GF_OK) status = allow_smem(convolve_chunk_kernel<8>, once[1], 2u * kConvolveRows * kMaxStateSize * 4u);
+    if (status == GF_OK) status = allow_smem(convolve_chunk_kernel<0>, once[2], 2u * kConvolveRows * kMaxStateSize * 4u);
+    if (status != GF_OK) return status;
+    if (p.tap_count <= 4u) convolve_chunk_kernel<4><<<grid, kConvolveThreads, smem, stream>>>(p);
+    else if (p.tap_count <= 8u) convolve_chunk_kernel<8><<<grid, kConvolveThreads, smem, stream>>>(p);
+    else convolve_chunk_kernel<0><<<grid, kConvolveThreads, smem, stream>>>(p);
     GF_CUDA(cudaGetLastError());
     return launch_by_state<false>(p, stream, false);
 }

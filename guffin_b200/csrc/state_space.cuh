@@ -27,8 +27,9 @@ struct StateSpace {
     uint32_t rows = 0, heads = 0, vdim = 0, state = 0, groups = 0, tap_count = 0, input_mask = 0;
     float* out = nullptr;                // [rows][heads * vdim]: passes: y * silu(gate); chunks: y
     // Chunks: the convolved inputs, x [rows][heads][vdim rounded up to 4], B and C [rows][groups][N rounded up to 4],
-    // and (dt, exp(decay * dt)) [rows][heads].
-    float *x = nullptr, *b = nullptr, *c = nullptr;
+    // (dt, decay * dt) [rows][heads], and the products of a row's C with the B of the rows of its four up to itself
+    // [rows][groups][4].
+    float *x = nullptr, *b = nullptr, *c = nullptr, *cb = nullptr;
     float2* steps = nullptr;
 
     __host__ __device__ uint32_t inner() const { return heads * vdim; }

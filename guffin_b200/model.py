@@ -95,6 +95,7 @@ lib.register({
     "gf_model_read_candidates": (i32, [vp, vp, u32]),
     "gf_model_read_logits": (i32, [vp, u32, vp]),
     "gf_model_read_kv": (i32, [vp, u32, u32, u32, vp, vp]),
+    "gf_model_read_state": (i32, [vp, u32, vp]),
     "gf_model_synchronize": (i32, [vp]),
     "gf_model_status": (i32, [vp, C.POINTER(u32)]),
     "gf_model_stream": (vp, [vp]),
@@ -252,6 +253,20 @@ class Model:
         """Committed cache rows of a latent-attention layer, [count, rank]."""
         out = np.empty((count, self.config["layers"][layer]["mixer"]["kv_rank"]), np.float32)
         check(self.L.gf_model_read_kv(self.handle, layer, first, count, out.ctypes.data, None))
+        return out
+
+    def read_keys_values(self, layer: int, first: int, count: int):
+        """Committed keys and values of a grouped-query attention layer, [count, kv_heads, dim] each."""
+        m = self.config["layers"][layer]["mixer"]
+        k, v = np.empty((count, m["kv_heads"], m["dim"]), np.float32), np.empty((count, m["kv_heads"], m["vdim"]), np.float32)
+        check(self.L.gf_model_read_kv(self.handle, layer, first, count, k.ctypes.data, v.ctypes.data))
+        return k, v
+
+    def read_state(self, layer: int) -> np.ndarray:
+        """The state of a recurrent layer after the committed tokens, [heads, vdim, N]."""
+        m = self.config["layers"][layer]["mixer"]
+        out = np.empty((m["heads"], m["vdim"], m["state"]), np.float32)
+        check(self.L.gf_model_read_state(self.handle, layer, out.ctypes.data))
         return out
 
     @property

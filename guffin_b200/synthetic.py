@@ -249,6 +249,86 @@ def zasevik_active_parameters(config: dict) -> int:
     return int(round(total))
 
 
+def tufirax_attention(heads, kv_heads, dim, scale=None, softcap=30.0, rot_dims=None, base=10000.0, ff=0, weights_of=None) -> dict:
+    """A layer of grouped-query attention and a gated feed-forward (none with ff = 0)."""
+    mixer = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=1.0 / math.sqrt(dim) if scale is None else scale, softcap=softcap,
+                 rot=dict(base=base, dims=dim if rot_dims is None else rot_dims))
+    return _tufirax_layer("attention", mixer, ff, weights_of)
+
+
+def tufirax_state_space(heads, vdim, state, groups=1, conv=4, norm_groups=1, ff=0, weights_of=None) -> dict:
+    """A state-space layer and a gated feed-forward (none with ff = 0)."""
+    return _tufirax_layer("mamba2", dict(heads=heads, vdim=vdim, state=state, groups=groups, conv=conv, norm_groups=norm_groups), ff, weights_of)
+
+
+def _tufirax_layer(kind, mixer, ff, weights_of) -> dict:
+    layer = dict(type=kind, mixer=mixer, mlp=dense_mlp(ff) if ff else None)
+    return layer if weights_of is None else dict(layer, weights_of=weights_of)
+
+
+def tufirax_config(width, vocab, layers, eps=1e-6) -> dict:
+    return dict(architecture="Tufirax", norm=dict(eps=eps), vocab=vocab, width=width, layers=layers)
+
+
+def tufirax_shapes(config: dict) -> dict:
+    """Tensor name -> shape of every tensor of a Tufirax configuration."""
+    W, shapes = config["width"], {"embed": (config["vocab"], config["width"])}
+    for i, layer in enumerate(config["layers"]):
+        if "weights_of" in layer:
+            continue
+        p, m = f"l{i}", layer["mixer"]
+        inner = m["heads"] * m["vdim"]
+        shapes[f"{p}.norm1"] = (W,)
+        if layer["type"] == "attention":
+            q, k = m["heads"] * m["dim"], m["kv_heads"] * m["dim"]
+            shapes.update({f"{p}.mix.q": (q, W), f"{p}.mix.k": (k, W), f"{p}.mix.q.norm": (q,), f"{p}.mix.k.norm": (k,), f"{p}.mix.sink": (m["heads"],),
+                           f"{p}.mix.g": (m["heads"], W)})
+        else:
+            channels = inner + 2 * m["groups"] * m["state"]
+            shapes.update({f"{p}.mix.in": (inner + channels + m["heads"], W), f"{p}.mix.conv": (channels, m["conv"]), f"{p}.mix.conv.b": (channels,),
+                           f"{p}.mix.dt_bias": (m["heads"],), f"{p}.mix.A_log": (m["heads"],), f"{p}.mix.D": (m["heads"],), f"{p}.mix.norm": (inner,)})
+        shapes[f"{p}.mix.o"] = (W, inner)
+        if layer["mlp"]:
+            ff = layer["mlp"]["ff"]
+            shapes.update({f"{p}.norm2": (W,), f"{p}.mlp.gate": (ff, W), f"{p}.mlp.up": (ff, W), f"{p}.mlp.down": (W, ff)})
+    shapes.update({"final.norm": (W,), "head": (config["vocab"], W)})
+    return shapes
+
+
+def iter_tufirax_weights(config: dict, seed: int):
+    """Yields (name, array): matrices as bfloat16 bits with entries of variance 1 / inputs (the token table's 1), vectors
+    as f32.  Step sizes lie between 0.001 and 0.3, decay rates between 1 and 16."""
+    rng = np.random.default_rng(seed)
+    for name, shape in tufirax_shapes(config).items():
+        if len(shape) == 2:
+            values = rng.standard_normal(shape, dtype=np.float32)
+            if name != "embed":
+                values *= np.float32(1.0 / math.sqrt(shape[1]))
+            bits = values.view(np.uint32)
+            yield name, ((bits + 0x7fff + ((bits >> 16) & 1)) >> 16).astype(np.uint16)
+        elif name.endswith(".sink"):
+            yield name, rng.normal(1.0, 1.0, shape).astype(np.float32)
+        elif name.endswith(".dt_bias"):
+            steps = np.exp(rng.uniform(math.log(0.001), math.log(0.3), shape))
+            yield name, (steps + np.log(-np.expm1(-steps))).astype(np.float32)      # softplus of it is the step
+        elif name.endswith(".A_log"):
+            yield name, np.log(rng.uniform(1.0, 16.0, shape)).astype(np.float32)
+        elif name.endswith(".conv.b"):
+            yield name, rng.normal(0.0, 0.2, shape).astype(np.float32)
+        else:
+            yield name, rng.uniform(0.5, 1.5, shape).astype(np.float32)
+
+
+def tufirax_active_parameters(config: dict) -> int:
+    """Matrix elements one token's pass multiplies with (a shared layer counts every time it runs; the head included)."""
+    shapes, total = tufirax_shapes(config), config["vocab"] * config["width"]
+    for i, layer in enumerate(config["layers"]):
+        while "weights_of" in config["layers"][i]:
+            i = config["layers"][i]["weights_of"]
+        total += sum(s[0] * s[1] for n, s in shapes.items() if n.startswith(f"l{i}.") and len(s) == 2 and not n.endswith(".conv"))
+    return total
+
+
 def model_weight_bytes(name: str, config: dict | None = None) -> int:
     """Native GGUF bytes one decode pass streams: every matrix once, the tied head included."""
     config = config or model_config(name)

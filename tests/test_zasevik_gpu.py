@@ -3,7 +3,6 @@ models of several shapes in both precisions, cut and batched in every way the pl
 import ctypes as C
 import json
 import os
-import struct
 import subprocess
 import sys
 
@@ -12,6 +11,7 @@ import pytest
 
 from guffin_b200 import synthetic as syn
 from oracle import zasevik as z
+from tests.layered import greedy_reference, limits_of, rel_l2, row_errors, tokens_for, within, write_folder
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
@@ -24,29 +24,8 @@ def gm(gf):
     return model
 
 
-def rel_l2(got, want):
-    return float(np.linalg.norm(np.asarray(got, np.float64) - want) / max(np.linalg.norm(want), 1e-30))
-
-
-def row_errors(got, want):
-    """Per row: root mean square of the difference over that of the wanted logits, means taken off."""
-    d, w = np.asarray(got, np.float64) - want, want - want.mean(1, keepdims=True)
-    d -= d.mean(1, keepdims=True)
-    return np.sqrt((d * d).mean(1) / (w * w).mean(1))
-
-
 def plain(config, weights, tokens, precision):
-    """The plain implementation's logits and the error a row may have: three times what rounding alone causes there, or
-    to the worst rows but a few."""
-    want = z.Reference(config, weights).extend(tokens)
-    if precision == "float32":
-        return want, np.full(len(tokens), 1e-4)
-    rounded = row_errors(z.Reference(config, weights, cast=z.bf16).extend(tokens), want)
-    return want, 3.0 * np.maximum(rounded, max(np.quantile(rounded, 0.98), 2e-3))
-
-
-def within(got, want, limits):
-    return bool((row_errors(got, want) <= limits).all())
+    return limits_of(z.Reference, z.bf16, config, weights, tokens, precision)
 
 
 # ------------------------------------------------------------------------------------------- operators
@@ -207,10 +186,6 @@ def make(gm, name, seed=None):
 PRECISIONS = ["float32", "bfloat16"]
 
 
-def tokens_for(config, count, seed=0):
-    return np.random.default_rng(seed).integers(0, config["vocab"], count).astype(np.uint32)
-
-
 @pytest.mark.parametrize("name", CONFIGS)
 @pytest.mark.parametrize("precision", PRECISIONS)
 def test_whole_prompts_and_rows(gm, name, precision):
@@ -363,17 +338,6 @@ def test_streams_equal_conversations_alone(gm, precision):
     assert within(streams.logits(2)[None], want[-1:], limits[-1:])
 
 
-def greedy_reference(config, weights, prompt, count):
-    ref, out, margins = z.Reference(config, weights), [], []
-    logits = ref.extend(prompt)[-1]
-    for _ in range(count):
-        out.append(int(np.argmax(logits)))
-        top = np.sort(logits)[-2:]
-        margins.append(top[1] - top[0])
-        logits = ref.extend(out[-1:])[-1]
-    return out, min(margins)
-
-
 @pytest.mark.parametrize("name", ["sharp attention", "every layer its own sizes"])
 def test_greedy_generation(gm, name):
     """The generation engine, the batch, the engine with a drafter, and the plain implementation choose the same tokens."""
@@ -381,7 +345,7 @@ def test_greedy_generation(gm, name):
     config, bits, weights = make(gm, name)
     plan = gm.Model.described(config, bits, 256, 4, "float32")
     prompts = [tokens_for(config, n, n) for n in (40, 3, 90)]
-    wanted = [greedy_reference(config, weights, p, 48) for p in prompts]
+    wanted = [greedy_reference(z.Reference, config, weights, p, 48) for p in prompts]
     assert all(margin > 1e-3 for _, margin in wanted) and (name != "sharp attention" or len(set(wanted[0][0])) > 10)
     options = ge.sampler_options(0.0)
     engine = ge.H1(plan, None, ge.H1Options(options, 0, 0, 0.0, 0, 0))
@@ -430,16 +394,6 @@ def test_what_a_layered_plan_does_not_offer(gm):
 
 # ------------------------------------------------------------------------------------------- folders and programs
 
-def write_folder(path, config, bits):
-    header, blob = {"__metadata__": {"format": "pt"}}, b""
-    for name, value in bits.items():
-        header[name] = dict(dtype="BF16", shape=list(value.shape), data_offsets=[len(blob), len(blob) + value.nbytes])
-        blob += value.tobytes()
-    text = json.dumps(header).encode()
-    (path / "config.json").write_text(json.dumps(config))
-    (path / "model.safetensors").write_bytes(struct.pack("<Q", len(text)) + text + blob)
-
-
 @pytest.mark.parametrize("precision", PRECISIONS)
 def test_trace_replay(gm, tmp_path, precision):
     config, bits, weights = make(gm, "experts")
@@ -470,7 +424,7 @@ def test_command_line(gm, tmp_path):
     config, bits, weights = make(gm, "every layer its own sizes")
     write_folder(tmp_path, config, bits)
     prompt = tokens_for(config, 40, 40)
-    want, _ = greedy_reference(config, weights, prompt, 10)
+    want, _ = greedy_reference(z.Reference, config, weights, prompt, 10)
     text = ",".join(str(t) for t in prompt)
     run = lambda *args: subprocess.run([sys.executable, "-m", "guffin_b200", *args], cwd=ROOT, capture_output=True, text=True, timeout=300)
     one = run("generate", "--model", str(tmp_path), "--tokens", text, "--max-tokens", "10", "--dtype", "float32")

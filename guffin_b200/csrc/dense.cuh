@@ -229,7 +229,7 @@ __device__ __forceinline__ float clamped_gate(float gate, float up, float limit)
     const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
     return g * sigmoid(1.702f * g) * (u + 1.0f);
 }
-__device__ __forceinline__ float silu(float z) { return z / (1.0f + expf(-z)); }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.0f + __expf(-z)); }      // to a few 1e-7
 __device__ __forceinline__ float gelu_tanh(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z))); }
 // One warp turns the (maximum, sum) pairs of a query's key partitions, and its sink, into the factors of the merge.
 __device__ __forceinline__ void merge_factors(const float* ml, uint32_t parts, float sink, float* factors) {

@@ -33,12 +33,11 @@ __device__ __forceinline__ uint32_t half_pair(float lo, float hi) {
 
 constexpr uint32_t kPrepareThreads = 256;
 
-// Cosine and sine of position * frequency: the turns in double, their remainder in f32.
-__device__ __forceinline__ float2 rotation(uint32_t position, double frequency) {
-    const double turns = (double)position * frequency * 0.15915494309189535;      // 1 / (2 pi)
-    float s, c;
-    sincospif((float)(2.0 * (turns - rint(turns))), &s, &c);
-    return make_float2(c, s);
+// Cosine and sine of a position's angle in pair i.
+__device__ __forceinline__ float2 rotation(const QueryKey& p, uint32_t position, uint32_t i) {
+    const uint32_t half = p.rotated / 2u;
+    const float2 a = p.turns[(size_t)(position % kTurnSpan) * half + i], b = p.spans[(size_t)(position / kTurnSpan) * half + i];
+    return make_float2(a.x * b.x - a.y * b.y, a.y * b.x + a.x * b.y);
 }
 
 // Dimension d of a head that starts at `first` of a projected row: normalised, turned.
@@ -65,7 +64,7 @@ __global__ void __launch_bounds__(kPrepareThreads) query_key_kernel(const __grid
     const uint32_t row = blockIdx.x, tid = threadIdx.x, half = p.rotated / 2u;
     const uint32_t q_width = p.heads * p.dim, k_width = p.kv_heads * p.dim;
     const uint32_t position = p.chain ? p.positions[0] + row : p.positions[row];
-    for (uint32_t i = tid; i < half; i += kPrepareThreads) turn[i] = rotation(position, p.frequencies[i]);
+    for (uint32_t i = tid; i < half; i += kPrepareThreads) turn[i] = rotation(p, position, i);
     pdl_wait();
     pdl_launch_dependents();
     const float *q = p.raw_q ? p.raw_q + (size_t)row * p.q_ld : nullptr, *k = p.raw_k + (size_t)row * p.k_ld, *v = p.raw_v + (size_t)row * p.v_ld;
@@ -159,14 +158,20 @@ __device__ __forceinline__ void merge_query(const GroupedAttention& p, uint32_t 
     merge_factors(pairs, p.parts, p.sink ? p.sink[head] : -INFINITY, factors);
     __syncwarp();
     const float gate = head_gate(p, row, head);
+#pragma unroll 1
     for (uint32_t d = lane * 4u; d < p.vdim; d += 128u) {              // a row's head is whole 16-byte pieces
         const float4* from = reinterpret_cast<const float4*>(p.partial_out + query * p.parts * p.row_head + d);
         float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-#pragma unroll 16
-        for (uint32_t part = 0; part < p.parts; ++part) {
-            const float4 x = __ldcg(from + part * (p.row_head / 4u));
-            const float f = factors[part];
-            v = make_float4(fmaf(x.x, f, v.x), fmaf(x.y, f, v.y), fmaf(x.z, f, v.z), fmaf(x.w, f, v.w));
+#pragma unroll 1
+        for (uint32_t first = 0; first < p.parts; first += 16u) {
+            float4 x[16];
+#pragma unroll
+            for (uint32_t i = 0; i < 16u; ++i) x[i] = first + i < p.parts ? __ldcg(from + (first + i) * (p.row_head / 4u)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+            for (uint32_t i = 0; i < 16u; ++i) {
+                const float f = first + i < p.parts ? factors[first + i] : 0.0f;
+                v = make_float4(fmaf(x[i].x, f, v.x), fmaf(x[i].y, f, v.y), fmaf(x[i].z, f, v.z), fmaf(x[i].w, f, v.w));
+            }
         }
         const float four[4] = {v.x * gate, v.y * gate, v.z * gate, v.w * gate};
 #pragma unroll
@@ -176,62 +181,91 @@ __device__ __forceinline__ void merge_query(const GroupedAttention& p, uint32_t 
     __syncwarp();
 }
 
-// The prologue of a fused pass: the block's queries (zeros behind them) and the pass's own keys and values of key/value
-// head `kv`, prepared from the projections.  Rows [first_row, first_row + query_rows) have queries here; with `own` all
-// of `rows` leave their cache rows in own_k and own_v, and with `publish` in the private rows too.
+// The prologue of a fused pass: the block's queries and the pass's own keys and values of key/value head `kv`, prepared
+// from the projections.  Rows [first_row, first_row + query_rows) have queries here; with `own` all of `rows` leave their
+// cache rows in own_k and own_v, and with `publish` in the private rows too.  Loops stay rolled: every block runs this
+// once, and instructions have to be fetched as well.
 struct FusedRows { uint32_t first_row, query_rows, rows, row0; bool own, publish; };
 template <int kThreads>
 __device__ __forceinline__ void prepare_fused(const GroupedAttention& p, const FusedRows& f, const float2* turns, uint32_t kv, uint32_t first_query, uint32_t queries,
                                               __half* q_tile, __half* own_k, __half* own_v, uint32_t stride) {
     constexpr uint32_t kWarps = kThreads / 32u, kItems = 16u + kGroupedFusedRows;
-    __shared__ float sums[kItems][kWarps];
+    __shared__ float sums[kItems][kWarps], factors[kItems];
     const QueryKey& in = p.prepare;
-    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, group = p.heads / p.kv_heads, half = in.rotated / 2u;
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, group = p.heads / p.kv_heads, half = in.rotated / 2u, couples = p.row_head / 2u;
     const uint32_t q_width = in.heads * in.dim, k_width = in.kv_heads * in.dim, items = f.query_rows + (f.own ? f.rows : 0u);
+#pragma unroll 1
     for (uint32_t item = 0; item < items; ++item) {
         const bool query = item < f.query_rows;
         const uint32_t row = f.row0 + (query ? f.first_row + item : item - f.query_rows), width = query ? q_width : k_width;
         const float* x = query ? in.raw_q + (size_t)row * in.q_ld : in.raw_k + (size_t)row * in.k_ld;
         float sum = 0.0f;
-#pragma unroll 8
-        for (uint32_t i = threadIdx.x; i < width; i += kThreads) sum = fmaf(x[i], x[i], sum);
+        if ((width | in.q_ld | in.k_ld) % 4u == 0u) {
+#pragma unroll 1
+            for (uint32_t i = tid * 4u; i < width; i += kThreads * 16u) {
+                float4 v[4];
+#pragma unroll
+                for (uint32_t j = 0; j < 4u; ++j)
+                    v[j] = i + j * kThreads * 4u < width ? *reinterpret_cast<const float4*>(x + i + j * kThreads * 4u) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                for (uint32_t j = 0; j < 4u; ++j) sum = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, fmaf(v[j].w, v[j].w, sum))));
+            }
+        } else {
+#pragma unroll 4
+            for (uint32_t i = tid; i < width; i += kThreads) sum = fmaf(x[i], x[i], sum);
+        }
         sum = warp_sum(sum);
         if (lane == 0) sums[item][warp] = sum;
     }
     __syncthreads();
-    auto inverse = [&](uint32_t item, uint32_t width) {
+    if (tid < items) {
         float sum = 0.0f;
 #pragma unroll
-        for (uint32_t w = 0; w < kWarps; ++w) sum += sums[item][w];
-        return 1.0f / sqrtf(sum / (float)width + in.eps);
-    };
-    for (uint32_t m = warp; m < 16u; m += kWarps) {
-        const uint32_t query = first_query + m;
-        const bool valid = query < queries;
-        const uint32_t r = valid ? query / group : 0u, first = (kv * group + query % group) * in.dim;
-        const float inv = valid ? inverse(r - f.first_row, q_width) : 0.0f;
-        const float* x = in.raw_q + (size_t)(f.row0 + r) * in.q_ld;
-#pragma unroll 4
-        for (uint32_t d = lane; d < p.row_head; d += 32u)
-            q_tile[m * stride + d] = valid && d < in.dim ? cache_half(in, turned(in, x, in.q_gain, inv, turns + r * half, first, d) * in.scale) : __float2half_rn(0.0f);
+        for (uint32_t w = 0; w < kWarps; ++w) sum += sums[tid][w];
+        factors[tid] = 1.0f / sqrtf(sum / (float)(tid < f.query_rows ? q_width : k_width) + in.eps);
+    }
+    __syncthreads();
+    // Couples of dimensions: those that turn together, then neighbours.
+    const uint32_t tile_queries = min(16u, queries - first_query), lines = tile_queries + (f.own ? f.rows : 0u);
+#pragma unroll 2
+    for (uint32_t i = tid; i < lines * couples; i += kThreads) {
+        const uint32_t line = i / couples, j = i % couples;
+        const bool query = line < tile_queries;
+        const uint32_t r = query ? (first_query + line) / group : line - tile_queries;
+        const uint32_t first = (query ? kv * group + (first_query + line) % group : kv) * in.dim;
+        const uint32_t d0 = j < half ? j : 2u * j, d1 = j < half ? j + half : 2u * j + 1u;       // 2 j = rotated + 2 (j - half)
+        const float* x = (query ? in.raw_q + (size_t)(f.row0 + r) * in.q_ld : in.raw_k + (size_t)(f.row0 + r) * in.k_ld) + first;
+        const float* gain = (query ? in.q_gain : in.k_gain) + first;
+        const float inv = factors[query ? r - f.first_row : f.query_rows + r];
+        float u = d0 < in.dim ? x[d0] * inv * gain[d0] : 0.0f, v = d1 < in.dim ? x[d1] * inv * gain[d1] : 0.0f;
+        if (j < half) {
+            const float2 turn = turns[r * half + j];
+            const float turned_u = u * turn.x - v * turn.y;
+            v = v * turn.x + u * turn.y;
+            u = turned_u;
+        }
+        const float scale = query ? in.scale : 1.0f;
+        const __half hu = cache_half(in, u * scale), hv = cache_half(in, v * scale);
+        __half* to = query ? q_tile + line * stride : own_k + r * stride;
+        to[d0] = hu;
+        to[d1] = hv;
+        if (!query && f.publish) {
+            __half* row = static_cast<__half*>(in.keys) + ((size_t)(f.row0 + r) * p.kv_heads + kv) * p.row_head;
+            row[d0] = hu;
+            row[d1] = hv;
+        }
     }
     if (!f.own) return;
-    for (uint32_t r = warp; r < f.rows; r += kWarps) {
-        const float inv = inverse(f.query_rows + r, k_width);
-        const float *x = in.raw_k + (size_t)(f.row0 + r) * in.k_ld, *v = in.raw_v + (size_t)(f.row0 + r) * in.v_ld + kv * in.vdim;
-        const size_t to = ((size_t)(f.row0 + r) * p.kv_heads + kv) * p.row_head;
-#pragma unroll 4
-        for (uint32_t d = lane; d < p.row_head; d += 32u) {
-            const __half key = d < in.dim ? cache_half(in, turned(in, x, in.k_gain, inv, turns + r * half, kv * in.dim, d)) : __float2half_rn(0.0f);
-            const __half value = d < in.vdim ? cache_half(in, v[d]) : __float2half_rn(0.0f);
-            own_k[r * stride + d] = key;
-            own_v[r * stride + d] = value;
-            if (f.publish) { static_cast<__half*>(in.keys)[to + d] = key; static_cast<__half*>(in.values)[to + d] = value; }
-        }
+#pragma unroll 1
+    for (uint32_t i = tid; i < f.rows * p.row_head; i += kThreads) {
+        const uint32_t r = i / p.row_head, d = i % p.row_head;
+        const __half value = cache_half(in, d < in.vdim ? in.raw_v[(size_t)(f.row0 + r) * in.v_ld + kv * in.vdim + d] : 0.0f);
+        own_v[r * stride + d] = value;
+        if (f.publish) static_cast<__half*>(in.values)[((size_t)(f.row0 + r) * p.kv_heads + kv) * p.row_head + d] = value;
     }
 }
 
-constexpr uint32_t kRowsWarps = 4;
+constexpr uint32_t kRowsWarps = 4, kRowsTile = 16;
 
 // A block serves sixteen queries of one key/value head -- (row, head of the group) pairs, heads fastest -- against one
 // partition of the keys; its warps take tiles of keys in turn, the next one copied while this one is used, and keep
@@ -240,7 +274,7 @@ template <int G>
 __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(const __grid_constant__ GroupedAttention p) {
     extern __shared__ __align__(16) uint8_t smem[];
     __shared__ float warp_top[kRowsWarps][16], warp_sum_of[kRowsWarps][16], scratch[kRowsWarps][kGroupedMaxParts * 3u];
-    constexpr uint32_t kTile = G <= 8 ? 32u : 16u;
+    constexpr uint32_t kTile = kRowsTile;
     const uint32_t stride = p.row_head + 8u, pieces = p.row_head / 8u;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, g = lane >> 2, t = lane & 3u;
     __half* q_tile = reinterpret_cast<__half*>(smem);
@@ -283,7 +317,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         copies_commit();
         float2* turns = reinterpret_cast<float2*>(own_rows + 2u * rows * stride);
         const uint32_t half = p.prepare.rotated / 2u;
-        for (uint32_t i = tid; i < rows * half; i += kRowsWarps * 32u) turns[i] = rotation(base + i / half, p.prepare.frequencies[i % half]);
+        for (uint32_t i = tid; i < rows * half; i += kRowsWarps * 32u) turns[i] = rotation(p.prepare, base + i / half, i % half);
         const uint32_t last_query = min(first_query + 15u, queries - 1u);
         FusedRows f;
         f.first_row = first_query / group; f.query_rows = last_query / group - f.first_row + 1u; f.rows = rows; f.row0 = chain ? 0u : z;
@@ -408,9 +442,11 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         if ((uint32_t)o * 8u >= p.row_head) break;
 #pragma unroll
         for (int i = 0; i < 2; ++i)
-            *reinterpret_cast<float2*>(parked + (warp * 16u + g + 8u * i) * parked_ld + o * 8u + 2u * t) = make_float2(acc[o][2 * i], acc[o][2 * i + 1]);
+            if (first_query + g + 8u * i < queries)
+                *reinterpret_cast<float2*>(parked + (warp * 16u + g + 8u * i) * parked_ld + o * 8u + 2u * t) = make_float2(acc[o][2 * i], acc[o][2 * i + 1]);
     }
     __syncthreads();
+#pragma unroll 1
     for (uint32_t m = warp; m < 16u; m += kRowsWarps) {
         const uint32_t query = first_query + m;
         if (query >= queries) break;
@@ -430,6 +466,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         } else if (lane == 0u) {
             *reinterpret_cast<float2*>(p.partial_ml + (((size_t)row * p.heads + head) * p.parts + part) * 2u) = make_float2(most, total);
         }
+#pragma unroll 1
         for (uint32_t d = lane; d < p.vdim; d += 32u) {
             float v = 0.0f;
 #pragma unroll
@@ -439,6 +476,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         }
     }
     if (p.parts == 1u || !last_to_arrive(p.counters + (size_t)blockIdx.z * gridDim.x + blockIdx.x, p.parts)) return;
+#pragma unroll 1
     for (uint32_t m = warp; m < 16u; m += kRowsWarps) {
         const uint32_t query = first_query + m;
         if (query >= queries) break;
@@ -524,7 +562,7 @@ int allow_smem(Kernel kernel, std::once_flag* once, uint32_t bytes) {
 
 template <int G>
 int launch_rows(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
-    constexpr uint32_t kTile = G <= 8 ? 32u : 16u;
+    constexpr uint32_t kTile = kRowsTile;
     static std::once_flag once[64];
     const int status = allow_smem(grouped_attention_kernel<G>, once, 200u * 1024u);
     if (status != GF_OK) return status;
@@ -538,7 +576,7 @@ int launch_rows(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
 
 int launch_query_key(QueryKey p, cudaStream_t stream, bool pdl) {
     if (!p.raw_k || !p.raw_v || (p.raw_q && (!p.q_gain || !p.q)) || !p.k_gain || !p.positions || !p.keys || !p.values || p.rows == 0 || p.heads == 0 || p.kv_heads == 0
-        || p.dim == 0 || p.vdim == 0 || p.row_head < p.dim || p.row_head < p.vdim || p.rotated > p.dim || p.rotated % 2u || (p.rotated && !p.frequencies))
+        || p.dim == 0 || p.vdim == 0 || p.row_head < p.dim || p.row_head < p.vdim || p.rotated > p.dim || p.rotated % 2u || (p.rotated && (!p.turns || !p.spans)))
         return fail(GF_ERR_INVALID, "query and key preparation: bad arguments");
     p.pairs = p.dim % 2u == 0u && p.vdim % 2u == 0u && p.rotated % 4u == 0u && p.q_ld % 2u == 0u && p.k_ld % 2u == 0u && p.v_ld % 2u == 0u ? 1u : 0u;
     return launch_kernel(query_key_kernel, dim3(p.rows), dim3(kPrepareThreads), p.rotated / 2u * sizeof(float2), stream, pdl, p);
@@ -546,14 +584,14 @@ int launch_query_key(QueryKey p, cudaStream_t stream, bool pdl) {
 
 uint32_t grouped_attention_parts(uint32_t rows, uint32_t heads, uint32_t kv_heads, uint32_t positions, bool chain) {
     const uint32_t queries = (chain ? rows : 1u) * (heads / kv_heads), blocks = (queries + 15u) / 16u * kv_heads * (chain ? 1u : rows);
-    // At least a tile for every warp of a partition.
-    const uint32_t most = std::max(1u, (positions + 127u) / 128u);
+    // Two tiles for every warp of a partition, and few partitions where they are short: the last block reads all of them.
+    const uint32_t most = std::max(1u, std::min((positions + 127u) / 128u, std::max(16u, positions / 512u)));
     return std::max(1u, std::min({most, kGroupedMaxParts, (uint32_t)sm_count() / std::max(1u, blocks)}));
 }
 
 int launch_grouped_attention(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
     if (p.fused ? (!grouped_attention_on_tensor_cores(p.row_head, p.f32 != 0u) || p.rows > kGroupedFusedRows || !p.prepare.raw_q || !p.prepare.raw_k || !p.prepare.raw_v
-                   || !p.prepare.keys || !p.prepare.values || p.prepare.row_head != p.row_head || p.prepare.vdim != p.vdim || (p.prepare.rotated && !p.prepare.frequencies))
+                   || !p.prepare.keys || !p.prepare.values || p.prepare.row_head != p.row_head || p.prepare.vdim != p.vdim || (p.prepare.rotated && (!p.prepare.turns || !p.prepare.spans)))
                 : !p.q)
         return fail(GF_ERR_INVALID, "grouped attention: bad arguments");
     if (!p.rings || !p.own_k || !p.own_v || !p.positions || !p.result.data || p.rows == 0 || p.heads == 0 || p.kv_heads == 0 || p.heads % p.kv_heads

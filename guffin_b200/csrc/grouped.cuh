@@ -12,13 +12,14 @@ namespace gf {
 __host__ __device__ inline uint32_t grouped_row_head(uint32_t dim, uint32_t vdim) { return ((dim > vdim ? dim : vdim) + 15u) / 16u * 16u; }
 
 // Projected rows to queries and cache rows: rmsnorm over the whole row, times the gain, then the first `rotated`
-// dimensions of every head turned by position * frequency in pairs (i, i + rotated / 2); queries times `scale`; values
-// as projected.
+// dimensions of every head turned by an angle that grows with the position, in pairs (i, i + rotated / 2); queries times
+// `scale`; values as projected.  A position's turn is the product of two tabulated ones.
+constexpr uint32_t kTurnSpan = 1024;
 struct QueryKey {
     const float *raw_q = nullptr, *raw_k = nullptr, *raw_v = nullptr;      // [rows][ld]; without raw_q the cache rows alone
     uint32_t q_ld = 0, k_ld = 0, v_ld = 0;
     const float *q_gain = nullptr, *k_gain = nullptr;
-    const double* frequencies = nullptr;           // [rotated / 2], radians per position
+    const float2 *turns = nullptr, *spans = nullptr;       // cosine and sine of positions 0 .. kTurnSpan - 1, and of multiples of it: [..][rotated / 2]
     const uint32_t* positions = nullptr;           // chain: position of row 0; else the position of every row
     bool chain = true;
     void *q = nullptr, *keys = nullptr, *values = nullptr;                 // [rows][heads][row_head], [rows][kv heads][row_head]

@@ -202,7 +202,8 @@ int Model::finalize_layered() {
     uint32_t q_width = 0, latent = 0, heads = 0, values = 0, ff = 0, top = 0, experts = 0, expert_ff = 0, shared_ff = 0, query_elements = 0;
     uint32_t k_width = 0, prepared = 0;
     size_t partial = 0, partial_pairs = 0;             // elements per row
-    p.frequencies.assign(s.layers.size(), nullptr);
+    p.turns.assign(s.layers.size(), {nullptr, nullptr});
+    std::map<std::pair<uint32_t, double>, std::pair<const float2*, const float2*>> rotations;
     for (uint32_t l = 0; l < s.layers.size(); ++l) {
         LayeredLayer& w = p.layers[l];
         const MixerSpec& m = s.layers[l].mixer;
@@ -240,10 +241,29 @@ int Model::finalize_layered() {
             prepared = std::max(prepared, m.heads * row_head);
             partial = std::max(partial, (size_t)m.heads * kGroupedMaxParts * row_head);
             partial_pairs = std::max<size_t>(partial_pairs, m.heads * kGroupedMaxParts * 2u);
-            std::vector<double> frequencies(std::max(1u, m.rotated / 2u), 0.0);
-            for (uint32_t i = 0; i < m.rotated / 2u; ++i) frequencies[i] = std::pow(m.rotation_base, -2.0 * (double)i / (double)m.rotated);
-            GF_TRY(plan_alloc(allocations_, &p.frequencies[l], frequencies.size()));
-            GF_CUDA(cudaMemcpy(p.frequencies[l], frequencies.data(), frequencies.size() * sizeof(double), cudaMemcpyHostToDevice));
+            // Angles in double; one pair of tables per (dimensions, base).
+            const uint32_t half = m.rotated / 2u, spans = c.context / kTurnSpan + 1u;
+            auto& tables = rotations[{m.rotated, m.rotation_base}];
+            if (half && !tables.first) {
+                auto tabulate = [&](uint32_t count, uint32_t step, const float2** out) -> int {
+                    std::vector<float2> host((size_t)count * half);
+                    for (uint32_t i = 0; i < half; ++i) {
+                        const double frequency = std::pow(m.rotation_base, -2.0 * (double)i / (double)m.rotated);
+                        for (uint32_t n = 0; n < count; ++n) {
+                            const double angle = (double)n * (double)step * frequency;
+                            host[(size_t)n * half + i] = make_float2((float)std::cos(angle), (float)std::sin(angle));
+                        }
+                    }
+                    float2* dev = nullptr;
+                    GF_TRY(plan_alloc(allocations_, &dev, host.size()));
+                    GF_CUDA(cudaMemcpy(dev, host.data(), host.size() * sizeof(float2), cudaMemcpyHostToDevice));
+                    *out = dev;
+                    return GF_OK;
+                };
+                GF_TRY(tabulate(kTurnSpan, 1u, &tables.first));
+                GF_TRY(tabulate(spans, kTurnSpan, &tables.second));
+            }
+            p.turns[l] = tables;
         } else {
             q_width = std::max(q_width, state_inputs_ld(m));
         }
@@ -393,7 +413,7 @@ int Model::encode_layers(uint32_t rows, bool logits, const LayeredRows& where) {
         QueryKey prepare;
         prepare.raw_q = p.raw_q; prepare.raw_k = prepare.raw_v = p.raw_k;
         prepare.q_ld = m.heads * m.dim; prepare.k_ld = prepare.v_ld = m.kv_heads * m.dim;
-        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.frequencies = p.frequencies[l];
+        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.turns = p.turns[l].first; prepare.spans = p.turns[l].second;
         prepare.positions = where.positions; prepare.chain = where.ring_stride == 0u;
         prepare.q = p.query; prepare.keys = caches_[l].private_k; prepare.values = caches_[l].private_v;
         prepare.rows = rows; prepare.heads = m.heads; prepare.kv_heads = m.kv_heads; prepare.dim = m.dim; prepare.vdim = m.vdim;
@@ -733,7 +753,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         QueryKey prepare;
         prepare.raw_q = last ? nullptr : a.raw_q; prepare.raw_k = prepare.raw_v = a.raw_k;
         prepare.q_ld = m.heads * m.dim; prepare.k_ld = prepare.v_ld = m.kv_heads * m.dim;
-        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.frequencies = p.frequencies[l]; prepare.positions = state_dev_;
+        prepare.q_gain = w.q_gain; prepare.k_gain = w.k_gain; prepare.turns = p.turns[l].first; prepare.spans = p.turns[l].second; prepare.positions = state_dev_;
         prepare.q = a.prepared_q; prepare.keys = a.private_rows[l]; prepare.values = a.private_values[l];
         prepare.rows = rows; prepare.heads = m.heads; prepare.kv_heads = m.kv_heads; prepare.dim = m.dim; prepare.vdim = m.vdim;
         prepare.row_head = row_head; prepare.rotated = m.rotated; prepare.f32 = f32 ? 1u : 0u;

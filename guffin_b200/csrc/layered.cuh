@@ -48,7 +48,7 @@ struct LayeredPlan {
     std::map<std::string, const TensorSlot*> slots;
     std::map<std::string, bool> bound;
     std::map<std::pair<TensorRole, uint32_t>, std::vector<float>> vectors;      // by role and layer, until finalized
-    std::vector<double*> frequencies;         // [layer]: of its rotation
+    std::vector<std::pair<const float2*, const float2*>> turns;      // [layer]: the tables of its rotation
 
     // ---- passes of a few rows
     float *residual[2] = {nullptr, nullptr}, *normed = nullptr, *raw_q = nullptr, *raw_latent = nullptr, *heads_out = nullptr, *projected = nullptr;

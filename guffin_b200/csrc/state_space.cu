@@ -8,7 +8,7 @@ namespace gf {
 
 namespace {
 
-constexpr uint32_t kMaxWarps = 4;
+constexpr uint32_t kMaxWarps = 4, kChunkWarps = 8;
 constexpr uint32_t kSmemLimit = 160u * 1024u;
 
 __device__ __forceinline__ void copy16(void* dst_smem, const void* src, bool valid) {      // zero-fills when not valid
@@ -56,7 +56,7 @@ __device__ __forceinline__ float convolve(const StateSpace& p, const float* raw,
         return back <= r ? raw[(size_t)(r - back) * p.raw_ld + inner + channel] : ring[(size_t)((base + r - back) & p.input_mask) * row + channel];
     };
     float sum = 0.0f;
-    if (kFew) {
+    if constexpr (kFew) {
         float v[4], w[4];
 #pragma unroll
         for (uint32_t j = 0; j < 4u; ++j) {                            // j taps before the last one
@@ -67,9 +67,10 @@ __device__ __forceinline__ float convolve(const StateSpace& p, const float* raw,
 #pragma unroll
         for (int j = 3; j >= 0; --j) sum = fmaf(w[j], v[j], sum);
         return silu(sum + bias);
+    } else {
+        for (uint32_t j = 0; j < p.tap_count; ++j) sum = fmaf(taps[j], value(p.tap_count - 1u - j), sum);
+        return silu(sum + p.tap_bias[channel]);
     }
-    for (uint32_t j = 0; j < p.tap_count; ++j) sum = fmaf(taps[j], value(p.tap_count - 1u - j), sum);
-    return silu(sum + p.tap_bias[channel]);
 }
 // dt and the logarithm of the decay.
 __device__ __forceinline__ float2 step_of(const StateSpace& p, const float* raw, uint32_t r, uint32_t head) {
@@ -77,18 +78,20 @@ __device__ __forceinline__ float2 step_of(const StateSpace& p, const float* raw,
     return make_float2(dt, p.decay[head] * dt);
 }
 
-// Sums part[0 .. 4 V) over the L lanes that share a column: every round halves the values a lane is left with.  Returns
-// how many it has, from `index` on.
+// Sums part[0 .. 4 V) over the L lanes that share a column: every round halves the values a lane is left with, so that
+// part[0 .. lane_values()) hold the sums of values lane_first(lane) on.  Lanes left with the same value: the first writes.
+template <int L, int V> constexpr uint32_t lane_values() { return L >= 4 * V ? 1u : 4u * V / L; }
+template <int L, int V> constexpr uint32_t lane_copies() { return L > 4 * V ? L / (4u * V) : 1u; }
 template <int L, int V>
-__device__ __forceinline__ uint32_t lane_sums(float (&part)[4 * V], uint32_t lane, uint32_t& index) {
+__device__ __forceinline__ uint32_t lane_first(uint32_t lane) { return lane % L / lane_copies<L, V>() * lane_values<L, V>(); }
+template <int L, int V>
+__device__ __forceinline__ void lane_sums(float (&part)[4 * V], uint32_t lane) {
     uint32_t count = 4u * V;
-    index = 0u;
 #pragma unroll
     for (uint32_t o = L / 2u; o > 0u; o >>= 1) {
         const bool upper = (lane & o) != 0u;
         if (count > 1u) {
             count /= 2u;
-            if (upper) index += count;
 #pragma unroll
             for (uint32_t i = 0; i < 2u * V; ++i) {
                 if (i >= count) break;
@@ -97,13 +100,6 @@ __device__ __forceinline__ uint32_t lane_sums(float (&part)[4 * V], uint32_t lan
             }
         } else part[0] += __shfl_xor_sync(0xffffffffu, part[0], o);
     }
-    return count;
-}
-// Whether a lane writes what lane_sums leaves it with (of lanes left with the same value, the first).
-template <int L, int V>
-__device__ __forceinline__ bool sums_writer(uint32_t ln) {
-    constexpr uint32_t kSame = L > 4 * V ? L / (4 * V) : 1;
-    return ln % kSame == 0u;
 }
 
 // A block holds some columns (of vdim) of one head's state in registers while it walks the tokens: L lanes share a
@@ -248,13 +244,11 @@ __global__ void __launch_bounds__(kMaxWarps * 32, 3) state_space_rows_kernel(con
             const uint32_t row = first + t;
             if (row >= kept) mine.store(s, states + ((base + row + 1u) % slots) * slot_elements);
         }
-        uint32_t index;
-        const uint32_t count = lane_sums<L, V>(part, lane, index);
+        lane_sums<L, V>(part, lane);
 #pragma unroll
-        for (uint32_t i = 0; i < 4u * V; ++i) {
-            if (i >= count) break;
-            const uint32_t t = (index + i) / V, k = mine.local + (index + i) % V;
-            if (!sums_writer<L, V>(mine.ln) || t >= live || c0 + k >= p.vdim) continue;
+        for (uint32_t i = 0; i < lane_values<L, V>(); ++i) {
+            const uint32_t at = lane_first<L, V>(lane) + i, t = at / V, k = mine.local + at % V;
+            if (mine.ln % lane_copies<L, V>() || t >= live || c0 + k >= p.vdim) continue;
             p.out[(size_t)(row0 + first + t) * inner + head * p.vdim + c0 + k] = fmaf(skip, x[t * columns + k], part[i]) * silu(gate[t * columns + k]);
         }
         __syncthreads();                                               // the tile's buffers are free again
@@ -287,7 +281,7 @@ __host__ __device__ inline ChunkLayout chunk_layout(uint32_t tile, uint32_t wide
 }
 
 template <int L, int NQ, int V>
-__global__ void __launch_bounds__(kMaxWarps * 32) state_space_chunk_kernel(const __grid_constant__ StateSpace p) {
+__global__ void __launch_bounds__(kChunkWarps * 32) state_space_chunk_kernel(const __grid_constant__ StateSpace p) {
     extern __shared__ __align__(16) uint8_t smem[];
     const Columns<L, NQ, V> mine(p);
     constexpr uint32_t kWide = Columns<L, NQ, V>::kWide, kTile = chunk_tile<(int)kWide>();
@@ -325,6 +319,9 @@ __global__ void __launch_bounds__(kMaxWarps * 32) state_space_chunk_kernel(const
         copies_commit();
     };
     const uint32_t tiles = (rows + kTile - 1u) / kTile;
+    const uint32_t lane_at = lane_first<L, V>(lane);                   // the values of every four tokens that this lane writes
+    const bool writes = mine.ln % lane_copies<L, V>() == 0u;
+    float* out = p.out + (size_t)(lane_at / V) * inner + head * p.vdim + c0 + mine.local + lane_at % V;
     fill(0u, 0u);
     for (uint32_t tile = 0; tile < tiles; ++tile) {
         const uint32_t first = tile * kTile;
@@ -401,22 +398,21 @@ __global__ void __launch_bounds__(kMaxWarps * 32) state_space_chunk_kernel(const
             float part[4 * V];
 #pragma unroll
             for (int i = 0; i < 4 * V; ++i) part[i] = pair_sum(sum[i / V][i % V]);
-            uint32_t index;
-            const uint32_t count = lane_sums<L, V>(part, lane, index);
+            lane_sums<L, V>(part, lane);
 #pragma unroll
-            for (uint32_t i = 0; i < 4u * V; ++i) {
-                if (i >= count) break;
-                const uint32_t t = t4 + (index + i) / V, k = mine.local + (index + i) % V, row = first + t;
-                if (!sums_writer<L, V>(mine.ln) || row >= rows || c0 + k >= p.vdim) continue;
+            for (uint32_t i = 0; i < lane_values<L, V>(); ++i) {
+                const uint32_t t = t4 + (lane_at + i) / V, k = mine.local + (lane_at + i) % V;
+                if (!writes || first + t >= rows || c0 + k >= p.vdim) continue;
                 const float4 f = m[t];
                 const float* x4 = x + t4 * columns + k;
                 float y = u[t] * part[i];
                 y = fmaf(f.x, x4[0], y);
                 y = fmaf(f.y, x4[columns], y);
                 y = fmaf(f.z, x4[2u * columns], y);
-                p.out[(size_t)row * inner + head * p.vdim + c0 + k] = fmaf(f.w, x4[3u * columns], y);
+                out[((t4 + i / V) * inner) + i % V] = fmaf(f.w, x4[3u * columns], y);
             }
         }
+        out += (size_t)kTile * inner;
         __syncthreads();                                               // the tile's buffers are free again
     }
     mine.store(s, states + ((base + rows) % slots) * slot_elements);
@@ -430,13 +426,17 @@ constexpr uint32_t kConvolveRows = 8, kConvolveThreads = 256;
 // Eight rows of one channel: emit(row, value).  T: taps at most (0: any number).
 template <int T, typename Emit>
 __device__ __forceinline__ void convolve_rows(const StateSpace& p, const float* ring, uint32_t base, uint32_t row, uint32_t live, uint32_t channel, Emit emit) {
-    if (T == 0) {
+    if constexpr (T == 0) {
         for (uint32_t r = 0; r < live; ++r) emit(r, convolve<false>(p, p.raw, ring, base, row + r, channel));
-        return;
-    }
-    constexpr int kBack = T > 0 ? T - 1 : 0;
-    float v[kBack + (int)kConvolveRows], w[T > 0 ? T : 1];
+    } else {
+    constexpr int kBack = T - 1;
+    float v[kBack + (int)kConvolveRows], w[T];
     const float* raw = p.raw + p.inner() + channel;
+    if (row >= (uint32_t)kBack && live == kConvolveRows) {
+        const float* from = raw + (size_t)(row - kBack) * p.raw_ld;
+#pragma unroll
+        for (int i = 0; i < kBack + (int)kConvolveRows; ++i) v[i] = from[(size_t)i * p.raw_ld];
+    } else
 #pragma unroll
     for (int i = 0; i < kBack + (int)kConvolveRows; ++i) {
         const int r = (int)row + i - kBack;                            // a row of the chunk, or behind it
@@ -455,6 +455,7 @@ __device__ __forceinline__ void convolve_rows(const StateSpace& p, const float* 
 #pragma unroll
         for (int j = T - 1; j >= 0; --j) sum = fmaf(w[j], v[kBack + r - j], sum);
         emit((uint32_t)r, silu(sum + bias));
+    }
     }
 }
 
@@ -528,7 +529,7 @@ int launch_recurrence(const StateSpace& p, cudaStream_t stream, bool pdl) {
     if (status != GF_OK) return status;
     // As many warps per block as still give most SMs a block; the block's columns are whole 16-byte pieces.
     const uint32_t sequences = p.ring_stride ? p.rows : 1u;
-    uint32_t warps = kMaxWarps;
+    uint32_t warps = kPass ? kMaxWarps : kChunkWarps;
     while (warps > 1u && (warps / 2u) * per_warp % 4u == 0u
            && ((uint64_t)p.heads * sequences * ((p.vdim + warps * per_warp - 1u) / (warps * per_warp)) * 5u < (uint64_t)sm_count() * 4u
                || (warps / 2u) * per_warp >= p.vdim))
@@ -540,17 +541,19 @@ int launch_recurrence(const StateSpace& p, cudaStream_t stream, bool pdl) {
     else return launch_kernel(state_space_chunk_kernel<L, NQ, V>, grid, dim3(warps * 32u), chunk_layout(chunk_tile<(int)kWide>(), kWide, columns).bytes, stream, pdl, p);
 }
 
+// Chunks hold half the columns a lane: twice the warps hide more of one another's waits.
 template <bool kPass>
 int launch_by_state(const StateSpace& p, cudaStream_t stream, bool pdl) {
+    constexpr int V = kPass ? 4 : 2;
     const uint32_t fours = p.state_row() / 4u;
-    if (fours <= 1u) return launch_recurrence<1, 1, 4, kPass>(p, stream, pdl);
-    if (fours <= 2u) return launch_recurrence<1, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 4u) return launch_recurrence<2, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 8u) return launch_recurrence<4, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 16u) return launch_recurrence<8, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 32u) return launch_recurrence<16, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 64u) return launch_recurrence<32, 2, 4, kPass>(p, stream, pdl);
-    if (fours <= 128u) return launch_recurrence<32, 4, 4, kPass>(p, stream, pdl);
+    if (fours <= 1u) return launch_recurrence<1, 1, V, kPass>(p, stream, pdl);
+    if (fours <= 2u) return launch_recurrence<1, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 4u) return launch_recurrence<2, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 8u) return launch_recurrence<4, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 16u) return launch_recurrence<8, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 32u) return launch_recurrence<16, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 64u) return launch_recurrence<32, 2, V, kPass>(p, stream, pdl);
+    if (fours <= 128u) return launch_recurrence<32, 4, V, kPass>(p, stream, pdl);
     return launch_recurrence<32, 8, 2, kPass>(p, stream, pdl);
 }
 

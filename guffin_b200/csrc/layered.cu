@@ -527,7 +527,7 @@ int Model::ensure_chunk_arena() {
         return bytes_alloc(allocations_, &o.data, o.bytes());
     };
     uint32_t query = 0, latent_out = 0, values = 0, latent = 0, query_elements = 0, row_elements = 0, ff = 0, shared_ff = 0, expert_ff = 0, experts = 0, top = 0, heads = 0;
-    size_t raw_q = 0, raw_k = 0, gates = 0, prepared = 0, x_elements = 0, bc_elements = 0, cb_elements = 0, step_elements = 0, y_elements = 0;      // per row
+    size_t raw_q = 0, raw_k = 0, gates = 0, prepared = 0, x_elements = 0, bc_elements = 0, step_elements = 0, y_elements = 0;      // per row
     for (const LayerSpec& l : s.layers) {
         const MixerSpec& m = l.mixer;
         values = std::max(values, m.inner());
@@ -541,8 +541,10 @@ int Model::ensure_chunk_arena() {
         } else {
             const StateSpace shape = p.state_space((uint32_t)(&l - s.layers.data()));
             raw_q = std::max<size_t>(raw_q, state_inputs_ld(m)); y_elements = std::max<size_t>(y_elements, m.inner());
-            x_elements = std::max<size_t>(x_elements, m.heads * shape.x_row()); bc_elements = std::max<size_t>(bc_elements, m.groups * shape.state_row());
-            step_elements = std::max<size_t>(step_elements, m.heads); cb_elements = std::max<size_t>(cb_elements, m.groups * 4u);
+            const StateChunk cut = state_space_chunk(shape);
+            x_elements = std::max<size_t>(x_elements, m.heads * ((m.vdim + cut.columns - 1u) / cut.columns) * cut.x_ld);
+            bc_elements = std::max<size_t>(bc_elements, m.groups * cut.n_ld);
+            step_elements = std::max<size_t>(step_elements, m.heads);
         }
         const FeedForwardSpec& f = l.mlp;
         if (f.kind == FeedForwardSpec::kDense) ff = std::max(ff, f.ff);
@@ -563,7 +565,7 @@ int Model::ensure_chunk_arena() {
         GF_TRY(plan_alloc(allocations_, &a.state_x, rows * x_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_b, rows * bc_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_c, rows * bc_elements));
-        GF_TRY(plan_alloc(allocations_, &a.state_cb, rows * cb_elements));
+        GF_TRY(plan_alloc(allocations_, &a.state_factors, rows * step_elements * kStateFactors));
         GF_TRY(plan_alloc(allocations_, &a.state_steps, rows * step_elements));
         GF_TRY(plan_alloc(allocations_, &a.state_y, rows * y_elements));
     }
@@ -789,7 +791,7 @@ int Model::chunk_layers(const uint32_t* tokens_host, uint32_t rows, bool logits)
         step.raw = a.raw_q; step.raw_ld = state_inputs_ld(m);
         step.taps = w.taps; step.tap_bias = w.tap_bias; step.step_bias = w.step_bias; step.decay = w.decay; step.skip = w.skip;
         step.rings = p.rings_dev + l; step.positions = state_dev_; step.slots = p.slots_dev; step.rows = rows; step.input_mask = caches_[l].ring_rows - 1u;
-        step.out = a.state_y; step.x = a.state_x; step.b = a.state_b; step.c = a.state_c; step.cb = a.state_cb; step.steps = a.state_steps;
+        step.out = a.state_y; step.x = a.state_x; step.b = a.state_b; step.c = a.state_c; step.factors = a.state_factors; step.error_flag = error_flag_; step.steps = a.state_steps;
         launches_ += 2;
         GF_TRY(launch_state_space_chunk(step, stream_));
         if (last) return GF_OK;

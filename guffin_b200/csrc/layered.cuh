@@ -81,7 +81,7 @@ struct LayeredPlan {
         std::vector<void*> private_rows, private_values;
         float *raw_q = nullptr, *raw_k = nullptr, *raw_gate = nullptr;
         void* prepared_q = nullptr;
-        float *state_x = nullptr, *state_b = nullptr, *state_c = nullptr, *state_cb = nullptr, *state_y = nullptr;
+        float *state_x = nullptr, *state_b = nullptr, *state_c = nullptr, *state_factors = nullptr, *state_y = nullptr;
         float2* state_steps = nullptr;
         KvPublishLayer* publish_layers = nullptr;
     } chunk;

@@ -1,5 +1,6 @@
 // State-space mixer (see state_space.cuh).
 #include "state_space.cuh"
+#include "tcgen05.cuh"
 
 #include <algorithm>
 #include <mutex>
@@ -8,17 +9,8 @@ namespace gf {
 
 namespace {
 
-constexpr uint32_t kMaxWarps = 4, kChunkWarps = 8;
-constexpr uint32_t kSmemLimit = 160u * 1024u;
-
-__device__ __forceinline__ void copy16(void* dst_smem, const void* src, bool valid) {      // zero-fills when not valid
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst_smem)), "l"(src), "r"(valid ? 16u : 0u) : "memory");
-}
-__device__ __forceinline__ void copy8(void* dst_smem, const void* src, bool valid) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(smem_u32(dst_smem)), "l"(src), "r"(valid ? 8u : 0u) : "memory");
-}
-__device__ __forceinline__ void copies_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void copies_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+constexpr uint32_t kMaxWarps = 4, kChunkWarps = 16;
+constexpr uint32_t kSmemLimit = 160u * 1024u, kChunkSmem = 200u * 1024u;
 
 // Two f32 values side by side in a register pair.
 using Pair = unsigned long long;
@@ -78,22 +70,22 @@ __device__ __forceinline__ float2 step_of(const StateSpace& p, const float* raw,
     return make_float2(dt, p.decay[head] * dt);
 }
 
-// Sums part[0 .. 4 V) over the L lanes that share a column: every round halves the values a lane is left with, so that
+// Sums part[0 .. M) over the L lanes that share a column: every round halves the values a lane is left with, so that
 // part[0 .. lane_values()) hold the sums of values lane_first(lane) on.  Lanes left with the same value: the first writes.
-template <int L, int V> constexpr uint32_t lane_values() { return L >= 4 * V ? 1u : 4u * V / L; }
-template <int L, int V> constexpr uint32_t lane_copies() { return L > 4 * V ? L / (4u * V) : 1u; }
-template <int L, int V>
-__device__ __forceinline__ uint32_t lane_first(uint32_t lane) { return lane % L / lane_copies<L, V>() * lane_values<L, V>(); }
-template <int L, int V>
-__device__ __forceinline__ void lane_sums(float (&part)[4 * V], uint32_t lane) {
-    uint32_t count = 4u * V;
+template <int L, int M> constexpr uint32_t lane_values() { return L >= M ? 1u : (uint32_t)(M / L); }
+template <int L, int M> constexpr uint32_t lane_copies() { return L > M ? (uint32_t)(L / M) : 1u; }
+template <int L, int M>
+__device__ __forceinline__ uint32_t lane_first(uint32_t lane) { return lane % L / lane_copies<L, M>() * lane_values<L, M>(); }
+template <int L, int M>
+__device__ __forceinline__ void lane_sums(float (&part)[M], uint32_t lane) {
+    uint32_t count = M;
 #pragma unroll
     for (uint32_t o = L / 2u; o > 0u; o >>= 1) {
         const bool upper = (lane & o) != 0u;
         if (count > 1u) {
             count /= 2u;
 #pragma unroll
-            for (uint32_t i = 0; i < 2u * V; ++i) {
+            for (uint32_t i = 0; i < M / 2u; ++i) {
                 if (i >= count) break;
                 const float keep = upper ? part[i + count] : part[i], send = upper ? part[i] : part[i + count];
                 part[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
@@ -244,11 +236,11 @@ __global__ void __launch_bounds__(kMaxWarps * 32, 3) state_space_rows_kernel(con
             const uint32_t row = first + t;
             if (row >= kept) mine.store(s, states + ((base + row + 1u) % slots) * slot_elements);
         }
-        lane_sums<L, V>(part, lane);
+        lane_sums<L, 4 * V>(part, lane);
 #pragma unroll
-        for (uint32_t i = 0; i < lane_values<L, V>(); ++i) {
-            const uint32_t at = lane_first<L, V>(lane) + i, t = at / V, k = mine.local + at % V;
-            if (mine.ln % lane_copies<L, V>() || t >= live || c0 + k >= p.vdim) continue;
+        for (uint32_t i = 0; i < lane_values<L, 4 * V>(); ++i) {
+            const uint32_t at = lane_first<L, 4 * V>(lane) + i, t = at / V, k = mine.local + at % V;
+            if (mine.ln % lane_copies<L, 4 * V>() || t >= live || c0 + k >= p.vdim) continue;
             p.out[(size_t)(row0 + first + t) * inner + head * p.vdim + c0 + k] = fmaf(skip, x[t * columns + k], part[i]) * silu(gate[t * columns + k]);
         }
         __syncthreads();                                               // the tile's buffers are free again
@@ -258,169 +250,207 @@ __global__ void __launch_bounds__(kMaxWarps * 32, 3) state_space_rows_kernel(con
 
 // ------------------------------------------------------------------ chunks
 
-// Four tokens at a time.  With a_t the logarithm of token t's decay and A_t their sums within the four,
-//   y_t = exp(A_t) C_t . S + sum over s <= t of exp(A_t - A_s) dt_s (C_t . B_s) x_s + skip x_t
-//   S  <- exp(A_3) S + sum over s of exp(A_3 - A_s) dt_s B_s x_s^T
-// so that a state's element costs nine multiply-adds per four tokens; the products C_t . B_s come with the inputs.
-template <int NL> constexpr uint32_t chunk_tile() { return NL <= 128 ? 32u : NL <= 256 ? 16u : NL <= 512 ? 8u : 4u; }
-struct ChunkLayout { uint32_t c, x, steps, cb, stage, doubled, m, u, w, whole, bytes; };
-__host__ __device__ inline ChunkLayout chunk_layout(uint32_t tile, uint32_t wide, uint32_t columns) {      // bytes; two stages, then one of each
+// Eight tokens at a time.  With a_t the logarithm of token t's decay and A_t their sums within the eight,
+//   y_t = exp(A_t) S . C_t + sum over s <= t of M_ts x_s        M_ts = exp(A_t - A_s) dt_s (C_t . B_s), plus skip for s = t
+//   S  <- exp(A_7) S + sum over s of exp(A_7 - A_s) dt_s x_s B_s^T
+// as products on the tensor cores, in pairs of tf32 values (a value's leading bits and what they leave out) so that they
+// are as exact as f32 ones.  A warp keeps 16 columns (of vdim) x 8 NT values (of N) of the state in accumulators, which
+// are the first operand of the read-out as they lie: an accumulator's neighbouring columns 2 t and 2 t + 1 count as the
+// operand's t and t + 4.
+// Helper warps have the next tile's inputs and factors copied and write the last tile's outputs meanwhile.
+constexpr uint32_t kHelpers = 4;
+struct ChunkLayout { uint32_t c, x, factors, stage, y, y_stage, bytes; };
+__host__ __device__ inline ChunkLayout chunk_layout(const StateChunk& k) {      // bytes; two stages each of inputs and of outputs
     ChunkLayout t;
-    t.c = tile * wide * 4u;
+    t.c = k.tile * k.n_ld * 4u;
     t.x = 2u * t.c;
-    t.cb = t.x + tile * columns * 4u;
-    t.steps = t.cb + tile * 16u;
-    t.stage = t.steps + tile * 8u;
-    t.doubled = 2u * t.stage;
-    t.m = t.doubled + tile * columns * 8u;
-    t.u = t.m + tile * 16u;
-    t.w = t.u + tile * 4u;
-    t.whole = t.w + tile * 4u;
-    t.bytes = t.whole + tile * 4u;
+    t.factors = t.x + k.tile * k.x_ld * 4u;
+    t.stage = t.factors + k.tile * kStateFactors * 4u;
+    t.y = 2u * t.stage;
+    t.y_stage = k.splits * k.tile * k.x_ld * 4u;
+    t.bytes = t.y + 2u * t.y_stage;
     return t;
 }
 
-template <int L, int NQ, int V>
-__global__ void __launch_bounds__(kChunkWarps * 32) state_space_chunk_kernel(const __grid_constant__ StateSpace p) {
+__device__ __forceinline__ void mma_tf32(float (&d)[4], const float (&a)[4], float b0, float b1) {
+    asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+                 : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
+                   "r"(__float_as_uint(b1)));
+}
+// The bits of a value that tf32 holds, and the rest.
+__device__ __forceinline__ float leading(float v) { return __uint_as_float(__float_as_uint(v) & 0xffffe000u); }
+struct Split4 {
+    float hi[4], lo[4];
+    __device__ __forceinline__ Split4(float a, float b, float c, float d) {
+        const float v[4] = {a, b, c, d};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) { hi[i] = leading(v[i]); lo[i] = v[i] - hi[i]; }
+    }
+};
+
+template <int NT>
+__global__ void __launch_bounds__((kChunkWarps + kHelpers) * 32) state_space_chunk_kernel(const __grid_constant__ StateSpace p, const __grid_constant__ StateChunk k) {
     extern __shared__ __align__(16) uint8_t smem[];
-    const Columns<L, NQ, V> mine(p);
-    constexpr uint32_t kWide = Columns<L, NQ, V>::kWide, kTile = chunk_tile<(int)kWide>();
-    const uint32_t tid = threadIdx.x, threads = blockDim.x, lane = tid & 31u, columns = mine.count, c0 = mine.first, rows = p.rows;
-    const ChunkLayout at = chunk_layout(kTile, kWide, columns);
-    const uint32_t head = blockIdx.x, group = head / (p.heads / p.groups), np = mine.np, inner = p.inner(), x_row = p.x_row();
+    __shared__ __align__(8) uint64_t full[2];                          // a stage's copies have landed
+    __shared__ volatile uint32_t abort_flag;
+    const uint32_t warp = threadIdx.x >> 5, lane = threadIdx.x & 31u, g = lane >> 2, t = lane & 3u, rows = p.rows;
+    const ChunkLayout at = chunk_layout(k);
+    const uint32_t head = blockIdx.x, c0 = blockIdx.y * k.columns, np = p.state_row(), inner = p.inner();
+    const uint32_t workers = k.columns / 16u * k.splits, tiles = (rows + k.tile - 1u) / k.tile;
+    const bool helper = warp >= workers;
+    const uint32_t split = warp % k.splits, own = warp / k.splits * 16u;      // a worker's part of N, and its columns from c0 + own on
     const uint32_t base = *p.positions, slots = *p.slots;
     const size_t slot_elements = p.slot_elements();
     float* states = static_cast<float*>(const_cast<void*>(p.rings->ring_k)) + (size_t)head * p.vdim * np;
-    Pair s[V][2 * NQ];
-    mine.load(s, states + (base % slots) * slot_elements, base > 0u);
-    const float skip = p.skip[head];
-
-    auto fill = [&](uint32_t tile, uint32_t stage) {                   // zeros behind the chunk's rows
-        uint8_t* to = smem + stage * at.stage;
-        const uint32_t first = tile * kTile;
-        for (uint32_t i = tid; i < kTile * (kWide / 4u); i += threads) {
-            const uint32_t t = i / (kWide / 4u), n = i % (kWide / 4u) * 4u, row = first + t;
-            const bool valid = row < rows && n < np;
-            const size_t from = valid ? ((size_t)row * p.groups + group) * np + n : 0u;
-            copy16(to + (t * kWide + n) * 4u, p.b + from, valid);
-            copy16(to + at.c + (t * kWide + n) * 4u, p.c + from, valid);
-        }
-        for (uint32_t i = tid; i < kTile * (columns / 4u); i += threads) {
-            const uint32_t t = i / (columns / 4u), k = i % (columns / 4u) * 4u, row = first + t;
-            const bool valid = row < rows && c0 + k < x_row;
-            copy16(to + at.x + (t * columns + k) * 4u, p.x + (valid ? ((size_t)row * p.heads + head) * x_row + c0 + k : 0u), valid);
-        }
-        if (tid < kTile) {
-            const bool valid = first + tid < rows;
-            const size_t row = valid ? first + tid : 0u;
-            copy16(to + at.cb + tid * 16u, p.cb + (row * p.groups + group) * 4u, valid);
-            copy8(to + at.steps + tid * 8u, p.steps + row * p.heads + head, valid);
-        }
-        copies_commit();
+    float s[NT][4];
+    auto state_at = [&](int j, int i) { return (size_t)(c0 + own + g + 8u * i) * np + (split * NT + j) * 8u + 2u * t; };
+    auto state_valid = [&](int j, int i) { return !helper && c0 + own + g + 8u * i < p.vdim && (split * NT + j) * 8u + 2u * t < np; };
+    {
+        const float* from = states + (base % slots) * slot_elements;
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                const float2 v = base > 0u && state_valid(j, i) ? *reinterpret_cast<const float2*>(from + state_at(j, i)) : make_float2(0.0f, 0.0f);
+                s[j][2 * i] = v.x;
+                s[j][2 * i + 1] = v.y;
+            }
+    }
+    const uint32_t all_rows = (rows + 7u) & ~7u;                        // the inputs have whole eights
+    if (threadIdx.x == 0) {
+        abort_flag = 0u;
+        mbar_init(&full[0], 1);
+        mbar_init(&full[1], 1);
+        fence_barrier_init();
+    }
+    __syncthreads();
+    // ---- helpers
+    auto fill = [&](uint32_t tile) {                                   // one thread: a tile's rows follow one another
+        uint8_t* to = smem + (tile & 1u) * at.stage;
+        uint64_t* bar = &full[tile & 1u];
+        const uint32_t first = tile * k.tile, count = min(k.tile, all_rows - first), group = head / (p.heads / p.groups);
+        const size_t vectors = ((size_t)group * all_rows + first) * k.n_ld, columns = (((size_t)head * gridDim.y + blockIdx.y) * all_rows + first) * k.x_ld;
+        mbar_expect_tx(bar, count * (2u * k.n_ld + k.x_ld + kStateFactors) * 4u);
+        bulk_load(to, p.b + vectors, count * k.n_ld * 4u, bar);
+        bulk_load(to + at.c, p.c + vectors, count * k.n_ld * 4u, bar);
+        bulk_load(to + at.x, p.x + columns, count * k.x_ld * 4u, bar);
+        bulk_load(to + at.factors, p.factors + ((size_t)head * all_rows + first) * kStateFactors, count * kStateFactors * 4u, bar);
     };
-    const uint32_t tiles = (rows + kTile - 1u) / kTile;
-    const uint32_t lane_at = lane_first<L, V>(lane);                   // the values of every four tokens that this lane writes
-    const bool writes = mine.ln % lane_copies<L, V>() == 0u;
-    float* out = p.out + (size_t)(lane_at / V) * inner + head * p.vdim + c0 + mine.local + lane_at % V;
-    fill(0u, 0u);
-    for (uint32_t tile = 0; tile < tiles; ++tile) {
-        const uint32_t first = tile * kTile;
-        if (tile + 1u < tiles) fill(tile + 1u, (tile + 1u) & 1u);
-        else copies_commit();
-        copies_wait<1>();
-        __syncthreads();
+    auto write = [&](uint32_t tile) {
+        const float* y = reinterpret_cast<const float*>(smem + at.y + (tile & 1u) * at.y_stage);
+        const uint32_t first = tile * k.tile, count = min(k.tile, rows - first), quads = k.columns / 4u, part_step = k.tile * k.x_ld;
+        for (uint32_t i = threadIdx.x - workers * 32u; i < count * quads; i += kHelpers * 32u) {
+            const uint32_t r = i / quads, column = i % quads * 4u;
+            const float* from = y + r * k.x_ld + column;
+            float4 v = *reinterpret_cast<const float4*>(from);
+#pragma unroll 4
+            for (uint32_t part = 1; part < k.splits; ++part) {
+                const float4 o = *reinterpret_cast<const float4*>(from + part * part_step);
+                v = make_float4(v.x + o.x, v.y + o.y, v.z + o.z, v.w + o.w);
+            }
+            float* out = p.out + (size_t)(first + r) * inner + head * p.vdim + c0 + column;
+            if (p.vdim % 4u == 0u) {
+                if (c0 + column < p.vdim) *reinterpret_cast<float4*>(out) = v;
+                continue;
+            }
+            const float four[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+            for (uint32_t j = 0; j < 4u; ++j)
+                if (c0 + column + j < p.vdim) out[j] = four[j];
+        }
+    };
+    // ---- workers
+    auto work = [&](uint32_t tile) {
         const uint8_t* from = smem + (tile & 1u) * at.stage;
         const float *b = reinterpret_cast<const float*>(from), *c = reinterpret_cast<const float*>(from + at.c), *x = reinterpret_cast<const float*>(from + at.x);
-        float4* m = reinterpret_cast<float4*>(smem + at.m);            // of x_0 .. x_3 of the four tokens, in y_t
-        float *u = reinterpret_cast<float*>(smem + at.u), *w = reinterpret_cast<float*>(smem + at.w), *whole = reinterpret_cast<float*>(smem + at.whole);
-        Pair* doubled = reinterpret_cast<Pair*>(smem + at.doubled);    // w_t x_t, twice
-        if (tid < kTile) {
-            const float2* steps = reinterpret_cast<const float2*>(from + at.steps) + (tid & ~3u);
-            const float* cb = reinterpret_cast<const float*>(from + at.cb) + tid * 4u;
-            const uint32_t q = tid & 3u;
-            float factors[4], behind = 0.0f, rest = 0.0f;              // sums of logarithms: (s, q], and (q, 3]
-#pragma unroll
-            for (int i = 3; i >= 0; --i) {
-                factors[i] = 0.0f;
-                if ((uint32_t)i > q) { rest += steps[i].y; continue; }
-                factors[i] = cb[i] * expf(behind) * steps[i].x;
-                if ((uint32_t)i == q) factors[i] += skip;
-                behind += steps[i].y;
-            }
-            m[tid] = make_float4(factors[0], factors[1], factors[2], factors[3]);
-            u[tid] = expf(behind);
-            w[tid] = expf(rest) * steps[q].x;
-            whole[tid] = expf(behind + rest);
-        }
-        __syncthreads();
-        for (uint32_t i = tid; i < kTile * columns; i += threads) {
-            const float v = x[i] * w[i / columns];
-            doubled[i] = pair_of(v, v);
-        }
-        __syncthreads();
+        const float* factors = reinterpret_cast<const float*>(from + at.factors);      // a row: M, exp(A_t), dt exp(A_7 - A_t), exp(A_7)
+        float* y = reinterpret_cast<float*>(smem + at.y + (tile & 1u) * at.y_stage);
 #pragma unroll 1
-        for (uint32_t t4 = 0; t4 < kTile && first + t4 < rows; t4 += 4u) {
-            Pair xw[4][V], sum[4][V];
+        for (uint32_t t0 = 0; t0 < k.tile && tile * k.tile + t0 < rows; t0 += 8u) {
+            const float* x_at = x + (t0 + t) * k.x_ld + own + g;
+            const float x0 = x_at[0], x1 = x_at[8], x2 = x_at[4u * k.x_ld], x3 = x_at[4u * k.x_ld + 8u];
+            const float* eight = factors + t0 * kStateFactors;
+            const float w0 = eight[t * kStateFactors + 9u], w1 = eight[(t + 4u) * kStateFactors + 9u], decay = eight[10];
+            const Split4 xw(x0 * w0, x1 * w0, x2 * w1, x3 * w1);
+            float y0[4] = {}, y1[4] = {}, y2[4] = {};
+            const float *c_at = c + (t0 + g) * k.n_ld + split * NT * 8u + 2u * t, *b_at = b + (t0 + t) * k.n_ld + split * NT * 8u + g;
+            float bh[NT][2], bl[NT][2];
 #pragma unroll
-            for (int q = 0; q < 4; ++q)
+            for (int j = 0; j < NT; ++j) {
+                const float2 cv = *reinterpret_cast<const float2*>(c_at + j * 8);
+                const float ch0 = leading(cv.x), ch1 = leading(cv.y);
+                const Split4 state(s[j][0], s[j][2], s[j][1], s[j][3]);
+                mma_tf32(y0, state.hi, ch0, ch1);
+                mma_tf32(y1, state.hi, cv.x - ch0, cv.y - ch1);
+                mma_tf32(y2, state.lo, ch0, ch1);
 #pragma unroll
-                for (int v = 0; v < V; v += 2) {
-                    const ulonglong2 two = *reinterpret_cast<const ulonglong2*>(doubled + (t4 + q) * columns + mine.local + v);
-                    xw[q][v] = two.x;
-                    xw[q][v + 1] = two.y;
-                }
-            const float decay = whole[t4 + 3u];
-            const Pair a = pair_of(decay, decay);
+                for (int i = 0; i < 4; ++i) s[j][i] *= decay;
 #pragma unroll
-            for (int j = 0; j < NQ; ++j) {
-                ulonglong2 bq[4], cq[4];
-#pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    cq[q] = *reinterpret_cast<const ulonglong2*>(c + (t4 + q) * kWide + mine.n(j));
-                    bq[q] = *reinterpret_cast<const ulonglong2*>(b + (t4 + q) * kWide + mine.n(j));
-                }
-#pragma unroll
-                for (int v = 0; v < V; ++v) {
-#pragma unroll
-                    for (int q = 0; q < 4; ++q) {
-                        sum[q][v] = j == 0 ? pair_mul(s[v][0], cq[q].x) : pair_fma(s[v][2 * j], cq[q].x, sum[q][v]);
-                        sum[q][v] = pair_fma(s[v][2 * j + 1], cq[q].y, sum[q][v]);
-                    }
-                    s[v][2 * j] = pair_mul(s[v][2 * j], a);
-                    s[v][2 * j + 1] = pair_mul(s[v][2 * j + 1], a);
-#pragma unroll
-                    for (int q = 0; q < 4; ++q) {
-                        s[v][2 * j] = pair_fma(bq[q].x, xw[q][v], s[v][2 * j]);
-                        s[v][2 * j + 1] = pair_fma(bq[q].y, xw[q][v], s[v][2 * j + 1]);
-                    }
+                for (int i = 0; i < 2; ++i) {
+                    const float v = b_at[j * 8 + i * 4u * k.n_ld];
+                    bh[j][i] = leading(v);
+                    bl[j][i] = v - bh[j][i];
                 }
             }
-            float part[4 * V];
+            // Products into the same accumulators as far apart as there are accumulators.
 #pragma unroll
-            for (int i = 0; i < 4 * V; ++i) part[i] = pair_sum(sum[i / V][i % V]);
-            lane_sums<L, V>(part, lane);
+            for (int j = 0; j < NT; ++j) mma_tf32(s[j], xw.hi, bh[j][0], bh[j][1]);
 #pragma unroll
-            for (uint32_t i = 0; i < lane_values<L, V>(); ++i) {
-                const uint32_t t = t4 + (lane_at + i) / V, k = mine.local + (lane_at + i) % V;
-                if (!writes || first + t >= rows || c0 + k >= p.vdim) continue;
-                const float4 f = m[t];
-                const float* x4 = x + t4 * columns + k;
-                float y = u[t] * part[i];
-                y = fmaf(f.x, x4[0], y);
-                y = fmaf(f.y, x4[columns], y);
-                y = fmaf(f.z, x4[2u * columns], y);
-                out[((t4 + i / V) * inner) + i % V] = fmaf(f.w, x4[3u * columns], y);
+            for (int j = 0; j < NT; ++j) mma_tf32(s[j], xw.hi, bl[j][0], bl[j][1]);
+#pragma unroll
+            for (int j = 0; j < NT; ++j) mma_tf32(s[j], xw.lo, bh[j][0], bh[j][1]);
+            const float u0 = eight[2u * t * kStateFactors + 8u], u1 = eight[(2u * t + 1u) * kStateFactors + 8u];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) y0[i] = (y0[i] + (y1[i] + y2[i])) * (i & 1 ? u1 : u0);
+            if (split == 0u) {
+                const Split4 xs(x0, x1, x2, x3);
+                const float m0 = eight[g * kStateFactors + t], m1 = eight[g * kStateFactors + t + 4u], mh0 = leading(m0), mh1 = leading(m1);
+                mma_tf32(y0, xs.hi, mh0, mh1);
+                mma_tf32(y0, xs.hi, m0 - mh0, m1 - mh1);
+                mma_tf32(y0, xs.lo, mh0, mh1);
             }
+            float* y_at = y + (split * k.tile + t0 + 2u * t) * k.x_ld + own + g;
+            y_at[0] = y0[0];
+            y_at[k.x_ld] = y0[1];
+            y_at[8] = y0[2];
+            y_at[k.x_ld + 8u] = y0[3];
         }
-        out += (size_t)kTile * inner;
-        __syncthreads();                                               // the tile's buffers are free again
+    };
+    const bool copier = warp == workers && lane == 0u;
+    if (copier) fill(0u);
+    bool ok = true;
+    for (uint32_t tile = 0; tile < tiles; ++tile) {
+        if (helper) {
+            if (copier && tile + 1u < tiles && abort_flag == 0u) fill(tile + 1u);
+            __syncwarp();
+            if (tile > 0u) write(tile - 1u);
+        } else {
+            if (ok && !wait_or_abort(&full[tile & 1u], (tile >> 1) & 1u, &abort_flag)) {
+                ok = false;
+                if (lane == 0) { abort_flag = 1u; atomicExch(p.error_flag, 1); }
+            }
+            work(tile);
+        }
+        __syncthreads();
     }
-    mine.store(s, states + ((base + rows) % slots) * slot_elements);
-    keep_inputs(p, p.raw, static_cast<float*>(const_cast<void*>(p.rings->ring_v)), base, rows - min(rows, p.tap_count - 1u), rows, head, c0, columns);
+    if (abort_flag != 0u && copier)                                    // copies already requested get a bounded chance to land
+        for (uint32_t tile = tiles > 2u ? tiles - 2u : 0u; tile < tiles; ++tile) mbar_wait(&full[tile & 1u], (tile >> 1) & 1u, 1u << 16);
+    if (helper) {
+        write(tiles - 1u);
+    } else {
+        float* to = states + ((base + rows) % slots) * slot_elements;
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int i = 0; i < 2; ++i)
+                if (state_valid(j, i)) *reinterpret_cast<float2*>(to + state_at(j, i)) = make_float2(s[j][2 * i], s[j][2 * i + 1]);
+    }
+    keep_inputs(p, p.raw, static_cast<float*>(const_cast<void*>(p.rings->ring_v)), base, rows - min(rows, p.tap_count - 1u), rows, head, c0, k.columns);
 }
 
-// The convolved inputs of eight rows, padding included: the first blocks take a group's B and C, its heads' steps, and
-// the products C_t . B_s within every four tokens; the others columns of x.
+// The convolved inputs of eight rows, padding and rows behind the chunk included (zeros): the first blocks take a group's B
+// and C and the factors of its heads, the others columns of x.
 constexpr uint32_t kConvolveRows = 8, kConvolveThreads = 256;
 
 // Eight rows of one channel: emit(row, value).  T: taps at most (0: any number).
@@ -460,50 +490,64 @@ __device__ __forceinline__ void convolve_rows(const StateSpace& p, const float* 
 }
 
 template <int T>
-__global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const __grid_constant__ StateSpace p) {
-    extern __shared__ float vectors[];                                 // [2][8][np]: B, C
-    const uint32_t np = p.state_row(), x_row = p.x_row(), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
-    const uint32_t base = p.positions[0], row = blockIdx.y * kConvolveRows, live = min(kConvolveRows, p.rows - row);
+__global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const __grid_constant__ StateSpace p, const __grid_constant__ StateChunk k) {
+    extern __shared__ float vectors[];                                 // [2][8][n_ld]: B, C
+    const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u;
+    const uint32_t base = p.positions[0], row = blockIdx.y * kConvolveRows, live = min(kConvolveRows, p.rows - row), all_rows = (p.rows + 7u) & ~7u;
     const float* ring = static_cast<const float*>(p.rings->ring_v);
     if (blockIdx.x >= p.groups) {
-        const uint32_t i = (blockIdx.x - p.groups) * kConvolveThreads + tid, all = p.heads * x_row, k = i % x_row;
-        if (i >= all) return;
-        float* out = p.x + (size_t)row * all + i;
-        if (k >= p.vdim) {
-            for (uint32_t r = 0; r < live; ++r) out[(size_t)r * all] = 0.0f;
-            return;
-        }
-        convolve_rows<T>(p, ring, base, row, live, i / x_row * p.vdim + k, [&](uint32_t r, float v) { out[(size_t)r * all] = v; });
+        const uint32_t i = (blockIdx.x - p.groups) * kConvolveThreads + tid, blocks = (p.vdim + k.columns - 1u) / k.columns;
+        const uint32_t head_block = i / k.x_ld, c = i % k.x_ld, head = head_block / blocks, column = head_block % blocks * k.columns + c;
+        if (head >= p.heads) return;
+        float* out = p.x + ((size_t)head_block * all_rows + row) * k.x_ld + c;
+        const bool valid = c < k.columns && column < p.vdim;
+        for (uint32_t r = valid ? live : 0u; r < kConvolveRows; ++r) out[r * k.x_ld] = 0.0f;
+        if (valid) convolve_rows<T>(p, ring, base, row, live, head * p.vdim + column, [&](uint32_t r, float v) { out[r * k.x_ld] = v; });
         return;
     }
-    const uint32_t group = blockIdx.x, per_group = p.heads / p.groups;
+    const uint32_t group = blockIdx.x, per_group = p.heads / p.groups, np = k.n_ld;
     for (uint32_t i = tid; i < 2u * np; i += kConvolveThreads) {
         const uint32_t which = i / np, n = i % np;
-        float *out = (which ? p.c : p.b) + ((size_t)row * p.groups + group) * np + n, *here = vectors + which * kConvolveRows * np + n;
-        if (n >= p.state) {
-            for (uint32_t r = 0; r < kConvolveRows; ++r) { here[r * np] = 0.0f; if (r < live) out[(size_t)r * p.groups * np] = 0.0f; }
-            continue;
-        }
-        for (uint32_t r = live; r < kConvolveRows; ++r) here[r * np] = 0.0f;
+        float *out = (which ? p.c : p.b) + ((size_t)group * all_rows + row) * np + n, *here = vectors + which * kConvolveRows * np + n;
+        const bool valid = n < p.state;
+        for (uint32_t r = valid ? live : 0u; r < kConvolveRows; ++r) { here[r * np] = 0.0f; out[r * np] = 0.0f; }
+        if (!valid) continue;
         convolve_rows<T>(p, ring, base, row, live, p.inner() + (which * p.groups + group) * p.state + n, [&](uint32_t r, float v) {
             here[r * np] = v;
-            out[(size_t)r * p.groups * np] = v;
+            out[r * np] = v;
         });
     }
-    for (uint32_t i = tid; i < live * per_group; i += kConvolveThreads) {
-        const uint32_t r = row + i / per_group, head = group * per_group + i % per_group;
-        p.steps[(size_t)r * p.heads + head] = step_of(p, p.raw, r, head);
+    for (uint32_t i = tid; i < kConvolveRows * per_group; i += kConvolveThreads) {
+        const uint32_t r = i / per_group, head = group * per_group + i % per_group;
+        p.steps[(size_t)(row + r) * p.heads + head] = r < live ? step_of(p, p.raw, row + r, head) : make_float2(0.0f, 0.0f);
+    }
+    __shared__ float cb[kConvolveRows * 8u];
+    __syncthreads();
+    for (uint32_t i = warp; i < kConvolveRows * 8u; i += kConvolveThreads / 32u) {
+        const uint32_t t = i / 8u, other = i % 8u;
+        if (other > t) continue;
+        const float *b = vectors + other * np, *c = vectors + (kConvolveRows + t) * np;
+        float sum = 0.0f;
+        for (uint32_t n = lane; n < np; n += 32u) sum = fmaf(c[n], b[n], sum);
+        sum = warp_sum(sum);
+        if (lane == 0) cb[i] = sum;
     }
     __syncthreads();
-    for (uint32_t i = warp; i < kConvolveRows * 4u; i += kConvolveThreads / 32u) {
-        const uint32_t t = i / 4u, s = i % 4u;
-        if (t >= live) break;
-        const float *b = vectors + ((t & ~3u) + s) * np, *c = vectors + (kConvolveRows + t) * np;
-        float sum = 0.0f;
-        if (s <= (t & 3u))
-            for (uint32_t n = lane; n < np; n += 32u) sum = fmaf(c[n], b[n], sum);
-        sum = warp_sum(sum);
-        if (lane == 0) p.cb[((size_t)(row + t) * p.groups + group) * 4u + s] = sum;
+    // The factors of every head: element (t, s) of M, and with s = t the row's exponentials.
+    for (uint32_t i = tid; i < per_group * kConvolveRows * 8u; i += kConvolveThreads) {
+        const uint32_t head = group * per_group + i / (kConvolveRows * 8u), t = i / 8u % kConvolveRows, s = i % 8u;
+        float between = 0.0f, before = 0.0f, behind = 0.0f, dt = 0.0f;
+#pragma unroll
+        for (uint32_t l = 0; l < 8u; ++l) {
+            const float2 step = p.steps[(size_t)(row + l) * p.heads + head];
+            if (l > s && l <= t) between += step.y;
+            (l <= t ? before : behind) += step.y;
+            if (l == s) dt = step.x;
+        }
+        float* out = p.factors + ((size_t)head * all_rows + row + t) * kStateFactors;
+        out[s] = s > t ? 0.0f : fmaf(cb[t * 8u + s] * dt, expf(between), s == t ? p.skip[head] : 0.0f);
+        if (s != t) continue;
+        *reinterpret_cast<float4*>(out + 8) = make_float4(expf(before), expf(behind) * dt, expf(before + behind), 0.0f);
     }
 }
 
@@ -519,42 +563,44 @@ int allow_smem(Kernel kernel, std::once_flag* once, uint32_t bytes) {
     return GF_OK;
 }
 
-template <int L, int NQ, int V, bool kPass>
-int launch_recurrence(const StateSpace& p, cudaStream_t stream, bool pdl) {
+template <int L, int NQ, int V>
+int launch_rows(const StateSpace& p, cudaStream_t stream, bool pdl) {
     constexpr uint32_t kWide = L * NQ * 4, per_warp = 32u / L * V;
     static std::once_flag once[64];
-    int status = GF_OK;
-    if constexpr (kPass) status = allow_smem(state_space_rows_kernel<L, NQ, V>, once, kSmemLimit);
-    else status = allow_smem(state_space_chunk_kernel<L, NQ, V>, once, kSmemLimit);
+    const int status = allow_smem(state_space_rows_kernel<L, NQ, V>, once, kSmemLimit);
     if (status != GF_OK) return status;
     // As many warps per block as still give most SMs a block; the block's columns are whole 16-byte pieces.
     const uint32_t sequences = p.ring_stride ? p.rows : 1u;
-    uint32_t warps = kPass ? kMaxWarps : kChunkWarps;
+    uint32_t warps = kMaxWarps;
     while (warps > 1u && (warps / 2u) * per_warp % 4u == 0u
            && ((uint64_t)p.heads * sequences * ((p.vdim + warps * per_warp - 1u) / (warps * per_warp)) * 5u < (uint64_t)sm_count() * 4u
                || (warps / 2u) * per_warp >= p.vdim))
         warps /= 2u;
-    while (!kPass && warps > 1u && chunk_layout(chunk_tile<(int)kWide>(), kWide, warps * per_warp).bytes > kSmemLimit) warps /= 2u;
     const uint32_t columns = warps * per_warp;
-    const dim3 grid(p.heads, (p.vdim + columns - 1u) / columns, sequences);
-    if constexpr (kPass) return launch_kernel(state_space_rows_kernel<L, NQ, V>, grid, dim3(warps * 32u), pass_smem(kWide, columns), stream, pdl, p);
-    else return launch_kernel(state_space_chunk_kernel<L, NQ, V>, grid, dim3(warps * 32u), chunk_layout(chunk_tile<(int)kWide>(), kWide, columns).bytes, stream, pdl, p);
+    return launch_kernel(state_space_rows_kernel<L, NQ, V>, dim3(p.heads, (p.vdim + columns - 1u) / columns, sequences), dim3(warps * 32u), pass_smem(kWide, columns),
+                         stream, pdl, p);
 }
 
-// Chunks hold half the columns a lane: twice the warps hide more of one another's waits.
-template <bool kPass>
-int launch_by_state(const StateSpace& p, cudaStream_t stream, bool pdl) {
-    constexpr int V = kPass ? 4 : 2;
-    const uint32_t fours = p.state_row() / 4u;
-    if (fours <= 1u) return launch_recurrence<1, 1, V, kPass>(p, stream, pdl);
-    if (fours <= 2u) return launch_recurrence<1, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 4u) return launch_recurrence<2, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 8u) return launch_recurrence<4, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 16u) return launch_recurrence<8, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 32u) return launch_recurrence<16, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 64u) return launch_recurrence<32, 2, V, kPass>(p, stream, pdl);
-    if (fours <= 128u) return launch_recurrence<32, 4, V, kPass>(p, stream, pdl);
-    return launch_recurrence<32, 8, 2, kPass>(p, stream, pdl);
+template <int NT>
+int launch_chunk(const StateSpace& p, const StateChunk& k, cudaStream_t stream) {
+    static std::once_flag once[64];
+    const int status = allow_smem(state_space_chunk_kernel<NT>, once, kChunkSmem);
+    if (status != GF_OK) return status;
+    state_space_chunk_kernel<NT><<<dim3(p.heads, (p.vdim + k.columns - 1u) / k.columns), (k.columns / 16u * k.splits + kHelpers) * 32u, chunk_layout(k).bytes, stream>>>(p, k);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
+}
+
+template <int T>
+int launch_convolution(const StateSpace& p, const StateChunk& k, cudaStream_t stream) {
+    static std::once_flag once[64];
+    const int status = allow_smem(convolve_chunk_kernel<T>, once, kChunkSmem);
+    if (status != GF_OK) return status;
+    const uint32_t x_all = p.heads * ((p.vdim + k.columns - 1u) / k.columns) * k.x_ld;
+    convolve_chunk_kernel<T><<<dim3(p.groups + (x_all + kConvolveThreads - 1u) / kConvolveThreads, (p.rows + kConvolveRows - 1u) / kConvolveRows), kConvolveThreads,
+                               2u * kConvolveRows * k.n_ld * 4u, stream>>>(p, k);
+    GF_CUDA(cudaGetLastError());
+    return GF_OK;
 }
 
 bool usable(const StateSpace& p) {
@@ -568,23 +614,45 @@ bool usable(const StateSpace& p) {
 int launch_state_space_rows(const StateSpace& p, cudaStream_t stream, bool pdl) {
     // Rows of the pass and the rows they look back at share the ring.
     if (!usable(p) || p.input_mask + 1u < p.tap_count - 1u + (p.ring_stride ? 1u : p.rows)) return fail(GF_ERR_INVALID, "state space: bad arguments");
-    return launch_by_state<true>(p, stream, pdl);
+    const uint32_t fours = p.state_row() / 4u;
+    if (fours <= 1u) return launch_rows<1, 1, 4>(p, stream, pdl);
+    if (fours <= 2u) return launch_rows<1, 2, 4>(p, stream, pdl);
+    if (fours <= 4u) return launch_rows<2, 2, 4>(p, stream, pdl);
+    if (fours <= 8u) return launch_rows<4, 2, 4>(p, stream, pdl);
+    if (fours <= 16u) return launch_rows<8, 2, 4>(p, stream, pdl);
+    if (fours <= 32u) return launch_rows<16, 2, 4>(p, stream, pdl);
+    if (fours <= 64u) return launch_rows<32, 2, 4>(p, stream, pdl);
+    if (fours <= 128u) return launch_rows<32, 4, 4>(p, stream, pdl);
+    return launch_rows<32, 8, 2>(p, stream, pdl);
+}
+
+StateChunk state_space_chunk(const StateSpace& p) {
+    StateChunk k;
+    k.per_warp = p.state <= 8u ? 8u : p.state <= 16u ? 16u : p.state <= 256u ? 32u : 64u;
+    k.splits = (p.state + k.per_warp - 1u) / k.per_warp;
+    uint32_t sixteens = std::max(1u, std::min((p.vdim + 15u) / 16u, kChunkWarps / k.splits));
+    while (sixteens > 1u && (uint64_t)p.heads * ((p.vdim + sixteens * 16u - 1u) / (sixteens * 16u)) * 5u < (uint64_t)sm_count() * 4u) sixteens = (sixteens + 1u) / 2u;
+    k.columns = sixteens * 16u;
+    // Row lengths that put a fragment's lanes into different banks.
+    k.n_ld = k.splits * k.per_warp + 8u;
+    k.x_ld = k.columns + 8u;
+    k.tile = 32u;
+    while (k.tile > 8u && chunk_layout(k).bytes > kChunkSmem) k.tile /= 2u;
+    return k;
 }
 
 int launch_state_space_chunk(const StateSpace& p, cudaStream_t stream) {
-    if (!usable(p) || p.ring_stride || !p.x || !p.b || !p.c || !p.steps || !p.cb || p.input_mask + 1u < p.tap_count - 1u) return fail(GF_ERR_INVALID, "state space: bad arguments");
-    const dim3 grid(p.groups + (p.heads * p.x_row() + kConvolveThreads - 1u) / kConvolveThreads, (p.rows + kConvolveRows - 1u) / kConvolveRows);
-    const uint32_t smem = 2u * kConvolveRows * p.state_row() * 4u;
-    static std::once_flag once[3][64];
-    int status = allow_smem(convolve_chunk_kernel<4>, once[0], 2u * kConvolveRows * kMaxStateSize * 4u);
-    if (status == GF_OK) status = allow_smem(convolve_chunk_kernel<8>, once[1], 2u * kConvolveRows * kMaxStateSize * 4u);
-    if (status == GF_OK) status = allow_smem(convolve_chunk_kernel<0>, once[2], 2u * kConvolveRows * kMaxStateSize * 4u);
+    if (!usable(p) || p.ring_stride || !p.x || !p.b || !p.c || !p.steps || !p.factors || !p.error_flag || p.input_mask + 1u < p.tap_count - 1u)
+        return fail(GF_ERR_INVALID, "state space: bad arguments");
+    const StateChunk k = state_space_chunk(p);
+    const int status = p.tap_count <= 4u ? launch_convolution<4>(p, k, stream) : p.tap_count <= 8u ? launch_convolution<8>(p, k, stream) : launch_convolution<0>(p, k, stream);
     if (status != GF_OK) return status;
-    if (p.tap_count <= 4u) convolve_chunk_kernel<4><<<grid, kConvolveThreads, smem, stream>>>(p);
-    else if (p.tap_count <= 8u) convolve_chunk_kernel<8><<<grid, kConvolveThreads, smem, stream>>>(p);
-    else convolve_chunk_kernel<0><<<grid, kConvolveThreads, smem, stream>>>(p);
-    GF_CUDA(cudaGetLastError());
-    return launch_by_state<false>(p, stream, false);
+    switch (k.per_warp) {
+        case 8u: return launch_chunk<1>(p, k, stream);
+        case 16u: return launch_chunk<2>(p, k, stream);
+        case 32u: return launch_chunk<4>(p, k, stream);
+        default: return launch_chunk<8>(p, k, stream);
+    }
 }
 
 }  // namespace gf

@@ -26,20 +26,25 @@ struct StateSpace {
     const uint32_t* slots = nullptr;
     uint32_t rows = 0, heads = 0, vdim = 0, state = 0, groups = 0, tap_count = 0, input_mask = 0;
     float* out = nullptr;                // [rows][heads * vdim]: passes: y * silu(gate); chunks: y
-    // Chunks: the convolved inputs, x [rows][heads][vdim rounded up to 4], B and C [rows][groups][N rounded up to 4],
-    // (dt, decay * dt) [rows][heads], and the products of a row's C with the B of the rows of its four up to itself
-    // [rows][groups][4].
-    float *x = nullptr, *b = nullptr, *c = nullptr, *cb = nullptr;
+    // Chunks (StateChunk k, the rows rounded up to eight): the convolved inputs, x [heads][blocks of columns][rows][x_ld], B
+    // and C [groups][rows][n_ld]; (dt, decay * dt) [rows][heads]; what a head's rows within their eight owe one another
+    // [heads][rows][kStateFactors].
+    float *x = nullptr, *b = nullptr, *c = nullptr, *factors = nullptr;
     float2* steps = nullptr;
+    int* error_flag = nullptr;           // set when a bounded wait for a copy gives up
 
     __host__ __device__ uint32_t inner() const { return heads * vdim; }
     __host__ __device__ uint32_t channels() const { return inner() + 2u * groups * state; }
     __host__ __device__ uint32_t state_row() const { return (state + 3u) & ~3u; }
-    __host__ __device__ uint32_t x_row() const { return (vdim + 3u) & ~3u; }
     __host__ __device__ uint32_t input_row() const { return (channels() + 3u) & ~3u; }
     __host__ __device__ size_t slot_elements() const { return (size_t)heads * vdim * state_row(); }
 };
-constexpr uint32_t kMaxStateSize = 1024;
+constexpr uint32_t kMaxStateSize = 1024, kStateFactors = 12;
+
+// How a chunk is cut up: a block takes `columns` of vdim of a head, `splits` warps share N by `per_warp` values, and `tile`
+// tokens are in shared memory at a time, in rows of n_ld and x_ld values.
+struct StateChunk { uint32_t columns = 0, splits = 0, per_warp = 0, tile = 0, n_ld = 0, x_ld = 0; };
+StateChunk state_space_chunk(const StateSpace& p);
 
 // Rows of a pass, convolution included.
 int launch_state_space_rows(const StateSpace& p, cudaStream_t stream, bool pdl);

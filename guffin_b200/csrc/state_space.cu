@@ -366,7 +366,7 @@ __global__ void __launch_bounds__((kChunkWarps + kHelpers) * 32) state_space_chu
         const float *b = reinterpret_cast<const float*>(from), *c = reinterpret_cast<const float*>(from + at.c), *x = reinterpret_cast<const float*>(from + at.x);
         const float* factors = reinterpret_cast<const float*>(from + at.factors);      // a row: M, exp(A_t), dt exp(A_7 - A_t), exp(A_7)
         float* y = reinterpret_cast<float*>(smem + at.y + (tile & 1u) * at.y_stage);
-#pragma unroll 1
+#pragma unroll 2
         for (uint32_t t0 = 0; t0 < k.tile && tile * k.tile + t0 < rows; t0 += 8u) {
             const float* x_at = x + (t0 + t) * k.x_ld + own + g;
             const float x0 = x_at[0], x1 = x_at[8], x2 = x_at[4u * k.x_ld], x3 = x_at[4u * k.x_ld + 8u];
@@ -403,12 +403,12 @@ __global__ void __launch_bounds__((kChunkWarps + kHelpers) * 32) state_space_chu
             const float u0 = eight[2u * t * kStateFactors + 8u], u1 = eight[(2u * t + 1u) * kStateFactors + 8u];
 #pragma unroll
             for (int i = 0; i < 4; ++i) y0[i] = (y0[i] + (y1[i] + y2[i])) * (i & 1 ? u1 : u0);
-            if (split == 0u) {
+            if (split < 3u) {                                          // the three terms, one a warp where there are as many
                 const Split4 xs(x0, x1, x2, x3);
                 const float m0 = eight[g * kStateFactors + t], m1 = eight[g * kStateFactors + t + 4u], mh0 = leading(m0), mh1 = leading(m1);
-                mma_tf32(y0, xs.hi, mh0, mh1);
-                mma_tf32(y0, xs.hi, m0 - mh0, m1 - mh1);
-                mma_tf32(y0, xs.lo, mh0, mh1);
+                if (split == 0u) mma_tf32(y0, xs.hi, mh0, mh1);
+                if (k.splits < 3u ? split == 0u : split == 1u) mma_tf32(y0, xs.hi, m0 - mh0, m1 - mh1);
+                if (k.splits < 3u ? split == 0u : split == 2u) mma_tf32(y0, xs.lo, mh0, mh1);
             }
             float* y_at = y + (split * k.tile + t0 + 2u * t) * k.x_ld + own + g;
             y_at[0] = y0[0];
@@ -506,6 +506,15 @@ __global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const 
         return;
     }
     const uint32_t group = blockIdx.x, per_group = p.heads / p.groups, np = k.n_ld;
+    // The steps of the first heads stay in shared memory.
+    constexpr uint32_t kNear = 64;
+    __shared__ float2 near[kConvolveRows * kNear];
+    for (uint32_t i = tid; i < kConvolveRows * per_group; i += kConvolveThreads) {
+        const uint32_t r = i / per_group, h = i % per_group;
+        const float2 step = r < live ? step_of(p, p.raw, row + r, group * per_group + h) : make_float2(0.0f, 0.0f);
+        if (h < kNear) near[r * kNear + h] = step;
+        else p.steps[(size_t)(row + r) * p.heads + group * per_group + h] = step;
+    }
     for (uint32_t i = tid; i < 2u * np; i += kConvolveThreads) {
         const uint32_t which = i / np, n = i % np;
         float *out = (which ? p.c : p.b) + ((size_t)group * all_rows + row) * np + n, *here = vectors + which * kConvolveRows * np + n;
@@ -516,10 +525,6 @@ __global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const 
             here[r * np] = v;
             out[r * np] = v;
         });
-    }
-    for (uint32_t i = tid; i < kConvolveRows * per_group; i += kConvolveThreads) {
-        const uint32_t r = i / per_group, head = group * per_group + i % per_group;
-        p.steps[(size_t)(row + r) * p.heads + head] = r < live ? step_of(p, p.raw, row + r, head) : make_float2(0.0f, 0.0f);
     }
     __shared__ float cb[kConvolveRows * 8u];
     __syncthreads();
@@ -535,11 +540,11 @@ __global__ void __launch_bounds__(kConvolveThreads) convolve_chunk_kernel(const 
     __syncthreads();
     // The factors of every head: element (t, s) of M, and with s = t the row's exponentials.
     for (uint32_t i = tid; i < per_group * kConvolveRows * 8u; i += kConvolveThreads) {
-        const uint32_t head = group * per_group + i / (kConvolveRows * 8u), t = i / 8u % kConvolveRows, s = i % 8u;
+        const uint32_t h = i / (kConvolveRows * 8u), head = group * per_group + h, t = i / 8u % kConvolveRows, s = i % 8u;
         float between = 0.0f, before = 0.0f, behind = 0.0f, dt = 0.0f;
 #pragma unroll
         for (uint32_t l = 0; l < 8u; ++l) {
-            const float2 step = p.steps[(size_t)(row + l) * p.heads + head];
+            const float2 step = h < kNear ? near[l * kNear + h] : p.steps[(size_t)(row + l) * p.heads + head];
             if (l > s && l <= t) between += step.y;
             (l <= t ? before : behind) += step.y;
             if (l == s) dt = step.x;

@@ -511,7 +511,7 @@ int launch_row_product(RowProduct p, cudaStream_t stream, bool pdl, uint32_t& la
     const bool single = p.input == kRowRouted || p.input == kRowExperts;
     uint32_t k_max = 0, sets = 0, widest = 0;
     // Groups per CTA from the shapes alone, so that a row's sums are added in the same order whatever the row count.
-    const uint32_t wanted = 3u * (uint32_t)sm_count();
+    const uint32_t wanted = 2u * (uint32_t)sm_count();              // what is resident at once
     for (uint32_t i = 0; i < p.count; ++i) {
         RowMatrix& m = p.m[i];
         if (!m.weight || !m.out || m.k == 0 || m.n == 0) return fail(GF_ERR_INVALID, "row product: bad matrix");

@@ -265,22 +265,24 @@ __device__ __forceinline__ void prepare_fused(const GroupedAttention& p, const F
     }
 }
 
-constexpr uint32_t kRowsWarps = 4, kRowsTile = 16;
+constexpr uint32_t kRowsTile = 16;
+template <int G> constexpr uint32_t rows_warps() { return G <= 8 ? 8u : 4u; }      // as many as have room for two tiles each
 
 // A block serves sixteen queries of one key/value head -- (row, head of the group) pairs, heads fastest -- against one
 // partition of the keys; its warps take tiles of keys in turn, the next one copied while this one is used, and keep
 // scores, weights and outputs in registers.  G = groups of sixteen dimensions a head has at most.
 template <int G>
-__global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(const __grid_constant__ GroupedAttention p) {
+__global__ void __launch_bounds__(rows_warps<G>() * 32) grouped_attention_kernel(const __grid_constant__ GroupedAttention p) {
     extern __shared__ __align__(16) uint8_t smem[];
-    __shared__ float warp_top[kRowsWarps][16], warp_sum_of[kRowsWarps][16], scratch[kRowsWarps][kGroupedMaxParts * 3u];
+    constexpr uint32_t kWarps = rows_warps<G>();
+    __shared__ float warp_top[kWarps][16], warp_sum_of[kWarps][16], scratch[kWarps][kGroupedMaxParts * 3u];
     constexpr uint32_t kTile = kRowsTile;
     const uint32_t stride = p.row_head + 8u, pieces = p.row_head / 8u;
     const uint32_t tid = threadIdx.x, warp = tid >> 5, lane = tid & 31u, g = lane >> 2, t = lane & 3u;
     __half* q_tile = reinterpret_cast<__half*>(smem);
     __half* tiles = q_tile + 16u * stride;                             // [warps][2][keys, values][kTile][stride]
     __half* mine = tiles + (size_t)warp * 4u * kTile * stride;
-    __half* own_rows = tiles + (size_t)kRowsWarps * 4u * kTile * stride;           // fused: [keys, values][rows][stride], then the turns
+    __half* own_rows = tiles + (size_t)kWarps * 4u * kTile * stride;           // fused: [keys, values][rows][stride], then the turns
     const bool chain = p.ring_stride == 0u;
     const uint32_t kv = blockIdx.z % p.kv_heads, z = blockIdx.z / p.kv_heads, part = blockIdx.y;
     const uint32_t group = p.heads / p.kv_heads, queries = (chain ? p.rows : 1u) * group, first_query = blockIdx.x * 16u;
@@ -288,7 +290,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
     const StreamRings rings = p.rings[(size_t)z * p.ring_stride];
     const uint32_t end = base + min(first_query + 15u, queries - 1u) / group + 1u;      // keys the block's last query sees
     const uint32_t all = (end + kTile - 1u) / kTile;
-    constexpr uint32_t step = kRowsWarps;
+    constexpr uint32_t step = kWarps;
     const uint32_t tile_begin = (uint32_t)((uint64_t)all * part / p.parts), tile_end = (uint32_t)((uint64_t)all * (part + 1u) / p.parts);
     const __half *ring_k = static_cast<const __half*>(rings.ring_k) + kv * p.row_head, *ring_v = static_cast<const __half*>(rings.ring_v) + kv * p.row_head;
     const size_t own_at = (size_t)(chain ? 0u : z) * cache_row + kv * p.row_head;
@@ -317,7 +319,7 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         copies_commit();
         float2* turns = reinterpret_cast<float2*>(own_rows + 2u * rows * stride);
         const uint32_t half = p.prepare.rotated / 2u;
-        for (uint32_t i = tid; i < rows * half; i += kRowsWarps * 32u) turns[i] = rotation(p.prepare, base + i / half, i % half);
+        for (uint32_t i = tid; i < rows * half; i += kWarps * 32u) turns[i] = rotation(p.prepare, base + i / half, i % half);
         const uint32_t last_query = min(first_query + 15u, queries - 1u);
         FusedRows f;
         f.first_row = first_query / group; f.query_rows = last_query / group - f.first_row + 1u; f.rows = rows; f.row0 = chain ? 0u : z;
@@ -325,14 +327,14 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         f.own = tile_end * kTile > base;
         pdl_wait();
         pdl_launch_dependents();
-        prepare_fused<kRowsWarps * 32>(p, f, turns, kv, first_query, queries, q_tile, my_k, my_v, stride);
+        prepare_fused<kWarps * 32>(p, f, turns, kv, first_query, queries, q_tile, my_k, my_v, stride);
     } else {
         pdl_wait();
         pdl_launch_dependents();
         if (tile_begin + warp < tile_end) load_tile(tile_begin + warp, 0u);
         copies_commit();
         const __half* q = static_cast<const __half*>(p.q);
-        for (uint32_t m = tid >> 3; m < 16u; m += kRowsWarps * 4u) {
+        for (uint32_t m = tid >> 3; m < 16u; m += kWarps * 4u) {
             const uint32_t query = first_query + m;
             const bool valid = query < queries;
             const size_t row = chain ? query / group : z;
@@ -447,15 +449,15 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
     }
     __syncthreads();
 #pragma unroll 1
-    for (uint32_t m = warp; m < 16u; m += kRowsWarps) {
+    for (uint32_t m = warp; m < 16u; m += kWarps) {
         const uint32_t query = first_query + m;
         if (query >= queries) break;
         const uint32_t row = chain ? query / group : z, head = kv * group + query % group;
-        float most = warp_top[0][m], factor[kRowsWarps], total = 0.0f;
+        float most = warp_top[0][m], factor[kWarps], total = 0.0f;
 #pragma unroll
-        for (uint32_t w = 1; w < kRowsWarps; ++w) most = fmaxf(most, warp_top[w][m]);
+        for (uint32_t w = 1; w < kWarps; ++w) most = fmaxf(most, warp_top[w][m]);
 #pragma unroll
-        for (uint32_t w = 0; w < kRowsWarps; ++w) {
+        for (uint32_t w = 0; w < kWarps; ++w) {
             factor[w] = warp_top[w][m] == -INFINITY ? 0.0f : expf(warp_top[w][m] - most);
             total += factor[w] * warp_sum_of[w][m];
         }
@@ -470,14 +472,14 @@ __global__ void __launch_bounds__(kRowsWarps * 32) grouped_attention_kernel(cons
         for (uint32_t d = lane; d < p.vdim; d += 32u) {
             float v = 0.0f;
 #pragma unroll
-            for (uint32_t w = 0; w < kRowsWarps; ++w) v = fmaf(parked[(w * 16u + m) * parked_ld + d], factor[w], v);
+            for (uint32_t w = 0; w < kWarps; ++w) v = fmaf(parked[(w * 16u + m) * parked_ld + d], factor[w], v);
             if (p.parts == 1u) store_operand(p.result, row, head * p.vdim + d, v * scale);
             else p.partial_out[(((size_t)row * p.heads + head) * p.parts + part) * p.row_head + d] = v;
         }
     }
     if (p.parts == 1u || !last_to_arrive(p.counters + (size_t)blockIdx.z * gridDim.x + blockIdx.x, p.parts)) return;
 #pragma unroll 1
-    for (uint32_t m = warp; m < 16u; m += kRowsWarps) {
+    for (uint32_t m = warp; m < 16u; m += kWarps) {
         const uint32_t query = first_query + m;
         if (query >= queries) break;
         merge_query(p, chain ? query / group : z, kv * group + query % group, scratch[warp]);
@@ -568,8 +570,8 @@ int launch_rows(const GroupedAttention& p, cudaStream_t stream, bool pdl) {
     if (status != GF_OK) return status;
     const bool chain = p.ring_stride == 0u;
     const uint32_t rows = chain ? p.rows : 1u, queries = rows * (p.heads / p.kv_heads);
-    const uint32_t smem = (16u + kRowsWarps * 4u * kTile + (p.fused ? 2u * rows : 0u)) * (p.row_head + 8u) * 2u + (p.fused ? rows * p.prepare.rotated * 4u : 0u);
-    return launch_kernel(grouped_attention_kernel<G>, dim3((queries + 15u) / 16u, p.parts, p.kv_heads * (chain ? 1u : p.rows)), dim3(kRowsWarps * 32u), smem, stream, pdl, p);
+    const uint32_t smem = (16u + rows_warps<G>() * 4u * kTile + (p.fused ? 2u * rows : 0u)) * (p.row_head + 8u) * 2u + (p.fused ? rows * p.prepare.rotated * 4u : 0u);
+    return launch_kernel(grouped_attention_kernel<G>, dim3((queries + 15u) / 16u, p.parts, p.kv_heads * (chain ? 1u : p.rows)), dim3(rows_warps<G>() * 32u), smem, stream, pdl, p);
 }
 
 }  // namespace

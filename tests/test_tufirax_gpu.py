@@ -29,11 +29,11 @@ def plain(config, weights, tokens, precision):
 
 attention, state_space = syn.tufirax_attention, syn.tufirax_state_space
 CONFIGS = {
-    "attention alone": syn.tufirax_config(40, 53, [attention(6, 3, 10, 0.5, 7.0, 4, 900.0), attention(6, 3, 10, 0.5, 7.0, 4, 900.0)], 1e-3),
+    "attention alone": syn.tufirax_config(45, 53, [attention(6, 3, 10, 0.5, 7.0, 4, 900.0), attention(6, 3, 10, 0.5, 7.0, 4, 900.0)], 1e-3),
     "one head": syn.tufirax_config(36, 50, [attention(1, 1, 24, 0.3, 3.0, 24, 77.0, ff=20), attention(1, 1, 7, 0.4, 50.0, 2, 10.0, ff=9)], 1e-5),
     "heads of their own": syn.tufirax_config(64, 80, [attention(5, 5, 20, 0.9, 4.0, 12, 5e4, ff=33), attention(12, 2, 40, 0.2, 12.0, 40, 300.0)]),
     "wide heads": syn.tufirax_config(72, 64, [attention(3, 1, 144, 0.08, 9.0, 64, 1e4, ff=40), attention(2, 2, 272, 0.06, 20.0, 16, 1e3)]),
-    "states alone": syn.tufirax_config(36, 48, [state_space(4, 6, 5, 2, 2, 3), state_space(4, 6, 5, 2, 2, 3)], 1e-4),
+    "states alone": syn.tufirax_config(37, 48, [state_space(4, 6, 5, 2, 2, 3), state_space(4, 6, 5, 2, 2, 3)], 1e-4),
     "states and feed-forwards": syn.tufirax_config(48, 60, [state_space(3, 20, 24, 1, 1, 1, ff=30), state_space(6, 9, 17, 3, 7, 2, ff=11), state_space(1, 5, 3, 1, 3, 5)]),
     "wide states": syn.tufirax_config(56, 72, [state_space(2, 70, 140, 2, 4, 7), state_space(8, 64, 128, 4, 4, 8), state_space(2, 33, 270, 1, 5, 6)]),
     "shared in turn": syn.tufirax_config(60, 90, [

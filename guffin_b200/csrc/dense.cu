@@ -325,34 +325,34 @@ __global__ void __launch_bounds__(kRowThreads) row_product_kernel(const __grid_c
                 __syncthreads();
             }
         } else {
-        // Warps share the parts: several to a part where there are fewer parts than warps.
-        uint32_t per = kRowWarps;
-        while (per > 1u && per * p.norm_parts > kRowWarps) per /= 2u;
-        for (int r = 0; r < R; ++r) {
-            const float* x = p.in + (size_t)r * p.in_ld;
-            for (uint32_t unit = warp; unit < per * p.norm_parts; unit += kRowWarps) {
-                const uint32_t first = unit / per * part;
-                float sum = 0.0f;
-                for (uint32_t i = (unit % per) * 32u + lane; i < part; i += per * 32u) {
-                    const float v = x[first + i];
-                    act[r * k_pad + first + i] = v;
-                    sum = fmaf(v, v, sum);
-                }
-                sum = warp_sum(sum);
-                if (lane == 0) route_scratch[unit] = sum;
-            }
-            __syncthreads();
-            for (uint32_t i = tid; i < k_pad; i += kRowThreads) {
-                float v = 0.0f;
-                if (i < p.width) {
+            // Warps share the parts: several to a part where there are fewer parts than warps.
+            uint32_t per = kRowWarps;
+            while (per > 1u && per * p.norm_parts > kRowWarps) per /= 2u;
+            for (int r = 0; r < R; ++r) {
+                const float* x = p.in + (size_t)r * p.in_ld;
+                for (uint32_t unit = warp; unit < per * p.norm_parts; unit += kRowWarps) {
+                    const uint32_t first = unit / per * part;
                     float sum = 0.0f;
-                    for (uint32_t s = 0; s < per; ++s) sum += route_scratch[i / part * per + s];
-                    v = act[r * k_pad + i] * norm_factor(sum, part, p.eps) * p.gain1[i];
+                    for (uint32_t i = (unit % per) * 32u + lane; i < part; i += per * 32u) {
+                        const float v = x[first + i];
+                        act[r * k_pad + first + i] = v;
+                        sum = fmaf(v, v, sum);
+                    }
+                    sum = warp_sum(sum);
+                    if (lane == 0) route_scratch[unit] = sum;
                 }
-                act[r * k_pad + i] = v;
+                __syncthreads();
+                for (uint32_t i = tid; i < k_pad; i += kRowThreads) {
+                    float v = 0.0f;
+                    if (i < p.width) {
+                        float sum = 0.0f;
+                        for (uint32_t s = 0; s < per; ++s) sum += route_scratch[i / part * per + s];
+                        v = act[r * k_pad + i] * norm_factor(sum, part, p.eps) * p.gain1[i];
+                    }
+                    act[r * k_pad + i] = v;
+                }
+                __syncthreads();
             }
-            __syncthreads();
-        }
         }
     } else if (p.input == kRowLatent) {
         for (int r = 0; r < R; ++r) {

@@ -256,8 +256,8 @@ __global__ void __launch_bounds__(kMaxWarps * 32, 3) state_space_rows_kernel(con
 // as products on the tensor cores, in pairs of tf32 values (a value's leading bits and what they leave out) so that they
 // are as exact as f32 ones.  A warp keeps 16 columns (of vdim) x 8 NT values (of N) of the state in accumulators, which
 // are the first operand of the read-out as they lie: an accumulator's neighbouring columns 2 t and 2 t + 1 count as the
-// operand's t and t + 4.
-// Helper warps have the next tile's inputs and factors copied and write the last tile's outputs meanwhile.
+// operand's t and t + 4.  Helper warps have the next
+// tile's inputs and factors copied and write the last tile's outputs meanwhile.
 constexpr uint32_t kHelpers = 4;
 struct ChunkLayout { uint32_t c, x, factors, stage, y, y_stage, bytes; };
 __host__ __device__ inline ChunkLayout chunk_layout(const StateChunk& k) {      // bytes; two stages each of inputs and of outputs
@@ -274,9 +274,8 @@ __host__ __device__ inline ChunkLayout chunk_layout(const StateChunk& k) {      
 
 __device__ __forceinline__ void mma_tf32(float (&d)[4], const float (&a)[4], float b0, float b1) {
     asm("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-                 : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)),
-                   "r"(__float_as_uint(b1)));
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(__float_as_uint(a[0])), "r"(__float_as_uint(a[1])), "r"(__float_as_uint(a[2])), "r"(__float_as_uint(a[3])), "r"(__float_as_uint(b0)), "r"(__float_as_uint(b1)));
 }
 // The bits of a value that tf32 holds, and the rest.
 __device__ __forceinline__ float leading(float v) { return __uint_as_float(__float_as_uint(v) & 0xffffe000u); }
@@ -459,33 +458,34 @@ __device__ __forceinline__ void convolve_rows(const StateSpace& p, const float* 
     if constexpr (T == 0) {
         for (uint32_t r = 0; r < live; ++r) emit(r, convolve<false>(p, p.raw, ring, base, row + r, channel));
     } else {
-    constexpr int kBack = T - 1;
-    float v[kBack + (int)kConvolveRows], w[T];
-    const float* raw = p.raw + p.inner() + channel;
-    if (row >= (uint32_t)kBack && live == kConvolveRows) {
-        const float* from = raw + (size_t)(row - kBack) * p.raw_ld;
+        constexpr int kBack = T - 1;
+        float v[kBack + (int)kConvolveRows], w[T];
+        const float* raw = p.raw + p.inner() + channel;
+        if (row >= (uint32_t)kBack && live == kConvolveRows) {
+            const float* from = raw + (size_t)(row - kBack) * p.raw_ld;
 #pragma unroll
-        for (int i = 0; i < kBack + (int)kConvolveRows; ++i) v[i] = from[(size_t)i * p.raw_ld];
-    } else
+            for (int i = 0; i < kBack + (int)kConvolveRows; ++i) v[i] = from[(size_t)i * p.raw_ld];
+        } else {
 #pragma unroll
-    for (int i = 0; i < kBack + (int)kConvolveRows; ++i) {
-        const int r = (int)row + i - kBack;                            // a row of the chunk, or behind it
-        v[i] = 0.0f;
-        if (i < kBack && (uint32_t)(kBack - i) >= p.tap_count) continue;
-        if (r >= 0) { if ((uint32_t)r < row + live) v[i] = raw[(size_t)r * p.raw_ld]; }
-        else if (base >= (uint32_t)-r) v[i] = ring[(size_t)((base + (uint32_t)r) & p.input_mask) * p.input_row() + channel];
-    }
+            for (int i = 0; i < kBack + (int)kConvolveRows; ++i) {
+                const int r = (int)row + i - kBack;                    // a row of the chunk, or behind it
+                v[i] = 0.0f;
+                if (i < kBack && (uint32_t)(kBack - i) >= p.tap_count) continue;
+                if (r >= 0) { if ((uint32_t)r < row + live) v[i] = raw[(size_t)r * p.raw_ld]; }
+                else if (base >= (uint32_t)-r) v[i] = ring[(size_t)((base + (uint32_t)r) & p.input_mask) * p.input_row() + channel];
+            }
+        }
 #pragma unroll
-    for (int j = 0; j < T; ++j) w[j] = (uint32_t)j < p.tap_count ? p.taps[(size_t)channel * p.tap_count + p.tap_count - 1u - j] : 0.0f;
-    const float bias = p.tap_bias[channel];
+        for (int j = 0; j < T; ++j) w[j] = (uint32_t)j < p.tap_count ? p.taps[(size_t)channel * p.tap_count + p.tap_count - 1u - j] : 0.0f;
+        const float bias = p.tap_bias[channel];
 #pragma unroll
-    for (int r = 0; r < (int)kConvolveRows; ++r) {
-        if ((uint32_t)r >= live) break;
-        float sum = 0.0f;
+        for (int r = 0; r < (int)kConvolveRows; ++r) {
+            if ((uint32_t)r >= live) break;
+            float sum = 0.0f;
 #pragma unroll
-        for (int j = T - 1; j >= 0; --j) sum = fmaf(w[j], v[kBack + r - j], sum);
-        emit((uint32_t)r, silu(sum + bias));
-    }
+            for (int j = T - 1; j >= 0; --j) sum = fmaf(w[j], v[kBack + r - j], sum);
+            emit((uint32_t)r, silu(sum + bias));
+        }
     }
 }
 

@@ -359,7 +359,7 @@ GF_API int gf_route(const float* logits_dev, uint32_t rows, uint32_t experts, ui
 
 /* ---- models described by a configuration file.  No counterpart in the reference, which serves the Gemma families
  * only.  `config_json` is the text of a config.json whose "architecture" names an entry of the registry
- * (gf_architectures, one name per line): "Zasevik" (a layered decoder: every layer names its mixer and its
+ * (gf_architectures, one name per line): "Zasevik" and "Tufirax" (layered decoders: every layer names its mixer and its
  * feed-forward with their sizes and constants; bf16 tensors bound by name), or "Gemma2" / "Gemma3" (the fields of
  * gf_model_config under their own names; tensors bound by kind).  A layered plan has the same passes, publication,
  * streams, candidate selection and generation engine as any other plan; tensor-parallel shards, the decode pass
@@ -404,6 +404,8 @@ GF_API int gf_model_prefill(gf_model* model, const uint32_t* tokens_host, uint32
  * plans as exact row passes.  Synchronises, and reports what gf_model_status would, when logits_host is given. */
 GF_API int gf_model_extend(gf_model* model, const uint32_t* tokens_host, uint32_t count, const uint32_t* want,
                            uint32_t want_count, float* logits_host);
+/* Takes published rows back, up to one pass.  A plan with recurrent layers holds the states after its last few positions
+ * (one more than the rows of a pass) and goes back no further than these, nor to before the end of a chunk. */
 GF_API int gf_model_truncate(gf_model* model, uint32_t position);
 /* gf_model_prefill ingests prompts of 65 tokens or more in chunks of up to 256 rows, every projection of
  * a chunk as one bf16 tensor-core GEMM (run_gemma3_resident_prefill's 128-row chunks,

@@ -36,6 +36,7 @@ CONFIGS = {
     "states alone": syn.tufirax_config(37, 48, [state_space(4, 6, 5, 2, 2, 3), state_space(4, 6, 5, 2, 2, 3)], 1e-4),
     "states and feed-forwards": syn.tufirax_config(48, 60, [state_space(3, 20, 24, 1, 1, 1, ff=30), state_space(6, 9, 17, 3, 7, 2, ff=11), state_space(1, 5, 3, 1, 3, 5)]),
     "wide states": syn.tufirax_config(56, 72, [state_space(2, 70, 140, 2, 4, 7), state_space(8, 64, 128, 4, 4, 8), state_space(2, 33, 270, 1, 5, 6)]),
+    "many heads": syn.tufirax_config(52, 66, [attention(20, 1, 12, 0.4, 8.0, 6, 500.0), state_space(70, 3, 9, 1, 11, 1), state_space(8, 64, 20, 2, 4, 2, ff=13)]),
     "shared in turn": syn.tufirax_config(60, 90, [
         state_space(4, 12, 20, 2, 4, 4), attention(4, 2, 18, 0.3, 6.0, 10, 2e3, ff=28), state_space(4, 12, 20, 2, 4, 4, weights_of=0),
         attention(4, 2, 18, 0.3, 6.0, 10, 2e3, ff=28, weights_of=1), attention(8, 1, 16, 0.25, 30.0, 16, 1e4), state_space(4, 12, 20, 2, 4, 4, weights_of=2),
@@ -86,7 +87,7 @@ def test_whole_prompts_and_rows(gm, name, precision):
     assert plan.status() == 0 and plan.position == 150
 
 
-@pytest.mark.parametrize("name", ["heads of their own", "states alone", "states and feed-forwards", "wide states", "shared in turn"])
+@pytest.mark.parametrize("name", ["heads of their own", "states alone", "states and feed-forwards", "wide states", "many heads", "shared in turn"])
 @pytest.mark.parametrize("precision", PRECISIONS)
 def test_portions_of_every_size(gm, name, precision):
     config, bits, weights = make(gm, name)
